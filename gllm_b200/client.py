@@ -252,8 +252,8 @@ class Client:
     def _install(self, model_id, kind, loaded, cfg, weights, tokenizer, device=None, dtype=None):
         from .backend import detect_backend
         from .engine.executor import EngineConfig, LLMEngine
-        from .models.decoder import DecoderModel
         from .models.encoder import EncoderModel
+        from .models.registry import decoder_class
         from .tokenizer import TokenizerHandle
         be = detect_backend(self._backend_name)
         dev = torch.device(device) if device is not None else be.device
@@ -273,8 +273,9 @@ class Client:
                     if self._weight_paging and cfg.is_moe and tp is None and not kv_kw.get("weight_quant"):
                         kv_kw["expert_slots"] = self.config.expert_slots or max(4 * cfg.num_experts_per_tok,
                                                                                 cfg.num_experts // 4)
-                    model = DecoderModel(cfg, weights, device=dev, dtype=dt,
-                                         max_positions=min(cfg.max_position_embeddings, self.config.max_model_len), **kv_kw)
+                    model = decoder_class(cfg)(cfg, weights, device=dev, dtype=dt,
+                                               max_positions=min(cfg.max_position_embeddings, self.config.max_model_len),
+                                               **kv_kw)
                     ec = EngineConfig(max_num_seqs=self.config.max_num_seqs, max_model_len=self.config.max_model_len,
                                       max_batch_tokens=self.config.max_batch_tokens,
                                       prefill_chunk=self.config.max_batch_tokens,
@@ -373,7 +374,7 @@ class Client:
         want_fp8 = pref in ("fp8", "fp8_e4m3") or (pref == "auto" and (variant.kivi or cfg.kv_cache_dtype in ("fp8", "fp8_e4m3")))
         self.kv_plan = {"variant": variant, "kv_cache_dtype": "fp8" if want_fp8 and dev.type == "cuda" else "bf16",
                         "bf16_bytes": bf16_per_token * tokens}
-        if want_fp8 and dev.type == "cuda" and not cfg.is_mla:
+        if want_fp8 and dev.type == "cuda" and not cfg.is_mla and not cfg.is_hybrid:
             return dict(kv_dtype=torch.float8_e4m3fn, kv_scale=float(self.config.kv_scale))
         return {}
 
@@ -549,7 +550,7 @@ class Client:
         lens = [len(s) for s in seqs]
         T = sum(lens)
         pages = [(n + 15) // 16 for n in lens]
-        kv = m.alloc_kv_cache(sum(pages) + 1)
+        kv = m.alloc_kv_cache(sum(pages) + 1, state_slots=len(seqs))
         bt = torch.zeros((len(seqs), max(pages)), dtype=torch.int32, device=dev)
         slot = torch.empty(T, dtype=torch.int32, device=dev)
         starts, p0, o = [], 0, 0
@@ -570,7 +571,7 @@ class Client:
             x = m.final_hidden(x)
         else:
             m.forward(batch, kv, return_hidden=True, capture_layers={layer})
-            x = m.captured[layer]
+            x = m.captured[layer].to(m.dtype)
         return ops.pool(x.contiguous(), q_start, q_len, pooling).float().cpu()
 
     def encode_to_layer(self, texts: Sequence[str], layer: int, pooling: str = "mean") -> torch.Tensor:

@@ -114,7 +114,8 @@ struct SoftmaxState {
 // One 16-token page: S = Q·Kᵀ (16x16), mask, online softmax, O += P·V.
 // k_smem / v_smem: shared addresses of the page's K and V tiles, each two 2 KB boxes
 // ([d half][token][64 bf16], 128-byte swizzle). Row r may attend tokens in [lo_r, hi_r).
-template <bool KV8>
+// kFW (bf16 pages): the softmax weights enter the second product as a bf16 value and its bf16 remainder.
+template <bool KV8, bool kFW = false>
 __device__ __forceinline__ void attend_page(const uint32_t (&qf)[8][4], uint32_t k_smem, uint32_t v_smem,
                                             int tok_base, int lo0, int hi0, int lo1, int hi1, float scale_log2,
                                             float (&o)[16][4], SoftmaxState& st) {
@@ -220,6 +221,14 @@ __device__ __forceinline__ void attend_page(const uint32_t (&qf)[8][4], uint32_t
     pf[2] = pack_bf16x2(s[1][0], s[1][1]);
     pf[3] = pack_bf16x2(s[1][2], s[1][3]);
   }
+  [[maybe_unused]] uint32_t pr[4];
+  if constexpr (kFW) {
+    auto rest = [](float a, float b) { return pack_bf16x2(a - bf16_round(a), b - bf16_round(b)); };
+    pr[0] = rest(s[0][0], s[0][1]);
+    pr[1] = rest(s[0][2], s[0][3]);
+    pr[2] = rest(s[1][0], s[1][1]);
+    pr[3] = rest(s[1][2], s[1][3]);
+  }
   if constexpr (KV8) {
     // V tile: [16 tokens][128 bytes]; a transposed 8x8 b16 matrix hands thread (g, t) the bytes
     // {tok 2t: features 2g, 2g+1 | tok 2t+1: features 2g, 2g+1} of a 16-feature block: bytes 0,2 are the even-feature
@@ -263,6 +272,10 @@ __device__ __forceinline__ void attend_page(const uint32_t (&qf)[8][4], uint32_t
       }
       mma_bf16_16816(o[2 * j], pf, b0, b1);
       mma_bf16_16816(o[2 * j + 1], pf, b2, b3);
+      if constexpr (kFW) {
+        mma_bf16_16816(o[2 * j], pr, b0, b1);
+        mma_bf16_16816(o[2 * j + 1], pr, b2, b3);
+      }
     }
   }
 }
@@ -304,6 +317,7 @@ __device__ __forceinline__ void softmax_t_finish(SoftmaxStateT& st) {
   }
 }
 // One page: tokens [tok_base, tok_base + 16) of which [lo, hi) may be attended (the same range for every head).
+template <bool kFW>
 __device__ __forceinline__ void attend_page_t(const uint32_t (&qt)[8][2], uint32_t k_smem, uint32_t v_smem, int tok_base,
                                               int lo, int hi, float scale_log2, float (&o)[8][4], SoftmaxStateT& st) {
   const int lane = threadIdx.x & 31;
@@ -352,6 +366,11 @@ __device__ __forceinline__ void attend_page_t(const uint32_t (&qt)[8][2], uint32
   // P^T as the B operand (k = token, n = head): the accumulator layout transposed 8 x 8 at a time
   const uint32_t pb0 = movmatrix_trans(pack_bf16x2(s0, s1));
   const uint32_t pb1 = movmatrix_trans(pack_bf16x2(s2, s3));
+  [[maybe_unused]] uint32_t pr0 = 0, pr1 = 0;
+  if constexpr (kFW) {
+    pr0 = movmatrix_trans(pack_bf16x2(s0 - bf16_round(s0), s1 - bf16_round(s1)));
+    pr1 = movmatrix_trans(pack_bf16x2(s2 - bf16_round(s2), s3 - bf16_round(s3)));
+  }
   {
     // A = V^T: transposed loads of (tokens 0-7 | 8-15) x (chunk 2 mt | 2 mt + 1)
     const int tok = (lane & 7) + ((lane >> 4) << 3);
@@ -369,6 +388,7 @@ __device__ __forceinline__ void attend_page_t(const uint32_t (&qt)[8][2], uint32
         o[mt][3] *= corrB;
       }
       mma_bf16_16816(o[mt], a, pb0, pb1);
+      if constexpr (kFW) mma_bf16_16816(o[mt], a, pr0, pr1);
     }
   }
 }
@@ -514,7 +534,7 @@ constexpr int kDecSmem = kDecWarps * kDecStages * 2 * kPageBytes + 1024 + 1024;
 // extra warps hide the latency of the per-fragment conversions
 constexpr int kDecSmem8 = kDecWarps * kDecStages * 2 * (kPageBytes / 2) + 1024 + 1024;
 
-template <bool KV8>
+template <bool KV8, bool kFW = false>
 __global__ void __launch_bounds__(kDecWarps * 32, KV8 ? 3 : 2)
 paged_decode_kernel(const __grid_constant__ CUtensorMap tmap_kv, const DecodeParams p) {
   constexpr int kTile = KvFmt<KV8>::kBytes;
@@ -535,7 +555,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmap_kv, const DecodePar
     ctx = p.max_blocks * kPage;
   }
   const int n_pages = (ctx + kPage - 1) / kPage;
-  const int first_tok = (p.window > 0 && ctx > p.window) ? ctx - p.window : 0;
+  const int first_tok = attn_first_key(ctx - 1, p.window);
   const int first_page = first_tok / kPage;
   // never more splits than the scratch was sized for: widen the split when the context is long
   const int span = n_pages - first_page;
@@ -622,10 +642,10 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmap_kv, const DecodePar
         attend_page_t8(qt, kaddr, kaddr + kTile, tok_base, first_tok, ctx, p.scale_log2,
                        *reinterpret_cast<float(*)[8][4]>(&o[0][0]), stt);
       else
-        attend_page_t(qt, kaddr, kaddr + kTile, tok_base, first_tok, ctx, p.scale_log2,
+        attend_page_t<kFW>(qt, kaddr, kaddr + kTile, tok_base, first_tok, ctx, p.scale_log2,
                       *reinterpret_cast<float(*)[8][4]>(&o[0][0]), stt);
     } else {
-      attend_page<KV8>(qf, kaddr, kaddr + kTile, tok_base, first_tok, ctx, first_tok, ctx, p.scale_log2, o, st);
+      attend_page<KV8, kFW>(qf, kaddr, kaddr + kTile, tok_base, first_tok, ctx, first_tok, ctx, p.scale_log2, o, st);
     }
     __syncwarp();
     const int nxt = i + kDecStages;
@@ -816,17 +836,14 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_kv, const PrefillP
   } else {
     hi0 = hi1 = ctx;
   }
-  if (p.window > 0) {
-    lo0 = max(0, hi0 - p.window);
-    lo1 = max(0, hi1 - p.window);
-  }
+  lo0 = attn_first_key(hi0 - 1, p.window);
+  lo1 = attn_first_key(hi1 - 1, p.window);
   if (row0 >= qlen) hi0 = lo0 = 0;
   if (row1 >= qlen) hi1 = lo1 = 0;
   // KV range needed by this CTA
   const int last_row = min(qblk * kPfRows + kPfRows, qlen) - 1;
   const int kv_hi = p.causal ? (pos0 + last_row + 1) : ctx;
-  int kv_lo = 0;
-  if (p.window > 0) kv_lo = max(0, (p.causal ? pos0 + qblk * kPfRows + 1 : ctx) - p.window);
+  const int kv_lo = attn_first_key((p.causal ? pos0 + qblk * kPfRows + 1 : ctx) - 1, p.window);
   const int page_lo = kv_lo / kPage;
   const int page_hi = (kv_hi + kPage - 1) / kPage;
   const int n_blocks = (page_hi - page_lo + kPfBlockPages - 1) / kPfBlockPages;
@@ -946,7 +963,7 @@ GLLM_API long long gllm_decode_scratch_floats(int batch, int n_q_heads, int max_
   return static_cast<long long>(batch) * n_q_heads * max_splits * (kHD + 1);
 }
 
-template <bool KV8>
+template <bool KV8, bool kFW = false>
 static int paged_decode_impl(const void* q, void* out, const void* kv_cache, int num_pages,
                              const int* block_tables, int max_blocks, const int* ctx_lens, int batch,
                              int n_q_heads, int n_kv_heads, float scale, int pages_per_split, int max_splits,
@@ -979,22 +996,28 @@ static int paged_decode_impl(const void* q, void* out, const void* kv_cache, int
   int dev = 0;
   cudaGetDevice(&dev);
   if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(paged_decode_kernel<KV8>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(paged_decode_kernel<KV8, kFW>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          KV8 ? kDecSmem8 : kDecSmem);
     if (e != cudaSuccess) { set_last_error("paged_decode: %s", cudaGetErrorString(e)); return -1; }
     attr_set[dev & 63] = true;
   }
   dim3 grid(p.max_splits, n_kv_heads, batch);
-  cudaError_t e = launch_kernel(paged_decode_kernel<KV8>, grid, dim3(kDecWarps * 32), KV8 ? kDecSmem8 : kDecSmem,
+  cudaError_t e = launch_kernel(paged_decode_kernel<KV8, kFW>, grid, dim3(kDecWarps * 32), KV8 ? kDecSmem8 : kDecSmem,
                                 (cudaStream_t)stream, true, 0, t, p);
   if (e != cudaSuccess) { (void)cudaGetLastError(); set_last_error("paged_decode launch: %s", cudaGetErrorString(e)); return -1; }
   return 0;
 }
 
+// full_weights: softmax weights as bf16 pairs in the second product.
 GLLM_API int gllm_paged_decode(const void* q, void* out, const void* kv_cache, int num_pages,
                                const int* block_tables, int max_blocks, const int* ctx_lens, int batch,
                                int n_q_heads, int n_kv_heads, float scale, int pages_per_split, int max_splits,
-                               float* scratch, int* counters, int window, const float* sinks, void* stream) {
+                               float* scratch, int* counters, int window, const float* sinks, int full_weights,
+                               void* stream) {
+  if (full_weights)
+    return paged_decode_impl<false, true>(q, out, kv_cache, num_pages, block_tables, max_blocks, ctx_lens, batch,
+                                          n_q_heads, n_kv_heads, scale, pages_per_split, max_splits, scratch, counters,
+                                          window, sinks, 1.f, stream);
   return paged_decode_impl<false>(q, out, kv_cache, num_pages, block_tables, max_blocks, ctx_lens, batch, n_q_heads,
                                   n_kv_heads, scale, pages_per_split, max_splits, scratch, counters, window, sinks,
                                   1.f, stream);

@@ -359,6 +359,15 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// First key position a query at `pos` may attend: `window` > 0 is a sliding window of that many tokens (the query's own
+// included), < 0 chunked attention (the keys of the query's own chunk of -window positions, counted from position 0 of
+// the sequence), 0 everything before it.
+__host__ __device__ __forceinline__ int attn_first_key(int pos, int window) {
+  if (window > 0) return pos - window + 1 > 0 ? pos - window + 1 : 0;
+  if (window < 0) return pos - pos % -window;
+  return 0;
+}
+
 // ---------------------------------------------------------------------------------------------
 // host side: tensor-map encoding through the driver entry point (no link-time libcuda dependency)
 // ---------------------------------------------------------------------------------------------

@@ -39,8 +39,11 @@ constexpr int kFaPTile = kFaRows * kFaKv * 2;  // 16 KB: 128 rows x 128 bytes
 constexpr int kFaOffK = 2 * kFaQTile;
 constexpr int kFaOffV = kFaOffK + kFaStages * kFaKvTile;
 constexpr int kFaOffP = kFaOffV + kFaStages * kFaKvTile;
-constexpr int kFaOffBar = kFaOffP + 2 * kFaPTile;
-constexpr int kFaSmem = kFaOffBar + 256 + 1024;
+// kFW (full weights): P is written as two bf16 tiles, the rounded value and its remainder, and the second product runs
+// over both, so the softmax weights keep 16 bits of mantissa
+template <bool kFW> constexpr int kFaOffBarOf = kFaOffP + (kFW ? 4 : 2) * kFaPTile;
+template <bool kFW> constexpr int kFaSmemOf = kFaOffBarOf<kFW> + 256 + 1024;
+static_assert(kFaSmemOf<true> <= 227 * 1024, "shared memory of one CTA");
 constexpr int kFaThreads = 320;
 constexpr int kFaTmemCols = 512;               // S_0, S_1: 64 columns each; O_0, O_1: 128 columns each (384 used)
 
@@ -96,12 +99,13 @@ struct FaTile {
   int j0, j1;
 };
 
+template <bool kFW>
 __global__ void __launch_bounds__(kFaThreads, 1)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
                   const FaParams p) {
   extern __shared__ uint8_t fa_smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(fa_smem_raw) + 1023) & ~uintptr_t(1023));
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + kFaOffBar);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + kFaOffBarOf<kFW>);
   uint64_t* q_full = bars;                 // 1
   uint64_t* k_full = bars + 1;             // 3
   uint64_t* k_empty = bars + 4;            // 3
@@ -146,7 +150,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     const int pos_first = ctx - qlen + ti.row0;
     const int pos_last = pos_first + ti.rows - 1;
     const int hi = p.causal ? min(ctx - 1, pos_last) : ctx - 1;
-    const int lo = (p.window > 0) ? max(0, pos_first - p.window + 1) : 0;
+    const int lo = attn_first_key(pos_first, p.window);
     ti.j0 = lo / kFaKv;
     ti.j1 = hi / kFaKv + 1;
   }
@@ -265,6 +269,8 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
           const uint64_t a = umma_desc_sw128(p_addr + t * kFaPTile + k * 32);
           const uint64_t b = umma_desc_sw128_mn(v_addr + stg * kFaKvTile + k * 2048, kFaKvTile / 2);
           umma_f16(tmem_base + 128 + t * kFaD, a, b, idesc_o, (j > tile[t].j0 || k > 0) ? 1u : 0u);
+          if constexpr (kFW)      // the remainders of the same 16 tokens
+            umma_f16(tmem_base + 128 + t * kFaD, umma_desc_sw128(p_addr + (2 + t) * kFaPTile + k * 32), b, idesc_o, 1u);
         }
       };
       // prologue: the first S of every tile whose range starts at J0
@@ -324,7 +330,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       const bool row_ok = row < ti.rows;
       const int pos = ctx - qlen + ti.row0 + (row_ok ? row : 0);
       const int hi = p.causal ? min(ctx - 1, pos) : ctx - 1;
-      const int lo = (p.window > 0) ? max(0, pos - p.window + 1) : 0;
+      const int lo = attn_first_key(pos, p.window);
       uint8_t* p_row = smem + kFaOffP + t * kFaPTile + (row >> 3) * 1024 + (row & 7) * 128;
       float m = -INFINITY, l = 0.f;
       bool ok = true;
@@ -357,6 +363,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         const float corr = ex2_approx(m - m_ref);        // m = -inf: 0
         float sum = 0.f;
         uint32_t pk[32];
+        [[maybe_unused]] uint32_t pr[kFW ? 32 : 1];
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
@@ -365,6 +372,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
             const float e1 = ex2_approx(__uint_as_float(sr[h][i + 1]) - m_ref);
             sum += e0 + e1;
             pk[h * 16 + (i >> 1)] = pack_bf16x2(e0, e1);
+            if constexpr (kFW) pr[h * 16 + (i >> 1)] = pack_bf16x2(e0 - bf16_round(e0), e1 - bf16_round(e1));
           }
         l = l * corr + sum;
         // the O accumulator: rescaled by the warp when any of its rows moved its maximum (never on the first tile:
@@ -388,6 +396,9 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         for (int ch = 0; ch < 8; ++ch) {
           const uint4 v = make_uint4(pk[ch * 4], pk[ch * 4 + 1], pk[ch * 4 + 2], pk[ch * 4 + 3]);
           *reinterpret_cast<uint4*>(p_row + ((ch ^ (row & 7)) << 4)) = v;
+          if constexpr (kFW)
+            *reinterpret_cast<uint4*>(p_row + 2 * kFaPTile + ((ch ^ (row & 7)) << 4)) =
+                make_uint4(pr[ch * 4], pr[ch * 4 + 1], pr[ch * 4 + 2], pr[ch * 4 + 3]);
         }
         fence_proxy_async_smem();
         tc_fence_before();
@@ -431,12 +442,13 @@ using namespace gllm;
 extern "C" int* gllm_error_word();
 
 // Causal (or bidirectional) flash attention over the paged bf16 KV cache for the query tokens of a prefill step.
-// q / out: [total_tokens, n_q_heads, 128] bf16, contiguous. Same semantics as gllm_paged_prefill.
+// q / out: [total_tokens, n_q_heads, 128] bf16, contiguous. Same semantics as gllm_paged_prefill. full_weights: softmax
+// weights as bf16 pairs.
 GLLM_API int gllm_paged_prefill_tc(const void* q, void* out, const void* kv_cache, int num_pages,
                                    const int* block_tables, int max_blocks, const int* q_start, const int* q_len,
                                    const int* ctx_lens, int num_seqs, int max_q_len, int total_tokens, int n_q_heads,
                                    int n_kv_heads, float scale, int causal, int window, const float* sinks,
-                                   void* stream) {
+                                   int full_weights, void* stream) {
   if (n_kv_heads <= 0 || n_q_heads % n_kv_heads != 0 || total_tokens <= 0) {
     set_last_error("paged_prefill_tc: heads %d / kv heads %d / tokens %d", n_q_heads, n_kv_heads, total_tokens);
     return -1;
@@ -461,17 +473,20 @@ GLLM_API int gllm_paged_prefill_tc(const void* q, void* out, const void* kv_cach
   p.num_pages = num_pages; p.window = window; p.causal = causal; p.sinks = sinks;
   p.err = gllm_error_word();
   p.wait_ns = static_cast<unsigned long long>(settings().wait_ns);
-  static bool attr_set[64] = {};
+  auto kern = full_weights ? fa_prefill_kernel<true> : fa_prefill_kernel<false>;
+  const int smem = full_weights ? kFaSmemOf<true> : kFaSmemOf<false>;
+  static bool attr_set[2][64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
-  if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(fa_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kFaSmem);
+  bool& set = attr_set[full_weights ? 1 : 0][dev & 63];
+  if (!set) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) { set_last_error("paged_prefill_tc: %s", cudaGetErrorString(e)); return -1; }
-    attr_set[dev & 63] = true;
+    set = true;
   }
   const int row_blocks = (max_q_len + kFaRows - 1) / kFaRows;
   dim3 grid(p.pair_heads ? row_blocks : (row_blocks + 1) / 2, p.pair_heads ? n_q_heads / 2 : n_q_heads, num_seqs);
-  cudaError_t e = launch_kernel(fa_prefill_kernel, grid, dim3(kFaThreads), kFaSmem, (cudaStream_t)stream, true, 0, tq,
+  cudaError_t e = launch_kernel(kern, grid, dim3(kFaThreads), smem, (cudaStream_t)stream, true, 0, tq,
                                 tkv, p);
   if (e != cudaSuccess) {
     (void)cudaGetLastError();

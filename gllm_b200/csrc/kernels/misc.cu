@@ -236,20 +236,23 @@ __global__ void rope_kv_write_kernel(const __nv_bfloat16* qkv, long long ld, int
 // Generic paged attention (CUDA cores) for head dims other than 128: one warp per (query token, head).
 // Used by small / encoder models; the tensor-core kernels cover head_dim 128.
 // ---------------------------------------------------------------------------------------------
-template <bool KV8>
-__global__ void paged_attention_generic_kernel(const __nv_bfloat16* q, __nv_bfloat16* out,
-                                               const void* kv_cache_v, const int* block_tables,
+template <typename T> __device__ __forceinline__ float exp_for(float x) { return __expf(x); }
+template <> __device__ __forceinline__ float exp_for<float>(float x) { return expf(x); }
+
+// T = float: fp32 queries, cache and output, full-precision exponentials.
+template <typename T, bool KV8>
+__global__ void paged_attention_generic_kernel(const T* q, T* out, const void* kv_cache_v, const int* block_tables,
                                                int max_blocks, const int* q_start, const int* q_len,
                                                const int* ctx_lens, int n_q, int n_kv, int D, float scale,
                                                int causal, int window, int num_pages, float kv_scale) {
-  const __nv_bfloat16* kv_cache = static_cast<const __nv_bfloat16*>(kv_cache_v);
+  const T* kv_cache = static_cast<const T*>(kv_cache_v);
   const uint8_t* kv_cache8 = static_cast<const uint8_t*>(kv_cache_v);
   auto ld_kv = [&](long long eoff) -> float {
     if (KV8) {
       const __half_raw h = __nv_cvt_fp8_to_halfraw(kv_cache8[eoff], __NV_E4M3);
       return __half2float(*reinterpret_cast<const __half*>(&h)) * kv_scale;
     }
-    return __bfloat162float(kv_cache[eoff]);
+    return static_cast<float>(kv_cache[eoff]);
   };
   const int seq = blockIdx.z, head = blockIdx.y;
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -260,12 +263,12 @@ __global__ void paged_attention_generic_kernel(const __nv_bfloat16* q, __nv_bflo
   const int tok = q_start[seq] + row;
   const int kvh = head / (n_q / n_kv);
   const int hi = causal ? (ctx - qlen + row + 1) : ctx;
-  const int lo = window > 0 ? max(0, hi - window) : 0;
+  const int lo = attn_first_key(hi - 1, window);
   const int per = (D + 31) / 32;
   float qv[8], acc[8];
   for (int i = 0; i < per; ++i) {
     const int d = lane + 32 * i;
-    qv[i] = d < D ? __bfloat162float(q[(static_cast<long long>(tok) * n_q + head) * D + d]) * scale : 0.f;
+    qv[i] = d < D ? static_cast<float>(q[(static_cast<long long>(tok) * n_q + head) * D + d]) * scale : 0.f;
     acc[i] = 0.f;
   }
   float mx = -INFINITY, l = 0.f;
@@ -282,7 +285,7 @@ __global__ void paged_attention_generic_kernel(const __nv_bfloat16* q, __nv_bflo
     }
     s = warp_sum(s);
     const float mn = fmaxf(mx, s);
-    const float c = __expf(mx - mn), pnew = __expf(s - mn);
+    const float c = exp_for<T>(mx - mn), pnew = exp_for<T>(s - mn);
     l = l * c + pnew;
     for (int i = 0; i < per; ++i) {
       const int d = lane + 32 * i;
@@ -292,7 +295,7 @@ __global__ void paged_attention_generic_kernel(const __nv_bfloat16* q, __nv_bflo
   }
   for (int i = 0; i < per; ++i) {
     const int d = lane + 32 * i;
-    if (d < D) out[(static_cast<long long>(tok) * n_q + head) * D + d] = __float2bfloat16_rn(l > 0.f ? acc[i] / l : 0.f);
+    if (d < D) out[(static_cast<long long>(tok) * n_q + head) * D + d] = static_cast<T>(l > 0.f ? acc[i] / l : 0.f);
   }
 }
 
@@ -685,10 +688,24 @@ GLLM_API int gllm_paged_attention_generic(const void* q, void* out, const void* 
                                           void* stream) {
   if (D > 256) { set_last_error("paged_attention_generic: head_dim %d > 256", D); return -1; }
   dim3 grid((max_q_len + 3) / 4, n_q, num_seqs);
-  paged_attention_generic_kernel<false><<<grid, 128, 0, (cudaStream_t)stream>>>(
+  paged_attention_generic_kernel<__nv_bfloat16, false><<<grid, 128, 0, (cudaStream_t)stream>>>(
       static_cast<const __nv_bfloat16*>(q), static_cast<__nv_bfloat16*>(out), kv_cache, block_tables, max_blocks,
       q_start, q_len, ctx_lens, n_q, n_kv, D, scale, causal, window, num_pages, 1.0f);
   CHECK_LAUNCH("paged_attention_generic");
+}
+
+// The same with fp32 queries, cache and output.
+GLLM_API int gllm_paged_attention_f32(const float* q, float* out, const float* kv_cache, int num_pages,
+                                      const int* block_tables, int max_blocks, const int* q_start, const int* q_len,
+                                      const int* ctx_lens, int num_seqs, int max_q_len, int n_q, int n_kv, int D,
+                                      float scale, int causal, int window, void* stream) {
+  if (D > 256) { set_last_error("paged_attention_f32: head_dim %d > 256", D); return -1; }
+  if (num_seqs <= 0 || max_q_len <= 0) return 0;
+  dim3 grid((max_q_len + 3) / 4, n_q, num_seqs);
+  paged_attention_generic_kernel<float, false><<<grid, 128, 0, (cudaStream_t)stream>>>(
+      q, out, kv_cache, block_tables, max_blocks, q_start, q_len, ctx_lens, n_q, n_kv, D, scale, causal, window,
+      num_pages, 1.0f);
+  CHECK_LAUNCH("paged_attention_f32");
 }
 
 // fp8 e4m3 KV cache (value = stored * kv_scale); any head_dim <= 256. Halves the cache footprint and the bytes
@@ -701,7 +718,7 @@ GLLM_API int gllm_paged_attention_fp8kv(const void* q, void* out, const void* kv
   if (D > 256) { set_last_error("paged_attention_fp8kv: head_dim %d > 256", D); return -1; }
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
   dim3 grid((max_q_len + 3) / 4, n_q, num_seqs);
-  paged_attention_generic_kernel<true><<<grid, 128, 0, (cudaStream_t)stream>>>(
+  paged_attention_generic_kernel<__nv_bfloat16, true><<<grid, 128, 0, (cudaStream_t)stream>>>(
       static_cast<const __nv_bfloat16*>(q), static_cast<__nv_bfloat16*>(out), kv_cache, block_tables, max_blocks,
       q_start, q_len, ctx_lens, n_q, n_kv, D, scale, causal, window, num_pages, kv_scale);
   CHECK_LAUNCH("paged_attention_fp8kv");

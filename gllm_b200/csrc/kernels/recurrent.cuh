@@ -1,0 +1,83 @@
+// Shared pieces of the recurrent mixers: the view of a step's sequences, the scalar functions of the recurrences, and
+// loads / stores that do not care whether a tensor is bf16 or fp32.
+#pragma once
+#include "common.cuh"
+
+namespace gllm {
+
+struct SeqView {
+  const int* q_start;   // [n] first flat row of the sequence (null: decode step, row = slot = sequence index)
+  const int* q_len;     // [n]
+  const int* ctx_lens;  // [n] tokens after this step
+  const int* slots;     // [n] state slot
+  int n;
+};
+struct SeqRows {
+  int row0, len, start, slot;   // first flat row, rows in this step, position of the first row, state slot
+};
+__device__ __forceinline__ SeqRows seq_rows(const SeqView& v, int i) {
+  SeqRows r;
+  const int ctx = v.ctx_lens[i];
+  if (v.q_start == nullptr) {
+    r.row0 = i; r.len = ctx > 0 ? 1 : 0; r.start = ctx - 1; r.slot = i;
+  } else {
+    r.row0 = v.q_start[i]; r.len = v.q_len[i]; r.start = ctx - r.len; r.slot = v.slots[i];
+  }
+  return r;
+}
+
+template <typename T> __device__ __forceinline__ float to_f(T v);
+template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// Four consecutive elements (the address must be aligned to four elements).
+template <typename T> __device__ __forceinline__ float4 load4(const T* p);
+template <> __device__ __forceinline__ float4 load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename T> __device__ __forceinline__ void store4(T* p, float4 v);
+template <> __device__ __forceinline__ void store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float log_sigmoid_f(float x) { return -softplus_f(-x); }
+__device__ __forceinline__ float silu_exact(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float gelu_tanh_exact(float x) {
+  return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+}
+
+// RG-LRU: gate pre-activations -> decay a and input b = sqrt(1 - a^2) * i * u; 1 - a^2 = -expm1(2 log a) keeps its
+// relative accuracy where a is close to 1.
+constexpr float kRglruC = 8.f;
+__device__ __forceinline__ void rglru_coeffs(float xr, float xi, float softplus_lam, float u, float& a, float& b) {
+  const float la = -kRglruC * sigmoid_f(xr) * softplus_lam;
+  a = expf(la);
+  b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(xi) * u;
+}
+
+// New convolution state of one channel: the last taps - 1 inputs (older ones from the old state, zeros before the
+// sequence's start). In place: entry j only reads entries at or behind j.
+template <typename T>
+__device__ __forceinline__ void advance_conv_state(const SeqRows& s, const T* z, long long ldz, float* conv_state,
+                                                   int width, int taps, int c) {
+  float* cs = conv_state + static_cast<long long>(s.slot) * (taps - 1) * width + c;
+  for (int j = 0; j < taps - 1; ++j) {
+    const int k = s.len - (taps - 1) + j;      // index among this step's rows
+    float v = 0.f;
+    if (k >= 0) v = to_f(z[static_cast<long long>(s.row0 + k) * ldz + c]);
+    else if (s.start > 0) v = cs[static_cast<long long>(taps - 1 + k) * width];
+    cs[static_cast<long long>(j) * width] = v;
+  }
+}
+
+}  // namespace gllm

@@ -158,7 +158,8 @@ PYBIND11_MODULE(_sched, m) {
              std::memcpy(d + 3 * n, p.dec_ctx_lens.data(), n * 4);
            })
       // packs the prefill side into caller-provided (pinned) buffers, no allocation:
-      //   pack = [tokens T | positions T | slot_mapping T | q_start S | q_len S | ctx_lens S | last_rows L | last_slots L]
+      //   pack = [tokens T | positions T | slot_mapping T | q_start S | q_len S | ctx_lens S | last_rows L | last_slots L |
+      //           slots S]
       //   bt   = [S, max_blocks]
       // and returns (T, S, L, max_q_len); L = chunks that reach the end of their prompt (they sample a token)
       .def("pack_prefill_into",
@@ -166,7 +167,7 @@ PYBIND11_MODULE(_sched, m) {
              const size_t T = p.pf_tokens.size(), S = p.prefill.size();
              size_t L = 0;
              for (auto& it : p.prefill) L += it.last ? 1 : 0;
-             if (static_cast<size_t>(pack.size()) < 3 * T + 3 * S + 2 * L ||
+             if (static_cast<size_t>(pack.size()) < 3 * T + 4 * S + 2 * L ||
                  static_cast<size_t>(bt.size()) < p.pf_block_tables.size())
                throw std::invalid_argument("prefill staging buffers too small");
              int32_t* d = pack.mutable_data();
@@ -188,6 +189,7 @@ PYBIND11_MODULE(_sched, m) {
                  ++k;
                }
              }
+             std::memcpy(slots + L, p.pf_slots.data(), S * 4);
              std::memcpy(bt.mutable_data(), p.pf_block_tables.data(), p.pf_block_tables.size() * 4);
              return py::make_tuple(T, S, L, max_q);
            });
@@ -206,6 +208,7 @@ PYBIND11_MODULE(_sched, m) {
       .def("add_request", &ContinuousBatcher::add_request, py::arg("id"), py::arg("prompt"), py::arg("params"),
            py::arg("session") = std::string())
       .def("abort", &ContinuousBatcher::abort)
+      .def("feed", &ContinuousBatcher::feed, py::arg("id"), py::arg("tokens"))
       .def("schedule", &ContinuousBatcher::schedule)
       .def("commit",
            [](ContinuousBatcher& self, const StepPlan& plan,

@@ -196,6 +196,26 @@ int64_t ContinuousBatcher::add_request(int64_t id, const std::vector<int32_t>& p
   return id;
 }
 
+void ContinuousBatcher::feed(int64_t id, const std::vector<int32_t>& tokens) {
+  if (tokens.empty()) throw std::invalid_argument("feed: no tokens");
+  auto it = seqs_.find(id);
+  const size_t have = it == seqs_.end() ? 0 : it->second->tokens.size();
+  if (it != seqs_.end() && !it->second->external) throw std::invalid_argument("feed: the request generates its own tokens");
+  if ((have + tokens.size() + page_size_ - 1) / page_size_ > static_cast<size_t>(max_blocks_))
+    throw std::length_error("SequenceTooLong");
+  if (it == seqs_.end()) {
+    auto s = std::make_unique<Sequence>();
+    s->id = id;
+    s->arrival = arrivals_++;
+    s->external = true;
+    it = seqs_.emplace(id, std::move(s)).first;
+    waiting_.push_back(id);
+  }
+  Sequence& s = *it->second;
+  s.tokens.insert(s.tokens.end(), tokens.begin(), tokens.end());
+  s.prompt_len = static_cast<int>(s.tokens.size());
+}
+
 bool ContinuousBatcher::is_eos(const Sequence& s, int32_t tok) const {
   for (int32_t e : s.sp.eos_ids)
     if (e == tok) return true;
@@ -232,7 +252,7 @@ void ContinuousBatcher::write_slot_table(const Sequence& s) {
 }
 
 void ContinuousBatcher::free_sequence(Sequence& s, bool to_prefix_cache) {
-  if (to_prefix_cache && cfg_.enable_prefix_cache && s.num_computed >= page_size_) {
+  if (to_prefix_cache && !s.external && cfg_.enable_prefix_cache && s.num_computed >= page_size_) {
     const int full = std::min<int>(s.num_computed / page_size_, static_cast<int>(s.block_table.size()));
     prefix_.insert(s.tokens.data(), s.num_computed, s.block_table.data(), full);
   }
@@ -462,11 +482,28 @@ StepPlan ContinuousBatcher::schedule() {
     ++plan.num_decode;
     --budget;
   }
+  // externally fed sequences with exactly one new token take a decode slot beside them
+  for (auto& kv : seqs_) {
+    Sequence& s = *kv.second;
+    if (!s.external || s.state != SeqState::Prefilling || s.num_computed == 0) continue;
+    if (static_cast<int>(s.tokens.size()) != s.num_computed + 1 || budget <= 0) continue;
+    if (!ensure_pages(s, s.num_computed + 1)) continue;
+    write_slot_table(s);
+    const int pos = s.num_computed;
+    plan.dec_tokens[s.slot] = s.tokens.back();
+    plan.dec_positions[s.slot] = pos;
+    plan.dec_slot_mapping[s.slot] = s.block_table[pos / page_size_] * page_size_ + pos % page_size_;
+    plan.dec_ctx_lens[s.slot] = pos + 1;
+    plan.dec_seq_ids[s.slot] = s.id;
+    ++plan.num_decode;
+    --budget;
+  }
   // sequences preempted above may still appear in the decode arrays: scrub them
   for (int sl = 0; sl < max_slots_; ++sl) {
     const int64_t id = plan.dec_seq_ids[sl];
     if (id < 0) continue;
     auto it = seqs_.find(id);
+    if (it != seqs_.end() && it->second->external && it->second->slot == sl) continue;
     if (it == seqs_.end() || it->second->state != SeqState::Running || it->second->slot != sl) {
       plan.dec_seq_ids[sl] = -1;
       plan.dec_ctx_lens[sl] = 0;
@@ -488,6 +525,7 @@ StepPlan ContinuousBatcher::schedule() {
     const int known = static_cast<int>(s.tokens.size());
     const int remaining = known - s.num_computed;
     if (remaining <= 0 || budget <= 0) return false;
+    if (s.external && plan.dec_seq_ids[s.slot] == s.id) return false;   // this token is in the decode part
     int cap = cfg_.prefill_chunk;
     if (cfg_.adaptive_chunk) {
       const double free_ratio = static_cast<double>(alloc_.num_free()) / std::max(1, num_total_pages());
@@ -512,7 +550,7 @@ StepPlan ContinuousBatcher::schedule() {
     item.slot = s.slot;
     item.start = s.num_computed;
     item.len = chunk;
-    item.last = (s.num_computed + chunk == known);
+    item.last = !s.external && (s.num_computed + chunk == known);
     const int q_start = static_cast<int>(plan.pf_tokens.size());
     for (int i = 0; i < chunk; ++i) {
       const int pos = s.num_computed + i;
@@ -590,7 +628,7 @@ StepPlan ContinuousBatcher::schedule() {
       // prefix reuse: bind shared full pages read-only; always leave at least one token to compute
       std::vector<int> shared;
       int matched = 0;
-      if (cfg_.enable_prefix_cache && s.block_table.empty()) {
+      if (cfg_.enable_prefix_cache && !s.external && s.block_table.empty()) {
         matched = prefix_.find_longest_prefix(s.tokens.data(), known - 1, &shared);
       }
       const int first_chunk = std::min(known - matched, std::min(budget, cfg_.prefill_chunk));
@@ -635,6 +673,10 @@ void ContinuousBatcher::commit(const StepPlan& plan, const int32_t* decode_token
     auto it = seqs_.find(id);
     if (it == seqs_.end()) continue;
     Sequence& s = *it->second;
+    if (s.external) {
+      s.num_computed += 1;
+      continue;
+    }
     if (s.state != SeqState::Running) continue;
     s.num_computed += 1;
     const int32_t tok = decode_tokens[sl];

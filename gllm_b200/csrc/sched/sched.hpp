@@ -108,6 +108,7 @@ struct Sequence {
   SamplingParams sp;
   int preemptions = 0;
   std::string session;
+  bool external = false;  // tokens come from the caller (ContinuousBatcher::feed), nothing is sampled or preempted
   int num_generated() const { return static_cast<int>(tokens.size()) - prompt_len; }
 };
 
@@ -195,6 +196,10 @@ class ContinuousBatcher {
   int64_t add_request(int64_t id, const std::vector<int32_t>& prompt, const SamplingParams& sp,
                       const std::string& session);
   bool abort(int64_t id);
+  // Externally fed sequence: `tokens` are appended to what the sequence knows (a new id is created and admitted like any
+  // request). schedule() runs what is not computed yet: one token behind computed ones goes through the decode slots,
+  // anything else as prefill chunks. Nothing is sampled; the sequence keeps its slot and pages until abort().
+  void feed(int64_t id, const std::vector<int32_t>& tokens);
   StepPlan schedule();
   // tokens sampled for the decode slots of the last plan (array of max_slots) and for the prefill
   // items that ended with `last` (in plan order).

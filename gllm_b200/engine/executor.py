@@ -46,6 +46,11 @@ class EngineConfig:
     pages_per_split: int = 32
     seed: int = 0
     order: int = S.ORDER_STRICT_REQUEST_ID
+    # admission limits of the batcher (None = its defaults): pages kept free when a request is admitted, the share of pages
+    # in use above which nobody is admitted, and the share of empty page space that has the same effect
+    watermark_pages: Optional[int] = None
+    emergency_pressure: Optional[float] = None
+    defrag_threshold: Optional[float] = None
     # swap tier: > 0 turns preemption from "recompute later" into "copy the victim's KV pages to pinned host memory and
     # bring them back when pages are free" (victims chosen by the HGAL policy); overflow goes to the NVMe file
     swap_space_pages: int = 0
@@ -121,10 +126,16 @@ class LLMEngine:
             ec.callbacks = chain
         if ec.callbacks is not None or getattr(model, "expert_pager", None) is not None:
             ec.use_cuda_graphs = False      # host decisions inside the forward (callback chain, expert paging): eager steps
+        self.recurrent = bool(getattr(model, "has_recurrent_state", False))
+        if self.recurrent or self.mc.is_hybrid:
+            self._check_hybrid(ec, lockstep_group, pp)
         self.max_blocks = (ec.max_model_len + 15) // 16
         self.num_pages = ec.num_pages or self._auto_pages()
-        self.kv_caches = model.alloc_kv_cache(self.num_pages)
+        self.kv_caches = model.alloc_kv_cache(self.num_pages, state_slots=ec.max_num_seqs)
         pc = S.PolicyConfig()
+        for name in ("watermark_pages", "emergency_pressure", "defrag_threshold"):
+            if getattr(ec, name) is not None:
+                setattr(pc, name, getattr(ec, name))
         pc.max_batch_size = ec.max_num_seqs
         pc.max_batch_tokens = ec.max_batch_tokens
         pc.prefill_chunk = ec.prefill_chunk
@@ -172,7 +183,7 @@ class LLMEngine:
         self.unhealthy: Optional[str] = None
         self.slot_params = np.zeros((self.ms, 4), dtype=np.float32)
         # prefill staging (allocated once: no per-step pinned allocation, concatenation or tensor construction)
-        pf_ints = 3 * ec.max_batch_tokens + 5 * self.ms + 64
+        pf_ints = 3 * ec.max_batch_tokens + 6 * self.ms + 64
         self.h_pf = torch.zeros(pf_ints, dtype=torch.int32, **pin)
         self.d_pf = torch.zeros(pf_ints, dtype=torch.int32, device=dev)
         self.h_pf_bt = torch.zeros((self.ms, self.max_blocks), dtype=torch.int32, **pin)
@@ -244,6 +255,25 @@ class LLMEngine:
         self.eagle = None                           # speculative.heads.EagleHead (attach_eagle): feature-level drafts
         self.eagle_depth = 0
         self._eagle_feat: Dict[int, torch.Tensor] = {}      # request -> hidden state behind its last committed token
+        # externally fed requests (feed_step): wanted positions and the logits gathered for them
+        self._feed_want: Dict[int, set] = {}
+        self._feed_out: Dict[tuple, torch.Tensor] = {}
+        self._fed: Dict[int, int] = {}
+        self._last_logits = None
+        self._graph_logits: Dict[tuple, torch.Tensor] = {}
+
+    def _check_hybrid(self, ec: EngineConfig, lockstep_group, pp):
+        """What a heterogeneous model (recurrent state, layers with different caches) cannot do, refused by name. A
+        prefix of pages cannot stand for a prefix of tokens (the state at its end is gone), so prefix pages are not
+        shared; preempted requests are recomputed."""
+        refused = {"pipeline stages": pp is not None, "lockstep groups": lockstep_group is not None,
+                   "swap_space_pages": ec.swap_space_pages > 0, "speculative_tokens": ec.speculative_tokens > 0,
+                   "mtp_depth": ec.mtp_depth > 0, "pd_role": ec.pd_role != "collocated",
+                   "kv_telemetry_every": ec.kv_telemetry_every > 0}
+        bad = [k for k, v in refused.items() if v]
+        if bad:
+            raise ValueError(f"not available for models with recurrent layers: {', '.join(bad)}")
+        ec.enable_prefix_cache = False
 
     # ------------------------------------------------------------------------------------------
     def generate_with_mtp(self, prompt_ids: List[int], max_tokens: int = 256, temperature: float = 0.0, top_k: int = 0,
@@ -287,16 +317,23 @@ class LLMEngine:
         """Draft with an EAGLE head: it continues the target's last hidden feature and the last token for ``depth``
         steps; the target verifies the chain in one forward, so the output stays the target's greedy output. Verify
         steps run eagerly (the feature behind the last kept token is read back from them).
+        Not for models with recurrent state (rejected drafts would have to be rolled back).
         Reference: EAGLE feature-head drafts (src/speculative/engine.rs:29-420)."""
+        if self.recurrent:
+            raise ValueError("speculative drafts are not available for models with recurrent layers")
         self.eagle, self.eagle_depth = head, int(depth)
 
     def _auto_pages(self) -> int:
         per_page = 16 * self.mc.kv_bytes_per_token(self.model.tp_size) * len(self.model.layer_ids) // max(
             self.mc.num_layers, 1)
+        if hasattr(self.model, "page_bytes"):
+            per_page = self.model.page_bytes()
         if self.device.type != "cuda":
             return max(64, min(4096, (self.cfg.max_num_seqs * self.cfg.max_model_len) // 16 + 8))
         free, total = torch.cuda.mem_get_info(self.device)
         budget = int(free - (1.0 - self.cfg.memory_fraction) * total)
+        if self.recurrent:
+            budget -= self.model.state_bytes(self.cfg.max_num_seqs)
         want = self.cfg.max_num_seqs * self.max_blocks + 64
         return int(max(64, min(want, budget // max(per_page, 1))))
 
@@ -350,6 +387,58 @@ class LLMEngine:
             return False
         self._vetoed[rid] = reason
         return True
+
+    # ---- externally fed requests ---------------------------------------------------------------------
+    def feed_step(self, entries):
+        """Run given tokens through the engine without sampling: ``entries`` = [(request id, tokens, want)], each request's
+        next tokens and the indices among them whose logits are returned. All entries are one batch; a request starts
+        at its first entry, may pause, and keeps its pages and slot until ``feed_end``. Returns one fp32 tensor
+        [len(want), vocab] (host) per entry. Prompt portions run as prefill chunks, single tokens behind computed ones
+        through the captured decode step, exactly as in generation."""
+        if self.pp is not None or self.lockstep is not None or (self.model.tp is not None and self.model.tp_size > 1):
+            raise ValueError("feed_step runs on one GPU (full-vocabulary logits)")
+        goal = {}
+        for rid, toks, want in entries:
+            rid = int(rid)
+            base = self._fed.get(rid, 0)
+            if rid in self.reqs and rid not in self._fed:
+                raise ValueError(f"request {rid} generates its own tokens")
+            if any(not 0 <= int(t) < self.mc.vocab_size for t in toks):
+                raise ValueError("token id outside the vocabulary")
+            if any(not 0 <= w < len(toks) for w in want):
+                raise ValueError("a wanted index lies outside the entry's tokens")
+            self.batcher.feed(rid, [int(t) for t in toks])
+            if rid not in self._fed:
+                self._next_id = max(self._next_id, rid) + 1
+                self.reqs[rid] = _ReqState(t_submit=time.perf_counter())
+                self._req_params[rid] = (0.0, 0, 1.0)
+                self._req_limits[rid] = (1 << 30, -1)
+            self._fed[rid] = goal[rid] = base + len(toks)
+            self._feed_want.setdefault(rid, set()).update(base + int(w) for w in want)
+        computed = lambda: {r: int(self.batcher.state_of(r)["num_computed"]) for r in goal}
+        have = computed()
+        while any(have[r] < g for r, g in goal.items()):
+            self.step()
+            now = computed()
+            if now == have:
+                raise RuntimeError("feed_step: no progress (not enough KV pages or slots for the live requests)")
+            have = now
+        out = []
+        for rid, toks, want in entries:
+            base = self._fed[int(rid)] - len(toks)
+            rows = [self._feed_out.pop((int(rid), base + int(w))).float() for w in want]
+            out.append(torch.stack(rows).cpu() if rows else torch.zeros((0, self.mc.vocab_size)))
+        self._feed_want.clear()
+        self._feed_out.clear()
+        return out
+
+    def feed_end(self, rid: int):
+        """An externally fed request is finished: its pages and its slot are given back."""
+        if self._fed.pop(int(rid), None) is None:
+            raise KeyError(f"request {rid} is not fed")
+        self.abort(int(rid), "end")
+        self._collect()
+        self.results.pop(int(rid), None)
 
     def has_work(self) -> bool:
         return bool(self.reqs)
@@ -410,6 +499,7 @@ class LLMEngine:
             return
         logits = self.model.forward(self._decode_batch(B), self.kv_caches, decode_ws=self.decode_ws,
                                     **({"callbacks": self.cfg.callbacks} if self.cfg.callbacks is not None else {}))
+        self._last_logits = logits
         self._sample(logits, self.d_params[:B], self.d_offsets[:B], self.d_out[:B])
         self.d_offsets[:B] += 1
         tm = getattr(self.model, "op_timer", None)
@@ -418,7 +508,8 @@ class LLMEngine:
 
     def decode_breakdown(self, B: int, replays: int = 3):
         """Per-op device milliseconds of one captured decode step of bucket ``B`` (event nodes inside a fresh graph of
-        the same step; the graph used for serving is left as it was)."""
+        the same step; the graph used for serving is left as it was). The replays advance recurrent states: for a model
+        that has them the running sequences are not usable afterwards."""
         from ..utils.tracing import GraphTimer
         key = self._graph_key(B)
         keep = self.graphs.get(key)
@@ -525,12 +616,18 @@ class LLMEngine:
             if g is not None:
                 self._note_variant_hit(key)
                 g.replay()
+                self._last_logits = self._graph_logits.get(key)
             else:     # lockstep: a capture (with its warm-up run) cannot happen on one rank alone; see precapture()
                 self._decode_body(B)
         else:
             self._decode_body(B)
             if self.cfg.callbacks is not None:
                 self._note_callback_veto(int(i) for i in plan.dec_seq_ids if i >= 0)
+        if self._feed_want:
+            for sl in active:
+                rid, pos = int(ids[sl]), int(plan.dec_positions[sl])
+                if pos in self._feed_want.get(rid, ()):
+                    self._feed_out[(rid, pos)] = self._last_logits[sl, :self.mc.vocab_size].clone()
         if self.d_status is not None:
             self.h_status.copy_(self.d_status, non_blocking=True)      # lands before the blocking copy below returns
         self.h_out.copy_(self.d_out, non_blocking=False)
@@ -757,11 +854,20 @@ class LLMEngine:
             self._graph_stream = torch.cuda.Stream(device=self.device)
             nv_.stream_splitk_workspace(self._graph_stream)
         s = self._graph_stream
+        held = None
+        if self.recurrent:
+            # the warm-up must not advance anybody's recurrent state (writing KV twice is harmless, a state update is
+            # not): it runs on empty slots
+            held = self.d_dec.clone()
+            self.d_dec[2 * self.ms:3 * self.ms] = -1
+            self.d_dec[3 * self.ms:] = 0
         s.wait_stream(torch.cuda.current_stream(self.device))
         with torch.cuda.stream(s):
             self._decode_body(B)
         torch.cuda.current_stream(self.device).wait_stream(s)
         torch.cuda.synchronize(self.device)
+        if held is not None:
+            self.d_dec.copy_(held)
         self.d_offsets[:B] -= 1
         g = torch.cuda.CUDAGraph()
         from ..ops import _native as nv
@@ -770,6 +876,8 @@ class LLMEngine:
             self._decode_body(B)
         self.launches_per_graph[B] = nv.CALLS[0] - n0
         self.graphs[self._graph_key(B)] = g
+        # the logits tensor of the graph stays referenced: its memory is then not reused inside the graph's pool
+        self._graph_logits[self._graph_key(B)] = self._last_logits
         self._register_variant(self._graph_key(B), g)
         return g
 
@@ -792,6 +900,7 @@ class LLMEngine:
         live = {v.key for v in self.variants.variants.values()}
         for k in [k for k in self.graphs if self._variant_key(k) not in live]:
             del self.graphs[k]                                         # evicted by the registry: drop the graph
+            self._graph_logits.pop(k, None)
 
     def _note_variant_hit(self, key):
         v = self.variants.variants.get(self._variant_key(key))
@@ -817,17 +926,28 @@ class LLMEngine:
         dev = self.device
         cuda = dev.type == "cuda"
         T, S_, n_last, max_q = plan.pack_prefill_into(self.h_pf.numpy(), self.h_pf_bt.numpy().reshape(-1))
-        used = 3 * T + 3 * S_ + 2 * n_last
+        used = 3 * T + 4 * S_ + 2 * n_last
         self.d_pf[:used].copy_(self.h_pf[:used], non_blocking=cuda)
         self.d_pf_bt[:S_].copy_(self.h_pf_bt[:S_], non_blocking=cuda)
         self.stats["h2d_bytes"] += used * 4 + S_ * self.max_blocks * 4
         dp = self.d_pf
         o = 3 * T + 3 * S_
         rows = dp[o:o + n_last] if n_last else None
+        fed = []            # (row, request, position) of the logits an externally fed request asks for
+        if self._feed_want:
+            row0 = 0
+            for it in plan.prefill:
+                want = self._feed_want.get(int(it.seq_id), ())
+                fed += [(row0 + i, int(it.seq_id), it.start + i) for i in range(it.len) if it.start + i in want]
+                row0 += it.len
+        if fed:
+            fr = torch.tensor([f[0] for f in fed], dtype=torch.int32, device=dev)
+            rows = fr if rows is None else torch.cat([rows, fr])
         batch = ForwardBatch(token_ids=dp[0:T], positions=dp[T:2 * T], slot_mapping=dp[2 * T:3 * T],
                              block_tables=self.d_pf_bt[:S_], ctx_lens=dp[3 * T + 2 * S_:3 * T + 3 * S_], is_decode=False,
                              q_start=dp[3 * T:3 * T + S_], q_len=dp[3 * T + S_:3 * T + 2 * S_],
-                             max_q_len=int(max_q), logits_rows=rows, want_mtp=self.mtp is not None)
+                             max_q_len=int(max_q), logits_rows=rows, want_mtp=self.mtp is not None,
+                             state_slots=dp[o + 2 * n_last:o + 2 * n_last + S_])
         self.stats["prefill_steps"] += 1
         self.stats["prefill_tokens"] += int(T)
         self.model.op_timer = getattr(self, "prefill_timer", None)   # utils.tracing.GraphTimer(eager=True) or None
@@ -846,6 +966,14 @@ class LLMEngine:
                 self._note_callback_veto(int(it.seq_id) for it in plan.prefill)
         finally:
             self.model.op_timer = None
+        for j, (_, rid, pos) in enumerate(fed):
+            self._feed_out[(rid, pos)] = logits[n_last + j, :self.mc.vocab_size]
+        if fed:
+            logits = logits[:n_last]
+        if n_last == 0:
+            if self.d_status is not None:
+                self.h_status.copy_(self.d_status, non_blocking=False)
+            return np.zeros(0, np.int32)
         last_slots = self.h_pf.numpy()[o + n_last:o + 2 * n_last]
         self._set_sampling_mode(self.slot_params[last_slots])
         self.h_pf_params.numpy()[:n_last] = self.slot_params[last_slots]

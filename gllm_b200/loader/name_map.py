@@ -49,6 +49,8 @@ class TensorRole(str, Enum):
     MOE_SHARED_GATE = "moe_shared_gate"
     MOE_SHARED_UP = "moe_shared_up"
     MOE_SHARED_DOWN = "moe_shared_down"
+    MIXER = "mixer"                # tensor of a token mixer (heterogeneous models: models/hybrid.py)
+    MIXER_NORM = "mixer_norm"
     CLASSIFIER = "classifier"
     POOLER = "pooler"
     UNKNOWN = "unknown"
@@ -107,6 +109,11 @@ _GLOBAL_RULES = [
 ]
 _GLOBAL_RULES = [(re.compile(p), c, r) for p, c, r in _GLOBAL_RULES]
 
+# Heterogeneous models (Zenevik): ``l<i>.mix.<name>``, ``l<i>.mlp.<name>``, ``l<i>.norm1|2``, ``embed``, ``head``, ``final.norm``
+_HYBRID_LAYER = re.compile(r"^l(\d+)\.(mix\.[\w.]+|mlp\.(?:gate|up|down)|norm[12])$")
+_HYBRID_GLOBAL = {"embed": ("embed_tokens", TensorRole.EMBEDDING), "head": ("lm_head", TensorRole.OUTPUT_HEAD),
+                  "final.norm": ("final_norm", TensorRole.FINAL_NORM)}
+
 _LAYER_PREFIX = re.compile(r"^(?:model\.|language_model\.|text_model\.|transformer\.|bert\.|roberta\.|encoder\.)*(?:layers|h|layer|blocks|blk|encoder\.layer)\.(\d+)\.(.+)$")
 # tensors of a multimodal checkpoint's towers and projectors are not the language model's: they have their own loaders
 _NOT_LANGUAGE = re.compile(r"(^|\.)(vision_tower|vision_model|visual|audio_tower|audio_model|multi_modal_projector|"
@@ -128,6 +135,15 @@ def match_tensor_role(name: str) -> Tuple[TensorRole, Optional[int], Optional[st
     The suffix kind is ``.weight`` / ``.bias`` / a quantisation companion (``.qweight``, ``.scales`` ...).
     Canonical names carry ``_bias`` for biases and the raw suffix for quantisation companions.
     """
+    if name in _HYBRID_GLOBAL:
+        canon, role = _HYBRID_GLOBAL[name]
+        return role, None, canon, ""
+    m = _HYBRID_LAYER.match(name)
+    if m:
+        rest = m.group(2)
+        role = TensorRole.MIXER if rest.startswith("mix.") else TensorRole.MIXER_NORM if rest.startswith("norm") else \
+            {"gate": TensorRole.FFN_GATE, "up": TensorRole.FFN_UP, "down": TensorRole.FFN_DOWN}[rest.split(".")[1]]
+        return role, int(m.group(1)), f"L{m.group(1)}.{rest}", ""
     stem, suffix = split_suffix(name)
     if _NOT_LANGUAGE.search(name):
         return TensorRole.UNKNOWN, None, None, suffix

@@ -33,6 +33,54 @@ class RopeScaling:
 
 
 @dataclass
+class MixerSpec:
+    """Token mixer of one layer of a heterogeneous model (``ModelConfig.layer_specs``).
+
+    attention: ``heads`` query and ``kv_heads`` key / value heads of size ``dim``, rotary on the first ``rot_dim``
+               dimensions, ``chunk`` > 0 = chunked mask (keys of the query's own chunk of that many positions),
+               ``row_qk_norm`` = RMS norm over the whole q / k projection, ``v_from_k`` = values are the projected keys.
+    rglru:     real-gated linear recurrent unit over ``width`` channels, gates in ``blocks`` diagonal blocks, behind a
+               causal convolution of ``taps`` taps.
+    gla:       gated linear attention, ``heads`` x (``dim`` key, ``vdim`` value) channels, decay sigmoid(z)^(1 / tau)
+               with z of rank ``decay_rank`` (0: taken from the weight)."""
+    kind: str = "attention"
+    heads: int = 0
+    kv_heads: int = 0
+    dim: int = 0
+    vdim: int = 0
+    scale: float = 0.0
+    rot_dim: int = 0
+    rot_base: float = 10000.0
+    chunk: int = 0
+    row_qk_norm: bool = False
+    v_from_k: bool = False
+    width: int = 0
+    blocks: int = 0
+    taps: int = 0
+    tau: float = 1.0
+    decay_rank: int = 0
+
+    def state_floats(self) -> int:
+        """fp32 words of recurrent state per sequence."""
+        if self.kind == "rglru":
+            return self.width * self.taps
+        if self.kind == "gla":
+            return self.heads * self.dim * self.vdim
+        return 0
+
+    def kv_elems(self) -> int:
+        """KV cache elements per token."""
+        return 2 * self.kv_heads * self.dim if self.kind == "attention" else 0
+
+
+@dataclass
+class LayerSpec:
+    mixer: MixerSpec
+    ff: int = 0             # intermediate size of the gated feed-forward, 0 = none
+    act: str = "gelu_tanh"
+
+
+@dataclass
 class ModelConfig:
     arch: str = "llama"
     kind: str = "chat"  # chat | embedding | reranker | classifier
@@ -72,6 +120,9 @@ class ModelConfig:
     logit_softcap: float = 0.0
     attn_scale: float = 0.0  # 0 -> 1/sqrt(head_dim)
     post_norm: bool = False  # encoder-style post-LN residual blocks
+    # Heterogeneous decoders (models/hybrid.py): one spec per layer; post-norm blocks x = norm(postln_alpha * x + f(x))
+    layer_specs: Optional[List[LayerSpec]] = None
+    postln_alpha: float = 1.0
     causal: bool = True
     # MoE
     num_experts: int = 0
@@ -145,6 +196,14 @@ class ModelConfig:
     def kv_size(self) -> int:
         return self.num_kv_heads * self.head_dim
 
+    @property
+    def is_hybrid(self) -> bool:
+        return self.layer_specs is not None
+
+    @property
+    def has_recurrent_state(self) -> bool:
+        return self.is_hybrid and any(l.mixer.state_floats() for l in self.layer_specs)
+
     def layer_is_moe(self, layer: int) -> bool:
         return self.is_moe and layer >= self.first_k_dense and (layer % max(self.moe_layer_freq, 1) == 0
                                                                  or self.moe_layer_freq <= 1)
@@ -187,6 +246,18 @@ class ModelConfig:
 
     def param_count(self) -> int:
         h, L = self.hidden_size, self.num_layers
+        if self.is_hybrid:
+            total = 2 * self.vocab_size * h
+            for l in self.layer_specs:
+                m = l.mixer
+                if m.kind == "attention":
+                    total += h * (2 * m.heads + m.kv_heads * (1 if m.v_from_k else 2)) * m.dim
+                elif m.kind == "rglru":
+                    total += 3 * h * m.width + 2 * m.width * m.width // m.blocks
+                else:
+                    total += h * m.heads * (2 * m.dim + 3 * m.vdim) + m.decay_rank * (h + m.heads * m.dim)
+                total += 3 * h * l.ff
+            return total
         attn = h * (self.q_size + 2 * self.kv_size) + self.q_size * h
         if self.is_mla:
             qd = self.qk_nope_head_dim + self.qk_rope_head_dim
@@ -207,6 +278,8 @@ class ModelConfig:
 
     def kv_bytes_per_token(self, tp: int = 1) -> int:
         esz = 1 if self.kv_cache_dtype in ("fp8", "fp8_e4m3") else 2
+        if self.is_hybrid:
+            return sum(l.mixer.kv_elems() for l in self.layer_specs) * esz
         if self.is_mla:
             return self.num_layers * (self.kv_lora_rank + self.qk_rope_head_dim) * esz
         return self.num_layers * 2 * max(1, self.num_kv_heads // tp) * self.head_dim * esz
@@ -218,6 +291,8 @@ class ModelConfig:
     @staticmethod
     def from_hf_dict(d: Dict[str, Any]) -> "ModelConfig":
         """HF ``config.json`` -> ModelConfig (keys per the reference's field registry)."""
+        if d.get("architecture") == "Zenevik":
+            return ModelConfig.from_zenevik_dict(d)
         tc = d.get("text_config") or d
         arch = (d.get("model_type") or tc.get("model_type") or "llama").lower()
         g = lambda *keys, default=None: next((tc[k] for k in keys if k in tc and tc[k] is not None), default)
@@ -305,6 +380,48 @@ class ModelConfig:
             cfg.quant = str(qc.get("quant_method", "")).lower()
             cfg.extra["quantization_config"] = qc
         return cfg
+
+    @staticmethod
+    def from_zenevik_dict(d: Dict[str, Any]) -> "ModelConfig":
+        """Zenevik ``config.json``: a list of layers, each with its own mixer (chunked attention, RG-LRU or gated linear
+        attention) and an optional dense feed-forward."""
+        specs = []
+        for i, l in enumerate(d["layers"]):
+            m, kind = l["mixer"], l["type"]
+            if kind == "attention":
+                if m.get("vdim", m["dim"]) != m["dim"]:
+                    raise ValueError(f"layer {i}: values are the projected keys, vdim {m['vdim']} must equal dim {m['dim']}")
+                rot = m.get("rot") or {}
+                spec = MixerSpec("attention", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                                 vdim=int(m["dim"]), scale=float(m["scale"]), rot_dim=int(rot.get("dims", 0)),
+                                 rot_base=float(rot.get("base", 10000.0)), chunk=int((m.get("mask") or {}).get("size", 0)),
+                                 row_qk_norm=True, v_from_k=True)
+            elif kind == "rglru":
+                spec = MixerSpec("rglru", width=int(m["width"]), blocks=int(m["blocks"]), taps=int(m["conv"]))
+            elif kind == "gla":
+                spec = MixerSpec("gla", heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), tau=float(m["tau"]))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            mlp = l.get("mlp")
+            if mlp is not None and mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            specs.append(LayerSpec(spec, ff=int(mlp["ff"]) if mlp else 0))
+        cfg = ModelConfig(arch="zenevik", hidden_size=int(d["width"]), num_layers=len(specs), vocab_size=int(d["vocab"]),
+                          rms_norm_eps=float(d["norm"]["eps"]), postln_alpha=float(d["postln_alpha"]),
+                          logit_softcap=float(d.get("logit_softcap") or 0.0), hidden_act="gelu_tanh",
+                          max_position_embeddings=int(d.get("max_positions", 1 << 20)), layer_specs=specs)
+        cfg.set_hybrid_dims()
+        return cfg
+
+    def set_hybrid_dims(self):
+        """The scalar head / feed-forward sizes of a heterogeneous model: the largest over its layers (they size shared
+        buffers; the layers use their specs). ``head_dim`` is 128 when any layer can use the head_dim-128 kernels."""
+        att = [l.mixer for l in self.layer_specs if l.mixer.kind == "attention"]
+        self.num_heads = max([m.heads for m in att], default=1)
+        self.num_kv_heads = max([m.kv_heads for m in att], default=1)
+        dims = [m.dim for m in att] or [64]
+        self.head_dim = 128 if 128 in dims else max(dims)
+        self.intermediate_size = max([l.ff for l in self.layer_specs] + [0])
 
     @staticmethod
     def from_json_file(path) -> "ModelConfig":

@@ -66,6 +66,8 @@ class Workspace:
 
 
 class DecoderModel:
+    has_recurrent_state = False
+
     def __init__(self, cfg: ModelConfig, src, *, device="cpu", dtype=torch.bfloat16, tp=None, max_positions=None,
                  fused: Optional[bool] = None, layers: Optional[range] = None, weight_quant: Optional[str] = None,
                  quant_group: int = 32, ep=None, kv_dtype=None, kv_scale: float = 1.0, expert_quant: Optional[str] = None,
@@ -287,8 +289,9 @@ class DecoderModel:
             return (num_pages, 16, self.cfg.kv_lora_rank + self.cfg.qk_rope_head_dim)
         return (num_pages, 2, self.n_kv_local, 16, self.cfg.head_dim)
 
-    def alloc_kv_cache(self, num_pages: int) -> List[torch.Tensor]:
-        """One cache per layer of this stage; a shared-KV layer's entry is its donor's tensor (no memory of its own)."""
+    def alloc_kv_cache(self, num_pages: int, state_slots: int = 1) -> List[torch.Tensor]:
+        """One cache per layer of this stage; a shared-KV layer's entry is its donor's tensor (no memory of its own).
+        ``state_slots`` sizes the recurrent state of models that have one; this class has none."""
         def one():
             if self.kv_dtype == torch.float8_e4m3fn:
                 return torch.zeros(self.kv_cache_shape(num_pages), dtype=torch.uint8, device=self.device).view(torch.float8_e4m3fn)

@@ -21,6 +21,7 @@ class ArchFamily(str, enum.Enum):
     DENSE_DECODER = "dense_decoder"
     MOE_DECODER = "moe_decoder"
     MLA_DECODER = "mla_decoder"
+    HYBRID_DECODER = "hybrid_decoder"
     ENCODER = "encoder"
     VISION = "vision"
     AUDIO = "audio"
@@ -29,11 +30,22 @@ class ArchFamily(str, enum.Enum):
 def family_of(cfg) -> ArchFamily:
     if not cfg.causal:
         return ArchFamily.ENCODER
+    if cfg.is_hybrid:
+        return ArchFamily.HYBRID_DECODER
     if cfg.is_mla:
         return ArchFamily.MLA_DECODER
     if cfg.is_moe:
         return ArchFamily.MOE_DECODER
     return ArchFamily.DENSE_DECODER
+
+
+def decoder_class(cfg):
+    """The class that runs a generating model of this configuration."""
+    if cfg.is_hybrid:
+        from .hybrid import HybridDecoder
+        return HybridDecoder
+    from .decoder import DecoderModel
+    return DecoderModel
 
 
 @dataclass

@@ -93,6 +93,9 @@ class RandomWeights:
 
     def shape_of(self, name: str):
         c = self.cfg
+        if c.is_hybrid:
+            from .hybrid import tensor_shapes
+            return tensor_shapes(c)[name]
         base = name.rsplit(".", 1)[-1]
         H, D = c.hidden_size, c.head_dim
         table = {
@@ -147,11 +150,17 @@ class RandomWeights:
     def get(self, name: str) -> torch.Tensor:
         base = name.rsplit(".", 1)[-1]
         shape = self.shape_of(name)
+        if self.cfg.is_hybrid:
+            from .hybrid import is_norm_weight
+            return self._gen(name, shape, ones=is_norm_weight(name))
         return self._gen(name, shape, ones=base.endswith("norm") or base == "altup_out_scale")
 
     def has(self, name: str) -> bool:
         c = self.cfg
         base = name.rsplit(".", 1)[-1]
+        if c.is_hybrid:
+            from .hybrid import tensor_shapes
+            return name in tensor_shapes(c)
         if base == "lm_head":
             return not c.tie_word_embeddings
         if base in ("q_norm", "k_norm"):
@@ -228,7 +237,7 @@ def _fold(w: torch.Tensor, norm_w: torch.Tensor, one_plus: bool) -> torch.Tensor
 def can_fuse(cfg: ModelConfig, tp: int = 1) -> bool:
     """The fused tcgen05 path needs head_dim 128 with full rotary, RMSNorm, SiLU/GELU-tanh GLU, causal."""
     inter = cfg.intermediate_size // tp
-    return (cfg.head_dim == 128 and cfg.norm_type == "rms" and cfg.rotary_dim == 128 and not cfg.is_mla
+    return (not cfg.is_hybrid and cfg.head_dim == 128 and cfg.norm_type == "rms" and cfg.rotary_dim == 128 and not cfg.is_mla
             and cfg.causal and not cfg.post_norm and (cfg.is_moe or inter % 64 == 0)
             and cfg.hidden_act in L.ACT_IDS and cfg.hidden_size % 8 == 0)
 

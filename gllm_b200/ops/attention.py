@@ -30,9 +30,16 @@ def _dequant_cache(kv_cache, kv_scale):
     return kv_cache.float() * kv_scale if kv_cache.dtype == torch.float8_e4m3fn else kv_cache
 
 
+def chunk_window(chunk: int) -> int:
+    """``window`` argument of chunked attention: a query attends the keys of its own chunk of ``chunk`` positions, chunks
+    counted from position 0 of the sequence."""
+    return -int(chunk)
+
+
 def attention_ref(q, kv_cache, block_tables, q_start, q_len, ctx_lens, n_q, n_kv, scale, causal=True, window=0,
                   sinks=None):
-    """q: [T, n_q*D]. Returns [T, n_q*D] in q.dtype. Works on any device (used as the oracle)."""
+    """q: [T, n_q*D]. Returns [T, n_q*D] in q.dtype. Works on any device (used as the oracle). ``window`` > 0: sliding
+    window; < 0: chunks of -window positions (``chunk_window``)."""
     D = kv_cache.shape[-1]
     out = torch.zeros_like(q)
     group = n_q // n_kv
@@ -52,6 +59,8 @@ def attention_ref(q, kv_cache, block_tables, q_start, q_len, ctx_lens, n_q, n_kv
             mask &= pos_k <= pos_q
             if window > 0:
                 mask &= pos_k > pos_q - window
+            elif window < 0:
+                mask &= pos_k // -window == pos_q // -window
         elif window > 0:
             mask &= pos_k >= ctx - window
         scores = scores.masked_fill(~mask[None], float("-inf"))
@@ -76,8 +85,9 @@ class DecodeWorkspace:
 
 
 def paged_decode(q, kv_cache, block_tables, ctx_lens, *, n_q, n_kv, scale=None, out=None, workspace=None,
-                 pages_per_split=32, window=0, sinks=None, kv_scale: float = 1.0):
-    """One query token per sequence. q: [B, n_q*D]; ctx_lens includes the token just written."""
+                 pages_per_split=32, window=0, sinks=None, kv_scale: float = 1.0, full_weights: bool = False):
+    """One query token per sequence. q: [B, n_q*D]; ctx_lens includes the token just written. ``full_weights``: the softmax
+    weights enter the second product as a bf16 pair (value + remainder, 16 bits of mantissa) instead of one bf16."""
     B = q.shape[0]
     D = kv_cache.shape[-1]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -89,7 +99,7 @@ def paged_decode(q, kv_cache, block_tables, ctx_lens, *, n_q, n_kv, scale=None, 
         out.copy_(attention_ref(q, _dequant_cache(kv_cache, kv_scale), block_tables, ar, ones, ctx_lens, n_q, n_kv, scale,
                                 True, window, sinks))
         return out
-    if D == 128 and n_q // n_kv <= 16:
+    if D == 128 and n_q // n_kv <= 16 and q.dtype == torch.bfloat16:
         max_blocks = block_tables.shape[1]
         if workspace is None:
             max_splits = max(1, (max_blocks + pages_per_split - 1) // pages_per_split)
@@ -105,17 +115,18 @@ def paged_decode(q, kv_cache, block_tables, ctx_lens, *, n_q, n_kv, scale=None, 
         rc = nv.lib().gllm_paged_decode(q.data_ptr(), out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
                                         block_tables.data_ptr(), max_blocks, ctx_lens.data_ptr(), B, n_q, n_kv,
                                         scale, pages_per_split, workspace.max_splits, workspace.scratch.data_ptr(),
-                                        workspace.counters.data_ptr(), window, nv.ptr(sinks), nv.stream_ptr())
+                                        workspace.counters.data_ptr(), window, nv.ptr(sinks), 1 if full_weights else 0,
+                                        nv.stream_ptr())
         nv.check(rc, "paged_decode")
         return out
     ar = torch.arange(B, dtype=torch.int32, device=q.device)
     ones = (ctx_lens > 0).to(torch.int32)
     return paged_prefill(q, kv_cache, block_tables, ar, ones, ctx_lens, max_q_len=1, n_q=n_q, n_kv=n_kv, scale=scale,
-                         out=out, window=window, kv_scale=kv_scale)
+                         out=out, window=window, kv_scale=kv_scale, full_weights=full_weights)
 
 
 def paged_prefill(q, kv_cache, block_tables, q_start, q_len, ctx_lens, *, max_q_len, n_q, n_kv, scale=None,
-                  out=None, causal=True, window=0, sinks=None, kv_scale: float = 1.0):
+                  out=None, causal=True, window=0, sinks=None, kv_scale: float = 1.0, full_weights: bool = False):
     """Variable-length (chunked) prefill. q: [T, n_q*D] flat tokens; sequence i owns rows
     [q_start[i], q_start[i]+q_len[i]) which are the last q_len[i] of its ctx_lens[i] cached tokens."""
     D = kv_cache.shape[-1]
@@ -127,6 +138,15 @@ def paged_prefill(q, kv_cache, block_tables, q_start, q_len, ctx_lens, *, max_q_
                                 causal, window, sinks))
         return out
     S = q_len.shape[0]
+    if q.dtype == torch.float32:
+        if sinks is not None or kv_cache.dtype != torch.float32:
+            raise NotImplementedError("fp32 attention: fp32 cache, no sinks")
+        rc = nv.lib().gllm_paged_attention_f32(q.data_ptr(), out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
+                                               block_tables.data_ptr(), block_tables.shape[1], q_start.data_ptr(),
+                                               q_len.data_ptr(), ctx_lens.data_ptr(), S, max_q_len, n_q, n_kv, D, scale,
+                                               1 if causal else 0, window, nv.stream_ptr())
+        nv.check(rc, "paged_attention_f32")
+        return out
     if kv_cache.dtype == torch.float8_e4m3fn and D == 128:
         rc = nv.lib().gllm_paged_prefill_fp8(q.data_ptr(), out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
                                              block_tables.data_ptr(), block_tables.shape[1], q_start.data_ptr(),
@@ -143,12 +163,13 @@ def paged_prefill(q, kv_cache, block_tables, q_start, q_len, ctx_lens, *, max_q_
                                                  1 if causal else 0, window, float(kv_scale), nv.stream_ptr())
         nv.check(rc, "paged_attention_fp8kv")
         return out
-    if D == 128 and nv.get_option("prefill_tc") != 0 and q.is_contiguous() and out.is_contiguous():
+    if D == 128 and (nv.get_option("prefill_tc") != 0 or full_weights) and q.is_contiguous() and out.is_contiguous():
         # tcgen05 flash attention (S and O accumulators in tensor memory)
         rc = nv.lib().gllm_paged_prefill_tc(q.data_ptr(), out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
                                             block_tables.data_ptr(), block_tables.shape[1], q_start.data_ptr(),
                                             q_len.data_ptr(), ctx_lens.data_ptr(), S, max_q_len, q.shape[0], n_q, n_kv,
-                                            scale, 1 if causal else 0, window, nv.ptr(sinks), nv.stream_ptr())
+                                            scale, 1 if causal else 0, window, nv.ptr(sinks), 1 if full_weights else 0,
+                                            nv.stream_ptr())
         nv.check(rc, "paged_prefill_tc")
     elif D == 128:
         rc = nv.lib().gllm_paged_prefill(q.data_ptr(), out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],

@@ -92,6 +92,9 @@ def glu(gu, act=0, *, out=None):
         return y
     if out is None:
         out = torch.empty((M, inter), dtype=gu.dtype, device=gu.device)
+    if gu.dtype == torch.float32:
+        nv.check(nv.lib().gllm_glu_f32(gu.data_ptr(), gu.stride(0), M, inter, act, out.data_ptr(), nv.stream_ptr()), "glu_f32")
+        return out
     rc = nv.lib().gllm_glu(gu.data_ptr(), gu.stride(0), M, inter, act, out.data_ptr(), nv.stream_ptr())
     nv.check(rc, "glu")
     return out

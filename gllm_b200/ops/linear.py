@@ -73,6 +73,13 @@ def row_scale_ref(row_ss, norm_dim, eps):
     return torch.rsqrt(ss / norm_dim + eps)
 
 
+def tensor_core_shape(a, w) -> bool:
+    """Whether bf16 operands fit the tcgen05 GEMM: row pitches and base addresses of 16-byte multiples (TMA), at least 8
+    columns, out-features a multiple of 32 (``pad_rows`` at load time)."""
+    return (a.stride(0) % 8 == 0 and w.stride(0) % 8 == 0 and a.shape[1] % 8 == 0 and w.shape[0] % 32 == 0
+            and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
+
+
 # --------------------------------------------------------------------------------------------
 # plain GEMM (+ RMSNorm-as-row-scale prologue, + bias)
 # --------------------------------------------------------------------------------------------
@@ -110,11 +117,20 @@ def gemm(a, w, *, out=None, out_dtype=torch.bfloat16, bias=None, row_ss=None, no
             out.copy_(res)
             return out
         return res
-    assert a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
+    assert a.dtype == w.dtype and a.dtype in (torch.bfloat16, torch.float32)
     assert a.stride(-1) == 1 and w.stride(-1) == 1
     _on_device(a, weight=w, bias=bias, row_ss=row_ss, out=out)
     if out is None:
         out = torch.empty((M, N), dtype=out_dtype, device=a.device)
+    if a.dtype == torch.float32 or not tensor_core_shape(a, w):
+        # true fp32 arithmetic, or operand rows that TMA cannot address: CUDA-core kernel
+        if row_ss is not None:
+            raise ValueError("gemm: the row-scale prologue needs the tensor-core kernel (bf16, rows of 16-byte multiples)")
+        rc = nv.lib().gllm_gemm_simt(a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M,
+                                     N, K, 1 if a.dtype == torch.float32 else 0, 1 if out.dtype == torch.float32 else 0,
+                                     nv.ptr(bias), float(softcap), nv.stream_ptr())
+        nv.check(rc, "gemm_simt")
+        return out
     bn = bn or _bn_for(N, M)
     nv.ensure_splitk_workspace(a.device)
     parts = 0 if row_ss is None else (row_ss.shape[1] if row_ss.dim() > 1 else 1)

@@ -1,0 +1,245 @@
+"""Recurrent token mixers (short convolution, RG-LRU, gated linear attention) and the ops of a residual stream kept in
+fp32: embedding rows, scaled post-norm, query / key preparation with a norm over the whole projection.
+
+CUDA path: ``csrc/kernels/recurrent.cu`` and ``csrc/kernels/simt.cu`` (bf16 or fp32 tensors, fp32 states). CPU path: an
+fp32 restatement of each op.
+
+The sequences of a step come as a ``SeqView``: sequence i owns rows [q_start, q_start + q_len) of the flat batch, the
+last q_len of its ctx tokens, and the state slot slots[i]; a decode view has one row per slot (row = slot, live where
+ctx > 0). Rows that start at position 0 start from zero state.
+"""
+from __future__ import annotations
+
+from ctypes import c_float, c_int, c_longlong, c_void_p
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import _native as nv
+
+P, I, L, F = c_void_p, c_int, c_longlong, c_float
+nv.register("gllm_embed_rows", I, [P, P, I, I, I, P, P, I, P])
+nv.register("gllm_scaled_add_norm", I, [P, L, P, L, I, P, I, I, F, F, P, P, P, I, P])
+nv.register("gllm_glu_f32", I, [P, L, I, I, I, P, P])
+nv.register("gllm_qk_row_norm_rope", I, [P, L, I, I, I, I, I, I, I, P, P, P, P, I, P, P, F, P, P, I, P])
+nv.register("gllm_short_conv", I, [P, P, P, P, I, I, P, L, I, P, P, P, I, I, P, P])
+nv.register("gllm_rglru_gates", I, [P, I, P, P, P, P, P, I, I, I, P, P, P])
+nv.register("gllm_rglru_scan", I, [P, P, P, P, I, P, P, P, L, P, L, I, P, P, I, I, P, P])
+nv.register("gllm_gla_step", I, [P, P, P, P, I, P, P, P, P, L, I, P, P, I, I, I, I, F, F, P, P, P])
+nv.register("gllm_head_norm_gate", I, [P, P, L, I, P, L, I, I, F, P, P])
+
+RGLRU_C = 8.0        # exponent of the RG-LRU decay: log a = -8 r softplus(lam)
+
+
+@dataclass
+class SeqView:
+    """Sequences of one step for the recurrent ops (see the module docstring)."""
+    ctx_lens: torch.Tensor
+    q_start: Optional[torch.Tensor] = None
+    q_len: Optional[torch.Tensor] = None
+    slots: Optional[torch.Tensor] = None
+    max_q_len: int = 1
+
+    @staticmethod
+    def of(batch) -> "SeqView":
+        if batch.is_decode:
+            return SeqView(batch.ctx_lens)
+        slots = batch.state_slots
+        if slots is None:       # stand-alone callers: sequence i keeps its state in slot i
+            slots = torch.arange(batch.q_len.shape[0], dtype=torch.int32, device=batch.q_len.device)
+        return SeqView(batch.ctx_lens, batch.q_start, batch.q_len, slots, batch.max_q_len)
+
+    @property
+    def n(self) -> int:
+        return int(self.ctx_lens.shape[0])
+
+    def ptrs(self):
+        return nv.ptr(self.q_start), nv.ptr(self.q_len), self.ctx_lens.data_ptr(), nv.ptr(self.slots), self.n
+
+    def rows(self):
+        """(first row, rows, start position, slot) of every sequence with rows in this step (host values)."""
+        for i in range(self.n):
+            ctx = int(self.ctx_lens[i])
+            if self.q_start is None:
+                if ctx > 0:
+                    yield i, 1, ctx - 1, i
+            elif int(self.q_len[i]) > 0:
+                n = int(self.q_len[i])
+                yield int(self.q_start[i]), n, ctx - n, int(self.slots[i])
+
+
+def _f32(t) -> int:
+    return 1 if t.dtype == torch.float32 else 0
+
+
+def embed_rows(ids, table, x, xb=None):
+    """x[m] = table[ids[m]] in fp32; ``xb`` (optional) the same rows in the table's dtype."""
+    M = ids.shape[0]
+    if not table.is_cuda:
+        rows = table[ids.long()]
+        x.copy_(rows.float())
+        if xb is not None:
+            xb.copy_(rows)
+        return x
+    nv.check(nv.lib().gllm_embed_rows(ids.data_ptr(), table.data_ptr(), table.shape[0], table.shape[1], _f32(table),
+                                      x.data_ptr(), nv.ptr(xb), M, nv.stream_ptr()), "embed_rows")
+    return x
+
+
+def scaled_add_norm(x, y, w, alpha, eps, *, rows=None, x_out=None, xb=None):
+    """h = alpha * x + y; h * rsqrt(mean(h^2) + eps) * w in fp32 into ``x_out`` (may be ``x``) and, cast, into ``xb``.
+    ``y`` None: the plain norm. ``rows`` (int32): which rows of x and y are normalised."""
+    M = x.shape[0] if rows is None else rows.shape[0]
+    H = x.shape[1]
+    if not x.is_cuda:
+        h = x.float() if rows is None else x[rows.long()].float()
+        h = alpha * h
+        if y is not None:
+            h = h + (y if rows is None else y[rows.long()]).float()
+        h = h * torch.rsqrt(h.pow(2).mean(-1, keepdim=True) + eps) * w
+        if x_out is not None:
+            x_out[:M].copy_(h)
+        if xb is not None:
+            xb[:M].copy_(h.to(xb.dtype))
+        return
+    nv.check(nv.lib().gllm_scaled_add_norm(
+        x.data_ptr(), x.stride(0), nv.ptr(y), 0 if y is None else y.stride(0), 1 if y is None else _f32(y), w.data_ptr(), M,
+        H, float(alpha), float(eps), nv.ptr(rows), nv.ptr(x_out), nv.ptr(xb), 0 if xb is None else _f32(xb),
+        nv.stream_ptr()), "scaled_add_norm")
+
+
+def qk_row_norm_rope(qk, *, n_q, n_kv, head_dim, rot_dim, v_from_k, positions, slot_mapping, cos_t, sin_t, q_w, k_w, eps,
+                     q_out, kv_cache):
+    """RMS norm over the whole q row and the whole k row -> RoPE on the first ``rot_dim`` dimensions of every head -> q
+    buffer and K pages; the V pages take the k row as projected (``v_from_k``) or the columns behind k."""
+    M = qk.shape[0]
+    nq, nk, D = n_q * head_dim, n_kv * head_dim, head_dim
+    if not qk.is_cuda:
+        q, k = qk[:, :nq].float(), qk[:, nq:nq + nk].float()
+        v = k if v_from_k else qk[:, nq + nk:nq + 2 * nk].float()
+        norm = lambda t, w: t if w is None else t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w
+        half = rot_dim // 2
+
+        def rot(t, heads):
+            t = t.reshape(M, heads, D)
+            if rot_dim == 0:
+                return t
+            c, s = cos_t[positions.long()][:, None], sin_t[positions.long()][:, None]
+            a, b = t[..., :half], t[..., half:rot_dim]
+            return torch.cat([a * c - b * s, b * c + a * s, t[..., rot_dim:]], -1)
+        q_out[:M].copy_(rot(norm(q, q_w), n_q).reshape(M, nq).to(q_out.dtype))
+        k = rot(norm(k, k_w), n_kv)
+        v = v.reshape(M, n_kv, D)
+        if slot_mapping is not None:
+            ok = slot_mapping >= 0
+            sl = slot_mapping[ok].long()
+            kv_cache[sl // 16, 0, :, sl % 16] = k[ok].to(kv_cache.dtype)
+            kv_cache[sl // 16, 1, :, sl % 16] = v[ok].to(kv_cache.dtype)
+        return q_out
+    nv.check(nv.lib().gllm_qk_row_norm_rope(
+        qk.data_ptr(), qk.stride(0), _f32(qk), M, n_q, n_kv, head_dim, rot_dim, 1 if v_from_k else 0, positions.data_ptr(),
+        nv.ptr(slot_mapping), nv.ptr(cos_t), nv.ptr(sin_t), cos_t.shape[0] if cos_t is not None else 1, nv.ptr(q_w),
+        nv.ptr(k_w), float(eps), q_out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0], nv.stream_ptr()),
+        "qk_row_norm_rope")
+    return q_out
+
+
+# --------------------------------------------------------------------------------------------
+# RG-LRU
+# --------------------------------------------------------------------------------------------
+def short_conv(sv: SeqView, z, w, b, state, out):
+    """Causal convolution per channel. z: [T, >= width] rows (a column slice is fine), w [width, taps] fp32, b [width] fp32,
+    state [slots, taps - 1, width] fp32 (read only here)."""
+    width, taps = w.shape
+    if not z.is_cuda:
+        for r0, n, start, slot in sv.rows():
+            hist = state[slot] if start > 0 else torch.zeros_like(state[slot])
+            zz = torch.cat([hist, z[r0:r0 + n, :width].float()])
+            u = sum(zz[j:j + n] * w[:, j] for j in range(taps)) + b
+            out[r0:r0 + n].copy_(u.to(out.dtype))
+        return out
+    nv.check(nv.lib().gllm_short_conv(*sv.ptrs(), sv.max_q_len, z.data_ptr(), z.stride(0), _f32(z), w.data_ptr(),
+                                      b.data_ptr(), state.data_ptr(), width, taps, out.data_ptr(), nv.stream_ptr()),
+             "short_conv")
+    return out
+
+
+def rglru_gates(u, w_r, b_r, w_i, b_i, lam, a_out, b_out):
+    """a = exp(-8 sigmoid(W_r u + b_r) softplus(lam)), b = sqrt(1 - a^2) sigmoid(W_i u + b_i) u, both fp32; the gate
+    matrices are block diagonal: w_r, w_i [blocks, bs, bs]."""
+    T, width = u.shape
+    nblk = w_r.shape[0]
+    if not u.is_cuda:
+        ub = u.float().reshape(T, nblk, -1)
+        r = torch.sigmoid(torch.einsum("tbi,boi->tbo", ub, w_r.float()).reshape(T, width) + b_r)
+        i = torch.sigmoid(torch.einsum("tbi,boi->tbo", ub, w_i.float()).reshape(T, width) + b_i)
+        la = -RGLRU_C * r * torch.nn.functional.softplus(lam)
+        a_out[:T].copy_(la.exp())
+        b_out[:T].copy_(torch.sqrt(-torch.expm1(2 * la)) * i * u.float())
+        return
+    nv.check(nv.lib().gllm_rglru_gates(u.data_ptr(), _f32(u), w_r.data_ptr(), b_r.data_ptr(), w_i.data_ptr(),
+                                       b_i.data_ptr(), lam.data_ptr(), T, width, nblk, a_out.data_ptr(),
+                                       b_out.data_ptr(), nv.stream_ptr()), "rglru_gates")
+
+
+def rglru_scan(sv: SeqView, a, b, y, z, state, conv_state, taps, out):
+    """S = a S + b along every sequence; out = S * gelu_tanh(y). Updates the recurrent state [slots, width] and moves the
+    convolution state forward over ``z``, the convolution's inputs."""
+    width = state.shape[1]
+    if not y.is_cuda:
+        for r0, n, start, slot in sv.rows():
+            S = state[slot].clone() if start > 0 else torch.zeros_like(state[slot])
+            g = torch.nn.functional.gelu(y[r0:r0 + n, :width].float(), approximate="tanh")
+            for i in range(n):
+                S = a[r0 + i] * S + b[r0 + i]
+                out[r0 + i].copy_((S * g[i]).to(out.dtype))
+            state[slot].copy_(S)
+            hist = conv_state[slot] if start > 0 else torch.zeros_like(conv_state[slot])
+            conv_state[slot].copy_(torch.cat([hist, z[r0:r0 + n, :width].float()])[n:])
+        return out
+    nv.check(nv.lib().gllm_rglru_scan(*sv.ptrs(), a.data_ptr(), b.data_ptr(), y.data_ptr(), y.stride(0), z.data_ptr(),
+                                      z.stride(0), _f32(y), state.data_ptr(), conv_state.data_ptr(), width, taps,
+                                      out.data_ptr(), nv.stream_ptr()), "rglru_scan")
+    return out
+
+
+# --------------------------------------------------------------------------------------------
+# gated linear attention
+# --------------------------------------------------------------------------------------------
+def gla_step(sv: SeqView, q, k, v, a1, w2, b2, *, heads, dim, vdim, tau, state, out):
+    """S = diag(alpha) S + k v^T, o = S^T (q dim^-1/2) per head, alpha = sigmoid(W_2 a1 + b_2)^(1/tau) per key channel.
+    q, k, v, a1: column slices of one projection buffer (same row pitch); out [T, heads * vdim] fp32; state
+    [slots, heads, dim, vdim] fp32."""
+    rank = w2.shape[1]
+    if not q.is_cuda:
+        for r0, n, start, slot in sv.rows():
+            S = state[slot].clone() if start > 0 else torch.zeros_like(state[slot])
+            qq = q[r0:r0 + n].float().reshape(n, heads, dim) * dim ** -0.5
+            kk = k[r0:r0 + n].float().reshape(n, heads, dim)
+            vv = v[r0:r0 + n].float().reshape(n, heads, vdim)
+            z = a1[r0:r0 + n].float() @ w2.float().t() + b2
+            al = torch.exp(torch.nn.functional.logsigmoid(z) / tau).reshape(n, heads, dim)
+            for i in range(n):
+                S = al[i][:, :, None] * S + kk[i][:, :, None] * vv[i][:, None, :]
+                out[r0 + i] = torch.einsum("hdv,hd->hv", S, qq[i]).reshape(-1)
+            state[slot].copy_(S)
+        return out
+    assert q.stride(0) == k.stride(0) == v.stride(0) == a1.stride(0)
+    nv.check(nv.lib().gllm_gla_step(*sv.ptrs(), q.data_ptr(), k.data_ptr(), v.data_ptr(), a1.data_ptr(), q.stride(0),
+                                    _f32(q), w2.data_ptr(), b2.data_ptr(), rank, heads, dim, vdim, 1.0 / tau, dim ** -0.5,
+                                    state.data_ptr(), out.data_ptr(), nv.stream_ptr()), "gla_step")
+    return out
+
+
+def head_norm_gate(o, g, w, *, heads, vdim, eps, out):
+    """Per-head RMS norm of o [T, heads * vdim] (fp32) with the shared weight w [vdim], times silu(g)."""
+    T = o.shape[0]
+    if not o.is_cuda:
+        h = o.reshape(T, heads, vdim)
+        h = (h * torch.rsqrt(h.pow(2).mean(-1, keepdim=True) + eps) * w).reshape(T, heads * vdim)
+        out.copy_((h * torch.nn.functional.silu(g.float())).to(out.dtype))
+        return out
+    nv.check(nv.lib().gllm_head_norm_gate(o.data_ptr(), g.data_ptr(), g.stride(0), _f32(g), w.data_ptr(), T, heads, vdim,
+                                          float(eps), out.data_ptr(), nv.stream_ptr()), "head_norm_gate")
+    return out
