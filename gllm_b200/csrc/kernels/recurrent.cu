@@ -33,9 +33,8 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const SeqView sv, const
   float acc = b[c];
   for (int j = 0; j < taps; ++j) {
     const int k = i - (taps - 1) + j;
-    float v = 0.f;
-    if (k >= 0) v = to_f(z[static_cast<long long>(s.row0 + k) * ldz + c]);
-    else if (s.start > 0) v = state[(static_cast<long long>(s.slot) * (taps - 1) + (taps - 1 + k)) * width + c];
+    const float v = k >= 0 ? to_f(z[static_cast<long long>(s.row0 + k) * ldz + c])
+                           : conv_history(state, s.slot, taps, width, s.start + k, c);
     acc = fmaf(w[static_cast<long long>(c) * taps + j], v, acc);
   }
   u[static_cast<long long>(s.row0 + i) * width + c] = from_f<T>(acc);
@@ -97,7 +96,7 @@ __global__ void __launch_bounds__(128) rglru_scan_kernel(const SeqView sv, const
     out[m * width + c] = from_f<T>(S * gelu_tanh_exact(to_f(y[m * ldy + c])));
   }
   state[static_cast<long long>(s.slot) * width + c] = S;
-  advance_conv_state(s, z, ldz, conv_state, width, taps, c);
+  advance_conv_ring(s, z, ldz, conv_state, width, taps, c);
 }
 
 // ---------------------------------------------------------------------------------------------

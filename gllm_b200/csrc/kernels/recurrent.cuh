@@ -65,19 +65,19 @@ __device__ __forceinline__ void rglru_coeffs(float xr, float xi, float softplus_
   b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(xi) * u;
 }
 
-// New convolution state of one channel: the last taps - 1 inputs (older ones from the old state, zeros before the
-// sequence's start). In place: entry j only reads entries at or behind j.
+// Convolution state: a ring of the last `taps` inputs per channel, [slots][taps][width] fp32, the input of position p in
+// entry p % taps. A decode step writes an entry nobody reads in that step, so readers and the writer need no order.
+__device__ __forceinline__ float conv_history(const float* ring, int slot, int taps, int width, int pos, int c) {
+  if (pos < 0) return 0.f;      // before the start of the sequence
+  return ring[(static_cast<long long>(slot) * taps + pos % taps) * width + c];
+}
+// The last inputs of this step's rows enter the ring (one channel; every reader of the old entries is done).
 template <typename T>
-__device__ __forceinline__ void advance_conv_state(const SeqRows& s, const T* z, long long ldz, float* conv_state,
-                                                   int width, int taps, int c) {
-  float* cs = conv_state + static_cast<long long>(s.slot) * (taps - 1) * width + c;
-  for (int j = 0; j < taps - 1; ++j) {
-    const int k = s.len - (taps - 1) + j;      // index among this step's rows
-    float v = 0.f;
-    if (k >= 0) v = to_f(z[static_cast<long long>(s.row0 + k) * ldz + c]);
-    else if (s.start > 0) v = cs[static_cast<long long>(taps - 1 + k) * width];
-    cs[static_cast<long long>(j) * width] = v;
-  }
+__device__ __forceinline__ void advance_conv_ring(const SeqRows& s, const T* z, long long ldz, float* ring, int width,
+                                                  int taps, int c) {
+  for (int i = s.len > taps ? s.len - taps : 0; i < s.len; ++i)
+    ring[(static_cast<long long>(s.slot) * taps + (s.start + i) % taps) * width + c] =
+        to_f(z[static_cast<long long>(s.row0 + i) * ldz + c]);
 }
 
 }  // namespace gllm

@@ -196,7 +196,7 @@ __global__ void __launch_bounds__(256) qk_row_norm_rope_kernel(const T* qkv, lon
   }
   const float rq = q_w ? 1.f / sqrtf(block_reduce_sum(sq, red) / nq + eps) : 1.f;
   const float rk = k_w ? 1.f / sqrtf(block_reduce_sum(sk, red) / nk + eps) : 1.f;
-  int pos = positions[m];
+  int pos = rot_dim > 0 ? positions[m] : 0;
   if (pos < 0 || pos >= max_pos) {
     if (err && threadIdx.x == 0) atomicCAS(err, 0, ERR_BAD_ARG);
     pos = 0;

@@ -14,8 +14,10 @@ chunks run as ordinary launches between decode replays.
 """
 from __future__ import annotations
 
+import gc
 import os
 import time
+import weakref
 from dataclasses import dataclass, field
 from typing import Callable, Dict, List, Optional
 
@@ -99,6 +101,28 @@ class _ReqState:
     hook: Optional[Callable] = None
     stream: Optional[Callable] = None
     n_out: int = 0
+
+
+_capture_streams: Dict[int, list] = {}      # device -> capture streams of engines that are gone
+
+
+def _take_capture_stream(engine):
+    """A capture stream with a split-K workspace of its own. The kernel library keeps a fixed number of workspaces, so a
+    stream goes back to the pool when its engine is collected."""
+    from ..ops import _native as nv
+    free = _capture_streams.setdefault(engine.device.index or 0, [])
+    if not free:
+        try:
+            s = torch.cuda.Stream(device=engine.device)
+            nv.stream_splitk_workspace(s)
+            free.append(s)
+        except RuntimeError:
+            gc.collect()                # engines held by reference cycles only
+            if not free:
+                raise
+    s = free.pop()
+    weakref.finalize(engine, free.append, s)
+    return s
 
 
 class LLMEngine:
@@ -850,9 +874,7 @@ class LLMEngine:
         # the graphs then share nothing with eager launches on other streams (prefill chunks), so the two may overlap.
         # Warm up outside capture so lazy initialisation (attribute setting, descriptor cache) is done.
         if getattr(self, "_graph_stream", None) is None:
-            from ..ops import _native as nv_
-            self._graph_stream = torch.cuda.Stream(device=self.device)
-            nv_.stream_splitk_workspace(self._graph_stream)
+            self._graph_stream = _take_capture_stream(self)
         s = self._graph_stream
         held = None
         if self.recurrent:

@@ -63,7 +63,7 @@ class MixerSpec:
     def state_floats(self) -> int:
         """fp32 words of recurrent state per sequence."""
         if self.kind == "rglru":
-            return self.width * self.taps
+            return self.width * (self.taps + 1)
         if self.kind == "gla":
             return self.heads * self.dim * self.vdim
         return 0

@@ -68,7 +68,7 @@ class HybridWorkspace:
     """Static activation buffers (CUDA graphs replay over them). ``take`` hands out a contiguous [T, n] view of a named
     buffer; ``f32`` buffers are fp32 whatever the compute dtype."""
 
-    F32 = ("f32",)
+    F32 = ("f32", "f32b", "y")
 
     def __init__(self, model: "HybridDecoder", tokens: int):
         dev, dt, H = model.device, model.dtype, model.cfg.hidden_size
@@ -86,7 +86,7 @@ class HybridWorkspace:
                     sizes["gu"] = l.w_gate_up.shape[0]
             for k, v in sizes.items():
                 need[k] = max(need.get(k, 0), v)
-        self.buf = {k: torch.zeros(tokens * n, dtype=torch.float32 if k in self.F32 or k == "y" else dt, device=dev)
+        self.buf = {k: torch.zeros(tokens * n, dtype=torch.float32 if k in self.F32 else dt, device=dev)
                     for k, n in need.items()}
         self.decode_ws = None
 

@@ -109,14 +109,15 @@ class RgLruMixer(_Mixer):
             self.w[g + "_b"] = self.vec(g + ".b").reshape(-1).contiguous()
         self.w["lam"] = self.vec("lam")
         self.w["wo"] = self.mat("o")
+        self.fused = R.rglru_fusable(m.width, m.blocks, m.taps, self.dtype, self.device)
 
     def workspace(self):
         m = self.spec
-        return {"proj": self.w["wyx"].shape[0], "mix": m.width, "q": m.width, "f32": 2 * m.width}
+        return {"proj": self.w["wyx"].shape[0], "mix": m.width, **({} if self.fused else {"q": m.width, "f32": 2 * m.width})}
 
     def state_shapes(self):
         m = self.spec
-        return {"rec": (m.width,), "conv": (m.taps - 1, m.width)}
+        return {"rec": (m.width,), "conv": (m.taps, m.width)}
 
     def forward(self, model, ws, batch, st, T):
         m, w = self.spec, self.w
@@ -125,10 +126,14 @@ class RgLruMixer(_Mixer):
         model.mark("rglru_in")
         sv = SeqView.of(batch)
         out = ws.take("mix", T, m.width)
-        u = R.short_conv(sv, z, w["conv"], w["conv_b"], st["conv"], ws.take("q", T, m.width))
-        ab = ws.take("f32", 2 * T, m.width)
-        R.rglru_gates(u, w["ra"], w["ra_b"], w["ri"], w["ri_b"], w["lam"], ab[:T], ab[T:])
-        R.rglru_scan(sv, ab[:T], ab[T:], y, z, st["rec"], st["conv"], m.taps, out)
+        if self.fused:
+            R.rglru_tile(sv, y, z, w["conv"], w["conv_b"], w["ra"], w["ra_b"], w["ri"], w["ri_b"], w["lam"], st["rec"],
+                         st["conv"], out)
+        else:
+            u = R.short_conv(sv, z, w["conv"], w["conv_b"], st["conv"], ws.take("q", T, m.width))
+            ab = ws.take("f32", 2 * T, m.width)
+            R.rglru_gates(u, w["ra"], w["ra_b"], w["ri"], w["ri_b"], w["lam"], ab[:T], ab[T:])
+            R.rglru_scan(sv, ab[:T], ab[T:], y, z, st["rec"], st["conv"], m.taps, out)
         model.mark("rglru")
         return L.gemm(out, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
 
@@ -144,9 +149,11 @@ class GlaMixer(_Mixer):
         self.w["a2_b"] = self.vec("a2.b")
         self.w["norm"] = self.vec("norm")
         self.w["wo"] = self.mat("o")
+        self.fused_decode, self.chunked = R.gla_fusable(m.dim, m.vdim, self.rank, self.w["wqkv"].shape[0], self.dtype,
+                                                        self.device)
 
     def workspace(self):
-        return {"proj": self.w["wqkv"].shape[0], "mix": self.nv, "f32": self.nv}
+        return {"proj": self.w["wqkv"].shape[0], "mix": self.nv, "f32": self.nv, **({"f32b": self.nk} if self.chunked else {})}
 
     def state_shapes(self):
         m = self.spec
@@ -163,10 +170,19 @@ class GlaMixer(_Mixer):
         q, k, v, g, a1 = parts
         model.mark("gla_in")
         sv = SeqView.of(batch)
-        acc = ws.take("f32", T, self.nv)
-        R.gla_step(sv, q, k, v, a1, w["a2"], w["a2_b"], heads=m.heads, dim=m.dim, vdim=m.vdim, tau=m.tau, state=st["rec"],
-                   out=acc)
-        out = R.head_norm_gate(acc, g, w["norm"], heads=m.heads, vdim=m.vdim, eps=self.eps, out=ws.take("mix", T, self.nv))
+        out = ws.take("mix", T, self.nv)
+        size = dict(heads=m.heads, dim=m.dim, vdim=m.vdim)
+        if batch.is_decode and self.fused_decode:
+            R.gla_decode(sv, q, k, v, g, a1, w["a2"], w["a2_b"], w["norm"], **size, tau=m.tau, eps=self.eps,
+                         state=st["rec"], out=out)
+        else:
+            acc = ws.take("f32", T, self.nv)
+            if not batch.is_decode and self.chunked:
+                R.gla_prefill(sv, q, k, v, a1, w["a2"], w["a2_b"], **size, tau=m.tau, decay=ws.take("f32b", T, self.nk),
+                              state=st["rec"], out=acc)
+            else:
+                R.gla_step(sv, q, k, v, a1, w["a2"], w["a2_b"], **size, tau=m.tau, state=st["rec"], out=acc)
+            R.head_norm_gate(acc, g, w["norm"], heads=m.heads, vdim=m.vdim, eps=self.eps, out=out)
         model.mark("gla")
         return L.gemm(out, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
 

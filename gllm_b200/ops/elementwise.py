@@ -139,6 +139,8 @@ def pool(h, seq_start, seq_len, mode="mean"):
             seg = h[st:st + n].float()
             out[s] = seg.mean(0) if m == 0 else (seg[0] if m == 1 else seg[-1])
         return out
+    if h.dtype != torch.bfloat16:
+        raise ValueError(f"pool: the kernel takes bf16 rows, got {h.dtype}")
     rc = nv.lib().gllm_pool(h.data_ptr(), seq_start.data_ptr(), seq_len.data_ptr(), S, h.shape[1], m, out.data_ptr(),
                             nv.stream_ptr())
     nv.check(rc, "pool")

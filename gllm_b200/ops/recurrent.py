@@ -26,7 +26,12 @@ nv.register("gllm_qk_row_norm_rope", I, [P, L, I, I, I, I, I, I, I, P, P, P, P, 
 nv.register("gllm_short_conv", I, [P, P, P, P, I, I, P, L, I, P, P, P, I, I, P, P])
 nv.register("gllm_rglru_gates", I, [P, I, P, P, P, P, P, I, I, I, P, P, P])
 nv.register("gllm_rglru_scan", I, [P, P, P, P, I, P, P, P, L, P, L, I, P, P, I, I, P, P])
+nv.register("gllm_rglru_tile_ok", I, [I, I, I])
+nv.register("gllm_rglru_tile", I, [P, P, P, P, I, P, P, L, P, P, P, P, P, P, P, I, I, I, P, P, P, I, P, P])
 nv.register("gllm_gla_step", I, [P, P, P, P, I, P, P, P, P, L, I, P, P, I, I, I, I, F, F, P, P, P])
+nv.register("gllm_gla_tile_ok", I, [I, I, I, L])
+nv.register("gllm_gla_decode", I, [P, I, P, P, P, P, P, L, P, P, P, I, I, I, I, F, F, F, P, P, P])
+nv.register("gllm_gla_prefill", I, [P, P, P, P, I, I, P, P, P, P, L, P, P, I, I, I, I, F, F, P, P, P, P])
 nv.register("gllm_head_norm_gate", I, [P, P, L, I, P, L, I, I, F, P, P])
 
 RGLRU_C = 8.0        # exponent of the RG-LRU decay: log a = -8 r softplus(lam)
@@ -96,7 +101,7 @@ def scaled_add_norm(x, y, w, alpha, eps, *, rows=None, x_out=None, xb=None):
         h = x.float() if rows is None else x[rows.long()].float()
         h = alpha * h
         if y is not None:
-            h = h + (y if rows is None else y[rows.long()]).float()
+            h = h + (y if rows is None else y[rows.long()])[:, :H].float()
         h = h * torch.rsqrt(h.pow(2).mean(-1, keepdim=True) + eps) * w
         if x_out is not None:
             x_out[:M].copy_(h)
@@ -148,14 +153,19 @@ def qk_row_norm_rope(qk, *, n_q, n_kv, head_dim, rot_dim, v_from_k, positions, s
 # --------------------------------------------------------------------------------------------
 # RG-LRU
 # --------------------------------------------------------------------------------------------
+def _conv_history(ring, start: int, taps: int):
+    """The taps - 1 inputs before position ``start`` from a slot's ring, zeros before the sequence's start."""
+    rows = [ring[p % taps] if p >= 0 else torch.zeros_like(ring[0]) for p in range(start - taps + 1, start)]
+    return torch.stack(rows) if rows else ring[:0]
+
+
 def short_conv(sv: SeqView, z, w, b, state, out):
     """Causal convolution per channel. z: [T, >= width] rows (a column slice is fine), w [width, taps] fp32, b [width] fp32,
-    state [slots, taps - 1, width] fp32 (read only here)."""
+    state [slots, taps, width] fp32: a ring, the input of position p in entry p % taps (read only here)."""
     width, taps = w.shape
     if not z.is_cuda:
         for r0, n, start, slot in sv.rows():
-            hist = state[slot] if start > 0 else torch.zeros_like(state[slot])
-            zz = torch.cat([hist, z[r0:r0 + n, :width].float()])
+            zz = torch.cat([_conv_history(state[slot], start, taps), z[r0:r0 + n, :width].float()])
             u = sum(zz[j:j + n] * w[:, j] for j in range(taps)) + b
             out[r0:r0 + n].copy_(u.to(out.dtype))
         return out
@@ -185,7 +195,7 @@ def rglru_gates(u, w_r, b_r, w_i, b_i, lam, a_out, b_out):
 
 def rglru_scan(sv: SeqView, a, b, y, z, state, conv_state, taps, out):
     """S = a S + b along every sequence; out = S * gelu_tanh(y). Updates the recurrent state [slots, width] and moves the
-    convolution state forward over ``z``, the convolution's inputs."""
+    convolution ring forward over ``z``, the convolution's inputs."""
     width = state.shape[1]
     if not y.is_cuda:
         for r0, n, start, slot in sv.rows():
@@ -195,12 +205,43 @@ def rglru_scan(sv: SeqView, a, b, y, z, state, conv_state, taps, out):
                 S = a[r0 + i] * S + b[r0 + i]
                 out[r0 + i].copy_((S * g[i]).to(out.dtype))
             state[slot].copy_(S)
-            hist = conv_state[slot] if start > 0 else torch.zeros_like(conv_state[slot])
-            conv_state[slot].copy_(torch.cat([hist, z[r0:r0 + n, :width].float()])[n:])
+            for i in range(max(0, n - taps), n):
+                conv_state[slot, (start + i) % taps].copy_(z[r0 + i, :width])
         return out
     nv.check(nv.lib().gllm_rglru_scan(*sv.ptrs(), a.data_ptr(), b.data_ptr(), y.data_ptr(), y.stride(0), z.data_ptr(),
                                       z.stride(0), _f32(y), state.data_ptr(), conv_state.data_ptr(), width, taps,
                                       out.data_ptr(), nv.stream_ptr()), "rglru_scan")
+    return out
+
+
+def rglru_fusable(width: int, blocks: int, taps: int, dtype, device) -> bool:
+    """Whether ``rglru_tile`` takes a layer of these sizes (bf16 on the GPU)."""
+    return device.type == "cuda" and dtype == torch.bfloat16 and bool(nv.lib().gllm_rglru_tile_ok(width, blocks, taps))
+
+
+def rglru_segments(width: int, blocks: int, n_seqs: int, max_q_len: int) -> int:
+    """Into how many time segments a prefill step is cut: as many as it takes to give every SM two tiles' worth of CTAs,
+    but not under four 64-token tiles per segment (a segmented step runs its gates twice)."""
+    ctas = blocks * -(-(width // blocks) // 32) * n_seqs
+    want = 296 // max(ctas, 1)
+    return max(1, min(want, max_q_len // 256, 16)) if want >= 4 else 1
+
+
+def rglru_tile(sv: SeqView, y, z, conv_w, conv_b, w_r, b_r, w_i, b_i, lam, state, ring, out, scratch=None, segments=None):
+    """Convolution, gates, recurrence and output gate of an RG-LRU layer in one pass (``csrc/kernels/rglru_tile.cu``):
+    the same result as ``short_conv`` + ``rglru_gates`` + ``rglru_scan``. y and z are column slices of one projection."""
+    width, taps = conv_w.shape
+    blocks = w_r.shape[0]
+    assert y.is_cuda and y.stride(0) == z.stride(0)
+    n_seg = 1
+    if sv.q_start is not None:
+        n_seg = segments or rglru_segments(width, blocks, sv.n, sv.max_q_len)
+        if n_seg > 1 and (scratch is None or scratch.numel() < 3 * sv.n * n_seg * width):
+            scratch = torch.empty(3 * sv.n * n_seg * width, dtype=torch.float32, device=y.device)
+    nv.check(nv.lib().gllm_rglru_tile(*sv.ptrs(), y.data_ptr(), z.data_ptr(), y.stride(0), conv_w.data_ptr(),
+                                      conv_b.data_ptr(), w_r.data_ptr(), b_r.data_ptr(), w_i.data_ptr(), b_i.data_ptr(),
+                                      lam.data_ptr(), width, blocks, taps, state.data_ptr(), ring.data_ptr(),
+                                      out.data_ptr(), n_seg, nv.ptr(scratch), nv.stream_ptr()), "rglru_tile")
     return out
 
 
@@ -229,6 +270,32 @@ def gla_step(sv: SeqView, q, k, v, a1, w2, b2, *, heads, dim, vdim, tau, state, 
     nv.check(nv.lib().gllm_gla_step(*sv.ptrs(), q.data_ptr(), k.data_ptr(), v.data_ptr(), a1.data_ptr(), q.stride(0),
                                     _f32(q), w2.data_ptr(), b2.data_ptr(), rank, heads, dim, vdim, 1.0 / tau, dim ** -0.5,
                                     state.data_ptr(), out.data_ptr(), nv.stream_ptr()), "gla_step")
+    return out
+
+
+def gla_fusable(dim: int, vdim: int, rank: int, pitch: int, dtype, device) -> tuple:
+    """(one-kernel decode step, chunked prefill): which bf16 kernels of ``csrc/kernels/gla_tile.cu`` take these sizes."""
+    if device.type != "cuda" or dtype != torch.bfloat16:
+        return False, False
+    ok = int(nv.lib().gllm_gla_tile_ok(dim, vdim, rank, pitch))
+    return bool(ok & 1), bool(ok & 2)
+
+
+def gla_decode(sv: SeqView, q, k, v, g, a1, w2, b2, norm_w, *, heads, dim, vdim, tau, eps, state, out):
+    """One token per slot: ``gla_step`` + ``head_norm_gate`` in one kernel. out [slots, heads * vdim] bf16."""
+    nv.check(nv.lib().gllm_gla_decode(sv.ctx_lens.data_ptr(), sv.n, q.data_ptr(), k.data_ptr(), v.data_ptr(), g.data_ptr(),
+                                      a1.data_ptr(), q.stride(0), w2.data_ptr(), b2.data_ptr(), norm_w.data_ptr(),
+                                      w2.shape[1], heads, dim, vdim, 1.0 / tau, dim ** -0.5, float(eps), state.data_ptr(),
+                                      out.data_ptr(), nv.stream_ptr()), "gla_decode")
+    return out
+
+
+def gla_prefill(sv: SeqView, q, k, v, a1, w2, b2, *, heads, dim, vdim, tau, decay, state, out):
+    """``gla_step`` over prompt portions in chunks of 64 tokens on tensor cores. ``decay`` [T, heads * dim] fp32 scratch."""
+    nv.check(nv.lib().gllm_gla_prefill(*sv.ptrs(), q.shape[0], q.data_ptr(), k.data_ptr(), v.data_ptr(), a1.data_ptr(),
+                                       q.stride(0), w2.data_ptr(), b2.data_ptr(), w2.shape[1], heads, dim, vdim, 1.0 / tau,
+                                       dim ** -0.5, decay.data_ptr(), state.data_ptr(), out.data_ptr(), nv.stream_ptr()),
+             "gla_prefill")
     return out
 
 
