@@ -51,6 +51,9 @@ def parse_args():
                     help="fp8: e4m3 KV cache (half the KV bytes); not the headline configuration, reported as invalid for it")
     ap.add_argument("--op-breakdown", action="store_true",
                     help="after the timed regions, time every op of one captured decode step with in-graph events")
+    ap.add_argument("--hybrid", nargs="?", const="2048,4096", default=None, metavar="WIDTHS",
+                    help="instead of the headline workload: prefill and decode throughput of the heterogeneous decoder "
+                         "(Zenevik) beside a dense decoder of equal size, per-op times against the roofline (one GPU)")
     ap.add_argument("--layers", type=int, default=0, help="debug only: a value other than 0 marks the result invalid")
     ap.add_argument("--no-baseline", action="store_true",
                     help="skip the NCCL baseline arm (unfused GEMM + ncclAllReduce) that vs_baseline is measured against")
@@ -129,6 +132,15 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}))
+        return 0
+
+    if args.hybrid:
+        from gllm_b200.utils import hybrid_bench
+        clocks = ClockSampler(0)
+        clocks.start()
+        res = hybrid_bench.main(args.hybrid.split(","), max(args.steps, 3), max(args.warmup, 3))
+        print(json.dumps({"metric": "hybrid_decoder_tokens_per_s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+                          "dtype": "bf16", "data": "synthetic", "clocks": clocks.stop(), "results": res}))
         return 0
 
     import numpy as np

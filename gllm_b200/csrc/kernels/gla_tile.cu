@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(256) gla_decode_kernel(const GlaDecodeParams p
     const bf16_t* wr = p.w2 + static_cast<long long>(head * p.dim + d) * p.rank;
     float z = p.b2[head * p.dim + d];
     for (int j = 0; j < p.rank; ++j) z = fmaf(__bfloat162float(wr[j]), a1s[j], z);
-    al[d] = expf(log_sigmoid_f(z) * p.inv_tau);
+    al[d] = decay_exp(log_sigmoid_f(z) * p.inv_tau);
   }
   __syncthreads();
   const int c = (tid % vq) * 4, rg = tid / vq;
@@ -165,28 +165,62 @@ struct GlaChunkParams {
   const float* decay;      // [rows, heads * dim] log2 decays
   int heads, dim, vdim;
   float qscale;
+  int vec_k, vec_v;        // 16-byte loads of the q / k and of the value tiles
   float* state;
   float* out;              // [rows, heads * vdim] fp32
 };
 
 constexpr int kGtKP = kGtSlice + 8;       // bf16 per row of the key tile
-constexpr int kGtBP = kGtSlice + 4;       // floats per row of the running sums
-constexpr int kGtVP = kGtV + 8;           // bf16 per row of the value and state tiles
-constexpr int kGtAP = kGtC + 4;           // floats per row of the score tile (aliases the running sums)
+constexpr int kGtBP = kGtSlice + 8;       // floats per row of the running sums
+constexpr int kGtVP = kGtV + 8;           // bf16 per row of the value tile
+constexpr int kGtAP = kGtC + 8;           // floats per row of the score tile (aliases the running sums)
 template <int NSL> constexpr int kGtSmem =
-    kGtC * kGtBP * 4 + kGtC * kGtKP * 2 + kGtC * kGtVP * 2 + NSL * 2 * kGtSlice * kGtVP * 2 + 256;
+    kGtC * kGtBP * 4 + 2 * kGtC * kGtKP * 2 + kGtC * kGtVP * 2 + NSL * 2 * kGtSlice * kGtV * 2 + 64;
+// Element offset in a state tile [rows][64] bf16: 16-byte chunks XOR-swizzled by the row.
+__device__ __forceinline__ int gt_state_off(int row, int col) {
+  return row * kGtV + ((((col >> 3) ^ row) & 7) << 3) + (col & 7);
+}
+// Rows [0, 64) x `cols` (a multiple of 8 for the 16-byte form) of a bf16 matrix into shared memory, zeros behind row n and
+// behind column `valid`. All loads of a thread are in flight together.
+template <int kCols, int kPitch>
+__device__ __forceinline__ void gt_load_tile(const bf16_t* src, long long ld, int n, int valid, bool vec, bf16_t* dst) {
+  if (vec) {
+    constexpr int kPer = kGtC * (kCols / 8) / kGtThreads;
+    uint4 v[kPer];
+#pragma unroll
+    for (int u = 0; u < kPer; ++u) {
+      const int i = threadIdx.x + u * kGtThreads, r = i / (kCols / 8), c = (i % (kCols / 8)) * 8;
+      v[u] = make_uint4(0, 0, 0, 0);
+      if (r < n && c < valid) v[u] = *reinterpret_cast<const uint4*>(src + r * ld + c);
+    }
+#pragma unroll
+    for (int u = 0; u < kPer; ++u) {
+      const int i = threadIdx.x + u * kGtThreads, r = i / (kCols / 8), c = (i % (kCols / 8)) * 8;
+      *reinterpret_cast<uint4*>(dst + r * kPitch + c) = v[u];
+    }
+  } else {
+#pragma unroll 8
+    for (int i = threadIdx.x; i < kGtC * (kCols / 2); i += kGtThreads) {
+      const int r = i / (kCols / 2), c = (i % (kCols / 2)) * 2;
+      uint32_t v = 0;
+      if (r < n && c < valid) v = *reinterpret_cast<const uint32_t*>(src + r * ld + c);
+      *reinterpret_cast<uint32_t*>(dst + r * kPitch + c) = v;
+    }
+  }
+}
 
 // NSL: key dimensions in slices of 128 (1 or 2)
 template <int NSL>
 __global__ void __launch_bounds__(kGtThreads, NSL == 1 ? 2 : 1) gla_chunk_kernel(const GlaChunkParams p) {
   extern __shared__ __align__(16) uint8_t gc_smem[];
-  float* b_s = reinterpret_cast<float*>(gc_smem);                       // [64][132] running sums
-  float* A_s = b_s;                                                     // [64][68] scores (after the slices)
+  float* b_s = reinterpret_cast<float*>(gc_smem);                       // [64][136] running sums
+  float* A_s = b_s;                                                     // [64][72] scores (after the slices)
   bf16_t* k_s = reinterpret_cast<bf16_t*>(b_s + kGtC * kGtBP);          // [64][136]
-  bf16_t* v_s = k_s + kGtC * kGtKP;                                     // [64][72]
-  bf16_t* s_hi = v_s + kGtC * kGtVP;                                    // [NSL * 128][72]
-  bf16_t* s_lo = s_hi + NSL * kGtSlice * kGtVP;
-  int* slow = reinterpret_cast<int*>(s_lo + NSL * kGtSlice * kGtVP);    // [4] diagonal blocks to be summed directly
+  bf16_t* q_s = k_s + kGtC * kGtKP;                                     // [64][136]
+  bf16_t* v_s = q_s + kGtC * kGtKP;                                     // [64][72]
+  bf16_t* s_hi = v_s + kGtC * kGtVP;                                    // [NSL * 128][64], swizzled
+  bf16_t* s_lo = s_hi + NSL * kGtSlice * kGtV;
+  int* slow = reinterpret_cast<int*>(s_lo + NSL * kGtSlice * kGtV);     // [4] diagonal blocks to be summed directly
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int v0 = blockIdx.x * kGtV, head = blockIdx.y;
   pdl_wait();
@@ -215,7 +249,7 @@ __global__ void __launch_bounds__(kGtThreads, NSL == 1 ? 2 : 1) gla_chunk_kernel
     for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
-        const int o = (sl * kGtSlice + warp * 16 + g + r * 8) * kGtVP + nt * 8 + t4 * 2;
+        const int o = gt_state_off(sl * kGtSlice + warp * 16 + g + r * 8, nt * 8 + t4 * 2);
         uint32_t hi, lo;
         split2(S[sl][nt][r * 2], S[sl][nt][r * 2 + 1], hi, lo);
         *reinterpret_cast<uint32_t*>(s_hi + o) = hi;
@@ -228,32 +262,28 @@ __global__ void __launch_bounds__(kGtThreads, NSL == 1 ? 2 : 1) gla_chunk_kernel
   for (int c0 = 0; c0 < s.len; c0 += kGtC) {
     const int n = min(kGtC, s.len - c0);
     const long long row0 = s.row0 + c0;
-    for (int i = tid; i < kGtC * (kGtV / 2); i += kGtThreads) {          // value tile
-      const int r = i / (kGtV / 2), c = (i % (kGtV / 2)) * 2;
-      uint32_t v = 0;
-      if (r < n && v0 + c < p.vdim)
-        v = *reinterpret_cast<const uint32_t*>(p.v + (row0 + r) * p.ld + head * p.vdim + v0 + c);
-      *reinterpret_cast<uint32_t*>(v_s + r * kGtVP + c) = v;
-    }
+    gt_load_tile<kGtV, kGtVP>(p.v + row0 * p.ld + head * p.vdim + v0, p.ld, n, p.vdim - v0, p.vec_v, v_s);
     float A[4][4] = {}, O[4][4] = {};
 #pragma unroll
     for (int sl = 0; sl < NSL; ++sl) {
       const int d0 = sl * kGtSlice, dn = min(kGtSlice, p.dim - d0);      // dims of this slice (a multiple of 16)
-      for (int i = tid; i < kGtC * (kGtSlice / 2); i += kGtThreads) {    // key tile
-        const int r = i / (kGtSlice / 2), c = (i % (kGtSlice / 2)) * 2;
-        uint32_t v = 0;
-        if (r < n && c < dn) v = *reinterpret_cast<const uint32_t*>(p.k + (row0 + r) * p.ld + head * p.dim + d0 + c);
-        *reinterpret_cast<uint32_t*>(k_s + r * kGtKP + c) = v;
-      }
+      gt_load_tile<kGtSlice, kGtKP>(p.k + row0 * p.ld + head * p.dim + d0, p.ld, n, dn, p.vec_k, k_s);
+      gt_load_tile<kGtSlice, kGtKP>(p.q + row0 * p.ld + head * p.dim + d0, p.ld, n, dn, p.vec_k, q_s);
       if (tid < 4) slow[tid] = 0;
       {                                                                  // running sums, 32 rows per thread
         const int c = tid & (kGtSlice - 1), r0 = (tid >> 7) * 32;
-        const float* dp = p.decay + (row0 + r0) * nk + head * p.dim + d0 + c;
+        const float* dp = p.decay + row0 * nk + head * p.dim + d0 + min(c, dn - 1);
         float run = 0.f;
-#pragma unroll 8
-        for (int r = 0; r < 32; ++r) {
-          if (r0 + r < n && c < dn) run += dp[static_cast<long long>(r) * nk];
-          b_s[(r0 + r) * kGtBP + c] = run;
+#pragma unroll
+        for (int rr = 0; rr < 32; rr += 16) {
+          float x[16];
+#pragma unroll
+          for (int r = 0; r < 16; ++r) x[r] = dp[static_cast<long long>(min(r0 + rr + r, n - 1)) * nk];
+#pragma unroll
+          for (int r = 0; r < 16; ++r) {
+            if (r0 + rr + r < n) run += x[r];
+            b_s[(r0 + rr + r) * kGtBP + c] = run;
+          }
         }
       }
       __syncthreads();
@@ -275,8 +305,6 @@ __global__ void __launch_bounds__(kGtThreads, NSL == 1 ? 2 : 1) gla_chunk_kernel
       // ---- scores against this slice's keys, and the state's read-out ----
       const bool direct = slow[I] != 0;
       const int i0 = I * 16 + g, i1 = i0 + 8;
-      const bf16_t* q0 = p.q + (row0 + i0) * p.ld + head * p.dim + d0;
-      const bf16_t* q1 = p.q + (row0 + i1) * p.ld + head * p.dim + d0;
       const float* ref_row = b_s + (I * 16 - 1) * kGtBP;                 // running sum in front of the block (I > 0)
       for (int ks = 0; ks < dn; ks += 16) {
         float2 ref[2], qh[4];                                            // columns ks + 2 t4, ks + 8 + 2 t4
@@ -286,13 +314,10 @@ __global__ void __launch_bounds__(kGtThreads, NSL == 1 ? 2 : 1) gla_chunk_kernel
           ref[u] = I > 0 ? *reinterpret_cast<const float2*>(ref_row + c) : make_float2(0.f, 0.f);
 #pragma unroll
           for (int r = 0; r < 2; ++r) {
-            float2 x = make_float2(0.f, 0.f);
-            if ((r ? i1 : i0) < n) {
-              x = ld_bf2((r ? q1 : q0) + c);
-              const float2 b = *reinterpret_cast<const float2*>(b_s + (r ? i1 : i0) * kGtBP + c);
-              x.x *= p.qscale * ex2_fast(b.x - ref[u].x);
-              x.y *= p.qscale * ex2_fast(b.y - ref[u].y);
-            }
+            float2 x = ld_bf2(q_s + (r ? i1 : i0) * kGtKP + c);          // zero behind the last row
+            const float2 b = *reinterpret_cast<const float2*>(b_s + (r ? i1 : i0) * kGtBP + c);
+            x.x *= p.qscale * ex2_fast(b.x - ref[u].x);
+            x.y *= p.qscale * ex2_fast(b.y - ref[u].y);
             qh[u * 2 + r] = x;
           }
         }
@@ -321,12 +346,12 @@ __global__ void __launch_bounds__(kGtThreads, NSL == 1 ? 2 : 1) gla_chunk_kernel
           const float2 r = ref[f >> 1];
           split2(qh[f].x * ex2_fast(r.x), qh[f].y * ex2_fast(r.y), ah[f], lo[f]);
         }
-        const int sr = (d0 + ks + (lane & 7) + (((lane >> 3) & 1) << 3)) * kGtVP + h * 32 + (lane >> 4) * 8;
+        const int sr = d0 + ks + (lane & 7) + (((lane >> 3) & 1) << 3);
 #pragma unroll
         for (int np = 0; np < 2; ++np) {
           uint32_t x0, x1, x2, x3, y0, y1, y2, y3;
-          ldsm_x4_t(smem_u32(s_hi + sr + np * 16), x0, x1, x2, x3);
-          ldsm_x4_t(smem_u32(s_lo + sr + np * 16), y0, y1, y2, y3);
+          ldsm_x4_t(smem_u32(s_hi + gt_state_off(sr, h * 32 + np * 16 + (lane >> 4) * 8)), x0, x1, x2, x3);
+          ldsm_x4_t(smem_u32(s_lo + gt_state_off(sr, h * 32 + np * 16 + (lane >> 4) * 8)), y0, y1, y2, y3);
           mma_bf16_16816(O[np * 2], ah, x0, x1);
           mma_bf16_16816(O[np * 2], ah, y0, y1);
           mma_bf16_16816(O[np * 2], lo, x0, x1);
@@ -342,7 +367,7 @@ __global__ void __launch_bounds__(kGtThreads, NSL == 1 ? 2 : 1) gla_chunk_kernel
           for (int e = 0; e < 4; ++e) {
             const int i = I * 16 + g + (e >> 1) * 8, j = I * 16 + nt2 * 8 + t4 * 2 + (e & 1);
             if (i >= n || j > i) continue;
-            const bf16_t* qr = p.q + (row0 + i) * p.ld + head * p.dim + d0;
+            const bf16_t* qr = q_s + i * kGtKP;
             float acc = 0.f;
             for (int d = 0; d < dn; ++d)
               acc = fmaf(__bfloat162float(qr[d]) * p.qscale * __bfloat162float(k_s[j * kGtKP + d]),
@@ -499,6 +524,9 @@ GLLM_API int gllm_gla_prefill(const int* q_start, const int* q_len, const int* c
   GlaChunkParams p = {};
   p.sv.q_start = q_start; p.sv.q_len = q_len; p.sv.ctx_lens = ctx_lens; p.sv.slots = slots; p.sv.n = n_seqs;
   p.q = static_cast<const bf16_t*>(q); p.k = static_cast<const bf16_t*>(k); p.v = static_cast<const bf16_t*>(v); p.ld = ld;
+  auto al16 = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
+  p.vec_k = (ld & 7) == 0 && (dim & 7) == 0 && al16(q) && al16(k);
+  p.vec_v = (ld & 7) == 0 && (vdim & 7) == 0 && al16(v);
   p.decay = decay; p.heads = heads; p.dim = dim; p.vdim = vdim; p.qscale = qscale; p.state = state; p.out = out;
   const bool two = dim > kGtSlice;
   auto kern = two ? gla_chunk_kernel<2> : gla_chunk_kernel<1>;

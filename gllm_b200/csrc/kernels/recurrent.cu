@@ -143,7 +143,7 @@ __global__ void __launch_bounds__(kGlaV* kGlaG) gla_step_kernel(const SeqView sv
       const T* wr = w2 + static_cast<long long>(head * dim + d) * rank;
       float z = b2[head * dim + d];
       for (int j = 0; j < rank; ++j) z = fmaf(to_f(wr[j]), a1s[j], z);
-      al[d] = expf(log_sigmoid_f(z) * inv_tau);
+      al[d] = decay_exp(log_sigmoid_f(z) * inv_tau);
     }
     __syncthreads();
     const float vv = live ? to_f(v[m * ld + head * vdim + col]) : 0.f;

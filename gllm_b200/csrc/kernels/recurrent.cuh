@@ -56,13 +56,17 @@ __device__ __forceinline__ float gelu_tanh_exact(float x) {
   return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
 }
 
-// RG-LRU: gate pre-activations -> decay a and input b = sqrt(1 - a^2) * i * u; 1 - a^2 = -expm1(2 log a) keeps its
-// relative accuracy where a is close to 1.
+// exp(x) for x <= 0 as a decay factor. A state remembers 1 / (1 - a) steps, so near 1 the distance to 1 must keep its
+// relative accuracy: it is taken from expm1 there.
+__device__ __forceinline__ float decay_exp(float x) { return x > -1.f ? 1.f + expm1f(x) : expf(x); }
+
+// RG-LRU: gate pre-activations -> decay a and input b = sqrt(1 - a^2) * i * u, 1 - a^2 = (1 - a) (2 - (1 - a)).
 constexpr float kRglruC = 8.f;
 __device__ __forceinline__ void rglru_coeffs(float xr, float xi, float softplus_lam, float u, float& a, float& b) {
   const float la = -kRglruC * sigmoid_f(xr) * softplus_lam;
-  a = expf(la);
-  b = sqrtf(-expm1f(2.f * la)) * sigmoid_f(xi) * u;
+  const float om = -expm1f(la);
+  a = decay_exp(la);
+  b = sqrtf(om * (2.f - om)) * sigmoid_f(xi) * u;
 }
 
 // Convolution state: a ring of the last `taps` inputs per channel, [slots][taps][width] fp32, the input of position p in

@@ -16,8 +16,8 @@
 namespace gllm {
 
 using bf16_t = __nv_bfloat16;
-constexpr int kRtRows = 64, kRtCh = 32, kRtThreads = 256, kRtTaps = 4;
-constexpr int kRtPitch = kRtCh + 1;      // floats per row of the decay / input tiles
+constexpr int kRtRows = 64, kRtCh = 32, kRtThreads = 256, kRtTaps = 4, kRtPre = 2;
+constexpr int kRtPitch = kRtCh + 8;      // floats per row of the decay / input tiles (pairs stored without bank conflicts)
 
 struct RtParams {
   SeqView sv;
@@ -40,15 +40,30 @@ struct RtParams {
   const float* seg_init;   // [seqs, n_seg, W] start states, or null (one segment: the slot's state)
 };
 
-// Gates at full fp32 arithmetic on the fast exponential units: relative errors of a few 1e-7.
-__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
-// 1 - exp(y) for y <= 0: a Taylor series where the difference would cancel.
-__device__ __forceinline__ float one_minus_exp(float y) {
-  if (y > -0.25f)
-    return -y * fmaf(y, fmaf(y, fmaf(y, fmaf(y, fmaf(y, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
-  return 1.f - __expf(y);
+// Gates in fp32 on the fast units (exponential, reciprocal, square root: relative errors of a few 1e-7).
+__device__ __forceinline__ float ex2_ap(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ float rcp_ap(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ float sqrt_ap(float x) { float y; asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+constexpr float kRtLog2e = 1.4426950408889634f;
+// sigmoid of a value that was multiplied by -log2(e)
+__device__ __forceinline__ float sigmoid_neg2(float x) { return rcp_ap(1.f + ex2_ap(x)); }
+// 1 - exp(y) for y <= 0, given e = exp(y): a Taylor series where the difference would cancel.
+__device__ __forceinline__ float one_minus_exp(float y, float e) {
+  const float t = fmaf(y, fmaf(y, fmaf(y, fmaf(y, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
+  return y > -0.125f ? -y * t : 1.f - e;
 }
-__device__ __forceinline__ float gelu_gate(float x) { return gelu_tanh_f(x); }
+// two fp32 multiply-adds in one instruction
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;"
+      : "=l"(reinterpret_cast<unsigned long long&>(d))
+      : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)),
+        "l"(reinterpret_cast<const unsigned long long&>(c)));
+  return d;
+}
+__device__ __forceinline__ float2 bf2_to_f2(uint32_t v) {
+  return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xFFFF0000u));
+}
 
 enum { RT_PREFILL = 0, RT_SUMMARY = 1, RT_DECODE = 2 };
 
@@ -62,21 +77,43 @@ __global__ void __launch_bounds__(kRtThreads, 2) rglru_tile_kernel(const RtParam
   float* b_s = a_s + kRtRows * kRtPitch;
   float* c_a = b_s + kRtRows * kRtPitch;                       // [8][32] per-warp products and end states
   float* c_b = c_a + 8 * kRtCh;
-  float* carry = c_b + 8 * kRtCh;                              // [2][32] state (and product) at the tile's start
+  float* carry = c_b + 8 * kRtCh;                              // [2][2][32] state and product at the tile's start (by tile parity)
+  float* cw_s = carry + 4 * kRtCh;                             // [5][bs_pad] convolution taps (oldest first) and bias
+  int* hist_s = reinterpret_cast<int*>(cw_s + 5 * p.bs_pad);   // decode: [64][4] ring entry of each older tap (-1: none),
+                                                               // and whether the row is live
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int blk = blockIdx.x / p.tiles_per_blk, c_in = (blockIdx.x % p.tiles_per_blk) * kRtCh;   // first channel in the block
   const int ch0 = blk * p.bs + c_in, nch = min(kRtCh, p.bs - c_in);
   const int kbase = blk * p.bs;
 
-  // gate weights of the CTA's channels: they do not depend on the kernel before this one
-  for (int i = tid; i < 2 * kRtCh * (p.bs_pad / 2); i += kRtThreads) {
-    const int r = i / (p.bs_pad / 2), k = (i % (p.bs_pad / 2)) * 2, o = r & (kRtCh - 1);
-    uint32_t v = 0;
-    if (o < nch && k < p.bs) {
-      const bf16_t* src = (r < kRtCh ? p.wr : p.wi) + (static_cast<long long>(blk) * p.bs + c_in + o) * p.bs + k;
-      v = *reinterpret_cast<const uint32_t*>(src);             // bs is even
+  // gate and convolution weights: they do not depend on the kernel before this one
+  if ((p.bs & 7) == 0) {
+    const int vecs = p.bs_pad / 8;
+#pragma unroll 8
+    for (int i = tid; i < 2 * kRtCh * vecs; i += kRtThreads) {
+      const int r = i / vecs, k = (i - r * vecs) * 8, o = r & (kRtCh - 1);
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (o < nch && k < p.bs)
+        v = __ldg(reinterpret_cast<const uint4*>((r < kRtCh ? p.wr : p.wi) +
+                                                 (static_cast<long long>(blk) * p.bs + c_in + o) * p.bs + k));
+      *reinterpret_cast<uint4*>(w_s + r * P + k) = v;
     }
-    *reinterpret_cast<uint32_t*>(w_s + r * P + k) = v;
+  } else {
+    for (int i = tid; i < 2 * kRtCh * (p.bs_pad / 2); i += kRtThreads) {
+      const int r = i / (p.bs_pad / 2), k = (i % (p.bs_pad / 2)) * 2, o = r & (kRtCh - 1);
+      uint32_t v = 0;
+      if (o < nch && k < p.bs)                                   // bs is even
+        v = *reinterpret_cast<const uint32_t*>((r < kRtCh ? p.wr : p.wi) +
+                                               (static_cast<long long>(blk) * p.bs + c_in + o) * p.bs + k);
+      *reinterpret_cast<uint32_t*>(w_s + r * P + k) = v;
+    }
+  }
+  for (int i = tid; i < 5 * p.bs_pad; i += kRtThreads) {         // missing taps are zero weights of older inputs
+    const int j = i / p.bs_pad, k = i - j * p.bs_pad, jj = j - (kRtTaps - p.taps);
+    float v = 0.f;
+    if (k < p.bs && j == 4) v = p.conv_b[kbase + k];
+    else if (k < p.bs && jj >= 0) v = p.conv_w[static_cast<long long>(kbase + k) * p.taps + jj];
+    cw_s[i] = v;
   }
   // this thread's gate columns: channels of its two accumulator tiles
   const int mrow = (warp & 3) * 16, half = warp >> 2, g = lane >> 2, t4 = lane & 3;
@@ -85,9 +122,9 @@ __global__ void __launch_bounds__(kRtThreads, 2) rglru_tile_kernel(const RtParam
   for (int e = 0; e < 4; ++e) {
     const int c = half * 16 + (e >> 1) * 8 + t4 * 2 + (e & 1);
     const bool ok = c < nch;
-    gbr[e] = ok ? p.br[ch0 + c] : 0.f;
-    gbi[e] = ok ? p.bi[ch0 + c] : 0.f;
-    gsp[e] = ok ? kRglruC * softplus_f(p.lam[ch0 + c]) : 0.f;
+    gbr[e] = ok ? -kRtLog2e * p.br[ch0 + c] : 0.f;
+    gbi[e] = ok ? -kRtLog2e * p.bi[ch0 + c] : 0.f;
+    gsp[e] = ok ? -kRglruC * softplus_f(p.lam[ch0 + c]) : 0.f;
   }
   pdl_wait();
   pdl_launch_dependents();
@@ -97,6 +134,16 @@ __global__ void __launch_bounds__(kRtThreads, 2) rglru_tile_kernel(const RtParam
   if (MODE == RT_DECODE) {
     t0 = blockIdx.y * kRtRows;
     t1 = min(t0 + kRtRows, p.sv.n);
+    for (int i = tid; i < kRtRows * 4; i += kRtThreads) {
+      const int r = i >> 2, j = i & 3;
+      const int ctx = t0 + r < t1 ? p.sv.ctx_lens[t0 + r] : 0;
+      const int pos = ctx - 1 - (kRtTaps - 1) + j;
+      int v;
+      if (j == 3) v = ctx > 0;
+      else v = (ctx > 0 && pos >= 0 && j >= kRtTaps - p.taps) ? pos % p.taps : -1;
+      hist_s[i] = v;
+    }
+    __syncthreads();
   } else {
     seq = blockIdx.y / p.n_seg;
     seg = blockIdx.y % p.n_seg;
@@ -114,67 +161,112 @@ __global__ void __launch_bounds__(kRtThreads, 2) rglru_tile_kernel(const RtParam
       carry[tid] = S;
       carry[kRtCh + tid] = 1.f;
     }
+    __syncthreads();                 // convolution weights
   }
+  // Inputs of a prefill work item (channel pair, 16 rows): rows r0 - 3 .. r0 + 15, all loads in flight at once. The first
+  // kRtPre items of a thread are fetched one tile ahead, behind the matrix products of the tile before.
+  const int npair = p.bs_pad / 2, nitem = npair * (kRtRows / 16);
+  auto fetch = [&](int it, int tile, uint32_t (&raw)[kRtTaps + 15]) {
+    const int tg = it / npair, k = (it - tg * npair) * 2;
+    const int c = kbase + min(k, p.bs - 2), first = tile + tg * 16 - (kRtTaps - 1);
+    const bf16_t* zp = p.z + static_cast<long long>(s.row0) * p.ld + c;
+    if (first >= 0 && first + kRtTaps + 15 <= t1) {
+      zp += static_cast<long long>(first) * p.ld;
+#pragma unroll
+      for (int j = 0; j < kRtTaps + 15; ++j) raw[j] = *reinterpret_cast<const uint32_t*>(zp + j * p.ld);
+    } else {
+#pragma unroll
+      for (int j = 0; j < kRtTaps + 15; ++j) {
+        raw[j] = *reinterpret_cast<const uint32_t*>(zp + min(max(first + j, 0), t1 - 1) * p.ld);
+        if (first + j >= t1) raw[j] = 0;
+      }
+    }
+  };
+  auto convolve = [&](int it, int tile, const uint32_t (&raw)[kRtTaps + 15]) {
+    const int tg = it / npair, k = (it - tg * npair) * 2, r0 = tg * 16;
+    const int c = kbase + min(k, p.bs - 2), first = tile + r0 - (kRtTaps - 1);   // columns behind the block: zero weights
+    float2 w[kRtTaps + 1];
+#pragma unroll
+    for (int j = 0; j < kRtTaps + 1; ++j) w[j] = *reinterpret_cast<const float2*>(cw_s + j * p.bs_pad + k);
+    float2 win[kRtTaps - 1];                                             // the three inputs in front of the next row
+#pragma unroll
+    for (int j = 0; j < kRtTaps - 1; ++j) win[j] = bf2_to_f2(raw[j]);
+    if (first < 0) {
+#pragma unroll
+      for (int j = 0; j < kRtTaps - 1; ++j)
+        win[j] = first + j > -p.taps ? make_float2(conv_history(p.ring, s.slot, p.taps, p.W, s.start + first + j, c),
+                                                   conv_history(p.ring, s.slot, p.taps, p.W, s.start + first + j, c + 1))
+                                     : make_float2(0.f, 0.f);
+    }
+    bf16_t* dst = u_s + r0 * P + k;
+#pragma unroll
+    for (int r = 0; r < 16; ++r) {
+      const float2 cur = bf2_to_f2(raw[r + kRtTaps - 1]);
+      const float2 x = fma2(w[0], win[0], fma2(w[1], win[1], fma2(w[2], win[2], fma2(w[3], cur, w[4]))));
+      win[0] = win[1];
+      win[1] = win[2];
+      win[2] = cur;
+      *reinterpret_cast<uint32_t*>(dst + r * P) = pack_bf16x2(x.x, x.y);
+    }
+  };
+  [[maybe_unused]] uint32_t pre[kRtPre][kRtTaps + 15];
+  if (MODE != RT_DECODE) {
+#pragma unroll
+    for (int i = 0; i < kRtPre; ++i)
+      if (tid + i * kRtThreads < nitem) fetch(tid + i * kRtThreads, t0, pre[i]);
+  }
+  [[maybe_unused]] int par = 0;
+
   for (int tile = t0; tile < t1; tile += kRtRows) {
     const int rows = min(kRtRows, t1 - tile);
-    // ---- convolution of the block's channels: work item = (channel pair, 8 rows) ----
-    const int npair = p.bs_pad / 2;
-    for (int it = tid; it < npair * 8; it += kRtThreads) {
-      const int k = (it % npair) * 2, r0 = (it / npair) * 8;
-      const bool live = k < p.bs;
-      const int c = kbase + k;
-      float w0[kRtTaps], w1[kRtTaps], b0 = 0.f, b1 = 0.f;      // missing taps are zero weights of older inputs
+    // ---- convolution of the block's channels ----
+    if (MODE == RT_DECODE) {
+      for (int it = tid; it < nitem; it += kRtThreads) {
+        const int tg = it / npair, k = (it - tg * npair) * 2, r0 = tg * 16;
+        const int c = kbase + min(k, p.bs - 2);
+        float2 w[kRtTaps + 1];
 #pragma unroll
-      for (int j = 0; j < kRtTaps; ++j) {
-        const int jj = j - (kRtTaps - p.taps);
-        w0[j] = live && jj >= 0 ? p.conv_w[static_cast<long long>(c) * p.taps + jj] : 0.f;
-        w1[j] = live && jj >= 0 ? p.conv_w[static_cast<long long>(c + 1) * p.taps + jj] : 0.f;
-      }
-      if (live) { b0 = p.conv_b[c]; b1 = p.conv_b[c + 1]; }
-      if (MODE == RT_DECODE) {
-        for (int r = r0; r < r0 + 8; ++r) {
-          float x0 = 0.f, x1 = 0.f;
-          const int m = tile + r;
-          const int ctx = r < rows ? p.sv.ctx_lens[m] : 0;
-          if (live && ctx > 0) {
-            const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.z + m * p.ld + c));
-            x0 = fmaf(w0[kRtTaps - 1], v.x, b0);
-            x1 = fmaf(w1[kRtTaps - 1], v.y, b1);
+        for (int j = 0; j < kRtTaps + 1; ++j) w[j] = *reinterpret_cast<const float2*>(cw_s + j * p.bs_pad + k);
+#pragma unroll
+        for (int rr = 0; rr < 16; rr += 4) {
+          float2 x[4][kRtTaps];
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            const int r = r0 + rr + q, m = min(tile + r, p.sv.n - 1);
+            x[q][kRtTaps - 1] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.z + m * p.ld + c));
 #pragma unroll
             for (int j = 0; j < kRtTaps - 1; ++j) {
-              if (j < kRtTaps - p.taps) continue;
-              const int pos = ctx - 1 - (kRtTaps - 1) + j;
-              x0 = fmaf(w0[j], conv_history(p.ring, m, p.taps, p.W, pos, c), x0);
-              x1 = fmaf(w1[j], conv_history(p.ring, m, p.taps, p.W, pos, c + 1), x1);
+              const int e = hist_s[r * 4 + j];
+              x[q][j] = *reinterpret_cast<const float2*>(p.ring + (static_cast<long long>(m) * p.taps + max(e, 0)) * p.W + c);
+              if (e < 0) x[q][j] = make_float2(0.f, 0.f);
             }
           }
-          *reinterpret_cast<uint32_t*>(u_s + r * P + k) = pack_bf16x2(x0, x1);
-        }
-      } else {
-        float2 win[kRtTaps + 7];                              // inputs of rows r0 - 3 .. r0 + 7
 #pragma unroll
-        for (int j = 0; j < kRtTaps + 7; ++j) {
-          const int i = tile + r0 - (kRtTaps - 1) + j;        // row within the portion
-          win[j] = make_float2(0.f, 0.f);
-          if (live && i < t1) {
-            if (i >= 0)
-              win[j] = __bfloat1622float2(
-                  *reinterpret_cast<const __nv_bfloat162*>(p.z + static_cast<long long>(s.row0 + i) * p.ld + c));
-            else if (i > -p.taps)
-              win[j] = make_float2(conv_history(p.ring, s.slot, p.taps, p.W, s.start + i, c),
-                                   conv_history(p.ring, s.slot, p.taps, p.W, s.start + i, c + 1));
+          for (int q = 0; q < 4; ++q) {
+            const int r = r0 + rr + q;
+            float x0 = w[kRtTaps].x, x1 = w[kRtTaps].y;
+#pragma unroll
+            for (int j = 0; j < kRtTaps; ++j) {
+              x0 = fmaf(w[j].x, x[q][j].x, x0);
+              x1 = fmaf(w[j].y, x[q][j].y, x1);
+            }
+            *reinterpret_cast<uint32_t*>(u_s + r * P + k) = hist_s[r * 4 + 3] ? pack_bf16x2(x0, x1) : 0u;
           }
         }
+      }
+    } else {
 #pragma unroll
-        for (int r = 0; r < 8; ++r) {
-          float x0 = b0, x1 = b1;
+      for (int i = 0; i < kRtPre; ++i)
+        if (tid + i * kRtThreads < nitem) convolve(tid + i * kRtThreads, tile, pre[i]);
+      for (int it = tid + kRtPre * kRtThreads; it < nitem; it += kRtThreads) {
+        uint32_t raw[kRtTaps + 15];
+        fetch(it, tile, raw);
+        convolve(it, tile, raw);
+      }
+      if (tile + kRtRows < t1) {
 #pragma unroll
-          for (int j = 0; j < kRtTaps; ++j) {
-            x0 = fmaf(w0[j], win[r + j].x, x0);
-            x1 = fmaf(w1[j], win[r + j].y, x1);
-          }
-          *reinterpret_cast<uint32_t*>(u_s + (r0 + r) * P + k) = pack_bf16x2(x0, x1);
-        }
+        for (int i = 0; i < kRtPre; ++i)
+          if (tid + i * kRtThreads < nitem) fetch(tid + i * kRtThreads, tile + kRtRows, pre[i]);
       }
     }
     // output-gate inputs of this thread's 8 (row, channel) pairs: fetched before the products that hide their latency
@@ -207,21 +299,27 @@ __global__ void __launch_bounds__(kRtThreads, 2) rglru_tile_kernel(const RtParam
         mma_bf16_16816(ai[1], a, b2, b3);
       }
     }
-    // ---- decays and inputs ----
+    // ---- decays and inputs (rows behind the last valid one are identities) ----
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int r = mrow + g + (e >> 1) * 8, cc = half * 16 + nt * 8 + t4 * 2 + (e & 1), q = nt * 2 + (e & 1);
-        float a = 1.f, b = 0.f;
-        if (r < rows && cc < nch) {
-          const float la = -sigmoid_fast(ar[nt][e] + gbr[q]) * gsp[q];
-          const float u = __bfloat162float(u_s[r * P + c_in + cc]);
-          a = __expf(la);
-          b = sqrtf(one_minus_exp(2.f * la)) * sigmoid_fast(ai[nt][e] + gbi[q]) * u;
+      for (int rh = 0; rh < 2; ++rh) {
+        const int r = mrow + g + rh * 8, cc = half * 16 + nt * 8 + t4 * 2;
+        const float2 u = bf2_to_f2(*reinterpret_cast<const uint32_t*>(u_s + r * P + min(c_in + cc, p.bs - 2)));
+        float2 a, b;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int q = nt * 2 + e;
+          const float la = sigmoid_neg2(fmaf(ar[nt][rh * 2 + e], -kRtLog2e, gbr[q])) * gsp[q];
+          // the distance of the decay to 1 keeps its relative accuracy (a state remembers 1 / (1 - a) steps)
+          const float om = one_minus_exp(la, ex2_ap(la * kRtLog2e)), av = 1.f - om;
+          const float bv = sqrt_ap(om * (1.f + av)) *
+                           sigmoid_neg2(fmaf(ai[nt][rh * 2 + e], -kRtLog2e, gbi[q])) * (e ? u.y : u.x);
+          if (e) { a.y = av; b.y = bv; } else { a.x = av; b.x = bv; }
         }
-        a_s[r * kRtPitch + cc] = a;
-        b_s[r * kRtPitch + cc] = b;
+        if (r >= rows) { a = make_float2(1.f, 1.f); b = make_float2(0.f, 0.f); }
+        *reinterpret_cast<float2*>(a_s + r * kRtPitch + cc) = a;
+        *reinterpret_cast<float2*>(b_s + r * kRtPitch + cc) = b;
       }
     __syncthreads();
 
@@ -230,13 +328,13 @@ __global__ void __launch_bounds__(kRtThreads, 2) rglru_tile_kernel(const RtParam
       for (int i = 0; i < 8; ++i) {
         const int r = warp * 8 + i, m = tile + r;
         if (r >= rows || lane >= nch) continue;
+        if (!hist_s[r * 4 + 3]) continue;
         const int ctx = p.sv.ctx_lens[m];
-        if (ctx <= 0) continue;
         const long long so = static_cast<long long>(m) * p.W + ch0 + lane;
         float S = ctx > 1 ? p.state[so] : 0.f;
         S = fmaf(a_s[r * kRtPitch + lane], S, b_s[r * kRtPitch + lane]);
         p.state[so] = S;
-        p.out[so] = __float2bfloat16_rn(S * gelu_gate(yv[i]));
+        p.out[so] = __float2bfloat16_rn(S * gelu_tanh_f(yv[i]));
         p.ring[(static_cast<long long>(m) * p.taps + (ctx - 1) % p.taps) * p.W + ch0 + lane] =
             __bfloat162float(p.z[m * p.ld + ch0 + lane]);
       }
@@ -254,7 +352,7 @@ __global__ void __launch_bounds__(kRtThreads, 2) rglru_tile_kernel(const RtParam
     c_a[warp * kRtCh + lane] = A;
     c_b[warp * kRtCh + lane] = B;
     __syncthreads();
-    float S = carry[lane], prod = carry[kRtCh + lane];
+    float S = carry[par * 2 * kRtCh + lane], prod = carry[par * 2 * kRtCh + kRtCh + lane];
     for (int w = 0; w < warp; ++w) {
       S = fmaf(c_a[w * kRtCh + lane], S, c_b[w * kRtCh + lane]);
       if (MODE == RT_SUMMARY) prod *= c_a[w * kRtCh + lane];
@@ -268,23 +366,23 @@ __global__ void __launch_bounds__(kRtThreads, 2) rglru_tile_kernel(const RtParam
         const int r = warp * 8 + i;
         S = fmaf(av[i], S, bv[i]);
         if (r < rows && lane < nch)
-          p.out[static_cast<long long>(s.row0 + tile + r) * p.W + ch0 + lane] = __float2bfloat16_rn(S * gelu_gate(yv[i]));
+          p.out[static_cast<long long>(s.row0 + tile + r) * p.W + ch0 + lane] = __float2bfloat16_rn(S * gelu_tanh_f(yv[i]));
       }
     }
-    __syncthreads();                 // every warp has read the carry of this tile
+    par ^= 1;
     if (warp == 7) {                 // rows behind the last valid one are identities: this is the tile's end state
-      carry[lane] = S;
-      carry[kRtCh + lane] = prod;
+      carry[par * 2 * kRtCh + lane] = S;
+      carry[par * 2 * kRtCh + kRtCh + lane] = prod;
     }
-    // the barrier behind the next tile's convolution orders this write before the next read
+    // the barriers of the next tile order this write before the next read
   }
   if (MODE == RT_DECODE) return;
   if (warp == 7 && lane < nch) {     // this warp wrote the carry itself
     if (MODE == RT_SUMMARY)
       p.seg_sum[(static_cast<long long>(seq) * p.n_seg + seg) * p.W + ch0 + lane] =
-          make_float2(carry[kRtCh + lane], carry[lane]);
+          make_float2(carry[par * 2 * kRtCh + kRtCh + lane], carry[par * 2 * kRtCh + lane]);
     else if (t1 == s.len)
-      p.state[static_cast<long long>(s.slot) * p.W + ch0 + lane] = carry[lane];
+      p.state[static_cast<long long>(s.slot) * p.W + ch0 + lane] = carry[par * 2 * kRtCh + lane];
   }
 }
 
@@ -326,10 +424,11 @@ static int rt_done(cudaError_t e, const char* what) {
   return -1;
 }
 static size_t rt_smem_bytes(int bs_pad) {
-  return static_cast<size_t>(kRtRows + 2 * kRtCh) * (bs_pad + 8) * 2 + sizeof(float) * (2 * kRtRows * kRtPitch + 16 * kRtCh + 2 * kRtCh);
+  return static_cast<size_t>(kRtRows + 2 * kRtCh) * (bs_pad + 8) * 2 + sizeof(float) * (2 * kRtRows * kRtPitch + 16 * kRtCh + 4 * kRtCh + 5 * bs_pad) +
+         kRtRows * 4 * 4;
 }
 
-// Whether the one-pass kernel takes a layer: even gate blocks that fit in shared memory, at most four taps.
+// Whether the one-pass kernel takes a layer: even gate blocks (and 16-byte aligned weights) that fit in shared memory, at most four taps.
 GLLM_API int gllm_rglru_tile_ok(int W, int nblk, int taps) {
   if (nblk <= 0 || W % nblk != 0 || (W & 1)) return 0;
   const int bs = W / nblk;

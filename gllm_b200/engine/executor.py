@@ -450,7 +450,7 @@ class LLMEngine:
         out = []
         for rid, toks, want in entries:
             base = self._fed[int(rid)] - len(toks)
-            rows = [self._feed_out.pop((int(rid), base + int(w))).float() for w in want]
+            rows = [self._feed_out[(int(rid), base + int(w))].float() for w in want]
             out.append(torch.stack(rows).cpu() if rows else torch.zeros((0, self.mc.vocab_size)))
         self._feed_want.clear()
         self._feed_out.clear()

@@ -200,6 +200,7 @@ class HybridDecoder:
         self.mark("begin")
         if hidden_in is None:
             R.embed_rows(batch.token_ids, self.embed, x, xb if two else None)
+            self.mark("embed")
         else:
             x.copy_(hidden_in.float())
             if two:
@@ -211,7 +212,7 @@ class HybridDecoder:
             if callbacks is not None and self._run_callbacks(callbacks, "pre", i, x, xb):
                 break
             y = lw.mixer.forward(self, ws, batch, kv_caches[i], T)
-            self.mark("mix_out")
+            self.mark("out_gemm")
             R.scaled_add_norm(x, y, lw.norm1, c.postln_alpha, c.rms_norm_eps, x_out=x, xb=xb if two else None)
             self.mark("norm")
             if lw.w_down is not None:
@@ -239,9 +240,9 @@ class HybridDecoder:
         else:
             gu = L.gemm(xb, lw.w_gate_up, out=ws.take("gu", T, lw.w_gate_up.shape[0]))
             act = ops.glu(gu, lw.act, out=ws.take("act", T, lw.w_down.shape[1]))
-        self.mark("gate_up")
+        self.mark("gate_up_gemm")
         y = L.gemm(act, lw.w_down, out=ws.take("y", T, lw.w_down.shape[0]))
-        self.mark("down")
+        self.mark("down_gemm")
         return y
 
     def _logits(self, x, rows=None):

@@ -77,6 +77,7 @@ class AttentionMixer(_Mixer):
     def forward(self, model, ws, batch, kv, T):
         m = self.spec
         qk = L.gemm(ws.xb[:T], self.w["wqk"], out=ws.take("proj", T, self.w["wqk"].shape[0]), bias=self.w["bqk"])
+        model.mark("in_gemm")
         cos, sin = model.rope_tables(m.rot_dim, m.rot_base)
         q = ws.take("q", T, self.nq)
         R.qk_row_norm_rope(qk, n_q=m.heads, n_kv=m.kv_heads, head_dim=m.dim, rot_dim=m.rot_dim, v_from_k=m.v_from_k,
@@ -123,7 +124,7 @@ class RgLruMixer(_Mixer):
         m, w = self.spec, self.w
         yx = L.gemm(ws.xb[:T], w["wyx"], out=ws.take("proj", T, w["wyx"].shape[0]), bias=w["byx"])
         y, z = yx[:, :m.width], yx[:, m.width:2 * m.width]
-        model.mark("rglru_in")
+        model.mark("in_gemm")
         sv = SeqView.of(batch)
         out = ws.take("mix", T, m.width)
         if self.fused:
@@ -168,13 +169,14 @@ class GlaMixer(_Mixer):
             parts.append(p[:, o:o + n])
             o += n
         q, k, v, g, a1 = parts
-        model.mark("gla_in")
+        model.mark("in_gemm")
         sv = SeqView.of(batch)
         out = ws.take("mix", T, self.nv)
         size = dict(heads=m.heads, dim=m.dim, vdim=m.vdim)
         if batch.is_decode and self.fused_decode:
             R.gla_decode(sv, q, k, v, g, a1, w["a2"], w["a2_b"], w["norm"], **size, tau=m.tau, eps=self.eps,
                          state=st["rec"], out=out)
+            model.mark("gla")
         else:
             acc = ws.take("f32", T, self.nv)
             if not batch.is_decode and self.chunked:
@@ -182,8 +184,9 @@ class GlaMixer(_Mixer):
                               state=st["rec"], out=acc)
             else:
                 R.gla_step(sv, q, k, v, a1, w["a2"], w["a2_b"], **size, tau=m.tau, state=st["rec"], out=acc)
+            model.mark("gla")
             R.head_norm_gate(acc, g, w["norm"], heads=m.heads, vdim=m.vdim, eps=self.eps, out=out)
-        model.mark("gla")
+            model.mark("gla_gate")
         return L.gemm(out, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
 
 

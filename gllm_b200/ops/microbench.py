@@ -6,7 +6,7 @@ warm-up; the achieved fraction of the measured peaks (``MEASURED_PEAKS.json`` at
 present) is printed as JSON.
 
 ops: bsgemm_mxfp8  bsgemm_nvfp4  gemm_prefill  gemm_prefill_glu  gemm_prefill_residual  gemm_prefill_qkv  gemm_decode  gemm_decode_trace  gemm_glu  gemm_qkv  decode_attn  prefill_attn  sample  qgemm_fp8  qgemm_fp4  qgemm_int4
-     mla_attn
+     mla_attn  rglru_prefill  rglru_decode  gla_prefill  gla_decode
 """
 from __future__ import annotations
 
@@ -343,6 +343,39 @@ def run(op: str, iters: int):
         params = torch.tensor([0.7, 50, 0.9, 0], device=dev).repeat(B, 1).contiguous()
         t = _time(lambda: ops.sample(lg, params, seed=1), iters)
         out.update(batch=B, vocab=V, us=t * 1e6, logits_gbs=B * V * 4 / t / 1e9)
+    elif op in ("rglru_prefill", "rglru_decode", "gla_prefill", "gla_decode"):
+        from . import recurrent as R
+        S, L = (4, 2048) if op.endswith("prefill") else (256, 1)
+        T, i32 = S * L, lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        sv = R.SeqView(i32([2048] * S)) if L == 1 else R.SeqView(i32([L] * S), i32([j * L for j in range(S)]), i32([L] * S),
+                                                                 i32(list(range(S))), L)
+        if op.startswith("rglru"):
+            W, nb, taps = 4096, 16, 4
+            bs = W // nb
+            yz, o = rnd(T, 2 * W), torch.empty(T, W, dtype=torch.bfloat16, device=dev)
+            wr, wi = rnd(nb, bs, bs) * 0.1, rnd(nb, bs, bs) * 0.1
+            f = lambda *n: torch.randn(*n, device=dev)
+            args = (f(W, taps), f(W), wr, f(W), wi, f(W), f(W) - 4)
+            st, ring = torch.zeros(S, W, device=dev), torch.zeros(S, taps, W, device=dev)
+            t = _time(lambda: R.rglru_tile(sv, yz[:, :W], yz[:, W:], *args, st, ring, o), iters)
+            by = T * W * 6 + 2 * W * bs * 2 + (T * W * (2 + taps) * 4 if L == 1 else 0)
+        else:
+            H, d, e, r = 16, 128, 256, 16
+            nk, nv_ = H * d, H * e
+            p = rnd(T, 2 * nk + 2 * nv_ + 32)
+            parts = [p[:, a:a + n] for a, n in ((0, nk), (nk, nk), (2 * nk, nv_), (2 * nk + nv_, nv_), (2 * nk + 2 * nv_, r))]
+            w2, b2, nw = rnd(nk, r) * 0.1, torch.randn(nk, device=dev), torch.ones(e, device=dev)
+            st, size = torch.zeros(S, H, d, e, device=dev), dict(heads=H, dim=d, vdim=e, tau=16.0)
+            q, k, v, g, a1 = parts
+            if L == 1:
+                o = torch.empty(T, nv_, dtype=torch.bfloat16, device=dev)
+                t = _time(lambda: R.gla_decode(sv, q, k, v, g, a1, w2, b2, nw, **size, eps=1e-5, state=st, out=o), iters)
+                by = T * H * d * e * 8 + T * (2 * nk + 3 * nv_) * 2
+            else:
+                o, dec = torch.empty(T, nv_, device=dev), torch.empty(T, nk, device=dev)
+                t = _time(lambda: R.gla_prefill(sv, q, k, v, a1, w2, b2, **size, decay=dec, state=st, out=o), iters)
+                by = T * (2 * nk + nv_) * 2 + T * nv_ * 4
+        out.update(seqs=S, len=L, us=t * 1e6, gbs=by / t / 1e9, frac_of_hbm_peak=by / t / 1e9 / hbm)
     else:
         raise SystemExit(f"unknown op {op}")
     from . import _native as nv
