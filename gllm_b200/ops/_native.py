@@ -58,6 +58,7 @@ _SIGNATURES = {
     "gllm_rope_kv_write": (I, [P, L, I, I, I, I, I, P, P, P, P, I, P, P, F, P, P, I, P]),
     "gllm_paged_attention_generic": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, F, I, I, P]),
     "gllm_paged_attention_f32": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, F, I, I, P]),
+    "gllm_attention_mma": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, F, I, I, P]),
     "gllm_gemm_simt": (I, [P, L, P, L, P, L, I, I, I, I, I, P, F, P]),
     "gllm_paged_attention_fp8kv": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, F, I, I, F, P]),
     "gllm_rope_kv_write_fp8": (I, [P, L, I, I, I, I, I, P, P, P, P, I, P, P, F, P, P, I, F, P]),

@@ -1,7 +1,7 @@
 """Paged attention ops over the 16-token-page KV cache ``[pages, 2, n_kv, 16, D]``.
 
-CUDA path: ``csrc/kernels/attention.cu`` (head_dim 128, TMA page gathers + tensor-core math) or the
-generic kernel in ``misc.cu`` for other head dims. CPU path / oracle: plain fp32 softmax attention with the
+CUDA path: ``csrc/kernels/attention.cu`` (head_dim 128, TMA page gathers + tensor-core math), ``attention_mma.cu`` (other
+multiples of 16, warp-level tensor cores) or the generic kernel in ``misc.cu`` (any head dim up to 256, fp32, fp8 pages). CPU path / oracle: plain fp32 softmax attention with the
 reference's semantics (src/compat/scalar_ops.rs:196-278,316-378): scale 1/sqrt(d), GQA head mapping
 ``kv_h = h // (Hq/Hkv)``, causal mask, max-subtracted softmax, optional sliding window and sinks.
 """
@@ -84,6 +84,22 @@ class DecodeWorkspace:
         self.counters = torch.zeros(max_batch * n_kv, dtype=torch.int32, device=device)
 
 
+def _mma_head(q, kv_cache, sinks) -> bool:
+    """Whether ``gllm_attention_mma`` takes the call: bf16, head dim a multiple of 16 other than 128, no sinks."""
+    D = kv_cache.shape[-1]
+    return (q.dtype == torch.bfloat16 and kv_cache.dtype == torch.bfloat16 and D % 16 == 0 and D <= 256 and D != 128
+            and sinks is None and q.is_contiguous())
+
+
+def _attention_mma(q, out, kv_cache, block_tables, q_start, q_len, ctx_lens, n_seqs, max_q_len, n_q, n_kv, scale, causal, window):
+    rc = nv.lib().gllm_attention_mma(q.data_ptr(), out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
+                                     block_tables.data_ptr(), block_tables.shape[1], nv.ptr(q_start), nv.ptr(q_len),
+                                     ctx_lens.data_ptr(), n_seqs, max_q_len, n_q, n_kv, kv_cache.shape[-1], scale,
+                                     1 if causal else 0, window, nv.stream_ptr())
+    nv.check(rc, "attention_mma")
+    return out
+
+
 def paged_decode(q, kv_cache, block_tables, ctx_lens, *, n_q, n_kv, scale=None, out=None, workspace=None,
                  pages_per_split=32, window=0, sinks=None, kv_scale: float = 1.0, full_weights: bool = False):
     """One query token per sequence. q: [B, n_q*D]; ctx_lens includes the token just written. ``full_weights``: the softmax
@@ -119,6 +135,8 @@ def paged_decode(q, kv_cache, block_tables, ctx_lens, *, n_q, n_kv, scale=None, 
                                         nv.stream_ptr())
         nv.check(rc, "paged_decode")
         return out
+    if _mma_head(q, kv_cache, sinks) and out.is_contiguous():
+        return _attention_mma(q, out, kv_cache, block_tables, None, None, ctx_lens, B, 1, n_q, n_kv, scale, True, window)
     ar = torch.arange(B, dtype=torch.int32, device=q.device)
     ones = (ctx_lens > 0).to(torch.int32)
     return paged_prefill(q, kv_cache, block_tables, ar, ones, ctx_lens, max_q_len=1, n_q=n_q, n_kv=n_kv, scale=scale,
@@ -177,6 +195,8 @@ def paged_prefill(q, kv_cache, block_tables, q_start, q_len, ctx_lens, *, max_q_
                                          q_len.data_ptr(), ctx_lens.data_ptr(), S, max_q_len, n_q, n_kv, scale,
                                          1 if causal else 0, window, nv.ptr(sinks), nv.stream_ptr())
         nv.check(rc, "paged_prefill")
+    elif _mma_head(q, kv_cache, sinks) and out.is_contiguous():
+        _attention_mma(q, out, kv_cache, block_tables, q_start, q_len, ctx_lens, S, max_q_len, n_q, n_kv, scale, causal, window)
     else:
         if sinks is not None:
             raise NotImplementedError("attention sinks need head_dim 128")

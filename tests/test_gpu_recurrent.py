@@ -165,6 +165,36 @@ def test_full_weight_attention(n_q, n_kv, window):
         assert rel(got, want[ctx - 1:ctx].cpu()) < 4e-3, ctx
 
 
+@pytest.mark.parametrize("D", [16, 48, 64, 80, 96, 176, 256])
+@pytest.mark.parametrize("n_q,n_kv", [(6, 3), (2, 2), (16, 1), (20, 1)])
+@pytest.mark.parametrize("window", [0, 70, ops.chunk_window(48), ops.chunk_window(100)])
+def test_attention_of_other_head_dims(D, n_q, n_kv, window):
+    """Warp-level tensor-core attention: three sequences of unequal portions and contexts, then decode rows with an empty
+    slot between them."""
+    lens, ctx = [150, 3, 70], [150, 90, 211]
+    pages = [(c + 15) // 16 for c in ctx]
+    kv = rand(sum(pages) + 5, 2, n_kv, 16, D, seed=1).to(DEV)
+    perm = torch.randperm(sum(pages) + 5, generator=torch.Generator().manual_seed(2))
+    bt = torch.zeros((3, max(pages)), dtype=torch.int32)
+    for i, n in enumerate(pages):
+        bt[i, :n] = perm[sum(pages[:i]):sum(pages[:i]) + n]
+    bt = bt.to(DEV)
+    starts = [0, 150, 153]
+    q = rand(sum(lens), n_q * D, seed=3).to(DEV)
+    want = ops.attention_ref(q.double(), kv.double(), bt, starts, lens, ctx, n_q, n_kv, 0.3, True, window)
+    ref = rel(want.to(BF), want.cpu())
+    got = ops.paged_prefill(q, kv, bt, i32(starts), i32(lens), i32(ctx), max_q_len=150, n_q=n_q, n_kv=n_kv, scale=0.3, window=window)
+    assert rel(got, want.cpu()) < 1.3 * ref
+    if window == 0:        # bidirectional
+        both = ops.attention_ref(q.double(), kv.double(), bt, starts, lens, ctx, n_q, n_kv, 0.3, False, 0)
+        got = ops.paged_prefill(q, kv, bt, i32(starts), i32(lens), i32(ctx), max_q_len=150, n_q=n_q, n_kv=n_kv, scale=0.3, causal=False)
+        assert rel(got, both.cpu()) < 1.3 * ref
+    dq = torch.stack([q[149], q[152], q[0], q[222]])
+    dbt = torch.stack([bt[0], bt[1], bt[0], bt[2]])
+    got = ops.paged_decode(dq, kv, dbt, i32([150, 90, 0, 211]), n_q=n_q, n_kv=n_kv, scale=0.3, window=window)
+    assert rel(got[[0, 1, 3]], want[[149, 152, 222]].cpu()) < 1.5 * ref
+
+
 def test_fp32_gemm_is_not_tf32():
     a, w = torch.randn(70, 333, device=DEV), torch.randn(45, 333, device=DEV)
     b = torch.randn(45, device=DEV)
