@@ -51,7 +51,7 @@ def parse_args():
                     help="fp8: e4m3 KV cache (half the KV bytes); not the headline configuration, reported as invalid for it")
     ap.add_argument("--op-breakdown", action="store_true",
                     help="after the timed regions, time every op of one captured decode step with in-graph events")
-    ap.add_argument("--hybrid", nargs="?", const="2048,4096", default=None, metavar="WIDTHS",
+    ap.add_argument("--hybrid", nargs="?", const="2048,2048d64,4096", default=None, metavar="SIZES",
                     help="instead of the headline workload: prefill and decode throughput of the heterogeneous decoder "
                          "(Zenevik) beside a dense decoder of equal size, per-op times against the roofline (one GPU)")
     ap.add_argument("--layers", type=int, default=0, help="debug only: a value other than 0 marks the result invalid")

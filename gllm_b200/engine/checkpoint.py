@@ -15,8 +15,15 @@ import torch
 FORMAT_VERSION = 1
 
 
+def _check(engine):
+    if engine.mc.is_hybrid:
+        raise ValueError("session snapshots hold pages of one shape per layer; a heterogeneous model has none to offer "
+                         "(its recurrent state does not outlive a request)")
+
+
 def save_sessions(engine, path: str) -> Dict[str, int]:
     """Writes {session id: tokens, per-layer page contents} for every session whose pages are still cached."""
+    _check(engine)
     b = engine.batcher
     out = {"version": FORMAT_VERSION, "page_size": 16, "layers": len(engine.kv_caches),
            "page_shape": tuple(engine.kv_caches[0].shape[1:]), "dtype": str(engine.kv_caches[0].dtype), "sessions": {}}
@@ -36,6 +43,7 @@ def save_sessions(engine, path: str) -> Dict[str, int]:
 
 def load_sessions(engine, path: str) -> Dict[str, int]:
     """Restores sessions into ``engine`` (same model geometry). Returns {session id: tokens restored}."""
+    _check(engine)
     snap = torch.load(path, map_location="cpu", weights_only=True)     # tensors, lists, dicts and scalars only
     if snap.get("version") != FORMAT_VERSION:
         raise ValueError("unknown session snapshot version")

@@ -296,8 +296,9 @@ class LLMEngine:
                    "kv_telemetry_every": ec.kv_telemetry_every > 0}
         bad = [k for k, v in refused.items() if v]
         if bad:
-            raise ValueError(f"not available for models with recurrent layers: {', '.join(bad)}")
-        ec.enable_prefix_cache = False
+            raise ValueError(f"not available for heterogeneous models: {', '.join(bad)}")
+        if self.recurrent:
+            ec.enable_prefix_cache = False
 
     # ------------------------------------------------------------------------------------------
     def generate_with_mtp(self, prompt_ids: List[int], max_tokens: int = 256, temperature: float = 0.0, top_k: int = 0,

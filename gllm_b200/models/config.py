@@ -525,6 +525,16 @@ def preset(name: str) -> ModelConfig:
                            kv_lora_rank=32, qk_nope_head_dim=32, qk_rope_head_dim=16, v_head_dim=32, num_experts=8,
                            num_experts_per_tok=2, moe_intermediate_size=128, num_shared_experts=1, first_k_dense=1,
                            router_scoring="sigmoid", max_position_embeddings=2048, eos_token_ids=[2])
+    if n in ("tiny-zenevik",):
+        att = MixerSpec("attention", heads=4, kv_heads=2, dim=128, vdim=128, scale=0.09, rot_dim=32, rot_base=1000.0, chunk=48,
+                        row_qk_norm=True, v_from_k=True)
+        lru = MixerSpec("rglru", width=192, blocks=3, taps=4)
+        gla = MixerSpec("gla", heads=2, dim=48, vdim=96, tau=4.0, decay_rank=8)
+        cfg = ModelConfig(arch="zenevik", hidden_size=256, num_layers=3, vocab_size=1024, rms_norm_eps=1e-6,
+                          postln_alpha=1.5, logit_softcap=20.0, hidden_act="gelu_tanh", max_position_embeddings=2048,
+                          layer_specs=[LayerSpec(att, ff=512), LayerSpec(lru), LayerSpec(gla, ff=256)], eos_token_ids=[2])
+        cfg.set_hybrid_dims()
+        return cfg
     if n in ("tiny-bert",):
         return ModelConfig(arch="bert", kind="embedding", hidden_size=128, num_layers=2, num_heads=2, num_kv_heads=2,
                            head_dim=64, intermediate_size=256, vocab_size=512, causal=False, norm_type="layer",

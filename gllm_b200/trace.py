@@ -4,7 +4,7 @@
 
 One JSON object per input line:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["b"]}
+    {"step": 7, "entries": [{"id": "r1", "tokens": [12, 40], "want": [1]}, {"id": "r2", "tokens": [9], "want": []}], "end": ["r2"]}
 
 ``entries``: the next tokens of each request and the indices among them whose logits are wanted; ``end``: requests that are
 finished after this step. The wanted logits of a step go to ``OUT/<step>.f32`` ([wanted, vocab], little-endian fp32, in the

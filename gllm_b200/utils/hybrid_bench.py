@@ -23,13 +23,15 @@ from .tracing import GraphTimer
 
 SIZES = {
     "2048": dict(hidden=2048, heads=16, kv=8, ff=6144, lru=2048, blocks=16, gla=8),
+    "2048d64": dict(hidden=2048, heads=32, kv=8, ff=6144, lru=2048, blocks=16, gla=8, dim=64),
     "4096": dict(hidden=4096, heads=32, kv=8, ff=12288, lru=4096, blocks=16, gla=16),
 }
 VOCAB, CHUNK, PROMPT, PROMPTS = 32768, 2048, 2048, 4
 
 
 def hybrid_config(s: dict) -> ModelConfig:
-    att = MixerSpec("attention", heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5, rot_dim=64,
+    att = MixerSpec("attention", heads=s["heads"], kv_heads=s["kv"], dim=s.get("dim", 128), vdim=s.get("dim", 128),
+                    scale=s.get("dim", 128) ** -0.5, rot_dim=s.get("dim", 128) // 2,
                     rot_base=10000.0, chunk=CHUNK, row_qk_norm=True, v_from_k=True)
     lru = MixerSpec("rglru", width=s["lru"], blocks=s["blocks"], taps=4)
     gla = MixerSpec("gla", heads=s["gla"], dim=128, vdim=256, tau=16.0, decay_rank=16)
@@ -42,7 +44,7 @@ def hybrid_config(s: dict) -> ModelConfig:
 
 def dense_config(s: dict) -> ModelConfig:
     return ModelConfig(arch="qwen3", hidden_size=s["hidden"], num_layers=6, num_heads=s["heads"], num_kv_heads=s["kv"],
-                       head_dim=128, intermediate_size=s["ff"], vocab_size=VOCAB, qk_norm=True, hidden_act="gelu_tanh",
+                       head_dim=s.get("dim", 128), intermediate_size=s["ff"], vocab_size=VOCAB, qk_norm=True, hidden_act="gelu_tanh",
                        max_position_embeddings=1 << 16)
 
 
@@ -120,10 +122,10 @@ def work(cfg: ModelConfig, T: int, decode: bool, rows: int) -> Dict[str, tuple]:
                 add("down_gemm", _gemm(T, H, l.ff, 4))
                 add("norm", (T * H * (4 + 4 + 4 + 2), 0))
     else:
-        nq, nk, L = cfg.num_heads * 128, cfg.num_kv_heads * 128, cfg.num_layers
+        nq, nk, L = cfg.num_heads * cfg.head_dim, cfg.num_kv_heads * cfg.head_dim, cfg.num_layers
         for _ in range(L):
             add("qkv_gemm", _gemm(T, nq + 2 * nk, H))
-            attend(cfg.num_heads, cfg.num_kv_heads, 128)
+            attend(cfg.num_heads, cfg.num_kv_heads, cfg.head_dim)
             add("o_proj", (_gemm(T, H, nq)[0] + T * H * 2, 2 * T * H * nq))
             add("gate_up_gemm", (T * H * 2 + 2 * cfg.intermediate_size * H * 2 + T * cfg.intermediate_size * 2,
                                  4 * T * cfg.intermediate_size * H))
@@ -205,7 +207,7 @@ def bench_model(model, steps: int, warmup: int, decode_sizes=(64, 256)) -> dict:
     return res
 
 
-def main(sizes=("2048", "4096"), steps: int = 10, warmup: int = 3) -> dict:
+def main(sizes=("2048", "2048d64", "4096"), steps: int = 10, warmup: int = 3) -> dict:
     out = {}
     for size in sizes:
         for name, cls, cfg in (("zenevik", HybridDecoder, hybrid_config(SIZES[size])),

@@ -288,6 +288,21 @@ def test_sampling_and_mixed_work_leave_the_state_alone():
     assert eng.results[rb].token_ids == Z.greedy(MIX, w, b, 30)
 
 
+def test_prefix_pages_are_shared_by_attention_only_models():
+    cfg = Z.config([Z.att(), Z.att(chunk=40, ff=48)])
+    w = Z.weights(cfg, seed=12)
+    eng = engine(cfg, w, ("cpu", torch.float32), max_len=128)
+    p = Z.tokens(cfg, 50, seed=12)
+    a = eng.generate_batch([p], max_tokens=4, temperature=0.0)[0]
+    b = eng.generate_batch([p[:40] + [1, 2]], max_tokens=4, temperature=0.0)[0]
+    assert b.telemetry.cached_prefix_tokens == 32
+    assert a.token_ids == Z.greedy(cfg, w, p, 4) and b.token_ids == Z.greedy(cfg, w, p[:40] + [1, 2], 4)
+    rec = engine(MIX, Z.weights(MIX), ("cpu", torch.float32), max_len=128)
+    q = Z.tokens(MIX, 50)
+    rec.generate_batch([q], max_tokens=2, temperature=0.0)
+    assert rec.generate_batch([q], max_tokens=2, temperature=0.0)[0].telemetry.cached_prefix_tokens == 0
+
+
 def test_refusals_by_name():
     w, mc = Z.weights(MIX), ModelConfig.from_hf_dict(MIX)
     with pytest.raises(ValueError, match="swap_space_pages"):
