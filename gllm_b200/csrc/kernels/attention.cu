@@ -506,6 +506,7 @@ struct DecodeParams {
   int* counters;    // [B, Hkv], zero before the first launch; the kernel leaves them zero
   int num_pages;
   int window;          // 0 = full attention
+  int keep;            // with a window: the first `keep` tokens stay visible
   const float* sinks;  // [Hq] learnable sink logits or null
   float v_scale;       // fp8 cache: value = stored * scale (the K scale is folded into scale_log2)
   int* err;
@@ -539,15 +540,20 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmap_kv, const DecodePar
     ctx = p.max_blocks * kPage;
   }
   const int n_pages = (ctx + kPage - 1) / kPage;
-  const int first_tok = attn_first_key(ctx - 1, p.window);
+  int first_tok = attn_first_key(ctx - 1, p.window);
+  if (p.keep >= first_tok) first_tok = 0;          // the kept tokens reach the window: one range
   const int first_page = first_tok / kPage;
+  // Pages in visiting order: those of the kept tokens [0, keep), then those of the window [first_tok, ctx). A page that
+  // holds tokens of both is visited once for each.
+  const int n_kept = first_tok > 0 ? (p.keep + kPage - 1) / kPage : 0;
   // never more splits than the scratch was sized for: widen the split when the context is long
-  const int span = n_pages - first_page;
+  const int span = n_pages - first_page + n_kept;
   const int pps = max(p.pages_per_split, (span + p.max_splits - 1) / p.max_splits);
   const int n_splits = (span + pps - 1) / pps;
   if (split >= n_splits) return;
-  const int p0 = first_page + split * pps;
-  const int p1 = min(p0 + pps, n_pages);
+  const int p0 = split * pps;
+  const int p1 = min(p0 + pps, span);
+  auto page_of = [&](int i) { return i < n_kept ? i : i - n_kept + first_page; };
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
@@ -594,7 +600,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmap_kv, const DecodePar
     const int i = base + lane;
     int page = 0;
     if (i < n_my) {
-      page = bt[p0 + warp + i * kDecWarps];
+      page = bt[page_of(p0 + warp + i * kDecWarps)];
       if (page < 0 || page >= p.num_pages) {
         if (p.err) atomicCAS(p.err, 0, ERR_BAD_PAGE);
         page = 0;
@@ -620,16 +626,18 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmap_kv, const DecodePar
     const bool got = mbar_wait(&my_bars[stg], (i / kDecStages) & 1, abort_flag, p.err, ERR_TIMEOUT_TMA_FULL);
     if (!__all_sync(0xffffffffu, got)) break;
     const uint32_t kaddr = smem_u32(my_ring + stg * 2 * kTile);
-    const int tok_base = (p0 + warp + i * kDecWarps) * kPage;
+    const int pi = p0 + warp + i * kDecWarps;
+    const int tok_base = page_of(pi) * kPage;
+    const int lo = pi < n_kept ? 0 : first_tok, hi = pi < n_kept ? p.keep : ctx;
     if (swapped) {
       if constexpr (KV8)
-        attend_page_t8(qt, kaddr, kaddr + kTile, tok_base, first_tok, ctx, p.scale_log2,
+        attend_page_t8(qt, kaddr, kaddr + kTile, tok_base, lo, hi, p.scale_log2,
                        *reinterpret_cast<float(*)[8][4]>(&o[0][0]), stt);
       else
-        attend_page_t<kFW>(qt, kaddr, kaddr + kTile, tok_base, first_tok, ctx, p.scale_log2,
+        attend_page_t<kFW>(qt, kaddr, kaddr + kTile, tok_base, lo, hi, p.scale_log2,
                       *reinterpret_cast<float(*)[8][4]>(&o[0][0]), stt);
     } else {
-      attend_page<KV8, kFW>(qf, kaddr, kaddr + kTile, tok_base, first_tok, ctx, first_tok, ctx, p.scale_log2, o, st);
+      attend_page<KV8, kFW>(qf, kaddr, kaddr + kTile, tok_base, lo, hi, lo, hi, p.scale_log2, o, st);
     }
     __syncwarp();
     const int nxt = i + kDecStages;
@@ -951,8 +959,12 @@ template <bool KV8, bool kFW = false>
 static int paged_decode_impl(const void* q, void* out, const void* kv_cache, int num_pages,
                              const int* block_tables, int max_blocks, const int* ctx_lens, int batch,
                              int n_q_heads, int n_kv_heads, float scale, int pages_per_split, int max_splits,
-                             float* scratch, int* counters, int window, const float* sinks, float kv_scale,
+                             float* scratch, int* counters, int window, int keep, const float* sinks, float kv_scale,
                              void* stream) {
+  if (keep > 0 && window < 0) {
+    set_last_error("paged_decode: kept tokens with a chunked mask");
+    return -1;
+  }
   if (n_q_heads % n_kv_heads != 0 || n_q_heads / n_kv_heads > 16) {
     set_last_error("paged_decode: group size %d/%d unsupported (must divide, <= 16)", n_q_heads, n_kv_heads);
     return -1;
@@ -974,7 +986,7 @@ static int paged_decode_impl(const void* q, void* out, const void* kv_cache, int
   p.max_splits = max_splits > 0 ? max_splits : 1;
   p.part_o = scratch;
   p.part_lse = scratch ? scratch + static_cast<long long>(batch) * n_q_heads * p.max_splits * kHD : nullptr;
-  p.counters = counters; p.num_pages = num_pages; p.window = window; p.sinks = sinks;
+  p.counters = counters; p.num_pages = num_pages; p.window = window; p.keep = keep; p.sinks = sinks;
   p.err = gllm_error_word();
   static bool attr_set[64] = {};   // per device: the attribute belongs to the device's copy of the kernel
   int dev = 0;
@@ -992,18 +1004,19 @@ static int paged_decode_impl(const void* q, void* out, const void* kv_cache, int
   return 0;
 }
 
-// full_weights: softmax weights as bf16 pairs in the second product.
+// full_weights: softmax weights as bf16 pairs in the second product. keep: the first `keep` tokens stay visible outside the
+// window.
 GLLM_API int gllm_paged_decode(const void* q, void* out, const void* kv_cache, int num_pages,
                                const int* block_tables, int max_blocks, const int* ctx_lens, int batch,
                                int n_q_heads, int n_kv_heads, float scale, int pages_per_split, int max_splits,
-                               float* scratch, int* counters, int window, const float* sinks, int full_weights,
+                               float* scratch, int* counters, int window, int keep, const float* sinks, int full_weights,
                                void* stream) {
   if (full_weights)
     return paged_decode_impl<false, true>(q, out, kv_cache, num_pages, block_tables, max_blocks, ctx_lens, batch,
                                           n_q_heads, n_kv_heads, scale, pages_per_split, max_splits, scratch, counters,
-                                          window, sinks, 1.f, stream);
+                                          window, keep, sinks, 1.f, stream);
   return paged_decode_impl<false>(q, out, kv_cache, num_pages, block_tables, max_blocks, ctx_lens, batch, n_q_heads,
-                                  n_kv_heads, scale, pages_per_split, max_splits, scratch, counters, window, sinks,
+                                  n_kv_heads, scale, pages_per_split, max_splits, scratch, counters, window, keep, sinks,
                                   1.f, stream);
 }
 // Same kernel over an fp8 (e4m3) cache of the same shape; cached value = stored byte * kv_scale.
@@ -1013,7 +1026,7 @@ GLLM_API int gllm_paged_decode_fp8(const void* q, void* out, const void* kv_cach
                                    float* scratch, int* counters, int window, const float* sinks, float kv_scale,
                                    void* stream) {
   return paged_decode_impl<true>(q, out, kv_cache, num_pages, block_tables, max_blocks, ctx_lens, batch, n_q_heads,
-                                 n_kv_heads, scale, pages_per_split, max_splits, scratch, counters, window, sinks,
+                                 n_kv_heads, scale, pages_per_split, max_splits, scratch, counters, window, 0, sinks,
                                  kv_scale, stream);
 }
 

@@ -1,4 +1,5 @@
-// Paged attention on warp-level tensor cores for head dims other than 128 (any multiple of 16 up to 256), bf16 cache.
+// Paged attention on warp-level tensor cores for head sizes other than 128 (keys and values: any multiples of 8 up to 256),
+// bf16 cache.
 //
 // The rows of a CTA's query tile are (token, query head of one KV head) pairs, so the heads of a group share every K / V
 // tile. K and V come in blocks of 64 tokens through a two-stage cp.async ring. Two forms of one kernel:
@@ -6,7 +7,9 @@
 //   decode    16 rows (a group of at most 16 heads and one token); the four warps share a block's tokens, 16 each, and
 //             merge their partial results at the end
 // Online softmax in the exp2 domain; the weights enter the second product as a bf16 value and its bf16 remainder (16 bits
-// of mantissa). Masks: causal with sliding window or chunks (attn_first_key), or none.
+// of mantissa). Masks: causal with sliding window (and kept first tokens) or chunks (attn_first_key), or none. Blocks outside
+// every row's range are skipped: the kept tokens' blocks come first, then the window's. `sinks`: one more logit per head in
+// the denominator.
 #include "mma.cuh"
 
 namespace gllm {
@@ -21,9 +24,10 @@ struct AmParams {
   const int* block_tables;
   int max_blocks;
   const int *q_start, *q_len, *ctx_lens;   // q_start null: decode, row = sequence index, one token where ctx > 0
-  int n_q, n_kv, group, D;
+  int n_q, n_kv, group, D, DV;
   float scale_log2;
-  int causal, window, num_pages;
+  int causal, window, keep, num_pages;
+  const float* sinks;
   int* err;
 };
 
@@ -38,7 +42,7 @@ __device__ __forceinline__ float am_ex2(float x) {
 
 template <int D16, bool SPLIT>
 __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParams p) {
-  constexpr int DP = D16 * 16, P = DP + 8;                 // padded head dim, bf16 per shared-memory row
+  constexpr int DP = D16 * 16, P = DP + 8;                 // padded head size, bf16 per shared-memory row
   constexpr int RT = SPLIT ? 16 : 64, NT = SPLIT ? 2 : 8;  // rows per CTA, 8-token score tiles per warp and block
   constexpr bool kQReg = D16 <= 8;
   extern __shared__ __align__(16) uint8_t am_smem[];
@@ -61,24 +65,34 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
   const int kv_lo = p.causal ? attn_first_key(pos0 + row0 / p.group, p.window) : attn_first_key(ctx - 1, p.window);
   const int kv_hi = p.causal ? min(ctx, pos0 + last_row / p.group + 1) : ctx;
   const int j0 = kv_lo / kAmTok, j1 = (kv_hi + kAmTok - 1) / kAmTok, n_pages = (ctx + 15) / 16;
+  // blocks in visiting order: those of the kept tokens in front of the window, then the window's
+  const int jk = min((p.keep + kAmTok - 1) / kAmTok, j0), nj = jk + j1 - j0;
+  auto block_of = [&](int i) { return i < jk ? i : j0 + i - jk; };
 
-  if (DP != p.D) {                                         // columns behind the head dim read as zero
-    const int extra = DP - p.D;
-    for (int i = tid; i < 4 * kAmTok * extra; i += kAmThreads) k_s[(i / extra) * P + p.D + i % extra] = __float2bfloat16_rn(0.f);
-  }
+  // columns behind the head size read as zero
+  auto zero_tail = [&](bf16_t* rows, int d) {
+    const int extra = DP - d;
+    for (int i = tid; i < 2 * kAmTok * extra; i += kAmThreads) rows[(i / extra) * P + d + i % extra] = __float2bfloat16_rn(0.f);
+  };
+  if (DP != p.D) zero_tail(k_s, p.D);
+  if (DP != p.DV) zero_tail(v_s, p.DV);
   const int* bt = p.block_tables + static_cast<long long>(seq) * p.max_blocks;
-  const int vecs = p.D / 8;
+  const int kvecs = p.D / 8, vecs = (p.D + p.DV) / 8;
+  const long long page_elems = static_cast<long long>(p.n_kv) * 16 * (p.D + p.DV), v_base = static_cast<long long>(p.n_kv) * 16 * p.D;
   auto load = [&](int j, int stage) {
     for (int i = tid; i < kAmTok * vecs; i += kAmThreads) {
-      const int r = i / vecs, c = (i - r * vecs) * 8, tok = j * kAmTok + r;
+      const int r = i / vecs, c8 = i - r * vecs, tok = j * kAmTok + r;
       int page = bt[min(tok >> 4, n_pages - 1)];
       if (page < 0 || page >= p.num_pages) {
         if (p.err) atomicCAS(p.err, 0, ERR_BAD_PAGE);
         page = 0;
       }
-      const long long o = ((static_cast<long long>(page) * 2 * p.n_kv + kvh) * 16 + (tok & 15)) * p.D + c;
-      cp_async16(k_s + (stage * kAmTok + r) * P + c, p.kv + o);
-      cp_async16(v_s + (stage * kAmTok + r) * P + c, p.kv + o + static_cast<long long>(p.n_kv) * 16 * p.D);
+      const bf16_t* pg = p.kv + page * page_elems;
+      const int row = kvh * 16 + (tok & 15);
+      if (c8 < kvecs) cp_async16(k_s + (stage * kAmTok + r) * P + c8 * 8, pg + static_cast<long long>(row) * p.D + c8 * 8);
+      else
+        cp_async16(v_s + (stage * kAmTok + r) * P + (c8 - kvecs) * 8,
+                   pg + v_base + static_cast<long long>(row) * p.DV + (c8 - kvecs) * 8);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -113,11 +127,11 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
   for (int i = 0; i < 2 * D16; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 
-  load(j0, 0);
-  for (int j = j0; j < j1; ++j) {
-    const int stage = (j - j0) & 1;
-    if (j + 1 < j1) {
-      load(j + 1, stage ^ 1);
+  load(block_of(0), 0);
+  for (int i = 0; i < nj; ++i) {
+    const int j = block_of(i), stage = i & 1;
+    if (i + 1 < nj) {
+      load(block_of(i + 1), stage ^ 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -126,7 +140,8 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
     const int tb = SPLIT ? warp * 16 : 0, tok0 = j * kAmTok + tb;       // this warp's tokens of the block
     const bf16_t* kb = k_s + (stage * kAmTok + tb) * P;
     const bf16_t* vb = v_s + (stage * kAmTok + tb) * P;
-    const bool some = (tok0 < hi[0] && tok0 + NT * 8 > lo[0]) || (tok0 < hi[1] && tok0 + NT * 8 > lo[1]);
+    const bool some = (tok0 < hi[0] && (tok0 + NT * 8 > lo[0] || tok0 < p.keep)) ||
+                      (tok0 < hi[1] && (tok0 + NT * 8 > lo[1] || tok0 < p.keep));
     if (__any_sync(0xffffffffu, some)) {
       float s[NT][4];
 #pragma unroll
@@ -155,7 +170,7 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int r = e >> 1, t = tok0 + nt * 8 + t4 * 2 + (e & 1);
-          const float x = (t >= lo[r] && t < hi[r]) ? s[nt][e] * p.scale_log2 : -INFINITY;
+          const float x = ((t >= lo[r] || t < p.keep) && t < hi[r]) ? s[nt][e] * p.scale_log2 : -INFINITY;
           s[nt][e] = x;
           mx[r] = fmaxf(mx[r], x);
         }
@@ -213,12 +228,17 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
   }
   auto store = [&](int row, int c, float x, float y) {
-    if (row >= qlen * p.group || c >= p.D) return;
+    if (row >= qlen * p.group || c >= p.DV) return;
     const long long t = first + row / p.group;
-    *reinterpret_cast<uint32_t*>(p.out + (t * p.n_q + kvh * p.group + row % p.group) * p.D + c) = pack_bf16x2(x, y);
+    *reinterpret_cast<uint32_t*>(p.out + (t * p.n_q + kvh * p.group + row % p.group) * p.DV + c) = pack_bf16x2(x, y);
+  };
+  // 1 / denominator of a row with maximum M (exp2 domain) and sum L over its keys
+  auto inverse = [&](int row, float M, float L) {
+    if (p.sinks && row < qlen * p.group) L += am_ex2(p.sinks[kvh * p.group + row % p.group] * 1.4426950408889634f - M);
+    return L > 0.f ? 1.f / L : 0.f;
   };
   if constexpr (!SPLIT) {
-    const float i0 = l[0] > 0.f ? 1.f / l[0] : 0.f, i1 = l[1] > 0.f ? 1.f / l[1] : 0.f;
+    const float i0 = inverse(wrow + g, m[0], l[0]), i1 = inverse(wrow + g + 8, m[1], l[1]);
 #pragma unroll
     for (int i = 0; i < 2 * D16; ++i) {
       store(wrow + g, i * 8 + t4 * 2, o[i][0] * i0, o[i][1] * i0);
@@ -242,7 +262,7 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
     __syncthreads();
     for (int i = tid; i < 16 * (DP / 2); i += kAmThreads) {
       const int r = i / (DP / 2), c = (i % (DP / 2)) * 2;
-      if (row0 + r >= qlen * p.group || c >= p.D) continue;
+      if (row0 + r >= qlen * p.group || c >= p.DV) continue;
       float M = -INFINITY;
 #pragma unroll
       for (int w = 0; w < 4; ++w) M = fmaxf(M, ml[(w * 16 + r) * 2]);
@@ -255,7 +275,7 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
         x += f * v.x;
         y += f * v.y;
       }
-      const float inv = L > 0.f ? 1.f / L : 0.f;
+      const float inv = inverse(row0 + r, M, L);
       store(row0 + r, c, x * inv, y * inv);
     }
   }
@@ -287,28 +307,30 @@ static int am_launch(const AmParams& p, dim3 grid, cudaStream_t s) {
   return 0;
 }
 
-// q / out [rows, n_q, D] bf16 contiguous; cache [pages, 2, n_kv, 16, D] bf16; D a multiple of 16, at most 256. q_start null:
-// a decode step (row = sequence index). max_q_len: the longest q_len.
+// q [rows, n_q, D], out [rows, n_q, DV] bf16 contiguous; pages of n_kv x 16 x D keys, then n_kv x 16 x DV values (bf16);
+// D and DV multiples of 8, at most 256. q_start null: a decode step (row = sequence index). max_q_len: the longest q_len.
 GLLM_API int gllm_attention_mma(const void* q, void* out, const void* kv, int num_pages, const int* block_tables,
                                 int max_blocks, const int* q_start, const int* q_len, const int* ctx_lens, int num_seqs,
-                                int max_q_len, int n_q, int n_kv, int D, float scale, int causal, int window, void* stream) {
+                                int max_q_len, int n_q, int n_kv, int D, int DV, float scale, int causal, int window, int keep,
+                                const float* sinks, void* stream) {
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
-  if (D <= 0 || D % 16 != 0 || D > 256 || n_kv <= 0 || n_q % n_kv != 0 || num_seqs > 65535 || n_kv > 65535) {
-    set_last_error("attention_mma: head dim %d, heads %d / %d", D, n_q, n_kv);
+  if (D <= 0 || D % 8 != 0 || D > 256 || DV <= 0 || DV % 8 != 0 || DV > 256 || n_kv <= 0 || n_q % n_kv != 0 ||
+      num_seqs > 65535 || n_kv > 65535 || (keep > 0 && window < 0)) {
+    set_last_error("attention_mma: head sizes %d / %d, heads %d / %d, window %d with %d kept", D, DV, n_q, n_kv, window, keep);
     return -1;
   }
   AmParams p = {};
   p.q = static_cast<const bf16_t*>(q); p.out = static_cast<bf16_t*>(out); p.kv = static_cast<const bf16_t*>(kv);
   p.block_tables = block_tables; p.max_blocks = max_blocks;
   p.q_start = q_start; p.q_len = q_len; p.ctx_lens = ctx_lens;
-  p.n_q = n_q; p.n_kv = n_kv; p.group = n_q / n_kv; p.D = D;
+  p.n_q = n_q; p.n_kv = n_kv; p.group = n_q / n_kv; p.D = D; p.DV = DV;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.causal = causal; p.window = window; p.num_pages = num_pages; p.err = gllm_error_word();
+  p.causal = causal; p.window = window; p.keep = keep; p.sinks = sinks; p.num_pages = num_pages; p.err = gllm_error_word();
   const int rows = max_q_len * p.group;
   const bool split = rows <= 16;
   dim3 grid(split ? 1 : (rows + 63) / 64, n_kv, num_seqs);
   auto s = static_cast<cudaStream_t>(stream);
-  const int d16 = D / 16;
+  const int d16 = ((D > DV ? D : DV) + 15) / 16;
 #define AM_CASE(N) \
   if (d16 <= N) return split ? am_launch<N, true>(p, grid, s) : am_launch<N, false>(p, grid, s)
   AM_CASE(1);

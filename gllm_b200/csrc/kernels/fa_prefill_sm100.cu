@@ -59,6 +59,7 @@ struct FaParams {
   float scale_log2;
   int num_pages;
   int window, causal;
+  int keep;                  // with a window: the first `keep` tokens stay visible
   const float* sinks;
   int* err;
   unsigned long long wait_ns;
@@ -93,7 +94,7 @@ __device__ __forceinline__ uint64_t umma_desc_sw128_mn(uint32_t smem_addr, uint3
   return d;
 }
 
-// KV token range of one query tile: tiles [j0, j1) of 64 tokens.
+// KV token range of one query tile: tiles [j0, j1) of 64 tokens, counted in visiting order (see `kv_tile_of`).
 struct FaTile {
   int head, row0, rows;   // rows = valid query rows (0: the tile does not exist)
   int j0, j1;
@@ -155,6 +156,21 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     ti.j1 = hi / kFaKv + 1;
   }
   if (tile[0].rows == 0) return;   // tile 1 never exists without tile 0
+  // Kept first tokens: their tiles in front of the window are visited first, then the window's; both query tiles take the
+  // window from the earlier start (masked where it is not theirs), so their ranges stay contiguous in visiting order.
+  int n_kept = 0, skipped = 0;
+  if (p.keep > 0) {
+    const int w0 = tile[1].rows ? min(tile[0].j0, tile[1].j0) : tile[0].j0;
+    n_kept = min((p.keep + kFaKv - 1) / kFaKv, w0);
+    skipped = w0 - n_kept;
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+      if (tile[t].rows > 0) {
+        tile[t].j0 = 0;
+        tile[t].j1 -= skipped;
+      }
+  }
+  auto kv_tile_of = [&](int v) { return v < n_kept ? v : v + skipped; };
   const int kvh = tile[0].head / p.group;
   const int J0 = tile[1].rows ? min(tile[0].j0, tile[1].j0) : tile[0].j0;
   const int J1 = tile[1].rows ? max(tile[0].j1, tile[1].j1) : tile[0].j1;
@@ -208,7 +224,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       // finite values), lanes 0..7 issue one box each
       int page = 0;
       if (lane < 4) {
-        const int pi = min(j * 4 + lane, n_pages - 1);
+        const int pi = min(kv_tile_of(j) * 4 + lane, n_pages - 1);
         page = bt[pi];
         if (page < 0 || page >= p.num_pages) {
           if (p.err) atomicCAS(p.err, 0, ERR_BAD_PAGE);
@@ -343,7 +359,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         tmem_ld_32x32(s_addr, sr[0]);
         tmem_ld_32x32(s_addr + 32, sr[1]);
         tmem_ld_wait();
-        const int t0 = j * kFaKv;
+        const int t0 = kv_tile_of(j) * kFaKv;
         const bool full_tile = t0 >= lo && t0 + kFaKv - 1 <= hi;
         float mx = -INFINITY;
 #pragma unroll
@@ -353,7 +369,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
             float x = __uint_as_float(sr[h][i]) * p.scale_log2;
             if (!full_tile) {
               const int tk = t0 + h * 32 + i;
-              if (tk < lo || tk > hi) x = -INFINITY;
+              if ((tk < lo && tk >= p.keep) || tk > hi) x = -INFINITY;
             }
             sr[h][i] = __float_as_uint(x);
             mx = fmaxf(mx, x);
@@ -443,12 +459,16 @@ extern "C" int* gllm_error_word();
 
 // Causal (or bidirectional) flash attention over the paged bf16 KV cache for the query tokens of a prefill step.
 // q / out: [total_tokens, n_q_heads, 128] bf16, contiguous. Same semantics as gllm_paged_prefill. full_weights: softmax
-// weights as bf16 pairs.
+// weights as bf16 pairs; keep: the first `keep` tokens stay visible outside the window.
 GLLM_API int gllm_paged_prefill_tc(const void* q, void* out, const void* kv_cache, int num_pages,
                                    const int* block_tables, int max_blocks, const int* q_start, const int* q_len,
                                    const int* ctx_lens, int num_seqs, int max_q_len, int total_tokens, int n_q_heads,
-                                   int n_kv_heads, float scale, int causal, int window, const float* sinks,
+                                   int n_kv_heads, float scale, int causal, int window, int keep, const float* sinks,
                                    int full_weights, void* stream) {
+  if (keep > 0 && window < 0) {
+    set_last_error("paged_prefill_tc: kept tokens with a chunked mask");
+    return -1;
+  }
   if (n_kv_heads <= 0 || n_q_heads % n_kv_heads != 0 || total_tokens <= 0) {
     set_last_error("paged_prefill_tc: heads %d / kv heads %d / tokens %d", n_q_heads, n_kv_heads, total_tokens);
     return -1;
@@ -470,7 +490,7 @@ GLLM_API int gllm_paged_prefill_tc(const void* q, void* out, const void* kv_cach
   p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads; p.group = n_q_heads / n_kv_heads;
   p.pair_heads = (p.group % 2 == 0) ? 1 : 0;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.num_pages = num_pages; p.window = window; p.causal = causal; p.sinks = sinks;
+  p.num_pages = num_pages; p.window = window; p.keep = keep; p.causal = causal; p.sinks = sinks;
   p.err = gllm_error_word();
   p.wait_ns = static_cast<unsigned long long>(settings().wait_ns);
   auto kern = full_weights ? fa_prefill_kernel<true> : fa_prefill_kernel<false>;

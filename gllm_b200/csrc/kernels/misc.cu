@@ -233,26 +233,16 @@ __global__ void rope_kv_write_kernel(const __nv_bfloat16* qkv, long long ld, int
 }
 
 // ---------------------------------------------------------------------------------------------
-// Generic paged attention (CUDA cores) for head dims other than 128: one warp per (query token, head).
-// Used by small / encoder models; the tensor-core kernels cover head_dim 128.
+// Paged attention over fp8 (e4m3) pages on CUDA cores, any head dim up to 256: one warp per (query token, head). Head dim
+// 128 has tensor-core kernels; bf16 and fp32 pages of other sizes are attention_mma.cu and attention_any.cu.
 // ---------------------------------------------------------------------------------------------
-template <typename T> __device__ __forceinline__ float exp_for(float x) { return __expf(x); }
-template <> __device__ __forceinline__ float exp_for<float>(float x) { return expf(x); }
-
-// T = float: fp32 queries, cache and output, full-precision exponentials.
-template <typename T, bool KV8>
-__global__ void paged_attention_generic_kernel(const T* q, T* out, const void* kv_cache_v, const int* block_tables,
-                                               int max_blocks, const int* q_start, const int* q_len,
-                                               const int* ctx_lens, int n_q, int n_kv, int D, float scale,
-                                               int causal, int window, int num_pages, float kv_scale) {
-  const T* kv_cache = static_cast<const T*>(kv_cache_v);
-  const uint8_t* kv_cache8 = static_cast<const uint8_t*>(kv_cache_v);
+__global__ void paged_attention_fp8kv_kernel(const __nv_bfloat16* q, __nv_bfloat16* out, const uint8_t* kv_cache,
+                                             const int* block_tables, int max_blocks, const int* q_start,
+                                             const int* q_len, const int* ctx_lens, int n_q, int n_kv, int D, float scale,
+                                             int causal, int window, int num_pages, float kv_scale) {
   auto ld_kv = [&](long long eoff) -> float {
-    if (KV8) {
-      const __half_raw h = __nv_cvt_fp8_to_halfraw(kv_cache8[eoff], __NV_E4M3);
-      return __half2float(*reinterpret_cast<const __half*>(&h)) * kv_scale;
-    }
-    return static_cast<float>(kv_cache[eoff]);
+    const __half_raw h = __nv_cvt_fp8_to_halfraw(kv_cache[eoff], __NV_E4M3);
+    return __half2float(*reinterpret_cast<const __half*>(&h)) * kv_scale;
   };
   const int seq = blockIdx.z, head = blockIdx.y;
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -285,7 +275,7 @@ __global__ void paged_attention_generic_kernel(const T* q, T* out, const void* k
     }
     s = warp_sum(s);
     const float mn = fmaxf(mx, s);
-    const float c = exp_for<T>(mx - mn), pnew = exp_for<T>(s - mn);
+    const float c = __expf(mx - mn), pnew = __expf(s - mn);
     l = l * c + pnew;
     for (int i = 0; i < per; ++i) {
       const int d = lane + 32 * i;
@@ -295,7 +285,7 @@ __global__ void paged_attention_generic_kernel(const T* q, T* out, const void* k
   }
   for (int i = 0; i < per; ++i) {
     const int d = lane + 32 * i;
-    if (d < D) out[(static_cast<long long>(tok) * n_q + head) * D + d] = static_cast<T>(l > 0.f ? acc[i] / l : 0.f);
+    if (d < D) out[(static_cast<long long>(tok) * n_q + head) * D + d] = static_cast<__nv_bfloat16>(l > 0.f ? acc[i] / l : 0.f);
   }
 }
 
@@ -681,33 +671,6 @@ GLLM_API int gllm_rope_kv_write_fp8(const void* qkv, long long ld, int M, int n_
   CHECK_LAUNCH("rope_kv_write_fp8");
 }
 
-GLLM_API int gllm_paged_attention_generic(const void* q, void* out, const void* kv_cache, int num_pages,
-                                          const int* block_tables, int max_blocks, const int* q_start,
-                                          const int* q_len, const int* ctx_lens, int num_seqs, int max_q_len,
-                                          int n_q, int n_kv, int D, float scale, int causal, int window,
-                                          void* stream) {
-  if (D > 256) { set_last_error("paged_attention_generic: head_dim %d > 256", D); return -1; }
-  dim3 grid((max_q_len + 3) / 4, n_q, num_seqs);
-  paged_attention_generic_kernel<__nv_bfloat16, false><<<grid, 128, 0, (cudaStream_t)stream>>>(
-      static_cast<const __nv_bfloat16*>(q), static_cast<__nv_bfloat16*>(out), kv_cache, block_tables, max_blocks,
-      q_start, q_len, ctx_lens, n_q, n_kv, D, scale, causal, window, num_pages, 1.0f);
-  CHECK_LAUNCH("paged_attention_generic");
-}
-
-// The same with fp32 queries, cache and output.
-GLLM_API int gllm_paged_attention_f32(const float* q, float* out, const float* kv_cache, int num_pages,
-                                      const int* block_tables, int max_blocks, const int* q_start, const int* q_len,
-                                      const int* ctx_lens, int num_seqs, int max_q_len, int n_q, int n_kv, int D,
-                                      float scale, int causal, int window, void* stream) {
-  if (D > 256) { set_last_error("paged_attention_f32: head_dim %d > 256", D); return -1; }
-  if (num_seqs <= 0 || max_q_len <= 0) return 0;
-  dim3 grid((max_q_len + 3) / 4, n_q, num_seqs);
-  paged_attention_generic_kernel<float, false><<<grid, 128, 0, (cudaStream_t)stream>>>(
-      q, out, kv_cache, block_tables, max_blocks, q_start, q_len, ctx_lens, n_q, n_kv, D, scale, causal, window,
-      num_pages, 1.0f);
-  CHECK_LAUNCH("paged_attention_f32");
-}
-
 // fp8 e4m3 KV cache (value = stored * kv_scale); any head_dim <= 256. Halves the cache footprint and the bytes
 // the attention streams; CUDA-core kernel.
 GLLM_API int gllm_paged_attention_fp8kv(const void* q, void* out, const void* kv_cache, int num_pages,
@@ -718,8 +681,8 @@ GLLM_API int gllm_paged_attention_fp8kv(const void* q, void* out, const void* kv
   if (D > 256) { set_last_error("paged_attention_fp8kv: head_dim %d > 256", D); return -1; }
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
   dim3 grid((max_q_len + 3) / 4, n_q, num_seqs);
-  paged_attention_generic_kernel<__nv_bfloat16, true><<<grid, 128, 0, (cudaStream_t)stream>>>(
-      static_cast<const __nv_bfloat16*>(q), static_cast<__nv_bfloat16*>(out), kv_cache, block_tables, max_blocks,
+  paged_attention_fp8kv_kernel<<<grid, 128, 0, (cudaStream_t)stream>>>(
+      static_cast<const __nv_bfloat16*>(q), static_cast<__nv_bfloat16*>(out), static_cast<const uint8_t*>(kv_cache), block_tables, max_blocks,
       q_start, q_len, ctx_lens, n_q, n_kv, D, scale, causal, window, num_pages, kv_scale);
   CHECK_LAUNCH("paged_attention_fp8kv");
 }

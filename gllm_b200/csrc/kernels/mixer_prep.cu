@@ -1,0 +1,330 @@
+// What lies between a mixer's input projection and its attention:
+//
+//   conv_qkv_prep    causal convolution over time on the projected q, k and v -> RMS norm of each q / k head -> RoPE on the
+//                    first dimensions of q and k -> q buffer, K page, V page; the last projected values enter the ring
+//                    of the sequence's slot. One pass: a warp owns one head's channels over a tile of tokens.
+//   latent_prep      RMS norm of the query latent (operand of the query up-projection) and of the key / value latent
+//                    (written to its page), one warp per token and part.
+//
+// Page layout of a layer with n_kv heads of key size D and value size DV: [n_kv][16][D] then [n_kv][16][DV]; of a latent
+// layer: [16][rank]. The convolution ring is the one of recurrent.cuh. Only the first tile of a sequence reads the ring (a
+// tile has at least taps - 1 tokens) and the same warp then writes it, so the entries need no ordering across CTAs.
+#include "recurrent.cuh"
+
+namespace gllm {
+
+struct ConvPrepParams {
+  SeqView sv;
+  const void* proj;          // [T, ld]: n_q * D q columns, n_kv * D k columns, n_kv * DV v columns
+  long long ld;
+  int n_q, n_kv, D, DV, rot_dim, taps, tile;
+  const float* conv;         // [channels, taps] (taps 0: no convolution)
+  const float *q_w, *k_w;    // [D] or null
+  float eps;
+  const int *positions, *slot_mapping;
+  const float *cos_t, *sin_t;
+  int max_pos;
+  float* ring;               // [slots][taps][channels]
+  void *q_out, *kv;
+  int num_pages;
+  int* err;
+};
+
+constexpr int kPrepWarps = 4;
+
+// VEC consecutive elements per lane and step, N steps; TAPS -1: any number (0: none), weights re-read per token.
+template <typename T, int VEC, int N, int TAPS>
+__global__ void __launch_bounds__(kPrepWarps * 32) conv_qkv_prep_kernel(const ConvPrepParams p) {
+  extern __shared__ float prep_smem[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int unit = blockIdx.x * kPrepWarps + warp;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (unit >= p.n_q + 2 * p.n_kv) return;
+  const SeqRows s = seq_rows(p.sv, blockIdx.z);
+  const int t0 = blockIdx.y * p.tile;
+  const int n = min(p.tile, s.len - t0);
+  if (n <= 0) return;
+  const int kind = unit < p.n_q ? 0 : unit < p.n_q + p.n_kv ? 1 : 2;          // q, k, v
+  const int head = kind == 0 ? unit : kind == 1 ? unit - p.n_q : unit - p.n_q - p.n_kv;
+  const int D = kind == 2 ? p.DV : p.D;
+  const int nq = p.n_q * p.D, nk = p.n_kv * p.D, channels = nq + nk + p.n_kv * p.DV;
+  const int col0 = kind == 0 ? head * p.D : kind == 1 ? nq + head * p.D : nq + nk + head * p.DV;
+  const T* proj = static_cast<const T*>(p.proj);
+  const int taps = TAPS >= 0 ? TAPS : p.taps;
+  float* stage = prep_smem + warp * max(p.D, p.DV);
+  const float* norm_w = kind == 0 ? p.q_w : kind == 1 ? p.k_w : nullptr;
+  const int rot = kind == 2 ? 0 : p.rot_dim, half = rot / 2;
+  auto el = [&](int j) { return (j * 32 + lane) * VEC; };
+  auto load = [&](const T* row, int j, float (&v)[VEC]) {
+    if constexpr (VEC == 2) {
+      if constexpr (sizeof(T) == 2) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + el(j)));
+        v[0] = f.x; v[1] = f.y;
+      } else {
+        const float2 f = *reinterpret_cast<const float2*>(row + el(j));
+        v[0] = f.x; v[1] = f.y;
+      }
+    } else {
+      v[0] = to_f(row[el(j)]);
+    }
+  };
+  constexpr int H = TAPS > 1 ? TAPS - 1 : 1;
+  [[maybe_unused]] float w[TAPS > 0 ? TAPS : 1][N * VEC], hist[H][N * VEC];        // hist[i]: the input i + 1 tokens ago
+  auto from_ring = [&](int pos, int j, int e) { return conv_history(p.ring, s.slot, taps, channels, pos, col0 + el(j) + e); };
+  if constexpr (TAPS > 0) {
+#pragma unroll
+    for (int j = 0; j < N; ++j)
+      if (el(j) < D)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const float* wc = p.conv + static_cast<long long>(col0 + el(j) + e) * TAPS;
+#pragma unroll
+          for (int t = 0; t < TAPS; ++t) w[t][j * VEC + e] = wc[t];
+        }
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i) {
+      const int t = t0 - 1 - i;       // row of the sequence
+#pragma unroll
+      for (int j = 0; j < N; ++j)
+        if (el(j) < D) {
+          float v[VEC];
+          if (t >= 0) {
+            load(proj + static_cast<long long>(s.row0 + t) * p.ld + col0, j, v);
+          } else {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[e] = from_ring(s.start + t, j, e);
+          }
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) hist[i][j * VEC + e] = v[e];
+        }
+    }
+  }
+  for (int t = t0; t < t0 + n; ++t) {
+    const long long m = s.row0 + t;
+    const T* row = proj + m * p.ld + col0;
+    float y[N * VEC];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+      if (el(j) >= D) continue;
+      float u[VEC];
+      load(row, j, u);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const int c = j * VEC + e;
+        float a = u[e];
+        if constexpr (TAPS > 0) {
+          a *= w[TAPS - 1][c];
+#pragma unroll
+          for (int i = 0; i < TAPS - 1; ++i) a = fmaf(w[TAPS - 2 - i][c], hist[i][c], a);
+#pragma unroll
+          for (int i = TAPS - 2; i > 0; --i) hist[i][c] = hist[i - 1][c];
+          if constexpr (TAPS > 1) hist[0][c] = u[e];
+        } else if (taps > 0) {
+          const float* wc = p.conv + static_cast<long long>(col0 + el(j) + e) * taps;
+          a *= wc[taps - 1];
+          for (int i = 1; i < taps; ++i) {
+            const float h = t - i >= 0 ? to_f(proj[(m - i) * p.ld + col0 + el(j) + e]) : from_ring(s.start + t - i, j, e);
+            a = fmaf(wc[taps - 1 - i], h, a);
+          }
+        }
+        y[c] = a;
+        ss += a * a;
+      }
+    }
+    if (norm_w) {
+      const float r = 1.f / sqrtf(warp_sum(ss) / D + p.eps);
+#pragma unroll
+      for (int j = 0; j < N; ++j)
+        if (el(j) < D)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) y[j * VEC + e] *= r * norm_w[el(j) + e];
+    }
+    if (rot > 0) {
+      int pos = p.positions[m];
+      if (pos < 0 || pos >= p.max_pos) {
+        if (p.err && lane == 0) atomicCAS(p.err, 0, ERR_BAD_ARG);
+        pos = 0;
+      }
+      const float* ct = p.cos_t + static_cast<long long>(pos) * half;
+      const float* st = p.sin_t + static_cast<long long>(pos) * half;
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < N; ++j)
+        if (el(j) < D)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) stage[el(j) + e] = y[j * VEC + e];
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < N; ++j)
+        if (el(j) < D)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) {
+            const int d = el(j) + e;
+            if (d < half) y[j * VEC + e] = y[j * VEC + e] * ct[d] - stage[d + half] * st[d];
+            else if (d < rot) y[j * VEC + e] = y[j * VEC + e] * ct[d - half] + stage[d - half] * st[d - half];
+          }
+    }
+    T* dst = nullptr;
+    if (kind == 0) {
+      dst = static_cast<T*>(p.q_out) + m * nq + col0;
+    } else {
+      const int slot = p.slot_mapping ? p.slot_mapping[m] : -1;
+      const int page = slot >= 0 ? slot / 16 : -1;
+      if (page >= p.num_pages) {
+        if (p.err && lane == 0) atomicCAS(p.err, 0, ERR_BAD_PAGE);
+      } else if (page >= 0) {
+        dst = static_cast<T*>(p.kv) + static_cast<long long>(page) * p.n_kv * 16 * (p.D + p.DV) +
+              (kind == 1 ? 0 : static_cast<long long>(p.n_kv) * 16 * p.D) + (static_cast<long long>(head) * 16 + slot % 16) * D;
+      }
+    }
+    if (dst) {
+#pragma unroll
+      for (int j = 0; j < N; ++j)
+        if (el(j) < D) {
+          if constexpr (VEC == 2 && sizeof(T) == 2)
+            *reinterpret_cast<uint32_t*>(dst + el(j)) = pack_bf16x2(y[j * 2], y[j * 2 + 1]);
+          else
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) dst[el(j) + e] = from_f<T>(y[j * VEC + e]);
+        }
+    }
+  }
+  if (taps > 1 && t0 == 0) {
+#pragma unroll
+    for (int j = 0; j < N; ++j)
+      if (el(j) < D)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) advance_conv_ring(s, proj, p.ld, p.ring, channels, taps, col0 + el(j) + e);
+  }
+}
+
+template <typename T>
+static cudaError_t conv_prep_launch(const ConvPrepParams& p, dim3 grid, bool vec, cudaStream_t s) {
+  const int dmax = p.D > p.DV ? p.D : p.DV;
+  const size_t smem = static_cast<size_t>(kPrepWarps) * dmax * sizeof(float);
+#define PREP(V, N, TP) return launch_kernel(conv_qkv_prep_kernel<T, V, N, TP>, grid, dim3(kPrepWarps * 32), smem, s, true, 0, p)
+#define PREP_TAPS(V, N)                  \
+  switch (p.taps) {                      \
+    case 2: PREP(V, N, 2);               \
+    case 3: PREP(V, N, 3);               \
+    case 4: PREP(V, N, 4);               \
+    default: PREP(V, N, -1);             \
+  }
+  if (vec && dmax <= 64) { PREP_TAPS(2, 1) }
+  if (vec && dmax <= 128) { PREP_TAPS(2, 2) }
+  if (vec && dmax <= 256) { PREP_TAPS(2, 4) }
+  PREP(1, 32, -1);
+#undef PREP_TAPS
+#undef PREP
+}
+
+// ---------------------------------------------------------------------------------------------
+// Latent attention: [T, ld] = query latent (q_rank columns) | key / value latent (kv_rank columns).
+// ---------------------------------------------------------------------------------------------
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(128) latent_prep_kernel(const T* proj, long long ld, int M, int q_rank, int kv_rank,
+                                                          const float* q_w, const float* kv_w, float eps, T* cq,
+                                                          const int* slot_mapping, T* cache, int num_pages, int* err) {
+  const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = unit >> 1;
+  const bool is_kv = unit & 1;
+  if (m >= M) return;
+  const int n = is_kv ? kv_rank : q_rank;
+  const T* row = proj + static_cast<long long>(m) * ld + (is_kv ? q_rank : 0);
+  const float* w = is_kv ? kv_w : q_w;
+  T* dst;
+  if (is_kv) {
+    const int slot = slot_mapping ? slot_mapping[m] : -1;
+    if (slot < 0) return;
+    if (slot / 16 >= num_pages) {
+      if (err && lane == 0) atomicCAS(err, 0, ERR_BAD_PAGE);
+      return;
+    }
+    dst = cache + static_cast<long long>(slot) * kv_rank;
+  } else {
+    dst = cq + static_cast<long long>(m) * q_rank;
+  }
+  float ss = 0.f;
+  if constexpr (VEC) {
+    for (int i = lane * 4; i < n; i += 128) {
+      const float4 v = load4(row + i);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int i = lane; i < n; i += 32) ss += to_f(row[i]) * to_f(row[i]);
+  }
+  const float r = 1.f / sqrtf(warp_sum(ss) / n + eps);
+  if constexpr (VEC) {
+    for (int i = lane * 4; i < n; i += 128) {
+      const float4 v = load4(row + i), g = load4(w + i);
+      store4(dst + i, make_float4(v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w));
+    }
+  } else {
+    for (int i = lane; i < n; i += 32) dst[i] = from_f<T>(to_f(row[i]) * r * w[i]);
+  }
+}
+
+}  // namespace gllm
+
+using namespace gllm;
+extern "C" int* gllm_error_word();
+using bf16_t = __nv_bfloat16;
+
+static int prep_done(cudaError_t e, const char* name) {
+  if (e == cudaSuccess) return 0;
+  (void)cudaGetLastError();
+  set_last_error("%s launch: %s", name, cudaGetErrorString(e));
+  return -1;
+}
+
+// q_start null: a decode step (row = slot = sequence index). ring may be null when taps <= 1.
+GLLM_API int gllm_conv_qkv_prep(const int* q_start, const int* q_len, const int* ctx_lens, const int* slots, int n_seqs,
+                                int max_q_len, const void* proj, long long ld, int is_f32, int n_q, int n_kv, int D, int DV,
+                                int rot_dim, int taps, const float* conv, const float* q_w, const float* k_w, float eps,
+                                const int* positions, const int* slot_mapping, const float* cos_t, const float* sin_t,
+                                int max_pos, float* ring, void* q_out, void* kv, int num_pages, void* stream) {
+  if (n_seqs <= 0 || max_q_len <= 0) return 0;
+  if (D <= 0 || DV <= 0 || D > 1024 || DV > 1024 || rot_dim > D || (rot_dim & 1) || (rot_dim > 0 && (!cos_t || !sin_t)) ||
+      taps < 0 || (taps > 0 && !conv) || (taps > 1 && !ring) || n_seqs > 65535) {
+    set_last_error("conv_qkv_prep: sizes %d / %d, rot_dim %d, taps %d, %d sequences", D, DV, rot_dim, taps, n_seqs);
+    return -1;
+  }
+  ConvPrepParams p = {};
+  p.sv = SeqView{q_start, q_len, ctx_lens, slots, n_seqs};
+  p.proj = proj; p.ld = ld; p.n_q = n_q; p.n_kv = n_kv; p.D = D; p.DV = DV; p.rot_dim = rot_dim; p.taps = taps;
+  p.tile = taps - 1 > 8 ? taps - 1 : 8;
+  p.conv = conv; p.q_w = q_w; p.k_w = k_w; p.eps = eps; p.positions = positions; p.slot_mapping = slot_mapping;
+  p.cos_t = cos_t; p.sin_t = sin_t; p.max_pos = max_pos; p.ring = ring; p.q_out = q_out; p.kv = kv;
+  p.num_pages = num_pages; p.err = gllm_error_word();
+  const int rows = q_start ? max_q_len : 1;
+  dim3 grid((n_q + 2 * n_kv + kPrepWarps - 1) / kPrepWarps, (rows + p.tile - 1) / p.tile, n_seqs);
+  if (grid.y > 65535) {
+    set_last_error("conv_qkv_prep: portion of %d tokens", rows);
+    return -1;
+  }
+  const bool vec = D % 2 == 0 && DV % 2 == 0 && ld % 2 == 0;
+  auto s = static_cast<cudaStream_t>(stream);
+  return prep_done(is_f32 ? conv_prep_launch<float>(p, grid, vec, s) : conv_prep_launch<bf16_t>(p, grid, vec, s), "conv_qkv_prep");
+}
+
+GLLM_API int gllm_latent_prep(const void* proj, long long ld, int is_f32, int M, int q_rank, int kv_rank, const float* q_w,
+                              const float* kv_w, float eps, void* cq, const int* slot_mapping, void* cache, int num_pages,
+                              void* stream) {
+  if (M <= 0) return 0;
+  const dim3 grid((2 * M + 3) / 4);
+  const bool vec = q_rank % 4 == 0 && kv_rank % 4 == 0 && ld % 4 == 0;
+  auto s = static_cast<cudaStream_t>(stream);
+  int* err = gllm_error_word();
+  cudaError_t e;
+#define LATENT(T, V)                                                                                                        \
+  e = launch_kernel(latent_prep_kernel<T, V>, grid, dim3(128), 0, s, true, 0, static_cast<const T*>(proj), ld, M, q_rank,   \
+                    kv_rank, q_w, kv_w, eps, static_cast<T*>(cq), slot_mapping, static_cast<T*>(cache), num_pages, err)
+  if (is_f32) { if (vec) LATENT(float, true); else LATENT(float, false); }
+  else { if (vec) LATENT(bf16_t, true); else LATENT(bf16_t, false); }
+#undef LATENT
+  return prep_done(e, "latent_prep");
+}

@@ -10,7 +10,7 @@
 //
 // Everything is sized for the worst case and driven by device-side counts, so the whole MoE layer can
 // sit inside a CUDA graph: no host round trip for the routing decision.
-#include "common.cuh"
+#include "recurrent.cuh"
 
 namespace gllm {
 
@@ -46,7 +46,7 @@ __global__ void moe_route_kernel(const float* logits, long long ld, int T, int E
   } else {  // sigmoid
     for (int i = 0; i < per; ++i) {
       const int e = lane + 32 * i;
-      score[i] = e < E ? 1.f / (1.f + __expf(-score[i])) : 0.f;
+      score[i] = e < E ? 1.f / (1.f + expf(-score[i])) : 0.f;
     }
   }
   for (int i = 0; i < per; ++i) {
@@ -147,13 +147,15 @@ __global__ void moe_plan_kernel(const int* counts, int e_local, int* offsets, in
   }
 }
 
-// One warp per (token, slot): claim a row in the expert's bucket and copy the hidden row there.
-__global__ void moe_scatter_kernel(const __nv_bfloat16* x, const float* row_ss, int ss_parts, const int* ids, int T,
-                                   int k, int hidden, int e0, int e_local, const int* offsets, int* cursors,
-                                   __nv_bfloat16* a_perm, float* ss_perm, int* dest_rows, int max_rows) {
+// One warp per (token, slot): claim a row in the expert's bucket and copy the hidden row there, times the pair's weight
+// when row_w is given (models that weight an expert's input instead of its output).
+template <typename T>
+__global__ void moe_scatter_kernel(const T* x, const float* row_ss, int ss_parts, const int* ids, const float* row_w, int tokens,
+                                   int k, int hidden, int e0, int e_local, const int* offsets, int* cursors, T* a_perm,
+                                   float* ss_perm, int* dest_rows, int max_rows) {
   const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
-  if (w >= T * k) return;
+  if (w >= tokens * k) return;
   const int t = w / k;
   const int e = ids[w] - e0;
   int dest = -1;
@@ -164,9 +166,22 @@ __global__ void moe_scatter_kernel(const __nv_bfloat16* x, const float* row_ss, 
   }
   if (lane == 0) dest_rows[w] = dest;
   if (dest < 0) return;
-  const uint4* src = reinterpret_cast<const uint4*>(x + static_cast<long long>(t) * hidden);
-  uint4* dst = reinterpret_cast<uint4*>(a_perm + static_cast<long long>(dest) * hidden);
-  for (int i = lane; i < hidden / 8; i += 32) dst[i] = src[i];
+  const T* src = x + static_cast<long long>(t) * hidden;
+  T* dst = a_perm + static_cast<long long>(dest) * hidden;
+  constexpr int kVec = 16 / sizeof(T);
+  if (!row_w && hidden % kVec == 0) {
+    for (int i = lane; i < hidden / kVec; i += 32) reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+  } else {
+    const float f = row_w ? row_w[w] : 1.f;
+    if (hidden % 4 == 0) {
+      for (int i = lane * 4; i < hidden; i += 128) {
+        const float4 v = load4(src + i);
+        store4(dst + i, make_float4(v.x * f, v.y * f, v.z * f, v.w * f));
+      }
+    } else {
+      for (int i = lane; i < hidden; i += 32) dst[i] = from_f<T>(to_f(src[i]) * f);
+    }
+  }
   if (ss_perm && lane == 0) {
     float s = 0.f;
     for (int p = 0; p < ss_parts; ++p) s += row_ss[static_cast<long long>(t) * ss_parts + p];
@@ -243,12 +258,13 @@ GLLM_API int gllm_moe_route(const float* logits, long long ld, int T, int E, int
 // Buckets the T*k routed (token, slot) pairs of local experts [e0, e0+e_local) into 128-row blocks.
 // counts / offsets (e_local+1) / cursors / blk_group (2 * max_blocks: experts, then row counts) / total_rows (1) are int32 device
 // buffers; counts must be zero on entry (the call re-zeroes nothing: the caller owns them).
-GLLM_API int gllm_moe_permute(const void* x, const float* row_ss, int ss_parts, const int* ids, int T, int k,
+// row_w: [T, k] factors of the copied rows, or null. is_f32: element type of x and a_perm (bf16 otherwise).
+GLLM_API int gllm_moe_permute(const void* x, int is_f32, const float* row_ss, int ss_parts, const int* ids, const float* row_w, int T, int k,
                               int hidden, int e0, int e_local, int* counts, int* offsets, int* cursors,
                               int* blk_group, int max_blocks, int* total_rows, void* a_perm, float* ss_perm,
                               int* dest_rows, void* stream) {
-  if (e_local > 512 || hidden % 8 != 0) {
-    set_last_error("moe_permute: e_local=%d (max 512), hidden %d must be a multiple of 8", e_local, hidden);
+  if (e_local > 512) {
+    set_last_error("moe_permute: e_local=%d (max 512)", e_local);
     return -1;
   }
   cudaStream_t s = (cudaStream_t)stream;
@@ -260,9 +276,14 @@ GLLM_API int gllm_moe_permute(const void* x, const float* row_ss, int ss_parts, 
   MOE_CHECK("moe_plan");
   const int threads = 256;
   const long long blocks = (static_cast<long long>(n) * 32 + threads - 1) / threads;
-  if (n > 0) moe_scatter_kernel<<<static_cast<unsigned>(blocks), threads, 0, s>>>(
-      static_cast<const __nv_bfloat16*>(x), row_ss, ss_parts, ids, T, k, hidden, e0, e_local, offsets, cursors,
-      static_cast<__nv_bfloat16*>(a_perm), ss_perm, dest_rows, max_blocks * kMoeBlockRows);
+  if (n > 0 && is_f32)
+    moe_scatter_kernel<float><<<static_cast<unsigned>(blocks), threads, 0, s>>>(
+        static_cast<const float*>(x), row_ss, ss_parts, ids, row_w, T, k, hidden, e0, e_local, offsets, cursors,
+        static_cast<float*>(a_perm), ss_perm, dest_rows, max_blocks * kMoeBlockRows);
+  else if (n > 0)
+    moe_scatter_kernel<__nv_bfloat16><<<static_cast<unsigned>(blocks), threads, 0, s>>>(
+        static_cast<const __nv_bfloat16*>(x), row_ss, ss_parts, ids, row_w, T, k, hidden, e0, e_local, offsets, cursors,
+        static_cast<__nv_bfloat16*>(a_perm), ss_perm, dest_rows, max_blocks * kMoeBlockRows);
   MOE_CHECK("moe_scatter");
   return 0;
 }

@@ -1,0 +1,189 @@
+// The step between two sublayers of a sandwich-norm block over a residual stream kept in fp32, one pass per row:
+//
+//   s = sublayer output (a projection's row, or the sum of the row's routed expert outputs)
+//   x += norm(s) * post_w;   x += add;   xb = norm(x) * pre_w      (each part optional)
+//
+// Norms are RMS or layer norms without bias, statistics in fp32; a layer norm takes its variance from the deviations. One
+// CTA per row, the row in registers, one barrier per reduction.
+#include "recurrent.cuh"
+
+namespace gllm {
+
+struct ResidualNormParams {
+  float* x;
+  long long ldx;
+  const void* y;
+  long long ldy;
+  const int* dest;        // [M, top] rows of y to sum (null: row m)
+  int top;
+  const float *post_w, *add, *pre_w;
+  void* xb;
+  long long ldb;
+  int hidden, layer;      // layer 1: layer norm, 0: RMS norm
+  float eps;
+  const int* rows;        // rows of x (then x is only read)
+};
+
+template <int THREADS>
+__device__ __forceinline__ float row_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+#pragma unroll
+  for (int i = 0; i < THREADS / 32; ++i) t += red[i];
+  return t;
+}
+
+// V elements per thread and step (4 needs a hidden size and pitches of multiples of 4), N steps
+template <typename TY, typename TB, int THREADS, int V, int N>
+__global__ void __launch_bounds__(THREADS) residual_norm_kernel(const ResidualNormParams p) {
+  __shared__ float red[4][THREADS / 32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long m = blockIdx.x;
+  const long long src = p.rows ? p.rows[m] : m;
+  float* xr = p.x + src * p.ldx;
+  const int H = p.hidden;
+  float h[N * V];
+  auto idx = [&](int n) { return (n * THREADS + static_cast<int>(threadIdx.x)) * V; };
+  auto load_f = [&](const float* q, int i, float (&o)[V]) {
+    if constexpr (V == 4) {
+      const float4 f = load4(q + i);
+      o[0] = f.x; o[1] = f.y; o[2] = f.z; o[3] = f.w;
+    } else {
+      o[0] = q[i];
+    }
+  };
+  // normalises h in place; which: reduction buffers to use
+  auto normalise = [&](const float* w, int which) {
+    float mean = 0.f;
+    if (p.layer) {
+      float s = 0.f;
+#pragma unroll
+      for (int n = 0; n < N; ++n)
+        if (idx(n) < H)
+#pragma unroll
+          for (int e = 0; e < V; ++e) s += h[n * V + e];
+      mean = row_sum<THREADS>(s, red[which]) / H;
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; ++n)
+      if (idx(n) < H)
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          h[n * V + e] -= mean;
+          ss += h[n * V + e] * h[n * V + e];
+        }
+    const float rs = 1.f / sqrtf(row_sum<THREADS>(ss, red[which + 1]) / H + p.eps);
+#pragma unroll
+    for (int n = 0; n < N; ++n)
+      if (idx(n) < H) {
+        float g[V];
+        load_f(w, idx(n), g);
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[n * V + e] *= rs * g[e];
+      }
+  };
+  if (p.y) {
+    const TY* y = static_cast<const TY*>(p.y);
+#pragma unroll
+    for (int i = 0; i < N * V; ++i) h[i] = 0.f;
+    const int cnt = p.dest ? p.top : 1;
+    for (int j = 0; j < cnt; ++j) {
+      const long long r = p.dest ? p.dest[m * p.top + j] : m;
+      if (r < 0) continue;
+      const TY* yr = y + r * p.ldy;
+#pragma unroll
+      for (int n = 0; n < N; ++n)
+        if (idx(n) < H) {
+          if constexpr (V == 4) {
+            const float4 f = load4(yr + idx(n));
+            h[n * 4] += f.x; h[n * 4 + 1] += f.y; h[n * 4 + 2] += f.z; h[n * 4 + 3] += f.w;
+          } else {
+            h[n] += to_f(yr[idx(n)]);
+          }
+        }
+    }
+    if (p.post_w) normalise(p.post_w, 0);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N * V; ++i) h[i] = 0.f;
+  }
+  const bool write_x = !p.rows && (p.y || p.add);
+#pragma unroll
+  for (int n = 0; n < N; ++n)
+    if (idx(n) < H) {
+      float xv[V];
+      load_f(xr, idx(n), xv);
+#pragma unroll
+      for (int e = 0; e < V; ++e) h[n * V + e] += xv[e];
+      if (p.add) {
+        load_f(p.add, idx(n), xv);
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[n * V + e] += xv[e];
+      }
+      if (write_x) {
+        if constexpr (V == 4) store4(xr + idx(n), make_float4(h[n * 4], h[n * 4 + 1], h[n * 4 + 2], h[n * 4 + 3]));
+        else xr[idx(n)] = h[n];
+      }
+    }
+  if (!p.pre_w) return;
+  normalise(p.pre_w, 2);
+  TB* xb = static_cast<TB*>(p.xb) + m * p.ldb;
+#pragma unroll
+  for (int n = 0; n < N; ++n)
+    if (idx(n) < H) {
+      if constexpr (V == 4) store4(xb + idx(n), make_float4(h[n * 4], h[n * 4 + 1], h[n * 4 + 2], h[n * 4 + 3]));
+      else xb[idx(n)] = from_f<TB>(h[n]);
+    }
+}
+
+template <typename TY, typename TB>
+static cudaError_t residual_norm_launch(const ResidualNormParams& p, int M, bool vec, cudaStream_t s) {
+  const dim3 grid(M);
+  if (vec) {
+    if (p.hidden <= 512) return launch_kernel(residual_norm_kernel<TY, TB, 128, 4, 1>, grid, dim3(128), 0, s, true, 0, p);
+    if (p.hidden <= 1024) return launch_kernel(residual_norm_kernel<TY, TB, 256, 4, 1>, grid, dim3(256), 0, s, true, 0, p);
+    if (p.hidden <= 2048) return launch_kernel(residual_norm_kernel<TY, TB, 256, 4, 2>, grid, dim3(256), 0, s, true, 0, p);
+    if (p.hidden <= 4096) return launch_kernel(residual_norm_kernel<TY, TB, 512, 4, 2>, grid, dim3(512), 0, s, true, 0, p);
+    return launch_kernel(residual_norm_kernel<TY, TB, 512, 4, 8>, grid, dim3(512), 0, s, true, 0, p);
+  }
+  if (p.hidden <= 1024) return launch_kernel(residual_norm_kernel<TY, TB, 256, 1, 4>, grid, dim3(256), 0, s, true, 0, p);
+  return launch_kernel(residual_norm_kernel<TY, TB, 512, 1, 32>, grid, dim3(512), 0, s, true, 0, p);
+}
+
+}  // namespace gllm
+
+using namespace gllm;
+
+GLLM_API int gllm_residual_norm(float* x, long long ldx, const void* y, long long ldy, int y_f32, const int* dest, int top,
+                                const float* post_w, const float* add, const float* pre_w, void* xb, int xb_f32, int M,
+                                int hidden, int layer, float eps, const int* rows, int ldb, void* stream) {
+  if (M <= 0) return 0;
+  if (hidden <= 0 || hidden > 16384 || (rows && y) || (pre_w && !xb) || (dest && top <= 0)) {
+    set_last_error("residual_norm: hidden %d (at most 16384), rows with y, or a missing output", hidden);
+    return -1;
+  }
+  ResidualNormParams p = {};
+  p.x = x; p.ldx = ldx; p.y = y; p.ldy = ldy; p.dest = dest; p.top = top;
+  p.post_w = post_w; p.add = add; p.pre_w = pre_w; p.xb = xb; p.ldb = ldb;
+  p.hidden = hidden; p.layer = layer; p.eps = eps; p.rows = rows;
+  const auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = hidden % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && ldb % 4 == 0 && aligned(x) && aligned(y) &&
+                   aligned(xb) && aligned(post_w) && aligned(add) && aligned(pre_w);
+  auto s = static_cast<cudaStream_t>(stream);
+  cudaError_t e;
+  using bf16_t = __nv_bfloat16;
+  if (y_f32 && xb_f32) e = residual_norm_launch<float, float>(p, M, vec, s);
+  else if (y_f32) e = residual_norm_launch<float, bf16_t>(p, M, vec, s);
+  else if (xb_f32) e = residual_norm_launch<bf16_t, float>(p, M, vec, s);
+  else e = residual_norm_launch<bf16_t, bf16_t>(p, M, vec, s);
+  if (e != cudaSuccess) {
+    (void)cudaGetLastError();
+    set_last_error("residual_norm launch: %s", cudaGetErrorString(e));
+    return -1;
+  }
+  return 0;
+}

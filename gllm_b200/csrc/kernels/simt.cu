@@ -22,15 +22,24 @@ __device__ __forceinline__ float block_reduce_sum(float v, float* red) {
 }
 
 // ---------------------------------------------------------------------------------------------
-// C[M, N] = A[M, K] B[N, K]^T (+ bias, soft cap): 64 x 64 tiles, 4 x 4 outputs per thread, fp32 FMAs.
+// C[M, N] = A[M, K] B[N, K]^T (+ bias, soft cap): 64 x 64 tiles, 4 x 4 outputs per thread, fp32 FMAs. With `groups`, the 128-row
+// block i of A multiplies the groups[i]-th [N, K] matrix of the stack B (negative: nothing), and only its first
+// block_rows[i] rows are there.
 // ---------------------------------------------------------------------------------------------
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const TI* A, long long lda, const TI* B, long long ldb, TO* C,
                                                         long long ldc, int M, int N, int K, const float* bias,
-                                                        float softcap) {
+                                                        float softcap, const int* groups, const int* block_rows) {
   constexpr int BK = 16;
   __shared__ float As[BK][68], Bs[BK][68];
   const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  if (groups) {
+    const int g = groups[m0 / 128];
+    if (g < 0) return;
+    B += static_cast<long long>(g) * N * ldb;
+    if (block_rows) M = min(M, m0 / 128 * 128 + block_rows[m0 / 128]);
+    if (m0 >= M) return;
+  }
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   const int lr = threadIdx.x >> 4, lk = threadIdx.x & 15;     // rows lr, lr + 16, ... of the tile, column lk
   float acc[4][4] = {};
@@ -151,8 +160,8 @@ __global__ void __launch_bounds__(256) scaled_add_norm_kernel(const float* x, lo
 // act(gate) * up in fp32 (the bf16 form is glu_kernel): gu [M, 2 I] = gate | up. act: 0 silu, 1 gelu_tanh.
 // ---------------------------------------------------------------------------------------------
 __global__ void glu_f32_kernel(const float* gu, long long ld, int inter, int act, float* out) {
-  const long long m = blockIdx.y;
-  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  const long long m = blockIdx.x;
+  const int i = blockIdx.y * blockDim.x + threadIdx.x;
   if (i >= inter) return;
   const float g = gu[m * ld + i], u = gu[m * ld + inter + i];
   float a;
@@ -280,30 +289,39 @@ extern "C" int* gllm_error_word();
 
 using bf16_t = __nv_bfloat16;
 
-// in_f32 / out_f32: element types of A and B / of C (bf16 otherwise).
-GLLM_API int gllm_gemm_simt(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M,
-                            int N, int K, int in_f32, int out_f32, const float* bias, float softcap, void* stream) {
+static int gemm_simt(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M, int N, int K,
+                     int in_f32, int out_f32, const float* bias, float softcap, const int* groups, const int* block_rows,
+                     void* stream) {
   if (M <= 0 || N <= 0 || K <= 0 || (M + 63) / 64 > 65535) {
     set_last_error("gemm_simt: bad problem M=%d N=%d K=%d", M, N, K);
     return -1;
   }
   dim3 grid((N + 63) / 64, (M + 63) / 64);
   auto s = static_cast<cudaStream_t>(stream);
-  if (in_f32 && out_f32)
-    gemm_simt_kernel<float, float><<<grid, 256, 0, s>>>(static_cast<const float*>(A), lda, static_cast<const float*>(B),
-                                                        ldb, static_cast<float*>(C), ldc, M, N, K, bias, softcap);
-  else if (in_f32)
-    gemm_simt_kernel<float, bf16_t><<<grid, 256, 0, s>>>(static_cast<const float*>(A), lda, static_cast<const float*>(B),
-                                                         ldb, static_cast<bf16_t*>(C), ldc, M, N, K, bias, softcap);
-  else if (out_f32)
-    gemm_simt_kernel<bf16_t, float><<<grid, 256, 0, s>>>(static_cast<const bf16_t*>(A), lda,
-                                                         static_cast<const bf16_t*>(B), ldb, static_cast<float*>(C), ldc,
-                                                         M, N, K, bias, softcap);
-  else
-    gemm_simt_kernel<bf16_t, bf16_t><<<grid, 256, 0, s>>>(static_cast<const bf16_t*>(A), lda,
-                                                          static_cast<const bf16_t*>(B), ldb, static_cast<bf16_t*>(C),
-                                                          ldc, M, N, K, bias, softcap);
+  auto run = [&](auto in, auto out) {
+    using TI = decltype(in);
+    using TO = decltype(out);
+    gemm_simt_kernel<TI, TO><<<grid, 256, 0, s>>>(static_cast<const TI*>(A), lda, static_cast<const TI*>(B), ldb,
+                                                  static_cast<TO*>(C), ldc, M, N, K, bias, softcap, groups, block_rows);
+  };
+  if (in_f32 && out_f32) run(float{}, float{});
+  else if (in_f32) run(float{}, bf16_t{});
+  else if (out_f32) run(bf16_t{}, float{});
+  else run(bf16_t{}, bf16_t{});
   SIMT_CHECK("gemm_simt");
+}
+
+// in_f32 / out_f32: element types of A and B / of C (bf16 otherwise).
+GLLM_API int gllm_gemm_simt(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M,
+                            int N, int K, int in_f32, int out_f32, const float* bias, float softcap, void* stream) {
+  return gemm_simt(A, lda, B, ldb, C, ldc, M, N, K, in_f32, out_f32, bias, softcap, nullptr, nullptr, stream);
+}
+
+// Grouped form: groups [M / 128] int32, block_rows [M / 128] int32 or null.
+GLLM_API int gllm_gemm_simt_grouped(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M,
+                                    int N, int K, int in_f32, int out_f32, const int* groups, const int* block_rows,
+                                    void* stream) {
+  return gemm_simt(A, lda, B, ldb, C, ldc, M, N, K, in_f32, out_f32, nullptr, 0.f, groups, block_rows, stream);
 }
 
 GLLM_API int gllm_embed_rows(const int* ids, const void* table, int vocab, int hidden, int is_f32, float* x, void* xb,
@@ -353,8 +371,8 @@ GLLM_API int gllm_scaled_add_norm(const float* x, long long ldx, const void* y, 
 
 GLLM_API int gllm_glu_f32(const float* gu, long long ld, int M, int inter, int act, float* out, void* stream) {
   if (M <= 0) return 0;
-  if (M > 65535 || act < 0 || act > 1) { set_last_error("glu_f32: rows %d / act %d", M, act); return -1; }
-  dim3 grid((inter + 255) / 256, M);
+  if (act < 0 || act > 1) { set_last_error("glu_f32: act %d", act); return -1; }
+  dim3 grid(M, (inter + 255) / 256);
   glu_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(gu, ld, inter, act, out);
   SIMT_CHECK("glu_f32");
 }

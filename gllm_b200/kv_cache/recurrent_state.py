@@ -25,3 +25,14 @@ class RecurrentState:
     @property
     def nbytes(self) -> int:
         return sum(t.numel() * 4 for t in self.t.values())
+
+
+class PagedWithState:
+    """Cache of a layer that has both: paged K / V and a recurrent state (attention behind a short convolution)."""
+
+    def __init__(self, pages: torch.Tensor, state: RecurrentState):
+        self.pages, self.state = pages, state
+
+    @property
+    def nbytes(self) -> int:
+        return self.pages.numel() * self.pages.element_size() + self.state.nbytes

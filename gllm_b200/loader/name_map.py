@@ -51,6 +51,7 @@ class TensorRole(str, Enum):
     MOE_SHARED_DOWN = "moe_shared_down"
     MIXER = "mixer"                # tensor of a token mixer (heterogeneous models: models/hybrid.py)
     MIXER_NORM = "mixer_norm"
+    LOOP_STEP = "loop_step"        # vector added to the residual stream before each pass of a looped range of layers
     CLASSIFIER = "classifier"
     POOLER = "pooler"
     UNKNOWN = "unknown"
@@ -109,10 +110,13 @@ _GLOBAL_RULES = [
 ]
 _GLOBAL_RULES = [(re.compile(p), c, r) for p, c, r in _GLOBAL_RULES]
 
-# Heterogeneous models (Zenevik): ``l<i>.mix.<name>``, ``l<i>.mlp.<name>``, ``l<i>.norm1|2``, ``embed``, ``head``, ``final.norm``
-_HYBRID_LAYER = re.compile(r"^l(\d+)\.(mix\.[\w.]+|mlp\.(?:gate|up|down)|norm[12])$")
+# Heterogeneous models: ``l<i>.mix.<name>``, ``l<i>.mlp.<name>`` (``mlp.e<j>.<name>``, ``mlp.router`` with experts),
+# ``l<i>.norm1|2`` (and ``norm1b|2b`` behind the sublayers), ``embed``, ``head``, ``final.norm``, ``loop.step``
+_HYBRID_LAYER = re.compile(r"^l(\d+)\.(mix\.[\w.]+|mlp\.(?:gate|up|down|router)|mlp\.e\d+\.(?:gate|up|down)|norm[12]b?)$")
 _HYBRID_GLOBAL = {"embed": ("embed_tokens", TensorRole.EMBEDDING), "head": ("lm_head", TensorRole.OUTPUT_HEAD),
-                  "final.norm": ("final_norm", TensorRole.FINAL_NORM)}
+                  "final.norm": ("final_norm", TensorRole.FINAL_NORM), "loop.step": ("loop_step", TensorRole.LOOP_STEP)}
+_HYBRID_MLP = {"gate": TensorRole.FFN_GATE, "up": TensorRole.FFN_UP, "down": TensorRole.FFN_DOWN, "router": TensorRole.MOE_ROUTER}
+_HYBRID_EXPERT = {"gate": TensorRole.MOE_EXPERT_GATE, "up": TensorRole.MOE_EXPERT_UP, "down": TensorRole.MOE_EXPERT_DOWN}
 
 _LAYER_PREFIX = re.compile(r"^(?:model\.|language_model\.|text_model\.|transformer\.|bert\.|roberta\.|encoder\.)*(?:layers|h|layer|blocks|blk|encoder\.layer)\.(\d+)\.(.+)$")
 # tensors of a multimodal checkpoint's towers and projectors are not the language model's: they have their own loaders
@@ -142,7 +146,7 @@ def match_tensor_role(name: str) -> Tuple[TensorRole, Optional[int], Optional[st
     if m:
         rest = m.group(2)
         role = TensorRole.MIXER if rest.startswith("mix.") else TensorRole.MIXER_NORM if rest.startswith("norm") else \
-            {"gate": TensorRole.FFN_GATE, "up": TensorRole.FFN_UP, "down": TensorRole.FFN_DOWN}[rest.split(".")[1]]
+            (_HYBRID_EXPERT if rest.count(".") == 2 else _HYBRID_MLP)[rest.rsplit(".", 1)[1]]
         return role, int(m.group(1)), f"L{m.group(1)}.{rest}", ""
     stem, suffix = split_suffix(name)
     if _NOT_LANGUAGE.search(name):

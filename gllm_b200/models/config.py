@@ -36,9 +36,15 @@ class RopeScaling:
 class MixerSpec:
     """Token mixer of one layer of a heterogeneous model (``ModelConfig.layer_specs``).
 
-    attention: ``heads`` query and ``kv_heads`` key / value heads of size ``dim``, rotary on the first ``rot_dim``
-               dimensions, ``chunk`` > 0 = chunked mask (keys of the query's own chunk of that many positions),
-               ``row_qk_norm`` = RMS norm over the whole q / k projection, ``v_from_k`` = values are the projected keys.
+    attention: ``heads`` query and ``kv_heads`` key / value heads of size ``dim`` (values: ``vdim``), rotary on the first
+               ``rot_dim`` dimensions; ``chunk`` > 0 = chunked mask (keys of the query's own chunk of that many positions),
+               ``window`` > 0 = the last ``window`` keys and the first ``keep_first`` of the sequence; ``row_qk_norm`` = RMS
+               norm over the whole q / k projection, ``head_qk_norm`` = over each head; ``v_from_k`` = values are the
+               projected keys; ``taps`` > 0 = causal convolution over time on q, k and v (before norm and rotation);
+               ``o_bias`` = the output projection has a bias (q, k and v always do).
+    latent:    attention over a shared latent of ``kv_rank`` channels per token, no positions: ``heads`` heads of ``dim`` query /
+               key and ``vdim`` value dimensions, queries of rank ``q_rank``, sliding ``window``, ``sink`` = a learned extra
+               logit per head in the softmax denominator.
     rglru:     real-gated linear recurrent unit over ``width`` channels, gates in ``blocks`` diagonal blocks, behind a
                causal convolution of ``taps`` taps.
     gla:       gated linear attention, ``heads`` x (``dim`` key, ``vdim`` value) channels, decay sigmoid(z)^(1 / tau)
@@ -59,9 +65,22 @@ class MixerSpec:
     taps: int = 0
     tau: float = 1.0
     decay_rank: int = 0
+    window: int = 0
+    keep_first: int = 0
+    head_qk_norm: bool = False
+    o_bias: bool = True
+    q_rank: int = 0
+    kv_rank: int = 0
+    sink: bool = False
+
+    @property
+    def value_dim(self) -> int:
+        return self.vdim or self.dim
 
     def state_floats(self) -> int:
         """fp32 words of recurrent state per sequence."""
+        if self.kind == "attention":
+            return self.taps * ((self.heads + self.kv_heads) * self.dim + self.kv_heads * self.value_dim)
         if self.kind == "rglru":
             return self.width * (self.taps + 1)
         if self.kind == "gla":
@@ -70,7 +89,22 @@ class MixerSpec:
 
     def kv_elems(self) -> int:
         """KV cache elements per token."""
-        return 2 * self.kv_heads * self.dim if self.kind == "attention" else 0
+        if self.kind == "latent":
+            return self.kv_rank
+        return self.kv_heads * (self.dim + self.value_dim) if self.kind == "attention" else 0
+
+
+@dataclass
+class MoeSpec:
+    """Mixture-of-experts feed-forward of one layer: ``top`` of ``experts`` gated feed-forwards of intermediate size ``ff``.
+    ``scoring``: sigmoid or softmax over the router logits; ``norm_topk``: the chosen scores are renormalised to sum 1;
+    ``scale_input``: the score multiplies the expert's input instead of its output."""
+    experts: int
+    top: int
+    ff: int
+    scoring: str = "softmax"
+    norm_topk: bool = True
+    scale_input: bool = False
 
 
 @dataclass
@@ -78,6 +112,7 @@ class LayerSpec:
     mixer: MixerSpec
     ff: int = 0             # intermediate size of the gated feed-forward, 0 = none
     act: str = "gelu_tanh"
+    moe: Optional[MoeSpec] = None
 
 
 @dataclass
@@ -120,9 +155,14 @@ class ModelConfig:
     logit_softcap: float = 0.0
     attn_scale: float = 0.0  # 0 -> 1/sqrt(head_dim)
     post_norm: bool = False  # encoder-style post-LN residual blocks
-    # Heterogeneous decoders (models/hybrid.py): one spec per layer; post-norm blocks x = norm(postln_alpha * x + f(x))
+    # Heterogeneous decoders (models/hybrid.py): one spec per layer. ``block``: "post" = post-norm blocks
+    # x = norm(postln_alpha * x + f(x)), "sandwich" = x = x + norm_b(f(norm_a(x))); ``norm_type`` rms or layer (no bias).
+    # ``loop`` = (start, stop, times): that range of layers runs ``times`` times in a row with the same weights, a learned
+    # vector added to the stream before each pass; every pass has its own cache and state.
     layer_specs: Optional[List[LayerSpec]] = None
     postln_alpha: float = 1.0
+    block: str = "post"
+    loop: Optional[tuple] = None
     causal: bool = True
     # MoE
     num_experts: int = 0
@@ -204,6 +244,18 @@ class ModelConfig:
     def has_recurrent_state(self) -> bool:
         return self.is_hybrid and any(l.mixer.state_floats() for l in self.layer_specs)
 
+    def layer_runs(self) -> List[tuple]:
+        """The layers of a heterogeneous model in the order they run: (layer, number of the pass that starts right before
+        it, or None)."""
+        n = len(self.layer_specs)
+        start, stop, times = self.loop or (0, 0, 0)
+        if stop <= start or times <= 0:
+            start, stop, times = n, n, 0
+        runs = [(i, None) for i in range(start)]
+        for t in range(times):
+            runs += [(i, t if i == start else None) for i in range(start, stop)]
+        return runs + [(i, None) for i in range(stop, n)]
+
     def layer_is_moe(self, layer: int) -> bool:
         return self.is_moe and layer >= self.first_k_dense and (layer % max(self.moe_layer_freq, 1) == 0
                                                                  or self.moe_layer_freq <= 1)
@@ -251,12 +303,17 @@ class ModelConfig:
             for l in self.layer_specs:
                 m = l.mixer
                 if m.kind == "attention":
-                    total += h * (2 * m.heads + m.kv_heads * (1 if m.v_from_k else 2)) * m.dim
+                    total += h * ((m.heads + m.kv_heads) * m.dim + (m.heads + (0 if m.v_from_k else m.kv_heads)) * m.value_dim)
+                elif m.kind == "latent":
+                    total += h * (m.q_rank + m.kv_rank + m.heads * m.vdim) + m.heads * (
+                        m.q_rank * m.dim + m.kv_rank * (m.dim + m.vdim))
                 elif m.kind == "rglru":
                     total += 3 * h * m.width + 2 * m.width * m.width // m.blocks
                 else:
                     total += h * m.heads * (2 * m.dim + 3 * m.vdim) + m.decay_rank * (h + m.heads * m.dim)
                 total += 3 * h * l.ff
+                if l.moe:
+                    total += h * l.moe.experts * (3 * l.moe.ff + 1)
             return total
         attn = h * (self.q_size + 2 * self.kv_size) + self.q_size * h
         if self.is_mla:
@@ -279,7 +336,7 @@ class ModelConfig:
     def kv_bytes_per_token(self, tp: int = 1) -> int:
         esz = 1 if self.kv_cache_dtype in ("fp8", "fp8_e4m3") else 2
         if self.is_hybrid:
-            return sum(l.mixer.kv_elems() for l in self.layer_specs) * esz
+            return sum(self.layer_specs[i].mixer.kv_elems() for i, _ in self.layer_runs()) * esz
         if self.is_mla:
             return self.num_layers * (self.kv_lora_rank + self.qk_rope_head_dim) * esz
         return self.num_layers * 2 * max(1, self.num_kv_heads // tp) * self.head_dim * esz
@@ -293,6 +350,8 @@ class ModelConfig:
         """HF ``config.json`` -> ModelConfig (keys per the reference's field registry)."""
         if d.get("architecture") == "Zenevik":
             return ModelConfig.from_zenevik_dict(d)
+        if d.get("architecture") == "Gorulorn":
+            return ModelConfig.from_gorulorn_dict(d)
         tc = d.get("text_config") or d
         arch = (d.get("model_type") or tc.get("model_type") or "llama").lower()
         g = lambda *keys, default=None: next((tc[k] for k in keys if k in tc and tc[k] is not None), default)
@@ -413,15 +472,48 @@ class ModelConfig:
         cfg.set_hybrid_dims()
         return cfg
 
+    @staticmethod
+    def from_gorulorn_dict(d: Dict[str, Any]) -> "ModelConfig":
+        """Gorulorn ``config.json``: sandwich-norm layers of windowed attention behind a short convolution or of windowed
+        latent attention, sparse feed-forwards, a range of layers that runs several times."""
+        specs = []
+        for i, l in enumerate(d["layers"]):
+            m, kind = l["mixer"], l["type"]
+            mask, rot, mlp = m.get("mask") or {}, m.get("rot") or {}, l.get("mlp")
+            size = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
+                        window=int(mask.get("size") or 0))
+            if kind == "attention":
+                mixer = MixerSpec("attention", kv_heads=int(m["kv_heads"]), rot_dim=int(rot.get("dims") or 0),
+                                  rot_base=float(rot.get("base", 10000.0)), keep_first=int(mask.get("keep_first") or 0),
+                                  taps=int(m.get("conv") or 0), head_qk_norm=True, o_bias=False, **size)
+            elif kind == "latent_attention":
+                mixer = MixerSpec("latent", q_rank=int(m["q_rank"]), kv_rank=int(m["kv_rank"]), sink=True, **size)
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            moe = None
+            if mlp is not None:
+                if mlp.get("kind", "moe") != "moe":
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+                moe = MoeSpec(experts=int(mlp["router"]["experts"]), top=int(mlp["router"]["top"]), ff=int(mlp["expert"]["ff"]),
+                              scoring="sigmoid", norm_topk=False, scale_input=True)
+            specs.append(LayerSpec(mixer, act="silu", moe=moe))
+        loop = d.get("loop")
+        cfg = ModelConfig(arch="gorulorn", hidden_size=int(d["width"]), num_layers=len(specs), vocab_size=int(d["vocab"]),
+                          rms_norm_eps=float(d["norm"]["eps"]), norm_type="layer", block="sandwich", hidden_act="silu",
+                          loop=(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None,
+                          max_position_embeddings=int(d.get("max_positions", 1 << 20)), layer_specs=specs)
+        cfg.set_hybrid_dims()
+        return cfg
+
     def set_hybrid_dims(self):
         """The scalar head / feed-forward sizes of a heterogeneous model: the largest over its layers (they size shared
         buffers; the layers use their specs). ``head_dim`` is 128 when any layer can use the head_dim-128 kernels."""
         att = [l.mixer for l in self.layer_specs if l.mixer.kind == "attention"]
         self.num_heads = max([m.heads for m in att], default=1)
         self.num_kv_heads = max([m.kv_heads for m in att], default=1)
-        dims = [m.dim for m in att] or [64]
+        dims = [m.dim for m in att if m.value_dim == m.dim] or [64]
         self.head_dim = 128 if 128 in dims else max(dims)
-        self.intermediate_size = max([l.ff for l in self.layer_specs] + [0])
+        self.intermediate_size = max([max(l.ff, l.moe.ff if l.moe else 0) for l in self.layer_specs] + [0])
 
     @staticmethod
     def from_json_file(path) -> "ModelConfig":
@@ -533,6 +625,17 @@ def preset(name: str) -> ModelConfig:
         cfg = ModelConfig(arch="zenevik", hidden_size=256, num_layers=3, vocab_size=1024, rms_norm_eps=1e-6,
                           postln_alpha=1.5, logit_softcap=20.0, hidden_act="gelu_tanh", max_position_embeddings=2048,
                           layer_specs=[LayerSpec(att, ff=512), LayerSpec(lru), LayerSpec(gla, ff=256)], eos_token_ids=[2])
+        cfg.set_hybrid_dims()
+        return cfg
+    if n in ("tiny-gorulorn",):
+        att = MixerSpec("attention", heads=4, kv_heads=2, dim=128, vdim=128, scale=0.09, rot_dim=48, rot_base=1000.0, window=50,
+                        keep_first=6, taps=4, head_qk_norm=True, o_bias=False)
+        lat = MixerSpec("latent", heads=3, dim=48, vdim=80, q_rank=96, kv_rank=160, scale=0.15, window=70, sink=True)
+        moe = MoeSpec(experts=9, top=2, ff=96, scoring="sigmoid", norm_topk=False, scale_input=True)
+        cfg = ModelConfig(arch="gorulorn", hidden_size=192, num_layers=3, vocab_size=1024, rms_norm_eps=1e-6, norm_type="layer",
+                          block="sandwich", loop=(1, 3, 2), hidden_act="silu", max_position_embeddings=2048,
+                          layer_specs=[LayerSpec(att, act="silu", moe=moe), LayerSpec(lat, act="silu", moe=moe),
+                                       LayerSpec(att, act="silu")], eos_token_ids=[2])
         cfg.set_hybrid_dims()
         return cfg
     if n in ("tiny-bert",):

@@ -1,11 +1,16 @@
-"""Heterogeneous decoders: every layer has its own token mixer (``models/mixers.py``) and an optional gated feed-forward,
-in post-norm blocks over a residual stream kept in fp32:
+"""Heterogeneous decoders: every layer has its own token mixer (``models/mixers.py``) and an optional feed-forward (gated, or
+a mixture of experts: ``models/moe.py::ExpertFF``), over a residual stream kept in fp32. Two kinds of block:
 
-    x = norm1(alpha * x + mixer(x));   x = norm2(alpha * x + ff(x))
+    post      x = norm1(alpha * x + mixer(x));         x = norm2(alpha * x + ff(x))
+    sandwich  x = x + norm1b(mixer(norm1(x)));         x = x + norm2b(ff(norm2(x)))
+
+A range of layers may run several times in a row with the same weights; a learned vector joins the stream before each pass,
+and each pass has its own cache and state (``ModelConfig.layer_runs``: "run" below is one execution of a layer).
 
 The model plugs into the engine like ``DecoderModel``: same ``ForwardBatch``, paged KV cache for its attention layers, and
-recurrent state in the batcher's sequence slots (``kv_cache/recurrent_state.py``) for the others. Two copies of the stream
-live in the workspace: ``x`` in fp32 (the residual sum and its norms) and ``xb`` in the compute dtype (the GEMM operand).
+recurrent state in the batcher's sequence slots (``kv_cache/recurrent_state.py``) for the others. The workspace holds the
+stream ``x`` in fp32 (the residual sum and its norms) and ``xb``, the next GEMM's operand in the compute dtype: the stream
+itself in post-norm blocks, its normalised rows in sandwich blocks.
 
 dtype bfloat16: tensor-core GEMMs with fp32 accumulation; positions, attention scores and weights, norms, gates, decays
 and states in fp32. dtype float32: every operation in true 32-bit arithmetic.
@@ -21,13 +26,15 @@ from .. import ops
 from ..engine.batch import ForwardBatch
 from ..ops import linear as L
 from ..ops import recurrent as R
+from ..ops.residual import residual_norm
 from .config import ModelConfig
 from .mixers import MIXERS, ROW_PAD, mixer_shapes, rope_table
+from .moe import ExpertFF
 from .weights import glu_tile_width, layer_prefix
 
 
 def is_norm_weight(name: str) -> bool:
-    return name.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2", "final_norm")
+    return name.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2", "norm1b", "norm2b", "final_norm")
 
 
 def tensor_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:
@@ -37,14 +44,23 @@ def tensor_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:
         return cached
     H = cfg.hidden_size
     s = {"embed_tokens": (cfg.vocab_size, H), "lm_head": (cfg.vocab_size, H), "final_norm": (H,)}
+    norms = ("", "b") if cfg.block == "sandwich" else ("",)
+    if cfg.loop:
+        s["loop_step"] = (cfg.loop[2], H)
     for i, l in enumerate(cfg.layer_specs):
         p = layer_prefix(i)
-        s[p + "norm1"] = (H,)
+        s.update({f"{p}norm1{b}": (H,) for b in norms})
         for n, shape in mixer_shapes(l.mixer, H).items():
             s[f"{p}mix.{n}"] = shape
+        if l.ff or l.moe:
+            s.update({f"{p}norm2{b}": (H,) for b in norms})
+        gated = lambda q, ff: {q + "gate": (ff, H), q + "up": (ff, H), q + "down": (H, ff)}
         if l.ff:
-            s[p + "norm2"] = (H,)
-            s[p + "mlp.gate"], s[p + "mlp.up"], s[p + "mlp.down"] = (l.ff, H), (l.ff, H), (H, l.ff)
+            s.update(gated(p + "mlp.", l.ff))
+        if l.moe:
+            s[p + "mlp.router"] = (l.moe.experts, H)
+            for e in range(l.moe.experts):
+                s.update(gated(f"{p}mlp.e{e}.", l.moe.ff))
     cfg.__dict__["_tensor_shapes"] = s
     return s
 
@@ -59,7 +75,10 @@ class HybridLayer:
     glu_fused: bool = False
     glu_bn: int = 128
     act: int = 1
-    moe: Optional[object] = None
+    moe: Optional[object] = None           # None: what the engine asks of other models' layers (expert balancing)
+    experts: Optional[ExpertFF] = None
+    norm1b: Optional[torch.Tensor] = None  # sandwich blocks: the norms behind the sublayers
+    norm2b: Optional[torch.Tensor] = None
     kv_donor: Optional[int] = None
     extra: Dict[str, torch.Tensor] = field(default_factory=dict)
 
@@ -74,7 +93,7 @@ class HybridWorkspace:
         dev, dt, H = model.device, model.dtype, model.cfg.hidden_size
         self.max_tokens = tokens
         self.x = torch.zeros((tokens, H), dtype=torch.float32, device=dev)
-        self.xb = self.x if dt == torch.float32 else torch.zeros((tokens, H), dtype=dt, device=dev)
+        self.xb = self.x if dt == torch.float32 and not model.sandwich else torch.zeros((tokens, H), dtype=dt, device=dev)
         need: Dict[str, int] = {}
         for l in model.layers:
             sizes = dict(l.mixer.workspace())
@@ -108,6 +127,10 @@ class HybridDecoder:
             raise ValueError(f"not available for heterogeneous decoders: {', '.join(sorted(bad))}")
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError(f"compute dtype {dtype}: bfloat16 or float32")
+        self.sandwich = cfg.block == "sandwich"
+        if cfg.block not in ("post", "sandwich") or (not self.sandwich and (
+                cfg.norm_type != "rms" or cfg.loop or any(l.moe for l in cfg.layer_specs))):
+            raise ValueError("heterogeneous decoder: looped layers, layer norms and experts are built for sandwich blocks")
         self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
         self.layer_ids = list(range(cfg.num_layers))
         self.kv_dtype, self.kv_scale = dtype, 1.0
@@ -132,10 +155,19 @@ class HybridDecoder:
             p = layer_prefix(i)
             lw = HybridLayer(MIXERS[spec.mixer.kind](spec.mixer, src, p, cfg.hidden_size, cfg.rms_norm_eps, dev, dtype),
                              norm1=f32(p + "norm1"), act=L.ACT_IDS[spec.act])
-            if spec.ff:
+            if spec.ff or spec.moe:
                 lw.norm2 = f32(p + "norm2")
+            if self.sandwich:
+                lw.norm1b = f32(p + "norm1b")
+                lw.norm2b = f32(p + "norm2b") if spec.ff or spec.moe else None
+            if spec.ff:
                 self._pack_ff(lw, to(p + "mlp.gate"), to(p + "mlp.up"), to(p + "mlp.down"))
+            if spec.moe:
+                lw.experts = ExpertFF(spec.moe, lw.act, src, p, cfg.hidden_size, dev, dtype)
             self.layers.append(lw)
+        self.runs = cfg.layer_runs()
+        steps = f32("loop_step") if any(t is not None for _, t in self.runs) else None
+        self.run_step = [None if t is None else steps[t] for _, t in self.runs]
 
     def _pack_ff(self, lw: HybridLayer, gate, up, down):
         inter, hidden = gate.shape
@@ -167,19 +199,21 @@ class HybridDecoder:
     def weight_bytes(self) -> int:
         ts = [self.embed, self.lm_head, self.final_norm]
         for l in self.layers:
-            ts += [t for t in list(l.mixer.w.values()) + [l.norm1, l.norm2, l.w_gate_up, l.w_down] if t is not None]
+            ts += [t for t in list(l.mixer.w.values()) + [l.norm1, l.norm2, l.norm1b, l.norm2b, l.w_gate_up, l.w_down]
+                   + (l.experts.tensors() if l.experts else []) if t is not None]
         return sum(t.numel() * t.element_size() for t in ts)
 
     def page_bytes(self) -> int:
         esz = 4 if self.dtype == torch.float32 else 2
-        return 16 * esz * sum(l.mixer.kv_elems() for l in self.cfg.layer_specs)
+        return 16 * esz * sum(self.cfg.layer_specs[i].mixer.kv_elems() for i, _ in self.runs)
 
     def state_bytes(self, slots: int) -> int:
-        return 4 * slots * sum(l.mixer.state_floats() for l in self.cfg.layer_specs)
+        return 4 * slots * sum(self.cfg.layer_specs[i].mixer.state_floats() for i, _ in self.runs)
 
     def alloc_kv_cache(self, num_pages: int, state_slots: int = 1) -> list:
-        """One entry per layer: paged K / V [pages, 2, kv_heads, 16, dim] or the layer's ``RecurrentState``."""
-        return [l.mixer.alloc(num_pages, state_slots) for l in self.layers]
+        """One entry per run: paged K / V [pages, 2, kv_heads, 16, dim], latent rows, the layer's ``RecurrentState``, or both
+        (``PagedWithState``)."""
+        return [self.layers[i].mixer.alloc(num_pages, state_slots) for i, _ in self.runs]
 
     def workspace(self, tokens: int) -> HybridWorkspace:
         if self._ws is None or self._ws.max_tokens < tokens:
@@ -190,39 +224,25 @@ class HybridDecoder:
     def forward(self, batch: ForwardBatch, kv_caches, *, hidden_in=None, decode_ws=None, return_hidden: bool = False,
                 capture_layers=None, callbacks=None):
         """fp32 logits [R, padded vocab], or (``return_hidden``) the fp32 residual stream [T, hidden] behind the last
-        layer. ``callbacks`` / ``capture_layers`` as in ``DecoderModel.forward``; captured streams are fp32."""
-        c = self.cfg
+        layer. ``callbacks`` / ``capture_layers`` as in ``DecoderModel.forward`` (a layer that runs several times counts each
+        time); captured streams are fp32."""
         T = batch.num_tokens
         ws = self.workspace(T)
         ws.decode_ws = decode_ws
         x, xb = ws.x[:T], ws.xb[:T]
-        two = ws.xb is not ws.x
+        copy = xb if ws.xb is not ws.x and not self.sandwich else None
         self.mark("begin")
         if hidden_in is None:
-            R.embed_rows(batch.token_ids, self.embed, x, xb if two else None)
+            R.embed_rows(batch.token_ids, self.embed, x, copy)
             self.mark("embed")
         else:
             x.copy_(hidden_in.float())
-            if two:
-                xb.copy_(hidden_in)
+            if copy is not None:
+                copy.copy_(hidden_in)
         self.callback_action, self.callback_info = None, {}
         self.captured = {}
-        stop = False
-        for i, lw in enumerate(self.layers):
-            if callbacks is not None and self._run_callbacks(callbacks, "pre", i, x, xb):
-                break
-            y = lw.mixer.forward(self, ws, batch, kv_caches[i], T)
-            self.mark("out_gemm")
-            R.scaled_add_norm(x, y, lw.norm1, c.postln_alpha, c.rms_norm_eps, x_out=x, xb=xb if two else None)
-            self.mark("norm")
-            if lw.w_down is not None:
-                y = self._feed_forward(lw, ws, T)
-                R.scaled_add_norm(x, y, lw.norm2, c.postln_alpha, c.rms_norm_eps, x_out=x, xb=xb if two else None)
-                self.mark("norm")
-            if capture_layers is not None and i in capture_layers:
-                self.captured[i] = x.clone()
-            if callbacks is not None and self._run_callbacks(callbacks, "post", i, x, xb):
-                break
+        layers = self._sandwich_layers if self.sandwich else self._post_layers
+        layers(x, xb, ws, batch, kv_caches, T, capture_layers or (), callbacks)
         if return_hidden:
             return x
         rows = batch.logits_rows
@@ -231,6 +251,64 @@ class HybridDecoder:
         logits = self._logits(x, rows)
         self.mark("lm_head")
         return logits
+
+    def _post_layers(self, x, xb, ws, batch, kv_caches, T, capture, callbacks):
+        c = self.cfg
+        copy = xb if ws.xb is not ws.x else None
+        for r, (i, _) in enumerate(self.runs):
+            lw = self.layers[i]
+            if callbacks is not None and self._run_callbacks(callbacks, "pre", r, x, copy):
+                break
+            y = lw.mixer.forward(self, ws, batch, kv_caches[r], T)
+            self.mark("out_gemm")
+            R.scaled_add_norm(x, y, lw.norm1, c.postln_alpha, c.rms_norm_eps, x_out=x, xb=copy)
+            self.mark("norm")
+            if lw.w_down is not None:
+                y = self._feed_forward(lw, ws, T)
+                R.scaled_add_norm(x, y, lw.norm2, c.postln_alpha, c.rms_norm_eps, x_out=x, xb=copy)
+                self.mark("norm")
+            if r in capture:
+                self.captured[r] = x.clone()
+            if callbacks is not None and self._run_callbacks(callbacks, "post", r, x, copy):
+                break
+
+    def _sandwich_layers(self, x, xb, ws, batch, kv_caches, T, capture, callbacks):
+        """One fused pass between two sublayers: norm behind the one, residual sum (with the vector of a pass that starts
+        here), norm in front of the next. It is split where somebody looks at the stream between two layers."""
+        norm = dict(kind=self.cfg.norm_type, eps=self.cfg.rms_norm_eps)
+        for r, (i, _) in enumerate(self.runs):
+            lw = self.layers[i]
+            last = r + 1 == len(self.runs)
+            if r == 0 or callbacks is not None or r - 1 in capture:      # not done by the pass behind the layer before
+                add = self.run_step[r]
+                if callbacks is not None:
+                    if add is not None:
+                        residual_norm(x, add=add, **norm)
+                        add = None
+                    if self._run_callbacks(callbacks, "pre", r, x, None):
+                        break
+                residual_norm(x, add=add, pre_w=lw.norm1, xb=xb, **norm)
+                self.mark("norm")
+            ahead = {}
+            if not (last or callbacks is not None or r in capture):
+                ahead = dict(add=self.run_step[r + 1], pre_w=self.layers[self.runs[r + 1][0]].norm1, xb=xb)
+            y = lw.mixer.forward(self, ws, batch, kv_caches[r], T)
+            self.mark("out_gemm")
+            routed = {}
+            if lw.norm2 is not None:
+                residual_norm(x, y, post_w=lw.norm1b, pre_w=lw.norm2, xb=xb, **norm)
+                self.mark("norm")
+                if lw.experts is not None:
+                    y, dest = lw.experts.forward(self, xb, T)
+                    routed = dict(dest=dest, top=lw.experts.spec.top)
+                else:
+                    y = self._feed_forward(lw, ws, T)
+            residual_norm(x, y, post_w=lw.norm1b if lw.norm2 is None else lw.norm2b, **routed, **ahead, **norm)
+            self.mark("norm")
+            if r in capture:
+                self.captured[r] = x.clone()
+            if callbacks is not None and self._run_callbacks(callbacks, "post", r, x, None):
+                break
 
     def _feed_forward(self, lw: HybridLayer, ws, T: int):
         xb = ws.xb[:T]
@@ -245,23 +323,30 @@ class HybridDecoder:
         self.mark("down_gemm")
         return y
 
-    def _logits(self, x, rows=None):
-        c = self.cfg
+    def _final_norm(self, x, rows=None):
         n = x.shape[0] if rows is None else rows.shape[0]
-        hn = torch.empty((n, c.hidden_size), dtype=self.dtype, device=self.device)
-        R.scaled_add_norm(x, None, self.final_norm, 1.0, c.rms_norm_eps, rows=rows, xb=hn)
-        return L.gemm(hn, self.lm_head, out_dtype=torch.float32, bn=256, softcap=float(c.logit_softcap or 0.0))
+        hn = torch.empty((n, self.cfg.hidden_size), dtype=self.dtype, device=self.device)
+        if self.sandwich:
+            residual_norm(x, pre_w=self.final_norm, xb=hn, rows=rows, kind=self.cfg.norm_type, eps=self.cfg.rms_norm_eps)
+        else:
+            R.scaled_add_norm(x, None, self.final_norm, 1.0, self.cfg.rms_norm_eps, rows=rows, xb=hn)
+        return hn
+
+    def _logits(self, x, rows=None):
+        return L.gemm(self._final_norm(x, rows), self.lm_head, out_dtype=torch.float32, bn=256,
+                      softcap=float(self.cfg.logit_softcap or 0.0))
 
     def _run_callbacks(self, callbacks, when: str, i: int, x, xb) -> bool:
-        """One port of the callback chain on the residual stream; True ends the layer loop."""
+        """One port of the callback chain on the residual stream (``xb``: its copy in the compute dtype, or None); True ends
+        the layer loop."""
         from ..engine.callbacks import CallbackAction
-        if i not in callbacks.layers_of_interest(self.cfg.num_layers):
+        if i not in callbacks.layers_of_interest(len(self.runs)):
             return False
         r = callbacks.run(when, i, x)
         self.callback_info.update(r.info)
         if r.hidden is not None:
             x.copy_(r.hidden.to(x.dtype))
-            if xb.data_ptr() != x.data_ptr():
+            if xb is not None:
                 xb.copy_(x)
         if r.action in (CallbackAction.EXIT_EARLY, CallbackAction.VETO):
             self.callback_action = r.action
@@ -276,6 +361,4 @@ class HybridDecoder:
         return self._logits(xr.float().contiguous())
 
     def final_hidden(self, x):
-        hn = torch.empty((x.shape[0], self.cfg.hidden_size), dtype=self.dtype, device=self.device)
-        R.scaled_add_norm(x.float(), None, self.final_norm, 1.0, self.cfg.rms_norm_eps, xb=hn)
-        return hn
+        return self._final_norm(x.float().contiguous())

@@ -1,9 +1,11 @@
-"""Token mixers of heterogeneous decoders: chunked / full attention with a whole-row query / key norm, RG-LRU and gated
-linear attention. Each class packs its layer's weights into the layouts of the ops and runs a step's tokens:
+"""Token mixers of heterogeneous decoders: attention (chunked, windowed with kept first tokens or full; query / key norm over
+the row or per head; optional short convolution), windowed latent attention, RG-LRU and gated linear attention. Each class
+packs its layer's weights into the layouts of the ops and runs a step's tokens:
 ``forward(model, ws, batch, cache, T) -> y [T, >= hidden]``, reading the layer input from ``ws.xb``.
 
-``cache`` is what ``alloc`` returned for the layer: paged K / V for attention, a ``RecurrentState`` for the others. All
-constants come from the layer's ``MixerSpec``, so other designs can combine the same mixers differently.
+``cache`` is what ``alloc`` returned for the layer: paged K / V (or latent rows) for attention, a ``RecurrentState`` for the
+recurrent mixers, both (``PagedWithState``) for attention behind a convolution. All constants come from the layer's
+``MixerSpec``, so other designs can combine the same mixers differently.
 """
 from __future__ import annotations
 
@@ -12,8 +14,9 @@ from typing import Dict, Optional, Tuple
 import torch
 
 from .. import ops
-from ..kv_cache.recurrent_state import RecurrentState
+from ..kv_cache.recurrent_state import PagedWithState, RecurrentState
 from ..ops import linear as L
+from ..ops import mla as MLA
 from ..ops import recurrent as R
 from ..ops.recurrent import SeqView
 from . import rope
@@ -58,44 +61,106 @@ class _Mixer:
 class AttentionMixer(_Mixer):
     def pack(self):
         m = self.spec
-        self.nq, self.nk = m.heads * m.dim, m.kv_heads * m.dim
+        self.dv = m.value_dim
+        self.nq, self.nk, self.nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * self.dv
         names = ("q", "k") if m.v_from_k else ("q", "k", "v")
         self.w["wqk"] = self.mat(*names)
         self.w["bqk"] = _pad_bias([self._src.get(self._p + n + ".b") for n in names], self.w["wqk"].shape[0], self.device)
         self.w["wo"] = self.mat("o")
-        self.w["bo"] = _pad_bias([self._src.get(self._p + "o.b")], self.w["wo"].shape[0], self.device)
-        self.w["q_norm"] = self.vec("q.norm") if m.row_qk_norm else None
-        self.w["k_norm"] = self.vec("k.norm") if m.row_qk_norm else None
+        self.w["bo"] = _pad_bias([self._src.get(self._p + "o.b")], self.w["wo"].shape[0], self.device) if m.o_bias else None
+        norm = m.row_qk_norm or m.head_qk_norm
+        self.w["q_norm"] = self.vec("q.norm") if norm else None
+        self.w["k_norm"] = self.vec("k.norm") if norm else None
+        self.w["conv"] = torch.cat([self.vec(n + ".conv") for n in names]).contiguous() if m.taps else None
+        if m.row_qk_norm and (m.taps or self.dv != m.dim) or m.v_from_k and not m.row_qk_norm or (m.keep_first and m.chunk):
+            raise ValueError("attention mixer: this combination of norm, values, convolution and mask is not built")
 
     def workspace(self):
-        return {"proj": self.w["wqk"].shape[0], "q": self.nq, "mix": self.nq}
+        return {"proj": self.w["wqk"].shape[0], "q": self.nq, "mix": self.spec.heads * self.dv}
+
+    def state_shapes(self):
+        return {"conv": (self.spec.taps, self.nq + self.nk + self.nv)} if self.spec.taps else None
 
     def alloc(self, num_pages, slots):
         m = self.spec
-        return torch.zeros((num_pages, 2, m.kv_heads, PAGE, m.dim), dtype=self.dtype, device=self.device)
+        shape = (2, m.kv_heads, PAGE, m.dim) if self.dv == m.dim else (PAGE * (self.nk + self.nv),)
+        kv = torch.zeros((num_pages,) + shape, dtype=self.dtype, device=self.device)
+        return PagedWithState(kv, RecurrentState(slots, self.state_shapes(), self.device)) if m.taps else kv
 
-    def forward(self, model, ws, batch, kv, T):
+    def forward(self, model, ws, batch, cache, T):
         m = self.spec
+        kv = cache.pages if m.taps else cache
         qk = L.gemm(ws.xb[:T], self.w["wqk"], out=ws.take("proj", T, self.w["wqk"].shape[0]), bias=self.w["bqk"])
         model.mark("in_gemm")
         cos, sin = model.rope_tables(m.rot_dim, m.rot_base)
         q = ws.take("q", T, self.nq)
-        R.qk_row_norm_rope(qk, n_q=m.heads, n_kv=m.kv_heads, head_dim=m.dim, rot_dim=m.rot_dim, v_from_k=m.v_from_k,
-                           positions=batch.positions, slot_mapping=batch.slot_mapping, cos_t=cos, sin_t=sin,
-                           q_w=self.w["q_norm"], k_w=self.w["k_norm"], eps=self.eps, q_out=q, kv_cache=kv)
+        common = dict(rot_dim=m.rot_dim, positions=batch.positions, slot_mapping=batch.slot_mapping, cos_t=cos, sin_t=sin,
+                      q_w=self.w["q_norm"], k_w=self.w["k_norm"], eps=self.eps, q_out=q, kv_cache=kv)
+        if m.row_qk_norm:
+            R.qk_row_norm_rope(qk, n_q=m.heads, n_kv=m.kv_heads, head_dim=m.dim, v_from_k=m.v_from_k, **common)
+        else:
+            R.conv_qkv_prep(SeqView.of(batch), qk, n_q=m.heads, n_kv=m.kv_heads, dim=m.dim, vdim=self.dv, conv=self.w["conv"],
+                            ring=cache.state["conv"] if m.taps else None, **common)
         model.mark("qk_prep")
-        o = ws.take("mix", T, self.nq)
-        window = ops.chunk_window(m.chunk) if m.chunk > 0 else 0
+        o = ws.take("mix", T, m.heads * self.dv)
+        mask = dict(window=ops.chunk_window(m.chunk) if m.chunk > 0 else m.window, keep_first=m.keep_first, dim=m.dim)
         if batch.is_decode:
             ops.paged_decode(q, kv, batch.block_tables, batch.ctx_lens, n_q=m.heads, n_kv=m.kv_heads, scale=m.scale, out=o,
-                             workspace=ws.decode_ws, window=window,
-                             pages_per_split=getattr(ws.decode_ws, "pages_per_split", 32), full_weights=True)
+                             workspace=ws.decode_ws, pages_per_split=getattr(ws.decode_ws, "pages_per_split", 32),
+                             full_weights=True, **mask)
         else:
             ops.paged_prefill(q, kv, batch.block_tables, batch.q_start, batch.q_len, batch.ctx_lens,
-                              max_q_len=batch.max_q_len, n_q=m.heads, n_kv=m.kv_heads, scale=m.scale, out=o, window=window,
-                              full_weights=True)
+                              max_q_len=batch.max_q_len, n_q=m.heads, n_kv=m.kv_heads, scale=m.scale, out=o,
+                              full_weights=True, **mask)
         model.mark("attention")
         return L.gemm(o, self.w["wo"], out=ws.take("y", T, self.w["wo"].shape[0]), bias=self.w["bo"])
+
+
+class LatentMixer(_Mixer):
+    """Latent attention without positions, in absorbed form: the key up-projection moves into the query, the value
+    up-projection behind the attention, and every head attends over the same cached latent rows."""
+
+    def pack(self):
+        m = self.spec
+        self.w["wdown"] = self.mat("dq", "dkv")
+        self.w["q_norm"], self.w["kv_norm"] = self.vec("dq.norm"), self.vec("dkv.norm")
+        self.w["wuq"] = self.mat("uq")
+        up = lambda n, d: self._src.get(self._p + n).to(self.device, self.dtype).reshape(m.heads, d, m.kv_rank)
+        self.w["wuk"] = up("uk", m.dim).contiguous()                           # [heads, dim, rank]
+        self.w["wuv"] = up("uv", m.vdim).transpose(1, 2).contiguous()          # [heads, rank, vdim]
+        self.w["sink"] = self.vec("sink") if m.sink else None
+        self.w["wo"] = self.mat("o")
+
+    def workspace(self):
+        m = self.spec
+        return {"proj": self.w["wdown"].shape[0], "cq": m.q_rank, "q": self.w["wuq"].shape[0], "qlat": m.heads * m.kv_rank,
+                "olat": m.heads * m.kv_rank, "mix": m.heads * m.vdim}
+
+    def alloc(self, num_pages, slots):
+        return torch.zeros((num_pages, PAGE, self.spec.kv_rank), dtype=self.dtype, device=self.device)
+
+    def forward(self, model, ws, batch, cache, T):
+        m, w = self.spec, self.w
+        p = L.gemm(ws.xb[:T], w["wdown"], out=ws.take("proj", T, w["wdown"].shape[0]))
+        model.mark("in_gemm")
+        cq = ws.take("cq", T, m.q_rank)
+        MLA.latent_prep(p, m.q_rank, m.kv_rank, w["q_norm"], w["kv_norm"], self.eps, batch.slot_mapping, cq, cache)
+        model.mark("latent_prep")
+        q = L.gemm(cq, w["wuq"], out=ws.take("q", T, w["wuq"].shape[0]))
+        model.mark("uq_gemm")
+        ql = ws.take("qlat", m.heads * T, m.kv_rank).view(m.heads, T, m.kv_rank)
+        torch.bmm(q[:, :m.heads * m.dim].unflatten(1, (m.heads, m.dim)).transpose(0, 1), w["wuk"], out=ql)
+        model.mark("uk_gemm")
+        ol = ws.take("olat", m.heads * T, m.kv_rank).view(m.heads, T, m.kv_rank)
+        rows = (None, None) if batch.is_decode else (batch.q_start, batch.q_len)
+        MLA.window_latent_attention(ql, cache, batch.block_tables, *rows, batch.ctx_lens,
+                                    max_q_len=1 if batch.is_decode else batch.max_q_len, scale=m.scale, window=m.window,
+                                    sinks=w["sink"], out=ol)
+        model.mark("latent_attention")
+        o = ws.take("mix", T, m.heads * m.vdim)
+        torch.bmm(ol, w["wuv"], out=o.unflatten(1, (m.heads, m.vdim)).transpose(0, 1))
+        model.mark("uv_gemm")
+        return L.gemm(o, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
 
 
 class RgLruMixer(_Mixer):
@@ -190,18 +255,31 @@ class GlaMixer(_Mixer):
         return L.gemm(out, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
 
 
-MIXERS = {"attention": AttentionMixer, "rglru": RgLruMixer, "gla": GlaMixer}
+MIXERS = {"attention": AttentionMixer, "latent": LatentMixer, "rglru": RgLruMixer, "gla": GlaMixer}
 
 
 def mixer_shapes(m: MixerSpec, hidden: int) -> Dict[str, Tuple[int, ...]]:
     """Checkpoint tensors of a mixer (names behind ``mix.``) and their shapes."""
     if m.kind == "attention":
-        nq, nk = m.heads * m.dim, m.kv_heads * m.dim
-        s = {"q": (nq, hidden), "q.b": (nq,), "k": (nk, hidden), "k.b": (nk,), "o": (hidden, nq), "o.b": (hidden,)}
+        nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.value_dim
+        s = {"q": (nq, hidden), "q.b": (nq,), "k": (nk, hidden), "k.b": (nk,), "o": (hidden, m.heads * m.value_dim)}
+        if m.o_bias:
+            s["o.b"] = (hidden,)
         if not m.v_from_k:
-            s.update({"v": (nk, hidden), "v.b": (nk,)})
+            s.update({"v": (nv, hidden), "v.b": (nv,)})
         if m.row_qk_norm:
             s.update({"q.norm": (nq,), "k.norm": (nk,)})
+        if m.head_qk_norm:
+            s.update({"q.norm": (m.dim,), "k.norm": (m.dim,)})
+        if m.taps:
+            s.update({n + ".conv": (s[n][0], m.taps) for n in ("q", "k", "v") if n in s})
+        return s
+    if m.kind == "latent":
+        s = {"dq": (m.q_rank, hidden), "dq.norm": (m.q_rank,), "uq": (m.heads * m.dim, m.q_rank), "dkv": (m.kv_rank, hidden),
+             "dkv.norm": (m.kv_rank,), "uk": (m.heads * m.dim, m.kv_rank), "uv": (m.heads * m.vdim, m.kv_rank),
+             "o": (hidden, m.heads * m.vdim)}
+        if m.sink:
+            s["sink"] = (m.heads,)
         return s
     if m.kind == "rglru":
         w, nb = m.width, m.blocks

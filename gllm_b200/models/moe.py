@@ -19,7 +19,7 @@ import torch
 from .. import ops
 from ..ops import linear as L
 from ..ops import moe as M
-from .config import ModelConfig
+from .config import ModelConfig, MoeSpec
 from .weights import _fold, layer_prefix, shard_range
 
 
@@ -511,3 +511,68 @@ class ExpertPager:
             out["faults"] += pg.handler.stats["faults"]
             out["resident_bytes"] += pg.resident_bytes()
         return out
+
+
+# --------------------------------------------------------------------------------------------------------------------
+# mixture of experts of a heterogeneous decoder's layer (models/hybrid.py)
+# --------------------------------------------------------------------------------------------------------------------
+class ExpertFF:
+    """One layer's experts, bf16 or true fp32: router -> top-k -> routed rows in per-expert blocks -> grouped gate / up and
+    down projections. ``forward`` returns the experts' rows and the place of each (token, pick) among them; the caller sums
+    them (``ops.residual.residual_norm`` does it together with the norm behind the sublayer)."""
+
+    def __init__(self, spec: MoeSpec, act: int, src, prefix: str, hidden: int, device, dtype):
+        if not spec.scale_input:
+            raise ValueError("expert outputs are summed unweighted: the spec must scale the experts' inputs")
+        self.spec, self.act, self.hidden = spec, act, hidden
+        get = lambda n: src.get(prefix + "mlp." + n).to(device, dtype)
+        self.router = L.pad_rows(get("router"), 32).contiguous()
+        self.fused = dtype == torch.bfloat16 and hidden % 8 == 0
+        pad = -spec.ff % 64 if self.fused else 0       # zero gate / up rows and down columns add nothing to the sums
+        self.inter = spec.ff + pad
+        rows = lambda w: torch.nn.functional.pad(w, (0, 0, 0, pad))
+        gus, downs = [], []
+        for e in range(spec.experts):
+            g, u, d = rows(get(f"e{e}.gate")), rows(get(f"e{e}.up")), torch.nn.functional.pad(get(f"e{e}.down"), (0, pad))
+            gus.append(L.interleave_gate_up(g, u) if self.fused else torch.cat([g, u], 0))
+            downs.append(L.pad_rows(d, 128))
+        self.w_gate_up, self.w_down = torch.cat(gus).contiguous(), torch.cat(downs).contiguous()
+        self.glu_bn = 256 if self.inter % 128 == 0 else 128
+
+    def tensors(self):
+        return [self.router, self.w_gate_up, self.w_down]
+
+    def workspace(self, model, T: int) -> M.MoeWorkspace:
+        holder = model.__dict__.setdefault("_expert_ws", {})
+        s = self.spec
+        key = (s.experts, s.top, self.inter)
+        ws = holder.get(key)
+        if ws is None or ws.ids.shape[0] < T:
+            n = max(T, 256)
+            ws = M.MoeWorkspace(n, s.top, self.hidden, self.inter, s.experts, model.device, model.dtype,
+                                out_cols=self.w_down.shape[0] // s.experts)
+            ws.logits = torch.zeros((n, self.router.shape[0]), dtype=torch.float32, device=model.device)
+            ws.gu = None if self.fused else torch.zeros((ws.max_rows, 2 * self.inter), dtype=model.dtype, device=model.device)
+            holder[key] = ws
+        return ws
+
+    def forward(self, model, h, T: int):
+        s = self.spec
+        ws = self.workspace(model, T)
+        logits = L.gemm(h, self.router, out=ws.logits[:T])
+        on_gpu = dict(out_ids=ws.ids[:T], out_w=ws.w[:T]) if h.is_cuda else {}
+        ids, w = M.route(logits[:, :s.experts], s.top, norm_topk=s.norm_topk, scoring=s.scoring, **on_gpu)
+        model.mark("moe_route")
+        M.permute(h, None, ids, ws, 0, s.experts, row_w=w)
+        model.mark("moe_permute")
+        if self.fused:
+            L.set_block_rows(ws.blk_rows if h.is_cuda else None)
+            L.gemm_glu(ws.a_perm, self.w_gate_up, act=self.act, out=ws.act, bn=self.glu_bn, mblk_group=ws.blk_group,
+                       num_groups=s.experts)
+        else:
+            L.gemm_grouped(ws.a_perm, self.w_gate_up, ws.blk_group, s.experts, out=ws.gu, block_rows=ws.blk_rows)
+            ops.glu(ws.gu, self.act, out=ws.act)
+        model.mark("moe_gate_up")
+        L.gemm_grouped(ws.act, self.w_down, ws.blk_group, s.experts, out=ws.y_perm, block_rows=ws.blk_rows)
+        model.mark("moe_down")
+        return ws.y_perm, ws.dest

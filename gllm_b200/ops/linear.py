@@ -273,8 +273,10 @@ def set_block_rows(rows):
         nv.check(nv.lib().gllm_gemm_set_block_rows(rows.data_ptr()), "gemm_set_block_rows")
 
 
-def gemm_grouped(a, w_stack, mblk_group, num_groups, *, out=None, bn=128, max_ctas=0):
-    """Grouped GEMM: rows [128i, 128i+128) of ``a`` multiply expert ``mblk_group[i]``'s [N,K] weight."""
+def gemm_grouped(a, w_stack, mblk_group, num_groups, *, out=None, bn=128, max_ctas=0, block_rows=None):
+    """Grouped GEMM: rows [128i, 128i+128) of ``a`` multiply expert ``mblk_group[i]``'s [N,K] weight; with ``block_rows``
+    only the first ``block_rows[i]`` of them exist. fp32 operands, and bf16 ones the tensor-core kernel cannot address, run
+    on CUDA cores."""
     M, K = a.shape
     N = w_stack.shape[0] // num_groups
     if not a.is_cuda:
@@ -290,7 +292,15 @@ def gemm_grouped(a, w_stack, mblk_group, num_groups, *, out=None, bn=128, max_ct
         return res
     _on_device(a, weight=w_stack, mblk_group=mblk_group, out=out)
     if out is None:
-        out = torch.empty((M, N), dtype=torch.bfloat16, device=a.device)
+        out = torch.empty((M, N), dtype=a.dtype, device=a.device)
+    if a.dtype == torch.float32 or not tensor_core_shape(a, w_stack) or N % 32:
+        rc = nv.lib().gllm_gemm_simt_grouped(a.data_ptr(), a.stride(0), w_stack.data_ptr(), w_stack.stride(0), out.data_ptr(),
+                                             out.stride(0), M, N, K, 1 if a.dtype == torch.float32 else 0,
+                                             1 if out.dtype == torch.float32 else 0, mblk_group.data_ptr(),
+                                             nv.ptr(block_rows), nv.stream_ptr())
+        nv.check(rc, "gemm_simt_grouped")
+        return out
+    set_block_rows(block_rows)
     rc = nv.lib().gllm_gemm_bf16_grouped(a.data_ptr(), a.stride(0), w_stack.data_ptr(), w_stack.stride(0),
                                          out.data_ptr(), out.stride(0), M, N, K, mblk_group.data_ptr(), num_groups,
                                          bn, nv.stream_ptr(), max_ctas)

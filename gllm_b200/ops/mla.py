@@ -1,6 +1,7 @@
 """Multi-head latent attention ops: latent cache write and attention over the latent cache.
 
-CUDA path: ``csrc/kernels/mla.cu``. CPU path / oracle: plain fp32 PyTorch of the same math.
+CUDA path: ``csrc/kernels/mla.cu`` and ``mla_decode.cu`` (latent with a rotated key part), ``mixer_prep.cu`` and
+``attention_any.cu`` (windowed latent attention without positions). CPU path / oracle: plain fp32 PyTorch of the same math.
 Reference parity: MlaKvCompress / MlaQAbsorb / MlaAttention
 (src/arch/auto_graph_fragments/build_graph.inc.rs:1486-1578).
 """
@@ -15,6 +16,8 @@ nv.register("gllm_mla_latent_write", I, [P, L, I, I, I, P, F, P, P, P, P, I, P, 
 nv.register("gllm_mla_attention", I, [P, P, P, I, P, I, P, P, P, P, I, I, I, I, F, I, P])
 nv.register("gllm_mla_decode_scratch_floats", L, [I, I, I])
 nv.register("gllm_mla_decode", I, [P, P, P, I, P, I, P, I, I, I, F, I, P, L, P])
+
+nv.register("gllm_latent_prep", I, [P, L, I, I, I, I, P, P, F, P, P, P, I, P])
 
 PAGE = 16
 
@@ -133,3 +136,52 @@ def latent_prefill(q, cache, block_tables, row_seq, positions, ctx_lens, *, n_he
         row_ctx = ctx_lens.index_select(0, row_seq.long()).to(torch.int32)
     return latent_decode(q, cache, tables.contiguous(), row_ctx.contiguous(), n_heads=n_heads, scale=scale,
                          max_ctx=max_ctx, out=out)
+
+
+# ------------------------------------------------------------------------------------------------------------------------------
+# windowed latent attention without positions: one normalised latent row per token is key and value of every head
+# ------------------------------------------------------------------------------------------------------------------------------
+def latent_prep(proj, q_rank, kv_rank, q_w, kv_w, eps, slot_mapping, cq, cache):
+    """proj [T, >= q_rank + kv_rank] = query latent | key / value latent; each RMS-normed with its weight: into ``cq``
+    [T, q_rank] and into the latent page [pages, 16, kv_rank] of the token's slot (negative: not written)."""
+    T = proj.shape[0]
+    if not proj.is_cuda:
+        norm = lambda t, w: t / torch.sqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w
+        cq[:T].copy_(norm(proj[:, :q_rank].float(), q_w).to(cq.dtype))
+        if slot_mapping is not None:
+            ok = slot_mapping >= 0
+            c = norm(proj[:, q_rank:q_rank + kv_rank].float(), kv_w)
+            cache.view(-1, kv_rank)[slot_mapping[ok].long()] = c[ok].to(cache.dtype)
+        return
+    nv.check(nv.lib().gllm_latent_prep(proj.data_ptr(), proj.stride(0), 1 if proj.dtype == torch.float32 else 0, T, q_rank, kv_rank,
+                                       q_w.data_ptr(), kv_w.data_ptr(), float(eps), cq.data_ptr(), nv.ptr(slot_mapping),
+                                       cache.data_ptr(), cache.shape[0], nv.stream_ptr()), "latent_prep")
+
+
+def window_latent_attention(q, cache, block_tables, q_start, q_len, ctx_lens, *, max_q_len, scale, window=0, sinks=None, out):
+    """q [heads, T, rank] (the query with the key up-projection absorbed); cache [pages, 16, rank]; out [heads, T, rank]: the
+    weighted latent of each head, causal with a sliding ``window`` (0: everything), ``sinks`` [heads] fp32 in the denominator.
+    ``q_start`` None: a decode step (row = sequence)."""
+    H, T, R = q.shape
+    S = ctx_lens.shape[0]
+    if not q.is_cuda:
+        if q_start is None:
+            q_start, q_len = torch.arange(S, dtype=torch.int32), (ctx_lens > 0).to(torch.int32)
+        for s in range(S):
+            ql, ctx, st = int(q_len[s]), int(ctx_lens[s]), int(q_start[s])
+            if ql <= 0 or ctx <= 0:
+                continue
+            rows = cache[block_tables[s, :(ctx + PAGE - 1) // PAGE].long()].reshape(-1, R)[:ctx].float()
+            sc = torch.einsum("hqd,kd->hqk", q[:, st:st + ql].float(), rows) * scale
+            pq, pk = torch.arange(ctx - ql, ctx)[:, None], torch.arange(ctx)[None, :]
+            ok = (pk <= pq) & ((pk > pq - window) if window > 0 else True)
+            sc = sc.masked_fill(~ok[None], float("-inf"))
+            if sinks is not None:
+                sc = torch.cat([sc, sinks.float().reshape(H, 1, 1).expand(H, ql, 1)], -1)
+            p = torch.softmax(sc, -1)[..., :ctx]
+            out[:, st:st + ql] = torch.einsum("hqk,kd->hqd", p, rows).to(out.dtype)
+        return out
+    from .attention import attention_any
+    strides = (q.stride(1), q.stride(0), out.stride(1), out.stride(0), PAGE * R, 0, R, 0, 0, R)
+    return attention_any(q, out, cache, strides, block_tables, q_start, q_len, ctx_lens, S, max_q_len, H, 1, R, R, scale, True,
+                         window, 0, sinks)

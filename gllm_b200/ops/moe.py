@@ -11,7 +11,7 @@ from . import _native as nv
 from ._native import F, I, L, P
 
 nv.register("gllm_moe_route", I, [P, L, I, I, I, I, I, P, F, P, P, P])
-nv.register("gllm_moe_permute", I, [P, P, I, P, I, I, I, I, I, P, P, P, P, I, P, P, P, P, P])
+nv.register("gllm_moe_permute", I, [P, I, P, I, P, P, I, I, I, I, I, P, P, P, P, I, P, P, P, P, P])
 nv.register("gllm_moe_combine", I, [P, P, P, I, I, I, P, P, P, P])
 
 BLOCK = 128
@@ -46,7 +46,7 @@ def route(logits, k, *, norm_topk=True, scoring="softmax", sel_bias=None, scale=
 class MoeWorkspace:
     """Worst-case-sized buffers for one MoE layer invocation (shared by all layers)."""
 
-    def __init__(self, max_tokens, k, hidden, inter, e_local, device, dtype):
+    def __init__(self, max_tokens, k, hidden, inter, e_local, device, dtype, out_cols=None):
         self.max_rows = max_tokens * k + e_local * (BLOCK - 1)
         self.max_rows = (self.max_rows + BLOCK - 1) // BLOCK * BLOCK
         self.max_blocks = self.max_rows // BLOCK
@@ -58,15 +58,16 @@ class MoeWorkspace:
         self.a_perm = torch.zeros((self.max_rows, hidden), dtype=dtype, device=device)
         self.ss_perm = torch.ones(self.max_rows, 1, dtype=torch.float32, device=device)
         self.act = torch.zeros((self.max_rows, inter), dtype=dtype, device=device)
-        self.y_perm = torch.zeros((self.max_rows, hidden), dtype=dtype, device=device)
+        self.y_perm = torch.zeros((self.max_rows, out_cols or hidden), dtype=dtype, device=device)
         self.dest = z(max_tokens * k)
         self.ids = z(max_tokens, k)
         self.w = torch.zeros((max_tokens, k), dtype=torch.float32, device=device)
         self.logits = None
 
 
-def permute(x, row_ss, ids, ws: MoeWorkspace, e0=0, e_local=None):
-    """Bucket (token, slot) pairs by local expert. Fills ws.a_perm / ss_perm / blk_group / dest."""
+def permute(x, row_ss, ids, ws: MoeWorkspace, e0=0, e_local=None, row_w=None):
+    """Bucket (token, slot) pairs by local expert. Fills ws.a_perm / ss_perm / blk_group / dest. ``row_w`` [T, k] fp32: the
+    copied rows are multiplied by it (models that weight an expert's input instead of its output)."""
     T, k = ids.shape
     H = x.shape[1]
     e_local = e_local if e_local is not None else ws.counts.shape[0]
@@ -86,7 +87,7 @@ def permute(x, row_ss, ids, ws: MoeWorkspace, e0=0, e_local=None):
                 d = int(offs[e]) + cursor[e]
                 cursor[e] += 1
                 ws.dest[i] = d
-                ws.a_perm[d] = x[i // k]
+                ws.a_perm[d] = x[i // k] if row_w is None else x[i // k].float() * row_w.reshape(-1)[i]
                 if row_ss is not None:
                     ws.ss_perm[d, 0] = row_ss[i // k].float().sum()
         blk = torch.full((ws.max_blocks,), -1, dtype=torch.int32)
@@ -101,7 +102,8 @@ def permute(x, row_ss, ids, ws: MoeWorkspace, e0=0, e_local=None):
         ws.blk_rows.copy_(rows)
         return
     parts = 0 if row_ss is None else (row_ss.shape[1] if row_ss.dim() > 1 else 1)
-    rc = nv.lib().gllm_moe_permute(x.data_ptr(), nv.ptr(row_ss), parts, ids.data_ptr(), T, k, H, e0, e_local,
+    rc = nv.lib().gllm_moe_permute(x.data_ptr(), 1 if x.dtype == torch.float32 else 0, nv.ptr(row_ss), parts,
+                                   ids.data_ptr(), nv.ptr(row_w), T, k, H, e0, e_local,
                                    ws.counts.data_ptr(), ws.offsets.data_ptr(), ws.cursors.data_ptr(),
                                    ws.blk_group.data_ptr(), ws.max_blocks, ws.total_rows.data_ptr(),
                                    ws.a_perm.data_ptr(), ws.ss_perm.data_ptr() if row_ss is not None else None,

@@ -32,6 +32,7 @@ nv.register("gllm_gla_step", I, [P, P, P, P, I, P, P, P, P, L, I, P, P, I, I, I,
 nv.register("gllm_gla_tile_ok", I, [I, I, I, L])
 nv.register("gllm_gla_decode", I, [P, I, P, P, P, P, P, L, P, P, P, I, I, I, I, F, F, F, P, P, P])
 nv.register("gllm_gla_prefill", I, [P, P, P, P, I, I, P, P, P, P, L, P, P, I, I, I, I, F, F, P, P, P, P])
+nv.register("gllm_conv_qkv_prep", I, [P, P, P, P, I, I, P, L, I, I, I, I, I, I, I, P, P, P, F, P, P, P, P, I, P, P, P, I, P])
 nv.register("gllm_head_norm_gate", I, [P, P, L, I, P, L, I, I, F, P, P])
 
 RGLRU_C = 8.0        # exponent of the RG-LRU decay: log a = -8 r softplus(lam)
@@ -147,6 +148,53 @@ def qk_row_norm_rope(qk, *, n_q, n_kv, head_dim, rot_dim, v_from_k, positions, s
         nv.ptr(slot_mapping), nv.ptr(cos_t), nv.ptr(sin_t), cos_t.shape[0] if cos_t is not None else 1, nv.ptr(q_w),
         nv.ptr(k_w), float(eps), q_out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0], nv.stream_ptr()),
         "qk_row_norm_rope")
+    return q_out
+
+
+def conv_qkv_prep(sv: "SeqView", qkv, *, n_q, n_kv, dim, vdim, rot_dim, conv, q_w, k_w, eps, positions, slot_mapping, cos_t, sin_t,
+                  ring, q_out, kv_cache):
+    """Attention layers with a short convolution: causal convolution per channel of the projected q | k | v rows (``conv``
+    [channels, taps] fp32, or None) -> RMS norm of each q / k head (weights [dim] shared by the heads, or None) -> RoPE on
+    the first ``rot_dim`` dimensions of q and k -> q buffer, K and V pages. ``ring`` [slots, taps, channels] fp32 keeps the
+    last projected values of each sequence: the one of position p in entry p % taps."""
+    M = qkv.shape[0]
+    nq, nk, nv_ = n_q * dim, n_kv * dim, n_kv * vdim
+    taps = 0 if conv is None else conv.shape[1]
+    if not qkv.is_cuda:
+        u = qkv[:, :nq + nk + nv_].float()
+        y = u
+        if taps:
+            y = torch.zeros_like(u)
+            for r0, n, start, slot in sv.rows():
+                z = torch.cat([_conv_history(ring[slot], start, taps), u[r0:r0 + n]])
+                y[r0:r0 + n] = sum(z[j:j + n] * conv[:, j] for j in range(taps))
+                for i in range(max(0, n - taps), n):
+                    ring[slot, (start + i) % taps] = u[r0 + i]
+        half = rot_dim // 2
+
+        def prep(t, heads, w):
+            t = t.reshape(M, heads, dim)
+            if w is not None:
+                t = t / torch.sqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w
+            if rot_dim == 0:
+                return t
+            c, s = cos_t[positions.long()][:, None], sin_t[positions.long()][:, None]
+            a, b = t[..., :half], t[..., half:rot_dim]
+            return torch.cat([a * c - b * s, b * c + a * s, t[..., rot_dim:]], -1)
+        q_out[:M].copy_(prep(y[:, :nq], n_q, q_w).reshape(M, nq).to(q_out.dtype))
+        if slot_mapping is not None:
+            from .attention import kv_views
+            kc, vc = kv_views(kv_cache, n_kv, dim)
+            ok = slot_mapping >= 0
+            sl = slot_mapping[ok].long()
+            kc[sl // 16, :, sl % 16] = prep(y[:, nq:nq + nk], n_kv, k_w)[ok].to(kv_cache.dtype)
+            vc[sl // 16, :, sl % 16] = y[:, nq + nk:].reshape(M, n_kv, vdim)[ok].to(kv_cache.dtype)
+        return q_out
+    nv.check(nv.lib().gllm_conv_qkv_prep(
+        *sv.ptrs(), sv.max_q_len, qkv.data_ptr(), qkv.stride(0), _f32(qkv), n_q, n_kv, dim, vdim, rot_dim, taps, nv.ptr(conv),
+        nv.ptr(q_w), nv.ptr(k_w), float(eps), positions.data_ptr(), nv.ptr(slot_mapping), nv.ptr(cos_t), nv.ptr(sin_t),
+        cos_t.shape[0] if cos_t is not None else 1, nv.ptr(ring), q_out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
+        nv.stream_ptr()), "conv_qkv_prep")
     return q_out
 
 

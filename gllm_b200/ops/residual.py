@@ -1,0 +1,57 @@
+"""The step between two sublayers of a sandwich-norm block, over a residual stream kept in fp32:
+
+    x = x + post_norm(y) (+ vector);   operand of the next sublayer = pre_norm(x)
+
+``y`` is the sublayer's output, either rows of a projection or, behind a mixture of experts, the sum of each token's routed
+rows. CUDA path: ``csrc/kernels/residual.cu``; CPU path: an fp32 restatement.
+"""
+from __future__ import annotations
+
+from ctypes import c_float, c_int, c_longlong, c_void_p
+
+import torch
+
+from . import _native as nv
+
+P, I, L, F = c_void_p, c_int, c_longlong, c_float
+nv.register("gllm_residual_norm", I, [P, L, P, L, I, P, I, P, P, P, P, I, I, I, I, F, P, I, P])
+
+KINDS = {"rms": 0, "layer": 1}
+
+
+def norm_ref(h, w, kind: str, eps: float):
+    h = h.float()
+    if kind == "layer":
+        h = h - h.mean(-1, keepdim=True)
+    return h / torch.sqrt(h.pow(2).mean(-1, keepdim=True) + eps) * w
+
+
+def residual_norm(x, y=None, *, kind: str, eps: float, post_w=None, add=None, pre_w=None, xb=None, rows=None, dest=None,
+                  top: int = 0):
+    """x (fp32 [T, H], in place) += norm(y) * post_w, then += ``add`` [H]; xb = norm(x) * pre_w in xb's dtype. ``kind``: rms
+    or layer (no bias). Everything but x is optional. With ``dest`` (int32 [T * top]) the sublayer output of token t is
+    sum_j y[dest[t * top + j]] (negative entries: nothing). ``rows`` (int32): only those rows of x are normalised, into
+    xb[0..], and x stays as it is (no y)."""
+    M = x.shape[0] if rows is None else rows.shape[0]
+    H = x.shape[1]
+    if not x.is_cuda:
+        if rows is not None:
+            xb[:M].copy_(norm_ref(x[rows.long()], pre_w, kind, eps).to(xb.dtype))
+            return
+        if y is not None:
+            if dest is not None:
+                d = dest[:M * top].reshape(M, top).long()
+                s = (y[d.clamp_min(0)][..., :H].float() * (d >= 0)[..., None]).sum(1)
+            else:
+                s = y[:M, :H].float()
+            x += s if post_w is None else norm_ref(s, post_w, kind, eps)
+        if add is not None:
+            x += add
+        if pre_w is not None:
+            xb[:M].copy_(norm_ref(x, pre_w, kind, eps).to(xb.dtype))
+        return
+    nv.check(nv.lib().gllm_residual_norm(
+        x.data_ptr(), x.stride(0), nv.ptr(y), 0 if y is None else y.stride(0), 1 if y is None or y.dtype == torch.float32 else 0,
+        nv.ptr(dest), int(top), nv.ptr(post_w), nv.ptr(add), nv.ptr(pre_w), nv.ptr(xb),
+        1 if xb is None or xb.dtype == torch.float32 else 0, M, H, KINDS[kind], float(eps), nv.ptr(rows),
+        0 if xb is None else xb.stride(0), nv.stream_ptr()), "residual_norm")
