@@ -108,6 +108,7 @@ class HybridWorkspace:
         self.buf = {k: torch.zeros(tokens * n, dtype=torch.float32 if k in self.F32 else dt, device=dev)
                     for k, n in need.items()}
         self.decode_ws = None
+        self.latent_scratch: dict = {}         # buffers of split latent decode steps
 
     def take(self, name: str, rows: int, cols: int) -> torch.Tensor:
         return self.buf[name][:rows * cols].view(rows, cols)

@@ -155,7 +155,7 @@ class LatentMixer(_Mixer):
         rows = (None, None) if batch.is_decode else (batch.q_start, batch.q_len)
         MLA.window_latent_attention(ql, cache, batch.block_tables, *rows, batch.ctx_lens,
                                     max_q_len=1 if batch.is_decode else batch.max_q_len, scale=m.scale, window=m.window,
-                                    sinks=w["sink"], out=ol)
+                                    sinks=w["sink"], out=ol, scratch=ws.latent_scratch)
         model.mark("latent_attention")
         o = ws.take("mix", T, m.heads * m.vdim)
         torch.bmm(ol, w["wuv"], out=o.unflatten(1, (m.heads, m.vdim)).transpose(0, 1))

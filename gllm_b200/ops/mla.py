@@ -1,11 +1,15 @@
 """Multi-head latent attention ops: latent cache write and attention over the latent cache.
 
-CUDA path: ``csrc/kernels/mla.cu`` and ``mla_decode.cu`` (latent with a rotated key part), ``mixer_prep.cu`` and
-``attention_any.cu`` (windowed latent attention without positions). CPU path / oracle: plain fp32 PyTorch of the same math.
+CUDA path: ``csrc/kernels/mla.cu`` and ``mla_decode.cu`` (latent with a rotated key part), ``mixer_prep.cu``,
+``latent_attention.cu`` and ``attention_any.cu`` (windowed latent attention without positions). CPU path / oracle: plain fp32
+PyTorch of the same math.
 Reference parity: MlaKvCompress / MlaQAbsorb / MlaAttention
 (src/arch/auto_graph_fragments/build_graph.inc.rs:1486-1578).
 """
 from __future__ import annotations
+
+import ctypes
+from typing import Optional
 
 import torch
 
@@ -17,6 +21,8 @@ nv.register("gllm_mla_attention", I, [P, P, P, I, P, I, P, P, P, P, I, I, I, I, 
 nv.register("gllm_mla_decode_scratch_floats", L, [I, I, I])
 nv.register("gllm_mla_decode", I, [P, P, P, I, P, I, P, I, I, I, F, I, P, L, P])
 
+nv.register("gllm_latent_attention_scratch", L, [I, I, I, I, P])
+nv.register("gllm_latent_attention", I, [P, L, L, P, L, L, P, I, P, I, P, P, P, I, I, I, I, F, I, P, I, P, P, P])
 nv.register("gllm_latent_prep", I, [P, L, I, I, I, I, P, P, F, P, P, P, I, P])
 
 PAGE = 16
@@ -158,10 +164,21 @@ def latent_prep(proj, q_rank, kv_rank, q_w, kv_w, eps, slot_mapping, cq, cache):
                                        cache.data_ptr(), cache.shape[0], nv.stream_ptr()), "latent_prep")
 
 
-def window_latent_attention(q, cache, block_tables, q_start, q_len, ctx_lens, *, max_q_len, scale, window=0, sinks=None, out):
+def latent_splits(n_seqs: int, heads: int, rank: int, keys: int) -> int:
+    """Into how many parts a decode step cuts the ``keys`` of each sequence: one wave of CTAs, at least two 64-token blocks
+    each."""
+    rows = 16 if heads <= 16 else 32 if heads <= 32 else 64
+    units = n_seqs * -(-heads // rows)
+    wave = 148 * (1 if rank > 256 else 2)
+    return max(1, min(wave // units, -(-keys // 128), 16))
+
+
+def window_latent_attention(q, cache, block_tables, q_start, q_len, ctx_lens, *, max_q_len, scale, window=0, sinks=None, out,
+                            scratch: Optional[dict] = None):
     """q [heads, T, rank] (the query with the key up-projection absorbed); cache [pages, 16, rank]; out [heads, T, rank]: the
     weighted latent of each head, causal with a sliding ``window`` (0: everything), ``sinks`` [heads] fp32 in the denominator.
-    ``q_start`` None: a decode step (row = sequence)."""
+    ``q_start`` None: a decode step (row = sequence). ``scratch``: a dict that keeps the buffers of split decode steps from
+    call to call (no splitting without it)."""
     H, T, R = q.shape
     S = ctx_lens.shape[0]
     if not q.is_cuda:
@@ -180,6 +197,25 @@ def window_latent_attention(q, cache, block_tables, q_start, q_len, ctx_lens, *,
                 sc = torch.cat([sc, sinks.float().reshape(H, 1, 1).expand(H, ql, 1)], -1)
             p = torch.softmax(sc, -1)[..., :ctx]
             out[:, st:st + ql] = torch.einsum("hqk,kd->hqd", p, rows).to(out.dtype)
+        return out
+    if (q.dtype == torch.bfloat16 and cache.dtype == q.dtype and R % 8 == 0 and R <= 512
+            and not (q.stride(0) | q.stride(1) | out.stride(0) | out.stride(1)) & 7):
+        splits, buf, cnt = 1, None, None
+        if q_start is None and scratch is not None:
+            keys = block_tables.shape[1] * PAGE
+            splits = latent_splits(S, H, R, min(keys, window + 64) if window > 0 else keys)
+        if splits > 1:
+            key = (S, H, R, splits)
+            if key not in scratch:
+                n_cnt = ctypes.c_int()
+                n = nv.lib().gllm_latent_attention_scratch(S, H, R, splits, ctypes.byref(n_cnt))
+                scratch[key] = (torch.empty(int(n), dtype=torch.float32, device=q.device),
+                                torch.zeros(n_cnt.value, dtype=torch.int32, device=q.device))
+            buf, cnt = scratch[key]
+        nv.check(nv.lib().gllm_latent_attention(
+            q.data_ptr(), q.stride(0), q.stride(1), out.data_ptr(), out.stride(0), out.stride(1), cache.data_ptr(), cache.shape[0],
+            block_tables.data_ptr(), block_tables.shape[1], nv.ptr(q_start), nv.ptr(q_len), ctx_lens.data_ptr(), S, max_q_len, H, R,
+            float(scale), window, nv.ptr(sinks), splits, nv.ptr(buf), nv.ptr(cnt), nv.stream_ptr()), "latent_attention")
         return out
     from .attention import attention_any
     strides = (q.stride(1), q.stride(0), out.stride(1), out.stride(0), PAGE * R, 0, R, 0, 0, R)

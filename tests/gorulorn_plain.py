@@ -184,13 +184,24 @@ def config(layers, width=64, vocab=96, eps=1e-6, loop=None):
 
 
 def weights(cfg, seed=0, sharp=2.0):
-    """Random weights, rounded to bf16. ``sharp`` scales the query weights (one key then stands out in a softmax)."""
+    """Random weights, rounded to bf16. ``sharp`` scales the query weights (one key then stands out in a softmax). With experts
+    every token id has one of four kinds, a strong direction of its embedding, and the router separates the chosen experts
+    of each kind from the others, so that 16-bit rounding does not decide who is chosen."""
     gen = torch.Generator().manual_seed(seed)
     rn = lambda *shape, s=1.0: torch.randn(shape, generator=gen) * s
     lin = lambda o, i, s=1.0: rn(o, i, s=s / math.sqrt(i))
     one = lambda n, s=1.0: s * (1 + 0.2 * rn(n))
     Wd, V = cfg["width"], cfg["vocab"]
     w = {"embed": rn(V, Wd), "head": lin(V, Wd, 2.0), "final.norm": one(Wd)}
+    kinds = torch.linalg.qr(rn(Wd, 4)).Q.T
+    if any(l["mlp"] for l in cfg["layers"]):
+        w["embed"] += 3 * math.sqrt(Wd) * kinds[torch.arange(V) % 4]
+
+    def router(E, top):
+        z = -2 - rn(4, E).abs()
+        for k in range(4):
+            z[k, torch.randperm(E, generator=gen)[:top]] = 0.5 + torch.rand(top, generator=gen)
+        return z.T @ kinds / math.sqrt(Wd) + lin(E, Wd, 0.2)
     if cfg.get("loop"):
         w["loop.step"] = rn(cfg["loop"]["times"], Wd, s=0.7)
     for n, layer in enumerate(cfg["layers"]):
@@ -209,7 +220,7 @@ def weights(cfg, seed=0, sharp=2.0):
         w.update({f"l{n}.norm1": one(Wd), f"l{n}.norm1b": one(Wd, 0.7)})
         if layer["mlp"]:
             f, E = layer["mlp"]["expert"]["ff"], layer["mlp"]["router"]["experts"]
-            w.update({f"l{n}.norm2": one(Wd), f"l{n}.norm2b": one(Wd, 0.7), f"l{n}.mlp.router": lin(E, Wd, 2.0)})
+            w.update({f"l{n}.norm2": 1 + 0.05 * rn(Wd), f"l{n}.norm2b": one(Wd, 0.7), f"l{n}.mlp.router": router(E, layer["mlp"]["router"]["top"])})
             for e in range(E):
                 w.update({f"l{n}.mlp.e{e}.gate": lin(f, Wd, 1.5), f"l{n}.mlp.e{e}.up": lin(f, Wd, 1.5),
                           f"l{n}.mlp.e{e}.down": lin(Wd, f)})

@@ -26,10 +26,10 @@ backend = pytest.mark.parametrize("be", BACKENDS)
 
 def tol(be, cfg=None, w=None, toks=None, want=None):
     """fp32: a fixed small limit. bf16: three times what rounding the projections to bf16 does to the plain statement
-    (a sharp softmax or a cancelling sum turns it into percents), at least 4e-2."""
+    (a sharp softmax or a cancelling sum turns it into percents), at least 2e-2."""
     if be[1] == torch.float32:
         return 2e-4
-    return 4e-2 if cfg is None else max(4e-2, 3 * Z.error(Z.rounded_forward(cfg, w, toks), want))
+    return 4e-2 if cfg is None else max(2e-2, 3 * Z.error(Z.rounded_forward(cfg, w, toks), want))
 
 
 @pytest.fixture(autouse=True)
@@ -206,6 +206,7 @@ EDGES = {"attention": Z.att(conv=1, window=23, keep=11, rot=4), "attention-pages
          "attention-128": Z.att(**BIG, conv=1, window=50, keep=19, rot=4), "attention-conv": Z.att(conv=3, window=30, keep=6, rot=4),
          "latent": Z.lat(window=23), "latent-pages": Z.lat(window=32), "latent-128": Z.lat(heads=2, dim=128, vdim=128, window=50),
          "latent-512": Z.lat(heads=2, kv_rank=512, window=37)}
+EDGE_SEEDS = dict(zip(EDGES, (13, 11, 8, 9, 10, 10, 13, 7)))        # weights with which every edge shows well
 
 
 @backend
@@ -214,7 +215,7 @@ def test_window_and_kept_edges(name, be):
     """Sharp scores over a small vocabulary: a window or a kept range that is one token longer or shorter changes the logits
     far beyond the tolerance, so the right edges pass and no others would."""
     cfg = Z.config([EDGES[name]], vocab=24)
-    w = Z.weights(cfg, seed=6, sharp=6.0)
+    w = Z.weights(cfg, seed=EDGE_SEEDS[name], sharp=6.0)
     toks = Z.tokens(cfg, 170, seed=5)
     want = Z.forward(cfg, w, toks)
     limit = tol(be, cfg, w, toks, want)
@@ -239,7 +240,7 @@ def test_far_keys_among_hundreds(name, be):
              "kept": Z.att(heads=4, kv_heads=2, dim=128, vdim=128, rot=0, conv=1, window=30, keep=8),
              "latent": Z.lat(heads=3, window=450), "latent-128": Z.lat(heads=4, dim=128, vdim=128, window=450)}[name]
     cfg = Z.config([layer], vocab=64)
-    w, toks = Z.weights(cfg, seed=10 if layer["type"] == "latent_attention" else 8, sharp=8.0), Z.tokens(cfg, 420, seed=6)
+    w, toks = Z.weights(cfg, seed=8 if layer["type"] == "latent_attention" else 11, sharp=8.0), Z.tokens(cfg, 420, seed=6)
     toks = [1 if t == 0 else t for t in toks]
     toks[3] = 0                        # the only token of its kind
     want = Z.forward(cfg, w, toks)
