@@ -52,8 +52,11 @@ struct FaParams {
   const int* q_start;        // [S]
   const int* q_len;          // [S]
   const int* ctx_lens;       // [S]
-  const int* block_tables;   // [S, max_blocks]
+  const int* block_tables;   // [S, max_blocks], or null: page i of sequence s is row block page_base[s] + i
+  const int* page_base;
   int max_blocks;
+  // where the 16 x 64 box of (page, K or V, kv head, column half) starts in the tensor map's rows and columns
+  int page_rows, kv_rows, head_rows, kv_cols, head_cols;
   int n_q_heads, n_kv_heads, group;
   int pair_heads;            // 1: the tiles are heads 2y, 2y+1 over the same rows; 0: row blocks 2x, 2x+1 of head y
   float scale_log2;
@@ -214,7 +217,8 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
           tma_load_2d(smem + t * kFaQTile + pn * (kFaQTile / 2), &tmap_q, q_full, tile[t].head * kFaD + pn * 64,
                       qstart + tile[t].row0);
     }
-    const int* bt = p.block_tables + static_cast<long long>(seq) * p.max_blocks;
+    const int* bt = p.block_tables ? p.block_tables + static_cast<long long>(seq) * p.max_blocks : nullptr;
+    const int base = bt ? 0 : p.page_base[seq];
     bool ok = true;
     int issued = 0;
     for (int j = J0; j < J1 && ok; ++j, ++issued) {
@@ -225,7 +229,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       int page = 0;
       if (lane < 4) {
         const int pi = min(kv_tile_of(j) * 4 + lane, n_pages - 1);
-        page = bt[pi];
+        page = bt ? bt[pi] : base + pi;
         if (page < 0 || page >= p.num_pages) {
           if (p.err) atomicCAS(p.err, 0, ERR_BAD_PAGE);
           page = 0;
@@ -243,9 +247,10 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         if (lane == 0) mbar_expect_tx(full, kFaKvTile);
         __syncwarp();
         if (lane < 8) {
-          const int row = ((my_page * 2 + kv) * p.n_kv_heads + kvh) * 16;
+          const int row = my_page * p.page_rows + kv * p.kv_rows + kvh * p.head_rows;
+          const int col = kv * p.kv_cols + kvh * p.head_cols + pn * 64;
           uint8_t* dst = smem + (kv ? kFaOffV : kFaOffK) + stg * kFaKvTile + pn * (kFaKvTile / 2) + (lane >> 1) * 2048;
-          tma_load_2d(dst, &tmap_kv, full, pn * 64, row);
+          tma_load_2d(dst, &tmap_kv, full, col, row);
         }
       }
     }
@@ -457,40 +462,23 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
 using namespace gllm;
 extern "C" int* gllm_error_word();
 
-// Causal (or bidirectional) flash attention over the paged bf16 KV cache for the query tokens of a prefill step.
-// q / out: [total_tokens, n_q_heads, 128] bf16, contiguous. Same semantics as gllm_paged_prefill. full_weights: softmax
-// weights as bf16 pairs; keep: the first `keep` tokens stay visible outside the window.
-GLLM_API int gllm_paged_prefill_tc(const void* q, void* out, const void* kv_cache, int num_pages,
-                                   const int* block_tables, int max_blocks, const int* q_start, const int* q_len,
-                                   const int* ctx_lens, int num_seqs, int max_q_len, int total_tokens, int n_q_heads,
-                                   int n_kv_heads, float scale, int causal, int window, int keep, const float* sinks,
-                                   int full_weights, void* stream) {
-  if (keep > 0 && window < 0) {
-    set_last_error("paged_prefill_tc: kept tokens with a chunked mask");
+// Launch with the geometry fields of `p` and the K / V tensor map set by the caller.
+static int fa_launch(FaParams p, const CUtensorMap& tkv, const void* q, int num_seqs, int max_q_len, int total_tokens,
+                     int full_weights, void* stream) {
+  if (p.keep > 0 && p.window < 0) {
+    set_last_error("prefill_tc: kept tokens with a chunked mask");
     return -1;
   }
-  if (n_kv_heads <= 0 || n_q_heads % n_kv_heads != 0 || total_tokens <= 0) {
-    set_last_error("paged_prefill_tc: heads %d / kv heads %d / tokens %d", n_q_heads, n_kv_heads, total_tokens);
+  if ((reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(p.out) & 15)) {
+    set_last_error("prefill_tc: q / out must be 16-byte aligned");
     return -1;
   }
-  if ((reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) {
-    set_last_error("paged_prefill_tc: q / out must be 16-byte aligned");
-    return -1;
-  }
-  CUtensorMap tq, tkv;
-  const uint64_t kv_rows = uint64_t(num_pages) * 2 * n_kv_heads * 16;
-  if (make_tmap_2d(&tkv, kv_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, kv_rows, kFaD, kFaD, 16, 64)) return -1;
-  const uint64_t q_cols = uint64_t(n_q_heads) * kFaD;
+  CUtensorMap tq;
+  const uint64_t q_cols = uint64_t(p.n_q_heads) * kFaD;
   if (make_tmap_2d(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, uint64_t(total_tokens), q_cols, q_cols, kFaRows, 64))
     return -1;
-  FaParams p = {};
-  p.out = static_cast<__nv_bfloat16*>(out);
-  p.q_start = q_start; p.q_len = q_len; p.ctx_lens = ctx_lens;
-  p.block_tables = block_tables; p.max_blocks = max_blocks;
-  p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads; p.group = n_q_heads / n_kv_heads;
+  p.group = p.n_q_heads / p.n_kv_heads;
   p.pair_heads = (p.group % 2 == 0) ? 1 : 0;
-  p.scale_log2 = scale * 1.4426950408889634f;
-  p.num_pages = num_pages; p.window = window; p.keep = keep; p.causal = causal; p.sinks = sinks;
   p.err = gllm_error_word();
   p.wait_ns = static_cast<unsigned long long>(settings().wait_ns);
   auto kern = full_weights ? fa_prefill_kernel<true> : fa_prefill_kernel<false>;
@@ -501,17 +489,66 @@ GLLM_API int gllm_paged_prefill_tc(const void* q, void* out, const void* kv_cach
   bool& set = attr_set[full_weights ? 1 : 0][dev & 63];
   if (!set) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) { set_last_error("paged_prefill_tc: %s", cudaGetErrorString(e)); return -1; }
+    if (e != cudaSuccess) { set_last_error("prefill_tc: %s", cudaGetErrorString(e)); return -1; }
     set = true;
   }
   const int row_blocks = (max_q_len + kFaRows - 1) / kFaRows;
-  dim3 grid(p.pair_heads ? row_blocks : (row_blocks + 1) / 2, p.pair_heads ? n_q_heads / 2 : n_q_heads, num_seqs);
-  cudaError_t e = launch_kernel(kern, grid, dim3(kFaThreads), smem, (cudaStream_t)stream, true, 0, tq,
-                                tkv, p);
+  dim3 grid(p.pair_heads ? row_blocks : (row_blocks + 1) / 2, p.pair_heads ? p.n_q_heads / 2 : p.n_q_heads, num_seqs);
+  cudaError_t e = launch_kernel(kern, grid, dim3(kFaThreads), smem, (cudaStream_t)stream, true, 0, tq, tkv, p);
   if (e != cudaSuccess) {
     (void)cudaGetLastError();
-    set_last_error("paged_prefill_tc launch: %s", cudaGetErrorString(e));
+    set_last_error("prefill_tc launch: %s", cudaGetErrorString(e));
     return -1;
   }
   return 0;
+}
+
+// Causal (or bidirectional) flash attention over the paged bf16 KV cache for the query tokens of a prefill step.
+// q / out: [total_tokens, n_q_heads, 128] bf16, contiguous. Same semantics as gllm_paged_prefill. full_weights: softmax
+// weights as bf16 pairs; keep: the first `keep` tokens stay visible outside the window.
+GLLM_API int gllm_paged_prefill_tc(const void* q, void* out, const void* kv_cache, int num_pages,
+                                   const int* block_tables, int max_blocks, const int* q_start, const int* q_len,
+                                   const int* ctx_lens, int num_seqs, int max_q_len, int total_tokens, int n_q_heads,
+                                   int n_kv_heads, float scale, int causal, int window, int keep, const float* sinks,
+                                   int full_weights, void* stream) {
+  if (n_kv_heads <= 0 || n_q_heads % n_kv_heads != 0 || total_tokens <= 0) {
+    set_last_error("paged_prefill_tc: heads %d / kv heads %d / tokens %d", n_q_heads, n_kv_heads, total_tokens);
+    return -1;
+  }
+  CUtensorMap tkv;
+  const uint64_t kv_rows = uint64_t(num_pages) * 2 * n_kv_heads * 16;
+  if (make_tmap_2d(&tkv, kv_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, kv_rows, kFaD, kFaD, 16, 64)) return -1;
+  FaParams p = {};
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.q_start = q_start; p.q_len = q_len; p.ctx_lens = ctx_lens;
+  p.block_tables = block_tables; p.max_blocks = max_blocks;
+  p.page_rows = 2 * n_kv_heads * 16; p.kv_rows = n_kv_heads * 16; p.head_rows = 16;
+  p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.num_pages = num_pages; p.window = window; p.keep = keep; p.causal = causal; p.sinks = sinks;
+  return fa_launch(p, tkv, q, num_seqs, max_q_len, total_tokens, full_weights, stream);
+}
+
+// The same over K / V rows that lie token by token: kv [16 * num_pages, n_kv_heads, 2, 128] bf16 (K, then V of each head),
+// token t of sequence s in row 16 * page_base[s] + t. Only tokens a query can see need to be there (page_base may be negative).
+GLLM_API int gllm_rows_prefill_tc(const void* q, void* out, const void* kv, int num_pages, const int* page_base,
+                                  const int* q_start, const int* q_len, const int* ctx_lens, int num_seqs, int max_q_len,
+                                  int total_tokens, int n_q_heads, int n_kv_heads, float scale, int window, const float* sinks,
+                                  int full_weights, void* stream) {
+  if (n_kv_heads <= 0 || n_q_heads % n_kv_heads != 0 || total_tokens <= 0 || num_pages <= 0 || !page_base) {
+    set_last_error("rows_prefill_tc: heads %d / kv heads %d / tokens %d", n_q_heads, n_kv_heads, total_tokens);
+    return -1;
+  }
+  CUtensorMap tkv;
+  const uint64_t cols = uint64_t(n_kv_heads) * 2 * kFaD;
+  if (make_tmap_2d(&tkv, kv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, uint64_t(num_pages) * 16, cols, cols, 16, 64)) return -1;
+  FaParams p = {};
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.q_start = q_start; p.q_len = q_len; p.ctx_lens = ctx_lens;
+  p.page_base = page_base; p.max_blocks = 1 << 26;
+  p.page_rows = 16; p.kv_cols = kFaD; p.head_cols = 2 * kFaD;
+  p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.num_pages = num_pages; p.window = window; p.causal = 1; p.sinks = sinks;
+  return fa_launch(p, tkv, q, num_seqs, max_q_len, total_tokens, full_weights, stream);
 }

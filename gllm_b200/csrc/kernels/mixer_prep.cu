@@ -5,6 +5,8 @@
 //                    of the sequence's slot. One pass: a warp owns one head's channels over a tile of tokens.
 //   latent_prep      RMS norm of the query latent (operand of the query up-projection) and of the key / value latent
 //                    (written to its page), one warp per token and part.
+//   latent_gather    the latent rows a prefill step can see, out of their pages into one matrix (operand of the key / value
+//                    up-projection).
 //
 // Page layout of a layer with n_kv heads of key size D and value size DV: [n_kv][16][D] then [n_kv][16][DV]; of a latent
 // layer: [16][rank]. The convolution ring is the one of recurrent.cuh. Only the first tile of a sequence reads the ring (a
@@ -268,6 +270,23 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const T* proj, long lo
   }
 }
 
+// Latent pages of each sequence from first_page[s] to its end -> rows of `out`, page i at page_base[s] + i.
+__global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* cache, int vecs, const int* block_tables, int max_blocks,
+                                                            const int* ctx_lens, const int* first_page, const int* page_base,
+                                                            uint4* out, int out_pages, int num_pages, int* err) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int s = blockIdx.y, i = first_page[s] + blockIdx.x, dst = page_base[s] + i;
+  if (i >= min((ctx_lens[s] + 15) / 16, max_blocks) || dst < 0 || dst >= out_pages) return;
+  int page = block_tables[static_cast<long long>(s) * max_blocks + i];
+  if (page < 0 || page >= num_pages) {
+    if (err && threadIdx.x == 0) atomicCAS(err, 0, ERR_BAD_PAGE);
+    page = 0;
+  }
+  for (int c = threadIdx.x; c < vecs; c += blockDim.x)
+    out[static_cast<long long>(dst) * vecs + c] = cache[static_cast<long long>(page) * vecs + c];
+}
+
 }  // namespace gllm
 
 using namespace gllm;
@@ -327,4 +346,18 @@ GLLM_API int gllm_latent_prep(const void* proj, long long ld, int is_f32, int M,
   else { if (vec) LATENT(bf16_t, true); else LATENT(bf16_t, false); }
 #undef LATENT
   return prep_done(e, "latent_prep");
+}
+
+// cache [num_pages, 16, R] and out [out_pages, 16, R] bf16 (R a multiple of 8).
+GLLM_API int gllm_latent_gather(const void* cache, int num_pages, int R, const int* block_tables, int max_blocks,
+                                const int* ctx_lens, const int* first_page, const int* page_base, int num_seqs, int max_pages,
+                                void* out, int out_pages, void* stream) {
+  if (num_seqs <= 0 || max_pages <= 0) return 0;
+  if (R % 8 != 0 || num_seqs > 65535) {
+    set_last_error("latent_gather: rank %d, %d sequences", R, num_seqs);
+    return -1;
+  }
+  return prep_done(launch_kernel(latent_gather_kernel, dim3(max_pages, num_seqs), dim3(128), 0, static_cast<cudaStream_t>(stream),
+                                 true, 0, static_cast<const uint4*>(cache), 2 * R, block_tables, max_blocks, ctx_lens, first_page,
+                                 page_base, static_cast<uint4*>(out), out_pages, num_pages, gllm_error_word()), "latent_gather");
 }

@@ -29,6 +29,7 @@ class ForwardBatch:
     causal: bool = True
     want_mtp: bool = False           # also run the model's multi-token-prediction heads on the logits rows
     state_slots: Optional[torch.Tensor] = None  # [S] int32 slot of each sequence's recurrent state (prefill; decode: the row)
+    host_spans: Optional[list] = None  # prefill: (first position, tokens) of each sequence, known to the host
     cp: Optional[object] = None      # parallel.context_parallel.CpPrefill: exchange of KV pages before each attention
 
     @property

@@ -970,7 +970,8 @@ class LLMEngine:
                              block_tables=self.d_pf_bt[:S_], ctx_lens=dp[3 * T + 2 * S_:3 * T + 3 * S_], is_decode=False,
                              q_start=dp[3 * T:3 * T + S_], q_len=dp[3 * T + S_:3 * T + 2 * S_],
                              max_q_len=int(max_q), logits_rows=rows, want_mtp=self.mtp is not None,
-                             state_slots=dp[o + 2 * n_last:o + 2 * n_last + S_])
+                             state_slots=dp[o + 2 * n_last:o + 2 * n_last + S_],
+                             host_spans=[(int(it.start), int(it.len)) for it in plan.prefill] if self.mc.is_hybrid else None)
         self.stats["prefill_steps"] += 1
         self.stats["prefill_tokens"] += int(T)
         self.model.op_timer = getattr(self, "prefill_timer", None)   # utils.tracing.GraphTimer(eager=True) or None

@@ -108,10 +108,19 @@ class HybridWorkspace:
         self.buf = {k: torch.zeros(tokens * n, dtype=torch.float32 if k in self.F32 else dt, device=dev)
                     for k, n in need.items()}
         self.decode_ws = None
+        self.spares: Dict[str, torch.Tensor] = {}
         self.latent_scratch: dict = {}         # buffers of split latent decode steps
 
     def take(self, name: str, rows: int, cols: int) -> torch.Tensor:
         return self.buf[name][:rows * cols].view(rows, cols)
+
+    def spare(self, name: str, rows: int, cols: int) -> torch.Tensor:
+        """A buffer of eager steps whose size is not bounded by the step's tokens: grows on demand."""
+        b = self.spares.get(name)
+        if b is None or b.numel() < rows * cols:
+            self.spares.pop(name, None)
+            b = self.spares[name] = torch.zeros(rows * cols, dtype=self.xb.dtype, device=self.xb.device)
+        return b[:rows * cols].view(rows, cols)
 
 
 class HybridDecoder:

@@ -117,8 +117,10 @@ class AttentionMixer(_Mixer):
 
 
 class LatentMixer(_Mixer):
-    """Latent attention without positions, in absorbed form: the key up-projection moves into the query, the value
-    up-projection behind the attention, and every head attends over the same cached latent rows."""
+    """Latent attention without positions. Absorbed form: the key up-projection moves into the query, the value up-projection
+    behind the attention, and every head attends over the same cached latent rows (decode steps, and any sizes). Prefill
+    steps with head sizes of 128 expand the keys and values of the rows they can see instead: a third of the products, on
+    the tcgen05 attention kernel."""
 
     def pack(self):
         m = self.spec
@@ -128,6 +130,10 @@ class LatentMixer(_Mixer):
         up = lambda n, d: self._src.get(self._p + n).to(self.device, self.dtype).reshape(m.heads, d, m.kv_rank)
         self.w["wuk"] = up("uk", m.dim).contiguous()                           # [heads, dim, rank]
         self.w["wuv"] = up("uv", m.vdim).transpose(1, 2).contiguous()          # [heads, rank, vdim]
+        self.expand = (self.dtype == torch.bfloat16 and self.device.type == "cuda" and m.dim == m.vdim == 128
+                       and m.kv_rank % 8 == 0)
+        if self.expand:
+            self.w["wukv"] = torch.stack([up("uk", 128), up("uv", 128)], 1).reshape(m.heads * 256, m.kv_rank).contiguous()
         self.w["sink"] = self.vec("sink") if m.sink else None
         self.w["wo"] = self.mat("o")
 
@@ -139,6 +145,17 @@ class LatentMixer(_Mixer):
     def alloc(self, num_pages, slots):
         return torch.zeros((num_pages, PAGE, self.spec.kv_rank), dtype=self.dtype, device=self.device)
 
+    def _span(self, batch, T: int):
+        """The expanded form's rows, or None when the step takes the absorbed form: decode steps, and portions so short that
+        expanding their windows costs more than it saves."""
+        if not self.expand or batch.is_decode or batch.host_spans is None:
+            return None
+        spans = batch.__dict__.setdefault("_latent_spans", {})       # the same for every layer with this window
+        if self.spec.window not in spans:
+            span = MLA.LatentSpan(batch.host_spans, self.spec.window, self.device)
+            spans[self.spec.window] = span if span.pages * PAGE <= 4 * T + 1024 else None
+        return spans[self.spec.window]
+
     def forward(self, model, ws, batch, cache, T):
         m, w = self.spec, self.w
         p = L.gemm(ws.xb[:T], w["wdown"], out=ws.take("proj", T, w["wdown"].shape[0]))
@@ -148,6 +165,17 @@ class LatentMixer(_Mixer):
         model.mark("latent_prep")
         q = L.gemm(cq, w["wuq"], out=ws.take("q", T, w["wuq"].shape[0]))
         model.mark("uq_gemm")
+        span = self._span(batch, T)
+        if span is not None:
+            lat = ws.spare("latent_rows", span.pages * PAGE, m.kv_rank)
+            MLA.latent_gather(cache, batch.block_tables, batch.ctx_lens, span, lat)
+            kv = L.gemm(lat, w["wukv"], out=ws.spare("latent_kv", span.pages * PAGE, m.heads * 256))
+            model.mark("ukv_gemm")
+            o = MLA.expanded_prefill(q, kv, span, batch.q_start, batch.q_len, batch.ctx_lens, max_q_len=batch.max_q_len,
+                                     heads=m.heads, scale=m.scale, window=m.window, sinks=w["sink"],
+                                     out=ws.take("mix", T, m.heads * 128))
+            model.mark("latent_prefill")
+            return L.gemm(o, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
         ql = ws.take("qlat", m.heads * T, m.kv_rank).view(m.heads, T, m.kv_rank)
         torch.bmm(q[:, :m.heads * m.dim].unflatten(1, (m.heads, m.dim)).transpose(0, 1), w["wuk"], out=ql)
         model.mark("uk_gemm")

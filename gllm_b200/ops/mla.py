@@ -23,6 +23,8 @@ nv.register("gllm_mla_decode", I, [P, P, P, I, P, I, P, I, I, I, F, I, P, L, P])
 
 nv.register("gllm_latent_attention_scratch", L, [I, I, I, I, P])
 nv.register("gllm_latent_attention", I, [P, L, L, P, L, L, P, I, P, I, P, P, P, I, I, I, I, F, I, P, I, P, P, P])
+nv.register("gllm_latent_gather", I, [P, I, I, P, I, P, P, P, I, I, P, I, P])
+nv.register("gllm_rows_prefill_tc", I, [P, P, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, P])
 nv.register("gllm_latent_prep", I, [P, L, I, I, I, I, P, P, F, P, P, P, I, P])
 
 PAGE = 16
@@ -221,3 +223,38 @@ def window_latent_attention(q, cache, block_tables, q_start, q_len, ctx_lens, *,
     strides = (q.stride(1), q.stride(0), out.stride(1), out.stride(0), PAGE * R, 0, R, 0, 0, R)
     return attention_any(q, out, cache, strides, block_tables, q_start, q_len, ctx_lens, S, max_q_len, H, 1, R, R, scale, True,
                          window, 0, sinks)
+
+
+class LatentSpan:
+    """Which latent rows a prefill step over ``spans`` = [(first position, tokens)] with a sliding ``window`` reads, laid out in
+    one matrix of 16-row pages: sequence s contributes its pages from ``first_page[s]`` (a whole 64-token block) to its end;
+    its page i is page ``page_base[s] + i`` of the matrix."""
+
+    def __init__(self, spans, window: int, device):
+        first = [(max(0, a - window + 1) // 64 * 4 if window > 0 else 0) for a, _ in spans]
+        count = [-(-(a + n) // PAGE) - f for (a, n), f in zip(spans, first)]
+        base, at = [], 0
+        for f, n in zip(first, count):
+            base.append(at - f)
+            at += n
+        self.pages, self.max_pages = at, max(count)
+        both = torch.tensor(first + base, dtype=torch.int32).to(device)
+        self.first_page, self.page_base = both[:len(first)], both[len(first):]
+
+
+def latent_gather(cache, block_tables, ctx_lens, span: LatentSpan, out):
+    """The rows of ``span`` out of the latent pages into ``out`` [span.pages * 16, rank] (CUDA, bf16)."""
+    nv.check(nv.lib().gllm_latent_gather(cache.data_ptr(), cache.shape[0], cache.shape[2], block_tables.data_ptr(),
+                                         block_tables.shape[1], ctx_lens.data_ptr(), span.first_page.data_ptr(),
+                                         span.page_base.data_ptr(), ctx_lens.shape[0], span.max_pages, out.data_ptr(), span.pages,
+                                         nv.stream_ptr()), "latent_gather")
+
+
+def expanded_prefill(q, kv, span: LatentSpan, q_start, q_len, ctx_lens, *, max_q_len, heads, scale, window, sinks, out):
+    """Attention of a prefill step over keys and values expanded from the latents (CUDA, bf16, head sizes 128): q, out
+    [T, heads * 128], kv [span.pages * 16, heads * 256] = key | value of each head. On the tcgen05 kernel."""
+    nv.check(nv.lib().gllm_rows_prefill_tc(q.data_ptr(), out.data_ptr(), kv.data_ptr(), span.pages, span.page_base.data_ptr(),
+                                           q_start.data_ptr(), q_len.data_ptr(), ctx_lens.data_ptr(), ctx_lens.shape[0], max_q_len,
+                                           q.shape[0], heads, heads, float(scale), window, nv.ptr(sinks), 1, nv.stream_ptr()),
+             "rows_prefill_tc")
+    return out
