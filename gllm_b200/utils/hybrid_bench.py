@@ -1,4 +1,6 @@
-"""Throughput of the heterogeneous decoder (Zenevik) beside a dense decoder of equal size: ``bench.py --hybrid``.
+"""Throughput of the heterogeneous decoders beside the closest other decoder of equal size: Zenevik beside a dense decoder
+(``bench.py --hybrid``), Gorulorn beside a mixture-of-experts decoder with the same sliding window (``bench.py --gorulorn``; its
+latent attention also beside the latent kernel of the MLA models, at the same heads, rank and number of keys).
 
 Both models have random weights, the same width, depth, attention heads, feed-forward and vocabulary. Prefill: one forward
 over 4 prompts of 2048 tokens. Decode: one captured step of B sequences at context 2048. Whole steps are timed with CUDA
@@ -13,7 +15,7 @@ from typing import Dict, List
 import torch
 
 from ..engine.batch import ForwardBatch
-from ..models.config import LayerSpec, MixerSpec, ModelConfig
+from ..models.config import LayerSpec, MixerSpec, ModelConfig, MoeSpec
 from ..models.decoder import DecoderModel
 from ..models.hybrid import HybridDecoder
 from ..models.weights import RandomWeights
@@ -26,7 +28,14 @@ SIZES = {
     "2048d64": dict(hidden=2048, heads=32, kv=8, ff=6144, lru=2048, blocks=16, gla=8, dim=64),
     "4096": dict(hidden=4096, heads=32, kv=8, ff=12288, lru=4096, blocks=16, gla=16),
 }
+# width, query / kv heads, heads and ranks of the latent layers, experts
+GORULORN_SIZES = {
+    "1024": dict(hidden=1024, heads=16, kv=4, lat=8, q_rank=512, kv_rank=256, experts=32, top=4, ff=512),
+    "2048": dict(hidden=2048, heads=32, kv=4, lat=16, q_rank=768, kv_rank=512, experts=64, top=8, ff=768),
+    "4096": dict(hidden=4096, heads=32, kv=8, lat=32, q_rank=1536, kv_rank=512, experts=64, top=8, ff=1536),
+}
 VOCAB, CHUNK, PROMPT, PROMPTS = 32768, 2048, 2048, 4
+WINDOW, KEEP = 1024, 64
 
 
 def hybrid_config(s: dict) -> ModelConfig:
@@ -48,6 +57,27 @@ def dense_config(s: dict) -> ModelConfig:
                        max_position_embeddings=1 << 16)
 
 
+def gorulorn_config(s: dict) -> ModelConfig:
+    """Six layers, the middle two run twice: four windowed attention and four latent attention runs."""
+    att = MixerSpec("attention", heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5, rot_dim=64, window=WINDOW,
+                    keep_first=KEEP, taps=4, head_qk_norm=True, o_bias=False)
+    lat = MixerSpec("latent", heads=s["lat"], dim=128, vdim=128, q_rank=s["q_rank"], kv_rank=s["kv_rank"], scale=128 ** -0.5,
+                    window=WINDOW, sink=True)
+    moe = MoeSpec(experts=s["experts"], top=s["top"], ff=s["ff"], scoring="sigmoid", norm_topk=False, scale_input=True)
+    cfg = ModelConfig(arch="gorulorn", hidden_size=s["hidden"], num_layers=6, vocab_size=VOCAB, rms_norm_eps=1e-5, norm_type="layer",
+                      block="sandwich", loop=(2, 4, 2), hidden_act="silu", max_position_embeddings=1 << 16,
+                      layer_specs=[LayerSpec(m, act="silu", moe=moe) for m in (att, lat) * 3])
+    cfg.set_hybrid_dims()
+    return cfg
+
+
+def moe_config(s: dict) -> ModelConfig:
+    return ModelConfig(arch="qwen3_moe", hidden_size=s["hidden"], num_layers=8, num_heads=s["heads"], num_kv_heads=s["kv"],
+                       head_dim=128, intermediate_size=s["ff"], vocab_size=VOCAB, qk_norm=True, sliding_window=WINDOW,
+                       num_experts=s["experts"], num_experts_per_tok=s["top"], moe_intermediate_size=s["ff"],
+                       max_position_embeddings=1 << 16)
+
+
 def _i32(v):
     return torch.tensor(v, dtype=torch.int32, device="cuda")
 
@@ -61,7 +91,7 @@ def prefill_batch() -> ForwardBatch:
                         ctx_lens=_i32([PROMPT] * PROMPTS), q_start=_i32([i * PROMPT for i in range(PROMPTS)]),
                         q_len=_i32([PROMPT] * PROMPTS), max_q_len=PROMPT,
                         logits_rows=_i32([(i + 1) * PROMPT - 1 for i in range(PROMPTS)]),
-                        state_slots=_i32(list(range(PROMPTS))))
+                        state_slots=_i32(list(range(PROMPTS))), host_spans=[(0, PROMPT)] * PROMPTS)
 
 
 def decode_batch(B: int) -> ForwardBatch:
@@ -86,12 +116,54 @@ def work(cfg: ModelConfig, T: int, decode: bool, rows: int) -> Dict[str, tuple]:
         e[1] += bf[1]
     H = cfg.hidden_size
 
-    def attend(heads, kv, d):
-        if decode:      # the whole context is visible
-            add("attention", (T * PROMPT * 2 * kv * d * 2 + T * heads * d * 4, 4 * T * PROMPT * heads * d))
+    def keys(window=0, keep=0):
+        """Keys a query sees: the last one of the prompt in decoding, on average over the prompt in prefill."""
+        window = window or PROMPT
+        see = [min(i + 1, window + min(keep, max(i + 1 - window, 0))) for i in range(PROMPT)]
+        return see[-1] if decode else sum(see) / PROMPT
+
+    def attend(heads, kv, d, window=0, keep=0):
+        n = keys(window, keep)
+        if decode:
+            add("attention", (T * n * 2 * kv * d * 2 + T * heads * d * 4, 4 * T * n * heads * d))
         else:
-            add("attention", (T * (2 * heads + 2 * kv) * d * 2, 4 * T * (PROMPT / 2) * heads * d))
-    if cfg.is_hybrid:
+            add("attention", (T * (2 * heads + 2 * kv) * d * 2, 4 * T * n * heads * d))
+
+    def experts(E, top, ff):
+        used = E * (1 - (1 - top / E) ** T)
+        rows = T * top
+        add("moe_route", _gemm(T, E, H, 4))
+        add("moe_permute", ((T + rows) * H * 2, 0))
+        add("moe_gate_up", (rows * (H + ff) * 2 + used * 2 * ff * H * 2, 4 * rows * ff * H))
+        add("moe_down", (rows * (H + ff) * 2 + used * ff * H * 2, 2 * rows * ff * H))
+    if cfg.block == "sandwich":
+        stream = T * H * (4 + 4 + 2)          # the residual sum read and written, the next operand written
+        for i, _ in cfg.layer_runs():
+            m, moe = cfg.layer_specs[i].mixer, cfg.layer_specs[i].moe
+            if m.kind == "attention":
+                nq, nk = m.heads * m.dim, m.kv_heads * m.dim
+                ring = T * (nq + 2 * nk) * (m.taps + 1) * 4 if decode else 0
+                add("in_gemm", _gemm(T, nq + 2 * nk, H))
+                add("qk_prep", (T * (2 * nq + 4 * nk) * 2 + ring, 0))
+                attend(m.heads, m.kv_heads, m.dim, m.window, m.keep_first)
+                add("out_gemm", _gemm(T, H, nq, 4))
+            else:
+                hd, r, n = m.heads * m.dim, m.kv_rank, keys(m.window)
+                add("in_gemm", _gemm(T, m.q_rank + r, H))
+                add("latent_prep", (T * (m.q_rank + r) * 4, 0))
+                add("uq_gemm", _gemm(T, hd, m.q_rank))
+                if decode:
+                    add("uk_gemm", (T * (hd + m.heads * r) * 2 + hd * r * 2, 2 * T * hd * r))
+                    add("uv_gemm", (T * (hd + m.heads * r) * 2 + hd * r * 2, 2 * T * hd * r))
+                    add("latent_attention", (T * n * r * 2 + T * m.heads * r * 4, 4 * T * n * m.heads * r))
+                else:
+                    add("ukv_gemm", _gemm(T, 2 * hd, r))
+                    add("latent_prefill", (T * 4 * hd * 2, 4 * T * n * hd))
+                add("out_gemm", _gemm(T, H, hd, 4))
+            add("norm", (stream + T * H * 4, 0))
+            experts(moe.experts, moe.top, moe.ff)
+            add("norm", (stream + T * H * 2 * moe.top, 0))
+    elif cfg.is_hybrid:
         for l in cfg.layer_specs:
             m = l.mixer
             if m.kind == "attention":
@@ -125,8 +197,12 @@ def work(cfg: ModelConfig, T: int, decode: bool, rows: int) -> Dict[str, tuple]:
         nq, nk, L = cfg.num_heads * cfg.head_dim, cfg.num_kv_heads * cfg.head_dim, cfg.num_layers
         for _ in range(L):
             add("qkv_gemm", _gemm(T, nq + 2 * nk, H))
-            attend(cfg.num_heads, cfg.num_kv_heads, cfg.head_dim)
+            attend(cfg.num_heads, cfg.num_kv_heads, cfg.head_dim, cfg.sliding_window)
             add("o_proj", (_gemm(T, H, nq)[0] + T * H * 2, 2 * T * H * nq))
+            if cfg.is_moe:
+                experts(cfg.num_experts, cfg.num_experts_per_tok, cfg.moe_intermediate_size)
+                add("moe_combine", (T * H * 2 * (cfg.num_experts_per_tok + 2), 0))
+                continue
             add("gate_up_gemm", (T * H * 2 + 2 * cfg.intermediate_size * H * 2 + T * cfg.intermediate_size * 2,
                                  4 * T * cfg.intermediate_size * H))
             add("down_proj", (_gemm(T, H, cfg.intermediate_size)[0] + T * H * 2, 2 * T * H * cfg.intermediate_size))
@@ -145,6 +221,19 @@ def _table(ms: Dict[str, float], algo: Dict[str, tuple], hbm: float, tf: float) 
     return rows
 
 
+def _timed(fn, steps: int, warmup: int) -> float:
+    for _ in range(max(warmup, 3)):
+        fn()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(steps):
+        fn()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / steps
+
+
 def bench_model(model, steps: int, warmup: int, decode_sizes=(64, 256)) -> dict:
     hbm, tf, _ = _peaks()
     cfg, res = model.cfg, {}
@@ -152,22 +241,14 @@ def bench_model(model, steps: int, warmup: int, decode_sizes=(64, 256)) -> dict:
     for c in kv:
         if isinstance(c, torch.Tensor):
             c.normal_()
-        else:
-            for t in c.t.values():
-                t.normal_()
+            continue
+        if hasattr(c, "pages"):
+            c.pages.normal_()
+        for t in getattr(c, "state", c).t.values():
+            t.normal_()
     model.workspace(PROMPT * PROMPTS)
 
-    def timed(fn):
-        for _ in range(max(warmup, 3)):
-            fn()
-        torch.cuda.synchronize()
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        e0.record()
-        for _ in range(steps):
-            fn()
-        e1.record()
-        torch.cuda.synchronize()
-        return e0.elapsed_time(e1) / steps
+    timed = lambda fn: _timed(fn, steps, warmup)
     b = prefill_batch()
     ms = timed(lambda: model.forward(b, kv))
     model.op_timer = GraphTimer(eager=True)
@@ -205,6 +286,46 @@ def bench_model(model, steps: int, warmup: int, decode_sizes=(64, 256)) -> dict:
                               "ops": _table(ops_ms, work(cfg, B, True, B), hbm, tf)}
         del graphs
     return res
+
+
+def mla_kernel(heads: int, steps: int, warmup: int, decode_sizes=(64, 256)) -> dict:
+    """The latent kernel of the MLA models (rank 512 + 64 rotated dimensions, no window) over WINDOW keys per row in decoding
+    and over whole prompts in prefill: ms and share of the roofline."""
+    from ..ops import mla as MLA
+    hbm, tf, _ = _peaks()
+    res = {}
+    for name, rows, keys in [("prefill", PROMPT * PROMPTS, None)] + [(f"decode_{B}", B, WINDOW) for B in decode_sizes]:
+        seqs = PROMPTS if keys is None else rows
+        per = PROMPT // 16
+        cache = torch.randn(seqs * per, 16, 576, device="cuda").to(torch.bfloat16)
+        bt = torch.arange(seqs * per, dtype=torch.int32, device="cuda").view(seqs, per)
+        if keys is None:
+            bt = bt.repeat_interleave(PROMPT, 0).contiguous()
+            ctx = torch.arange(1, PROMPT + 1, dtype=torch.int32, device="cuda").repeat(PROMPTS)
+        else:
+            ctx = torch.full((rows,), keys, dtype=torch.int32, device="cuda")
+        q = torch.randn(rows, heads * 576, device="cuda").to(torch.bfloat16)
+        out = torch.empty(rows, heads * 512, dtype=torch.bfloat16, device="cuda")
+        ms = _timed(lambda: MLA.latent_decode(q, cache, bt, ctx, n_heads=heads, scale=0.05, max_ctx=PROMPT, out=out), steps, warmup)
+        n = float(ctx.sum())
+        by = (n if keys else PROMPT * PROMPTS) * 576 * 2 + rows * heads * 1088 * 2
+        roof = max(by / (hbm * 1e9), 2 * n * heads * 1088 / (tf * 1e12)) * 1e3
+        res[name] = {"ms": round(ms, 4), "roofline": round(roof / ms, 3)}
+    return res
+
+
+def gorulorn_main(sizes=tuple(GORULORN_SIZES), steps: int = 10, warmup: int = 3) -> dict:
+    out = {}
+    for size in sizes:
+        s = GORULORN_SIZES[size]
+        for name, cls, cfg in (("gorulorn", HybridDecoder, gorulorn_config(s)), ("moe", DecoderModel, moe_config(s))):
+            src = RandomWeights(cfg, "cuda", torch.bfloat16, seed=0)
+            model = cls(cfg, src, device="cuda", dtype=torch.bfloat16, max_positions=PROMPT)
+            out[f"{name}-{size}"] = bench_model(model, steps, warmup)
+            del model, src
+            torch.cuda.empty_cache()
+        out[f"mla-kernel-{size}"] = mla_kernel(s["lat"], steps, warmup)
+    return out
 
 
 def main(sizes=("2048", "2048d64", "4096"), steps: int = 10, warmup: int = 3) -> dict:
