@@ -202,10 +202,187 @@ __global__ void __launch_bounds__(kPrepWarps * 32) conv_qkv_prep_kernel(const Co
   }
 }
 
+// The same for heads of 32, 64, 128 or 256 channels (keys and values alike), up to four taps, rotary halves of whole 8-channel
+// groups: a lane owns 8 consecutive channels of one head, 32 / LPH heads share a warp, the rotary partner is a shuffle away.
+template <typename T> __device__ __forceinline__ void load8(const T* p, float (&v)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      v[2 * i] = __uint_as_float(w[i] << 16);
+      v[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
+    }
+  } else {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+}
+template <typename T> __device__ __forceinline__ void store8(T* p, const float (&v)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
+                                              pack_bf16x2(v[6], v[7]));
+  } else {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  }
+}
+
+template <typename T, int LPH, int TAPS>
+__global__ void __launch_bounds__(kPrepWarps * 32) conv_qkv_prep8_kernel(const ConvPrepParams p) {
+  constexpr int D = LPH * 8, HPW = 32 / LPH, H = TAPS > 1 ? TAPS - 1 : 1;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int units = p.n_q + 2 * p.n_kv;
+  const int unit = (blockIdx.x * kPrepWarps + warp) * HPW + lane / LPH;
+  const bool live = unit < units;
+  pdl_wait();
+  pdl_launch_dependents();
+  if ((blockIdx.x * kPrepWarps + warp) * HPW >= units) return;          // the whole warp
+  const SeqRows s = seq_rows(p.sv, blockIdx.z);
+  const int t0 = blockIdx.y * p.tile;
+  const int n = min(p.tile, s.len - t0);
+  if (n <= 0) return;
+  const int u = live ? unit : 0;
+  const int kind = u < p.n_q ? 0 : u < p.n_q + p.n_kv ? 1 : 2;
+  const int d0 = (lane % LPH) * 8, col0 = u * D + d0;                   // heads of q, k and v follow one another
+  const int channels = units * D;
+  const T* proj = static_cast<const T*>(p.proj) + col0;
+  float w[TAPS > 0 ? TAPS : 1][8], hist[H][8], g[8];
+  if constexpr (TAPS > 0) {
+    float flat[8 * TAPS];                 // the lane's channels follow one another
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) {
+      float f[8];
+      load8(p.conv + static_cast<long long>(col0) * TAPS + i * 8, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) flat[i * 8 + e] = f[e];
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e)
+#pragma unroll
+      for (int t = 0; t < TAPS; ++t) w[t][e] = flat[e * TAPS + t];
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i) {
+      const int t = t0 - 1 - i;
+      if (t >= 0) {
+        load8(proj + static_cast<long long>(s.row0 + t) * p.ld, hist[i]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) hist[i][e] = conv_history(p.ring, s.slot, TAPS, channels, s.start + t, col0 + e);
+      }
+    }
+  }
+  const float* norm_w = kind == 0 ? p.q_w : kind == 1 ? p.k_w : nullptr;
+  if (norm_w) {
+    load8(norm_w + d0, g);
+  } else {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] = 1.f;
+  }
+  const int half = p.rot_dim / 2, hl = half / 8;
+  const bool rot = kind != 2 && d0 < p.rot_dim, upper = d0 >= half;
+  const int partner = rot ? (upper ? lane - hl : lane + hl) : lane, fi = upper ? d0 - half : d0;
+  const long long page_elems = static_cast<long long>(p.n_kv) * 32 * D;
+  const int kv_off = kind == 1 ? (u - p.n_q) * 16 * D + d0 : kind == 2 ? (u - p.n_q) * 16 * D + d0 : 0;   // values behind the keys
+#pragma unroll 4
+  for (int i = 0; i < n; ++i) {
+    const long long m = s.row0 + t0 + i;
+    float y[8];
+    load8(proj + m * p.ld, y);
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        float a = y[e] * w[TAPS - 1][e];
+#pragma unroll
+        for (int k = 0; k < TAPS - 1; ++k) a = fmaf(w[TAPS - 2 - k][e], hist[k][e], a);
+#pragma unroll
+        for (int k = TAPS - 2; k > 0; --k) hist[k][e] = hist[k - 1][e];
+        if constexpr (TAPS > 1) hist[0][e] = y[e];
+        y[e] = a;
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (norm_w) {
+      const float r = 1.f / sqrtf(ss * (1.f / D) + p.eps);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] *= r * g[e];
+    }
+    if (half > 0) {
+      float z[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) z[e] = __shfl_sync(0xffffffffu, y[e], partner);
+      if (rot) {
+        int pos = p.positions[m];
+        if (pos < 0 || pos >= p.max_pos) {
+          if (p.err) atomicCAS(p.err, 0, ERR_BAD_ARG);
+          pos = 0;
+        }
+        float c[8], sn[8];
+        load8(p.cos_t + static_cast<long long>(pos) * half + fi, c);
+        load8(p.sin_t + static_cast<long long>(pos) * half + fi, sn);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = y[e] * c[e] + (upper ? z[e] : -z[e]) * sn[e];
+      }
+    }
+    if (!live) continue;
+    if (kind == 0) {
+      store8(static_cast<T*>(p.q_out) + m * p.n_q * D + col0, y);
+    } else {
+      const int slot = p.slot_mapping ? p.slot_mapping[m] : -1, page = slot >= 0 ? slot / 16 : -1;
+      if (page >= p.num_pages) {
+        if (p.err) atomicCAS(p.err, 0, ERR_BAD_PAGE);
+      } else if (page >= 0) {
+        store8(static_cast<T*>(p.kv) + page * page_elems + kv_off + (slot % 16) * D, y);
+      }
+    }
+  }
+  if (TAPS > 1 && t0 == 0 && live) {
+    for (int i = s.len > TAPS ? s.len - TAPS : 0; i < s.len; ++i) {
+      float v[8];
+      load8(proj + static_cast<long long>(s.row0 + i) * p.ld, v);
+      store8(p.ring + (static_cast<long long>(s.slot) * TAPS + (s.start + i) % TAPS) * channels + col0, v);
+    }
+  }
+}
+
+template <typename T, int LPH>
+static cudaError_t conv_prep8_launch(const ConvPrepParams& p, dim3 grid, cudaStream_t s) {
+  grid.x = (p.n_q + 2 * p.n_kv + kPrepWarps * 32 / LPH - 1) / (kPrepWarps * 32 / LPH);
+#define PREP8(TP) return launch_kernel(conv_qkv_prep8_kernel<T, LPH, TP>, grid, dim3(kPrepWarps * 32), 0, s, true, 0, p)
+  switch (p.taps) {
+    case 0: PREP8(0);
+    case 1: PREP8(1);
+    case 2: PREP8(2);
+    case 3: PREP8(3);
+    default: PREP8(4);
+  }
+#undef PREP8
+}
+
+template <typename T>
+static bool conv_prep8_ok(const ConvPrepParams& p) {
+  const auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  return p.D == p.DV && (p.D == 32 || p.D == 64 || p.D == 128 || p.D == 256) && p.taps <= 4 && p.rot_dim % 16 == 0 &&
+         p.ld % 8 == 0 && al(p.proj) && al(p.q_out) && al(p.kv) && al(p.ring) && al(p.q_w) && al(p.k_w) && al(p.cos_t) && al(p.sin_t) && al(p.conv);
+}
+
 template <typename T>
 static cudaError_t conv_prep_launch(const ConvPrepParams& p, dim3 grid, bool vec, cudaStream_t s) {
   const int dmax = p.D > p.DV ? p.D : p.DV;
   const size_t smem = static_cast<size_t>(kPrepWarps) * dmax * sizeof(float);
+  if (conv_prep8_ok<T>(p)) {
+    switch (p.D) {
+      case 32: return conv_prep8_launch<T, 4>(p, grid, s);
+      case 64: return conv_prep8_launch<T, 8>(p, grid, s);
+      case 128: return conv_prep8_launch<T, 16>(p, grid, s);
+      default: return conv_prep8_launch<T, 32>(p, grid, s);
+    }
+  }
 #define PREP(V, N, TP) return launch_kernel(conv_qkv_prep_kernel<T, V, N, TP>, grid, dim3(kPrepWarps * 32), smem, s, true, 0, p)
 #define PREP_TAPS(V, N)                  \
   switch (p.taps) {                      \
@@ -315,11 +492,12 @@ GLLM_API int gllm_conv_qkv_prep(const int* q_start, const int* q_len, const int*
   ConvPrepParams p = {};
   p.sv = SeqView{q_start, q_len, ctx_lens, slots, n_seqs};
   p.proj = proj; p.ld = ld; p.n_q = n_q; p.n_kv = n_kv; p.D = D; p.DV = DV; p.rot_dim = rot_dim; p.taps = taps;
-  p.tile = taps - 1 > 8 ? taps - 1 : 8;
+  const int rows = q_start ? max_q_len : 1;
+  p.tile = rows >= 1024 ? 32 : rows >= 128 ? 16 : 8;
+  if (p.tile < taps - 1) p.tile = taps - 1;
   p.conv = conv; p.q_w = q_w; p.k_w = k_w; p.eps = eps; p.positions = positions; p.slot_mapping = slot_mapping;
   p.cos_t = cos_t; p.sin_t = sin_t; p.max_pos = max_pos; p.ring = ring; p.q_out = q_out; p.kv = kv;
   p.num_pages = num_pages; p.err = gllm_error_word();
-  const int rows = q_start ? max_q_len : 1;
   dim3 grid((n_q + 2 * n_kv + kPrepWarps - 1) / kPrepWarps, (rows + p.tile - 1) / p.tile, n_seqs);
   if (grid.y > 65535) {
     set_last_error("conv_qkv_prep: portion of %d tokens", rows);
