@@ -790,6 +790,8 @@ class LLMEngine:
     def export_prefix_pages(self, tokens: List[int]):
         """(number of cached full pages, their KV [layers, pages, ...]) of the longest cached prefix of ``tokens`` in this
         pool, or (0, None): what a peer needs to continue the same conversation (KV distribution modes)."""
+        if self.mc.is_hybrid:              # the layers' pages have different shapes: they are not handed on
+            return 0, None
         n_full = len(tokens) // 16
         have = list(self.batcher.lookup_prefix_pages([int(t) for t in tokens[:n_full * 16]])) if n_full else []
         if not have:
@@ -842,7 +844,7 @@ class LLMEngine:
         zigzag = n_full >= 4 * cp_size          # balanced causal work once every rank gets two chunks of some size
         ok = (cp_size > 1 and self.cfg.enable_prefix_cache
               and CpPrefill.every_rank_has_tokens(n_full * 16, cp_size, zigzag)
-              and not self.mc.is_mla and self.pp is None
+              and not self.mc.is_mla and not self.mc.is_hybrid and self.pp is None
               and len(self.batcher.lookup_prefix_pages(prompt[:n_full * 16])) == 0
               and self.batcher.num_free_pages >= n_full + (len(prompt) + int(kw.get("max_tokens", 256))) // 16 + 2)
         if cp_size > 1:

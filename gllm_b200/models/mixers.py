@@ -124,6 +124,10 @@ class LatentMixer(_Mixer):
 
     def pack(self):
         m = self.spec
+        # the batched up-projections are library products: full 32-bit accumulation, no reduced-precision modes
+        torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
+        if self.dtype == torch.float32:
+            torch.backends.cuda.matmul.allow_tf32 = False
         self.w["wdown"] = self.mat("dq", "dkv")
         self.w["q_norm"], self.w["kv_norm"] = self.vec("dq.norm"), self.vec("dkv.norm")
         self.w["wuq"] = self.mat("uq")
