@@ -25,6 +25,7 @@
 
 #include "common.cuh"
 #include "mma.cuh"
+#include "score_mod.cuh"
 
 namespace gllm {
 
@@ -99,10 +100,25 @@ struct SoftmaxState {
 // k_smem / v_smem: shared addresses of the page's K and V tiles, each two 2 KB boxes
 // ([d half][token][64 bf16], 128-byte swizzle). Row r may attend tokens in [lo_r, hi_r).
 // kFW (bf16 pages): the softmax weights enter the second product as a bf16 value and its bf16 remainder.
-template <bool KV8, bool kFW = false>
+// Soft cap and distance bias of a decode step's scores: `pos` is the query's position, `head0` the first head of the group.
+struct DecodeMod {
+  ScoreMod m;
+  int pos, head0, group;
+};
+// Scores of two heads (ha, hb: indices in the group) against tokens t0 and t1, raw -> log2 domain.
+__device__ __forceinline__ void modify_scores(const DecodeMod& d, int ha, int hb, int t0, int t1, float& a0, float& b0, float& a1,
+                                              float& b1) {
+  const int A = d.head0 + (ha < d.group ? ha : 0), B = d.head0 + (hb < d.group ? hb : 0);
+  a0 = score_cap(d.m, a0) + score_bias(d.m, A, d.pos - t0);
+  a1 = score_cap(d.m, a1) + score_bias(d.m, A, d.pos - t1);
+  b0 = score_cap(d.m, b0) + score_bias(d.m, B, d.pos - t0);
+  b1 = score_cap(d.m, b1) + score_bias(d.m, B, d.pos - t1);
+}
+
+template <bool KV8, bool kFW = false, bool MOD = false>
 __device__ __forceinline__ void attend_page(const uint32_t (&qf)[8][4], uint32_t k_smem, uint32_t v_smem,
                                             int tok_base, int lo0, int hi0, int lo1, int hi1, float scale_log2,
-                                            float (&o)[16][4], SoftmaxState& st) {
+                                            float (&o)[16][4], SoftmaxState& st, const DecodeMod* mod = nullptr) {
   const int lane = threadIdx.x & 31;
   float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
   if constexpr (KV8) {
@@ -132,6 +148,14 @@ __device__ __forceinline__ void attend_page(const uint32_t (&qf)[8][4], uint32_t
       mma_bf16_16816(s[0], qf[ks], b0, b1);
       mma_bf16_16816(s[1], qf[ks], b2, b3);
     }
+  }
+  if constexpr (MOD) {
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) {
+      const int t = tok_base + nt * 8 + (lane & 3) * 2;
+      modify_scores(*mod, lane >> 2, (lane >> 2) + 8, t, t + 1, s[nt][0], s[nt][2], s[nt][1], s[nt][3]);
+    }
+    scale_log2 = 1.f;
   }
   // mask + scale (log2 domain); pages that every row of the warp may attend in full skip the mask tests
   float mx0 = -INFINITY, mx1 = -INFINITY;
@@ -301,9 +325,10 @@ __device__ __forceinline__ void softmax_t_finish(SoftmaxStateT& st) {
   }
 }
 // One page: tokens [tok_base, tok_base + 16) of which [lo, hi) may be attended (the same range for every head).
-template <bool kFW>
+template <bool kFW, bool MOD = false>
 __device__ __forceinline__ void attend_page_t(const uint32_t (&qt)[8][2], uint32_t k_smem, uint32_t v_smem, int tok_base,
-                                              int lo, int hi, float scale_log2, float (&o)[8][4], SoftmaxStateT& st) {
+                                              int lo, int hi, float scale_log2, float (&o)[8][4], SoftmaxStateT& st,
+                                              const DecodeMod* mod = nullptr) {
   const int lane = threadIdx.x & 31;
   const int g = lane >> 2;
   float sa[4] = {0.f, 0.f, 0.f, 0.f}, sb[4] = {0.f, 0.f, 0.f, 0.f};   // two accumulation chains over the 8 k-steps
@@ -322,9 +347,11 @@ __device__ __forceinline__ void attend_page_t(const uint32_t (&qt)[8][2], uint32
     }
   }
   // c0: (token g, head 2t)  c1: (token g, head 2t + 1)  c2, c3: token g + 8
+  const int t0 = tok_base + g, t1 = t0 + 8;
+  if constexpr (MOD) scale_log2 = 1.f;
   float s0 = (sa[0] + sb[0]) * scale_log2, s1 = (sa[1] + sb[1]) * scale_log2;
   float s2 = (sa[2] + sb[2]) * scale_log2, s3 = (sa[3] + sb[3]) * scale_log2;
-  const int t0 = tok_base + g, t1 = t0 + 8;
+  if constexpr (MOD) modify_scores(*mod, 2 * (lane & 3), 2 * (lane & 3) + 1, t0, t1, s0, s1, s2, s3);
   if (t0 < lo || t0 >= hi) s0 = s1 = -INFINITY;
   if (t1 < lo || t1 >= hi) s2 = s3 = -INFINITY;
   float mxA = fmaxf(s0, s2), mxB = fmaxf(s1, s3);
@@ -509,6 +536,7 @@ struct DecodeParams {
   int keep;            // with a window: the first `keep` tokens stay visible
   const float* sinks;  // [Hq] learnable sink logits or null
   float v_scale;       // fp8 cache: value = stored * scale (the K scale is folded into scale_log2)
+  ScoreMod mod;        // MOD kernels: soft cap and distance bias
   int* err;
 };
 
@@ -519,7 +547,7 @@ constexpr int kDecSmem = kDecWarps * kDecStages * 2 * kPageBytes + 1024 + 1024;
 // extra warps hide the latency of the per-fragment conversions
 constexpr int kDecSmem8 = kDecWarps * kDecStages * 2 * (kPageBytes / 2) + 1024 + 1024;
 
-template <bool KV8, bool kFW = false>
+template <bool KV8, bool kFW = false, bool MOD = false>
 __global__ void __launch_bounds__(kDecWarps * 32, KV8 ? 3 : 2)
 paged_decode_kernel(const __grid_constant__ CUtensorMap tmap_kv, const DecodeParams p) {
   constexpr int kTile = KvFmt<KV8>::kBytes;
@@ -608,6 +636,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmap_kv, const DecodePar
     }
     return page;
   };
+  [[maybe_unused]] DecodeMod dm;
+  if constexpr (MOD) dm = DecodeMod{p.mod, ctx - 1, kvh * p.group, p.group};
   int ids = fetch_ids(0);        // pages [0, 32) of this warp
   int ids_next = 0;              // pages [32 * c + 32, 32 * c + 64): fetched one chunk ahead
   if (n_my > 32) ids_next = fetch_ids(32);
@@ -634,10 +664,10 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmap_kv, const DecodePar
         attend_page_t8(qt, kaddr, kaddr + kTile, tok_base, lo, hi, p.scale_log2,
                        *reinterpret_cast<float(*)[8][4]>(&o[0][0]), stt);
       else
-        attend_page_t<kFW>(qt, kaddr, kaddr + kTile, tok_base, lo, hi, p.scale_log2,
-                      *reinterpret_cast<float(*)[8][4]>(&o[0][0]), stt);
+        attend_page_t<kFW, MOD>(qt, kaddr, kaddr + kTile, tok_base, lo, hi, p.scale_log2,
+                                *reinterpret_cast<float(*)[8][4]>(&o[0][0]), stt, &dm);
     } else {
-      attend_page<KV8, kFW>(qf, kaddr, kaddr + kTile, tok_base, lo, hi, lo, hi, p.scale_log2, o, st);
+      attend_page<KV8, kFW, MOD>(qf, kaddr, kaddr + kTile, tok_base, lo, hi, lo, hi, p.scale_log2, o, st, &dm);
     }
     __syncwarp();
     const int nxt = i + kDecStages;
@@ -955,12 +985,12 @@ GLLM_API long long gllm_decode_scratch_floats(int batch, int n_q_heads, int max_
   return static_cast<long long>(batch) * n_q_heads * max_splits * (kHD + 1);
 }
 
-template <bool KV8, bool kFW = false>
+template <bool KV8, bool kFW = false, bool MOD = false>
 static int paged_decode_impl(const void* q, void* out, const void* kv_cache, int num_pages,
                              const int* block_tables, int max_blocks, const int* ctx_lens, int batch,
                              int n_q_heads, int n_kv_heads, float scale, int pages_per_split, int max_splits,
                              float* scratch, int* counters, int window, int keep, const float* sinks, float kv_scale,
-                             void* stream) {
+                             void* stream, float softcap = 0.f, const float* bias = nullptr, int nb = 0) {
   if (keep > 0 && window < 0) {
     set_last_error("paged_decode: kept tokens with a chunked mask");
     return -1;
@@ -987,30 +1017,40 @@ static int paged_decode_impl(const void* q, void* out, const void* kv_cache, int
   p.part_o = scratch;
   p.part_lse = scratch ? scratch + static_cast<long long>(batch) * n_q_heads * p.max_splits * kHD : nullptr;
   p.counters = counters; p.num_pages = num_pages; p.window = window; p.keep = keep; p.sinks = sinks;
+  p.mod = make_score_mod(scale, softcap, bias, nb);
   p.err = gllm_error_word();
   static bool attr_set[64] = {};   // per device: the attribute belongs to the device's copy of the kernel
   int dev = 0;
   cudaGetDevice(&dev);
   if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(paged_decode_kernel<KV8, kFW>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(paged_decode_kernel<KV8, kFW, MOD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          KV8 ? kDecSmem8 : kDecSmem);
     if (e != cudaSuccess) { set_last_error("paged_decode: %s", cudaGetErrorString(e)); return -1; }
     attr_set[dev & 63] = true;
   }
   dim3 grid(p.max_splits, n_kv_heads, batch);
-  cudaError_t e = launch_kernel(paged_decode_kernel<KV8, kFW>, grid, dim3(kDecWarps * 32), KV8 ? kDecSmem8 : kDecSmem,
+  cudaError_t e = launch_kernel(paged_decode_kernel<KV8, kFW, MOD>, grid, dim3(kDecWarps * 32), KV8 ? kDecSmem8 : kDecSmem,
                                 (cudaStream_t)stream, true, 0, t, p);
   if (e != cudaSuccess) { (void)cudaGetLastError(); set_last_error("paged_decode launch: %s", cudaGetErrorString(e)); return -1; }
   return 0;
 }
 
 // full_weights: softmax weights as bf16 pairs in the second product. keep: the first `keep` tokens stay visible outside the
-// window.
+// window. softcap, bias [n_q_heads][nb]: capped and biased scores (with full weights).
 GLLM_API int gllm_paged_decode(const void* q, void* out, const void* kv_cache, int num_pages,
                                const int* block_tables, int max_blocks, const int* ctx_lens, int batch,
                                int n_q_heads, int n_kv_heads, float scale, int pages_per_split, int max_splits,
                                float* scratch, int* counters, int window, int keep, const float* sinks, int full_weights,
-                               void* stream) {
+                               float softcap, const float* bias, int nb, void* stream) {
+  if (softcap > 0.f || bias) {
+    if (!full_weights || (bias && nb <= 0)) {
+      set_last_error("paged_decode: capped or biased scores need full weights");
+      return -1;
+    }
+    return paged_decode_impl<false, true, true>(q, out, kv_cache, num_pages, block_tables, max_blocks, ctx_lens, batch,
+                                                n_q_heads, n_kv_heads, scale, pages_per_split, max_splits, scratch, counters,
+                                                window, keep, sinks, 1.f, stream, softcap, bias, nb);
+  }
   if (full_weights)
     return paged_decode_impl<false, true>(q, out, kv_cache, num_pages, block_tables, max_blocks, ctx_lens, batch,
                                           n_q_heads, n_kv_heads, scale, pages_per_split, max_splits, scratch, counters,

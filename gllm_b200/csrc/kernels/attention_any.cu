@@ -3,8 +3,10 @@
 //
 // Keys and values are addressed by strides, so the same kernel covers K / V pages ([kv head][16][D] then [kv head][16][DV])
 // and latent pages ([16][rank], one row per token that is key and value of every head). Masks: causal with a sliding window
-// and kept first tokens, or chunks (attn_first_key), or none. `sinks`: one more logit per head in the denominator.
+// and kept first tokens, or chunks (attn_first_key), or none. Scores may be soft-capped and biased by distance
+// (score_mod.cuh). `sinks`: one more logit per head in the denominator.
 #include "recurrent.cuh"
+#include "score_mod.cuh"
 
 namespace gllm {
 
@@ -22,8 +24,14 @@ struct AnyAttnParams {
   float scale;
   int causal, window, keep, num_pages;
   const float* sinks;
+  float softcap;
+  const float* bias;                                    // [n_q][nb] by distance, the last entry for every longer one
+  int nb;
   int* err;
 };
+
+template <typename T> __device__ __forceinline__ float any_tanh(float x) { return tanh_score(x); }
+template <> __device__ __forceinline__ float any_tanh<float>(float x) { return tanhf(x); }
 
 template <typename T> __device__ __forceinline__ float any_exp(float x) { return __expf(x); }
 template <> __device__ __forceinline__ float any_exp<float>(float x) { return expf(x); }
@@ -74,6 +82,8 @@ __global__ void __launch_bounds__(128) attention_any_kernel(const AnyAttnParams 
       if (d < p.D) s = fmaf(qv[j], to_f(kp[d]), s);
     }
     s = warp_sum(s);
+    if (p.softcap > 0.f) s = p.softcap * any_tanh<T>(s / p.softcap);
+    if (p.bias) s += p.bias[static_cast<long long>(head) * p.nb + min(max(hi - 1 - t, 0), p.nb - 1)];
     const float mn = fmaxf(mx, s);
     const float c = any_exp<T>(mx - mn), w = any_exp<T>(s - mn);
     l = l * c + w;
@@ -114,10 +124,11 @@ extern "C" int* gllm_error_word();
 GLLM_API int gllm_attention_any(const void* q, void* out, const void* kv, const long long* strides, int is_f32, int num_pages,
                                 const int* block_tables, int max_blocks, const int* q_start, const int* q_len,
                                 const int* ctx_lens, int num_seqs, int max_q_len, int n_q, int n_kv, int D, int DV,
-                                float scale, int causal, int window, int keep, const float* sinks, void* stream) {
+                                float scale, int causal, int window, int keep, const float* sinks, float softcap,
+                                const float* bias, int nb, void* stream) {
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
   if (D <= 0 || DV <= 0 || D > 1024 || DV > 1024 || n_kv <= 0 || n_q % n_kv != 0 || num_seqs > 65535 || n_q > 65535 ||
-      (keep > 0 && window < 0)) {
+      (keep > 0 && window < 0) || (bias && (nb <= 0 || !causal))) {
     set_last_error("attention_any: head sizes %d / %d (at most 1024), heads %d / %d", D, DV, n_q, n_kv);
     return -1;
   }
@@ -129,7 +140,8 @@ GLLM_API int gllm_attention_any(const void* q, void* out, const void* kv, const 
   p.block_tables = block_tables; p.max_blocks = max_blocks;
   p.q_start = q_start; p.q_len = q_len; p.ctx_lens = ctx_lens;
   p.n_q = n_q; p.group = n_q / n_kv; p.D = D; p.DV = DV; p.scale = scale;
-  p.causal = causal; p.window = window; p.keep = keep; p.num_pages = num_pages; p.sinks = sinks; p.err = gllm_error_word();
+  p.causal = causal; p.window = window; p.keep = keep; p.num_pages = num_pages; p.sinks = sinks;
+  p.softcap = softcap; p.bias = bias; p.nb = nb; p.err = gllm_error_word();
   dim3 grid((max_q_len + 3) / 4, n_q, num_seqs);
   auto s = static_cast<cudaStream_t>(stream);
   cudaError_t e = is_f32 ? any_launch<float>(p, grid, s) : any_launch<__nv_bfloat16>(p, grid, s);

@@ -9,8 +9,9 @@
 // Online softmax in the exp2 domain; the weights enter the second product as a bf16 value and its bf16 remainder (16 bits
 // of mantissa). Masks: causal with sliding window (and kept first tokens) or chunks (attn_first_key), or none. Blocks outside
 // every row's range are skipped: the kept tokens' blocks come first, then the window's. `sinks`: one more logit per head in
-// the denominator.
+// the denominator. MOD: scores soft-capped and biased by distance (score_mod.cuh).
 #include "mma.cuh"
+#include "score_mod.cuh"
 
 namespace gllm {
 
@@ -28,6 +29,7 @@ struct AmParams {
   float scale_log2;
   int causal, window, keep, num_pages;
   const float* sinks;
+  ScoreMod mod;
   int* err;
 };
 
@@ -40,7 +42,7 @@ __device__ __forceinline__ float am_ex2(float x) {
   return y;
 }
 
-template <int D16, bool SPLIT>
+template <int D16, bool SPLIT, bool MOD>
 __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParams p) {
   constexpr int DP = D16 * 16, P = DP + 8;                 // padded head size, bf16 per shared-memory row
   constexpr int RT = SPLIT ? 16 : 64, NT = SPLIT ? 2 : 8;  // rows per CTA, 8-token score tiles per warp and block
@@ -101,12 +103,18 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
   const int wrow = row0 + (SPLIT ? 0 : warp * 16);
   const bf16_t* qp[2];
   int lo[2], hi[2];
+  [[maybe_unused]] int head[2];
+  [[maybe_unused]] float far[2];                           // bias of every key at the table's end and behind
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int row = wrow + g + r * 8;
     const bool ok = row < qlen * p.group;
     const int t = ok ? row / p.group : 0, hd = kvh * p.group + (ok ? row % p.group : 0);
     qp[r] = p.q + (static_cast<long long>(first + t) * p.n_q + hd) * p.D;
+    if constexpr (MOD) {
+      head[r] = hd;
+      far[r] = score_bias(p.mod, hd, p.mod.nb);
+    }
     hi[r] = ok ? (p.causal ? min(ctx, pos0 + t + 1) : ctx) : 0;
     lo[r] = ok ? (p.causal ? attn_first_key(pos0 + t, p.window) : attn_first_key(ctx - 1, p.window)) : 0;
   }
@@ -165,12 +173,19 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
         }
       }
       float mx[2] = {-INFINITY, -INFINITY};
+      [[maybe_unused]] bool is_far[2];
+      if constexpr (MOD)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) is_far[r] = hi[r] - 1 - (tok0 + NT * 8 - 1) >= p.mod.nb - 1;
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int r = e >> 1, t = tok0 + nt * 8 + t4 * 2 + (e & 1);
-          const float x = ((t >= lo[r] || t < p.keep) && t < hi[r]) ? s[nt][e] * p.scale_log2 : -INFINITY;
+          float y;
+          if constexpr (MOD) y = score_cap(p.mod, s[nt][e]) + (is_far[r] ? far[r] : score_bias(p.mod, head[r], hi[r] - 1 - t));
+          else y = s[nt][e] * p.scale_log2;
+          const float x = ((t >= lo[r] || t < p.keep) && t < hi[r]) ? y : -INFINITY;
           s[nt][e] = x;
           mx[r] = fmaxf(mx[r], x);
         }
@@ -286,7 +301,7 @@ __global__ void __launch_bounds__(kAmThreads) attention_mma_kernel(const AmParam
 using namespace gllm;
 extern "C" int* gllm_error_word();
 
-template <int D16, bool SPLIT>
+template <int D16, bool SPLIT, bool MOD>
 static int am_launch(const AmParams& p, dim3 grid, cudaStream_t s) {
   constexpr int smem_ring = 4 * kAmTok * (D16 * 16 + 8) * 2, smem_merge = 4 * 16 * (D16 * 16 + 2) * 4;
   constexpr int smem = SPLIT && smem_merge > smem_ring ? smem_merge : smem_ring;
@@ -294,11 +309,11 @@ static int am_launch(const AmParams& p, dim3 grid, cudaStream_t s) {
   int dev = 0;
   cudaGetDevice(&dev);
   if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(attention_mma_kernel<D16, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(attention_mma_kernel<D16, SPLIT, MOD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) { set_last_error("attention_mma: %s", cudaGetErrorString(e)); return -1; }
     attr_set[dev & 63] = true;
   }
-  cudaError_t e = launch_kernel(attention_mma_kernel<D16, SPLIT>, grid, dim3(kAmThreads), smem, s, true, 0, p);
+  cudaError_t e = launch_kernel(attention_mma_kernel<D16, SPLIT, MOD>, grid, dim3(kAmThreads), smem, s, true, 0, p);
   if (e != cudaSuccess) {
     (void)cudaGetLastError();
     set_last_error("attention_mma launch: %s", cudaGetErrorString(e));
@@ -312,10 +327,10 @@ static int am_launch(const AmParams& p, dim3 grid, cudaStream_t s) {
 GLLM_API int gllm_attention_mma(const void* q, void* out, const void* kv, int num_pages, const int* block_tables,
                                 int max_blocks, const int* q_start, const int* q_len, const int* ctx_lens, int num_seqs,
                                 int max_q_len, int n_q, int n_kv, int D, int DV, float scale, int causal, int window, int keep,
-                                const float* sinks, void* stream) {
+                                const float* sinks, float softcap, const float* bias, int nb, void* stream) {
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
   if (D <= 0 || D % 8 != 0 || D > 256 || DV <= 0 || DV % 8 != 0 || DV > 256 || n_kv <= 0 || n_q % n_kv != 0 ||
-      num_seqs > 65535 || n_kv > 65535 || (keep > 0 && window < 0)) {
+      num_seqs > 65535 || n_kv > 65535 || (keep > 0 && window < 0) || (bias && (nb <= 0 || !causal))) {
     set_last_error("attention_mma: head sizes %d / %d, heads %d / %d, window %d with %d kept", D, DV, n_q, n_kv, window, keep);
     return -1;
   }
@@ -326,13 +341,17 @@ GLLM_API int gllm_attention_mma(const void* q, void* out, const void* kv, int nu
   p.n_q = n_q; p.n_kv = n_kv; p.group = n_q / n_kv; p.D = D; p.DV = DV;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.causal = causal; p.window = window; p.keep = keep; p.sinks = sinks; p.num_pages = num_pages; p.err = gllm_error_word();
+  p.mod = make_score_mod(scale, softcap, bias, nb);
+  const bool mod = softcap > 0.f || bias;
   const int rows = max_q_len * p.group;
   const bool split = rows <= 16;
   dim3 grid(split ? 1 : (rows + 63) / 64, n_kv, num_seqs);
   auto s = static_cast<cudaStream_t>(stream);
   const int d16 = ((D > DV ? D : DV) + 15) / 16;
 #define AM_CASE(N) \
-  if (d16 <= N) return split ? am_launch<N, true>(p, grid, s) : am_launch<N, false>(p, grid, s)
+  if (d16 <= N)   \
+  return mod ? (split ? am_launch<N, true, true>(p, grid, s) : am_launch<N, false, true>(p, grid, s)) \
+             : (split ? am_launch<N, true, false>(p, grid, s) : am_launch<N, false, false>(p, grid, s))
   AM_CASE(1);
   AM_CASE(2);
   AM_CASE(4);

@@ -342,6 +342,11 @@ __device__ __forceinline__ float bf16_round(float x) { return __bfloat162float(_
 // Activations on the fast-math units (ex2 + rcp, a few ulp: far below the bf16 rounding of the result). An IEEE
 // division here made the SwiGLU epilogue of a 256 x 192 tile cost 43 k clocks (measured), longer than many main loops.
 __device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
+// Activation of a projection's output columns: 1 silu, 2 square of relu.
+__device__ __forceinline__ float store_act(float x, int act) {
+  const float r = fmaxf(x, 0.f);
+  return act == 1 ? silu_f(x) : act == 2 ? r * r : x;
+}
 __device__ __forceinline__ float gelu_tanh_f(float x) {
   // 0.5 x (1 + tanh y) = x * sigmoid(2 y),  y = sqrt(2/pi) (x + 0.044715 x^3)
   const float k0 = 0.7978845608028654f, k1 = 0.044715f;

@@ -25,7 +25,7 @@
 //
 // Every wait is bounded (settings().wait_ns); a wait that runs out raises the status word, all roles leave their
 // loops, the producer waits (bounded) for its copies in flight and the TMEM columns are freed.
-#include "common.cuh"
+#include "score_mod.cuh"
 
 namespace gllm {
 
@@ -64,6 +64,7 @@ struct FaParams {
   int window, causal;
   int keep;                  // with a window: the first `keep` tokens stay visible
   const float* sinks;
+  ScoreMod mod;              // MOD kernels: soft cap and distance bias
   int* err;
   unsigned long long wait_ns;
 };
@@ -97,13 +98,46 @@ __device__ __forceinline__ uint64_t umma_desc_sw128_mn(uint32_t smem_addr, uint3
   return d;
 }
 
+// 64 raw scores of one row against tokens t0 ..: soft cap, then the bias by distance (`n0`: distance to t0, `far`: the bias
+// at the table's end). The choice between the forms of tanh is the warp's, so it costs one vote.
+__device__ __forceinline__ void modify_scores(const ScoreMod& m, int head, int n0, float far, uint32_t (&sr)[2][32]) {
+  float big = 0.f;
+#pragma unroll
+  for (int h = 0; h < 2; ++h)
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      const float z = __uint_as_float(sr[h][i]) * m.in;
+      sr[h][i] = __float_as_uint(z);
+      big = fmaxf(big, fabsf(z));
+    }
+  const bool is_far = n0 - (kFaKv - 1) >= m.nb - 1;
+  auto each = [&](auto f) {
+    if (__all_sync(0xffffffffu, is_far)) {
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int i = 0; i < 32; ++i) sr[h][i] = __float_as_uint(f(__uint_as_float(sr[h][i])) + far);
+    } else {
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+          sr[h][i] = __float_as_uint(f(__uint_as_float(sr[h][i])) + score_bias(m, head, n0 - h * 32 - i));
+    }
+  };
+  const float out = m.out;
+  if (out <= 0.f) each([](float z) { return z; });
+  else if (__all_sync(0xffffffffu, big <= kTanhSmall)) each([out](float z) { return out * tanh_small(z); });
+  else each([out](float z) { return out * tanh_score(z); });
+}
+
 // KV token range of one query tile: tiles [j0, j1) of 64 tokens, counted in visiting order (see `kv_tile_of`).
 struct FaTile {
   int head, row0, rows;   // rows = valid query rows (0: the tile does not exist)
   int j0, j1;
 };
 
-template <bool kFW>
+template <bool kFW, bool MOD>
 __global__ void __launch_bounds__(kFaThreads, 1)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
                   const FaParams p) {
@@ -354,6 +388,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       const int lo = attn_first_key(pos, p.window);
       uint8_t* p_row = smem + kFaOffP + t * kFaPTile + (row >> 3) * 1024 + (row & 7) * 128;
       float m = -INFINITY, l = 0.f;
+      [[maybe_unused]] const float far = MOD ? score_bias(p.mod, ti.head, p.mod.nb) : 0.f;
       bool ok = true;
       for (int j = ti.j0; j < ti.j1; ++j) {
         const int c = j - ti.j0;
@@ -367,11 +402,12 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         const int t0 = kv_tile_of(j) * kFaKv;
         const bool full_tile = t0 >= lo && t0 + kFaKv - 1 <= hi;
         float mx = -INFINITY;
+        if constexpr (MOD) modify_scores(p.mod, ti.head, pos - t0, far, sr);
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            float x = __uint_as_float(sr[h][i]) * p.scale_log2;
+            float x = MOD ? __uint_as_float(sr[h][i]) : __uint_as_float(sr[h][i]) * p.scale_log2;
             if (!full_tile) {
               const int tk = t0 + h * 32 + i;
               if ((tk < lo && tk >= p.keep) || tk > hi) x = -INFINITY;
@@ -481,12 +517,17 @@ static int fa_launch(FaParams p, const CUtensorMap& tkv, const void* q, int num_
   p.pair_heads = (p.group % 2 == 0) ? 1 : 0;
   p.err = gllm_error_word();
   p.wait_ns = static_cast<unsigned long long>(settings().wait_ns);
-  auto kern = full_weights ? fa_prefill_kernel<true> : fa_prefill_kernel<false>;
+  const bool mod = p.mod.out > 0.f || p.mod.bias;
+  if (mod && (!full_weights || !p.causal)) {
+    set_last_error("prefill_tc: capped or biased scores need causal attention with full weights");
+    return -1;
+  }
+  auto kern = mod ? fa_prefill_kernel<true, true> : full_weights ? fa_prefill_kernel<true, false> : fa_prefill_kernel<false, false>;
   const int smem = full_weights ? kFaSmemOf<true> : kFaSmemOf<false>;
-  static bool attr_set[2][64] = {};
+  static bool attr_set[3][64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
-  bool& set = attr_set[full_weights ? 1 : 0][dev & 63];
+  bool& set = attr_set[mod ? 2 : full_weights ? 1 : 0][dev & 63];
   if (!set) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) { set_last_error("prefill_tc: %s", cudaGetErrorString(e)); return -1; }
@@ -510,7 +551,7 @@ GLLM_API int gllm_paged_prefill_tc(const void* q, void* out, const void* kv_cach
                                    const int* block_tables, int max_blocks, const int* q_start, const int* q_len,
                                    const int* ctx_lens, int num_seqs, int max_q_len, int total_tokens, int n_q_heads,
                                    int n_kv_heads, float scale, int causal, int window, int keep, const float* sinks,
-                                   int full_weights, void* stream) {
+                                   int full_weights, float softcap, const float* bias, int nb, void* stream) {
   if (n_kv_heads <= 0 || n_q_heads % n_kv_heads != 0 || total_tokens <= 0) {
     set_last_error("paged_prefill_tc: heads %d / kv heads %d / tokens %d", n_q_heads, n_kv_heads, total_tokens);
     return -1;
@@ -526,6 +567,7 @@ GLLM_API int gllm_paged_prefill_tc(const void* q, void* out, const void* kv_cach
   p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.num_pages = num_pages; p.window = window; p.keep = keep; p.causal = causal; p.sinks = sinks;
+  p.mod = make_score_mod(scale, softcap, bias, nb);
   return fa_launch(p, tkv, q, num_seqs, max_q_len, total_tokens, full_weights, stream);
 }
 

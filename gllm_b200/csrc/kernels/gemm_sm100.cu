@@ -158,6 +158,7 @@ struct GemmParams {
   long long ar_ll_res_off, ar_ll_res_bytes;     // same for the result slots ([M][n_pad] bf16)
   int ar_drop_flags;          // test hook: leave the tile flags unset (push) / the tiles unsent (ll): the waits run out
   float softcap;              // EPI_STORE, unsplit launches only: out = softcap * tanh(out / softcap) (0 = off)
+  int act, act_cols;          // EPI_STORE: columns [0, act_cols) of the result pass store_act(act) (0 = off)
   // Grouped GEMMs: rows that exist in every 128-row block (the rest of a block is padding: a block of an expert with
   // 16 routed rows has 112 of them). When given, the producer loads only ceil(rows / 32) * 32 rows of the A tile
   // (32-row boxes through the third tensor map) and the epilogue neither reads nor stores the padding rows.
@@ -421,6 +422,9 @@ __device__ __forceinline__ void apply_unit_epilogue(const GemmParams& p, int m, 
             v[j] *= rs;
             if (p.b_scale) v[j] *= p.b_scale[n0 + j];
             if (p.bias) v[j] += p.bias[n0 + j];
+            if constexpr (EPI == EPI_STORE) {
+              if (p.act && n0 + j < p.act_cols) v[j] = store_act(v[j], p.act);
+            }
           }
           if constexpr (EPI == EPI_RESIDUAL) {
             // pre_residual: the 4 residual values of this lane, loaded by the caller ahead of a long-latency phase
@@ -2070,6 +2074,11 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
 #pragma unroll
                   for (int j = 0; j < 32; ++j) v[j] = p.softcap * tanhf(v[j] * inv_cap);
                 }
+                if (p.act) {
+#pragma unroll
+                  for (int j = 0; j < 32; ++j)
+                    if (n0 + j < p.act_cols) v[j] = store_act(v[j], p.act);
+                }
               }
               if (p.scatter_meta) {
                 if (row_ok) {
@@ -2956,6 +2965,17 @@ GLLM_API int gllm_gemm_bf16_softcap(const void* A, long long lda, const void* B,
   p.softcap = softcap;
   p.err = gllm_error_word();
   return dispatch_gemm<EPI_STORE, false>(A, lda, B, ldb, N, p, bn, (cudaStream_t)stream, 0, 1);
+}
+
+// gllm_gemm_bf16 with an activation on columns [0, act_cols) of the result (1 silu, 2 square of relu).
+GLLM_API int gllm_gemm_bf16_act(const void* A, long long lda, const void* B, long long ldb, void* out, long long ldo, int M,
+                                int N, int K, int out_f32, const float* bias, int bn, int act, int act_cols, void* stream) {
+  GemmParams p = {};
+  p.M = M; p.N = N; p.K = K;
+  p.out = out; p.ldo = ldo; p.out_f32 = out_f32; p.bias = bias;
+  p.act = act; p.act_cols = act_cols;
+  p.err = gllm_error_word();
+  return dispatch_gemm<EPI_STORE, false>(A, lda, B, ldb, N, p, bn, (cudaStream_t)stream, 0, 0);
 }
 
 // out[M,N] = A · Bᵀ (+bias) + residual ; row_ss_out[M, ceil(N/bn)] receives per-tile sums of squares.

@@ -1,9 +1,10 @@
-// Windowed latent attention in absorbed form on warp-level tensor cores: every head attends over the same cached latent rows
-// (one per token, rank R, key and value at once), so the rows of a query tile are (token, head) pairs and each latent tile
-// is read once for all of them. bf16 latents, R a multiple of 8 up to 512.
+// Latent attention in absorbed form on warp-level tensor cores: every head attends over the same cached rows (one per token: RK
+// channels are its key, the first R of them, the latent, its value; the rest is a rotated key part), so the rows of a query tile
+// are (token, head) pairs and each tile of the cache is read once for all of them. bf16, R up to 512, RK up to 576, multiples
+// of 8. Causal, with a sliding window or without.
 //
 // Eight warps work on RG groups of 16 rows; the CS = 8 / RG warps of a group share its work, first by tokens, then by columns:
-//   scores   warp (g, c): 16 rows x 64 / CS tokens of the block over all R channels
+//   scores   warp (g, c): 16 rows x 64 / CS tokens of the block over all RK channels
 //   softmax  online, exp2 domain; row maxima through shared memory; the weights go to shared memory as a bf16 value and its
 //            bf16 remainder (16 bits of mantissa)
 //   values   warp (g, c): 16 rows x every CS-th 16-column tile over the block's 64 tokens
@@ -19,12 +20,12 @@ constexpr int kLaTok = 64, kLaThreads = 256, kLaPs = kLaTok + 8;
 struct LatentAttnParams {
   const bf16_t* q;
   bf16_t* out;
-  const bf16_t* kv;                                     // [pages][16][R]
+  const bf16_t* kv;                                     // [pages][16][RK]
   long long q_tok, q_head, o_tok, o_head;               // strides in elements
   const int* block_tables;
   int max_blocks;
   const int *q_start, *q_len, *ctx_lens;                // q_start null: decode, row = sequence index, one token where ctx > 0
-  int heads, R, window, num_pages, splits;
+  int heads, R, RK, window, num_pages, splits;
   float scale_log2;
   const float* sinks;
   float *part_o, *part_ml;                              // [units][splits][rows][R], [units][splits][rows][2]
@@ -38,15 +39,16 @@ __device__ __forceinline__ float la_ex2(float x) {
   return y;
 }
 
-template <int RP, int RG> struct LaShape {
-  static constexpr int P = RP + 8, CS = 8 / RG, RT = RG * 16, TW = kLaTok / CS, NT = TW / 8, NC = RP / (16 * CS);
+// RP: key channels, padded; RV: value channels, padded
+template <int RP, int RV, int RG> struct LaShape {
+  static constexpr int P = RP + 8, CS = 8 / RG, RT = RG * 16, TW = kLaTok / CS, NT = TW / 8, NC = RV / (16 * CS);
   static constexpr int kKv = 2 * kLaTok * P * 2, kQ = RT * P * 2, kP = 2 * RT * kLaPs * 2, kRed = 2 * CS * RT * 4;
   static constexpr int kSmem = kKv + kQ + kP + kRed + 16;
 };
 
-template <int RP, int RG>
+template <int RP, int RV, int RG>
 __global__ void __launch_bounds__(kLaThreads) latent_attention_kernel(const LatentAttnParams p) {
-  using Sh = LaShape<RP, RG>;
+  using Sh = LaShape<RP, RV, RG>;
   constexpr int P = Sh::P, CS = Sh::CS, RT = Sh::RT, NT = Sh::NT, NC = Sh::NC;
   extern __shared__ __align__(16) uint8_t la_smem[];
   bf16_t* kv_s = reinterpret_cast<bf16_t*>(la_smem);                       // [2][64][P]
@@ -68,18 +70,18 @@ __global__ void __launch_bounds__(kLaThreads) latent_attention_kernel(const Late
     if (p.err && tid == 0) atomicCAS(p.err, 0, ERR_BAD_ARG);
     ctx = p.max_blocks * 16;
   }
-  const int first = p.q_start ? p.q_start[seq] : seq, pos0 = ctx - qlen, R = p.R;
+  const int first = p.q_start ? p.q_start[seq] : seq, pos0 = ctx - qlen, R = p.R, RK = p.RK;
   const int last_row = min(row0 + RT, n_rows) - 1;
   const int kv_lo = attn_first_key(pos0 + row0 / p.heads, p.window), kv_hi = min(ctx, pos0 + last_row / p.heads + 1);
   const int blk0 = kv_lo / kLaTok, blks = (kv_hi + kLaTok - 1) / kLaTok - blk0, n_pages = (ctx + 15) / 16;
   const int j0 = blk0 + blks * split / p.splits, j1 = blk0 + blks * (split + 1) / p.splits;
 
-  // columns behind the rank read as zero
-  const int r32 = min((R + 31) / 32 * 32, P);
-  for (int i = tid; i < (2 * kLaTok + RT) * (r32 - R); i += kLaThreads)
-    (i / (r32 - R) < 2 * kLaTok ? kv_s + (i / (r32 - R)) * P : q_s + (i / (r32 - R) - 2 * kLaTok) * P)[R + i % (r32 - R)] =
+  // columns behind the key read as zero
+  const int r32 = min((RK + 31) / 32 * 32, P);
+  for (int i = tid; i < (2 * kLaTok + RT) * (r32 - RK); i += kLaThreads)
+    (i / (r32 - RK) < 2 * kLaTok ? kv_s + (i / (r32 - RK)) * P : q_s + (i / (r32 - RK) - 2 * kLaTok) * P)[RK + i % (r32 - RK)] =
         __float2bfloat16_rn(0.f);
-  const int vecs = R / 8;
+  const int vecs = RK / 8;
   for (int r = warp; r < RT; r += 8) {                  // query rows (rows behind the last one are zero)
     const int row = row0 + r;
     const bf16_t* src = p.q + (row % p.heads) * p.q_head + static_cast<long long>(first + row / p.heads) * p.q_tok;
@@ -101,7 +103,7 @@ __global__ void __launch_bounds__(kLaThreads) latent_attention_kernel(const Late
     for (int k = 0; k < kLaTok / 8; ++k) {
       const int r = warp + 8 * k;
       const long long pg = __shfl_sync(0xffffffffu, page, r >> 4);
-      const bf16_t* src = p.kv + (pg * 16 + (r & 15)) * R;
+      const bf16_t* src = p.kv + (pg * 16 + (r & 15)) * RK;
       bf16_t* dst = kv_s + (stage * kLaTok + r) * P;
       for (int c = lane; c < vecs; c += 32)
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst + c * 8)), "l"(src + c * 8) : "memory");
@@ -122,7 +124,7 @@ __global__ void __launch_bounds__(kLaThreads) latent_attention_kernel(const Late
   for (int i = 0; i < 2 * NC; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const uint32_t qa = smem_u32(q_s + (rg * 16 + (lane & 15)) * P + (lane >> 4) * 8);
-  const int ksteps2 = (R + 31) / 32;                    // pairs of 16-channel steps
+  const int ksteps2 = (RK + 31) / 32;                   // pairs of 16-channel steps
 
   if (j0 < j1) load(j0, 0);
   for (int j = j0; j < j1; ++j) {
@@ -312,22 +314,23 @@ __global__ void __launch_bounds__(kLaThreads) latent_attention_kernel(const Late
   if (tid == 0) p.counters[unit] = 0;
 }
 
-template <int RP, int RG>
+template <int RP, int RV, int RG>
 static cudaError_t la_launch(const LatentAttnParams& p, int rows, int n_seqs, cudaStream_t s) {
-  constexpr int smem = LaShape<RP, RG>::kSmem;
+  constexpr int smem = LaShape<RP, RV, RG>::kSmem;
+  static_assert(smem <= 227 * 1024, "shared memory of one CTA");
   static bool attr_set[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<RP, RG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<RP, RV, RG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return e;
     attr_set[dev & 63] = true;
   }
   const dim3 grid((rows + RG * 16 - 1) / (RG * 16), p.splits, n_seqs);
-  return launch_kernel(latent_attention_kernel<RP, RG>, grid, dim3(kLaThreads), smem, s, true, 0, p);
+  return launch_kernel(latent_attention_kernel<RP, RV, RG>, grid, dim3(kLaThreads), smem, s, true, 0, p);
 }
 
-static int la_row_groups(int rows) { return rows <= 16 ? 1 : rows <= 32 ? 2 : 4; }
+static int la_row_groups(int rows, int RK) { return rows <= 16 ? 1 : rows <= 32 || RK > 512 ? 2 : 4; }
 
 }  // namespace gllm
 
@@ -335,24 +338,24 @@ using namespace gllm;
 extern "C" int* gllm_error_word();
 
 // Scratch of a decode step with `splits` parts per key range: floats (part_o, part_ml); *counters = int32 counters needed.
-GLLM_API long long gllm_latent_attention_scratch(int num_seqs, int heads, int R, int splits, int* counters) {
-  const int rt = la_row_groups(heads) * 16;
+GLLM_API long long gllm_latent_attention_scratch(int num_seqs, int heads, int R, int RK, int splits, int* counters) {
+  const int rt = la_row_groups(heads, RK) * 16;
   const long long units = static_cast<long long>(num_seqs) * ((heads + rt - 1) / rt);
   if (counters) *counters = static_cast<int>(units);
   return splits > 1 ? units * splits * rt * (R + 2) : 0;
 }
 
 // q, out: element (head, token, c) at head * head_stride + token * tok_stride + c, both strides multiples of 8. cache
-// [num_pages, 16, R] bf16. q_start null: a decode step. splits > 1 (decode steps): scratch and zeroed counters as above.
+// [num_pages, 16, RK] bf16; q has RK columns, out R. q_start null: a decode step. splits > 1 (decode steps): scratch and zeroed counters as above.
 GLLM_API int gllm_latent_attention(const void* q, long long q_head, long long q_tok, void* out, long long o_head, long long o_tok,
                                    const void* cache, int num_pages, const int* block_tables, int max_blocks,
                                    const int* q_start, const int* q_len, const int* ctx_lens, int num_seqs, int max_q_len,
-                                   int heads, int R, float scale, int window, const float* sinks, int splits, float* scratch,
+                                   int heads, int R, int RK, float scale, int window, const float* sinks, int splits, float* scratch,
                                    int* counters, void* stream) {
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
-  if (R <= 0 || R % 8 != 0 || R > 512 || heads <= 0 || num_seqs > 65535 || splits < 1 || splits > 64 || window < 0 ||
+  if (R <= 0 || R % 8 != 0 || R > 512 || RK < R || RK % 8 != 0 || RK > 576 || heads <= 0 || num_seqs > 65535 || splits < 1 || splits > 64 || window < 0 ||
       ((q_head | q_tok | o_head | o_tok) & 7) || (splits > 1 && (q_start || !scratch || !counters))) {
-    set_last_error("latent_attention: rank %d (a multiple of 8, at most 512), %d heads, %d splits", R, heads, splits);
+    set_last_error("latent_attention: rank %d of %d channels (multiples of 8, at most 512 of 576), %d heads, %d splits", R, RK, heads, splits);
     return -1;
   }
   LatentAttnParams p = {};
@@ -360,10 +363,10 @@ GLLM_API int gllm_latent_attention(const void* q, long long q_head, long long q_
   p.q_tok = q_tok; p.q_head = q_head; p.o_tok = o_tok; p.o_head = o_head;
   p.block_tables = block_tables; p.max_blocks = max_blocks;
   p.q_start = q_start; p.q_len = q_len; p.ctx_lens = ctx_lens;
-  p.heads = heads; p.R = R; p.window = window; p.num_pages = num_pages; p.splits = splits;
+  p.heads = heads; p.R = R; p.RK = RK; p.window = window; p.num_pages = num_pages; p.splits = splits;
   p.scale_log2 = scale * 1.4426950408889634f; p.sinks = sinks; p.err = gllm_error_word();
   const int rows = (q_start ? max_q_len : 1) * heads;
-  const int rg = la_row_groups(rows);
+  const int rg = la_row_groups(rows, RK);
   if (splits > 1) {
     const long long units = static_cast<long long>(num_seqs) * ((rows + rg * 16 - 1) / (rg * 16));
     p.part_o = scratch;
@@ -372,10 +375,13 @@ GLLM_API int gllm_latent_attention(const void* q, long long q_head, long long q_
   }
   auto s = static_cast<cudaStream_t>(stream);
   cudaError_t e;
-#define LA_RANK(RP) e = rg == 1 ? la_launch<RP, 1>(p, rows, num_seqs, s) : rg == 2 ? la_launch<RP, 2>(p, rows, num_seqs, s) : la_launch<RP, 4>(p, rows, num_seqs, s)
-  if (R <= 128) LA_RANK(128);
-  else if (R <= 256) LA_RANK(256);
-  else LA_RANK(512);
+#define LA_RANK(RP, RV) e = rg == 1 ? la_launch<RP, RV, 1>(p, rows, num_seqs, s) : rg == 2 ? la_launch<RP, RV, 2>(p, rows, num_seqs, s) : la_launch<RP, RV, 4>(p, rows, num_seqs, s)
+  if (RK <= 128) LA_RANK(128, 128);
+  else if (R <= 128 && RK <= 192) LA_RANK(192, 128);
+  else if (RK <= 256) LA_RANK(256, 256);
+  else if (R <= 256 && RK <= 320) LA_RANK(320, 256);
+  else if (RK <= 512) LA_RANK(512, 512);
+  else e = rg == 1 ? la_launch<576, 512, 1>(p, rows, num_seqs, s) : la_launch<576, 512, 2>(p, rows, num_seqs, s);
 #undef LA_RANK
   if (e != cudaSuccess) {
     (void)cudaGetLastError();

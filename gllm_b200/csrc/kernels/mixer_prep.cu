@@ -5,11 +5,13 @@
 //                    of the sequence's slot. One pass: a warp owns one head's channels over a tile of tokens.
 //   latent_prep      RMS norm of the query latent (operand of the query up-projection) and of the key / value latent
 //                    (written to its page), one warp per token and part.
+//   latent_rope_prep the same for latent layers with a rotated key part and directly projected queries: latent norm and
+//                    rotated key part (written to the page), rotated query parts of all heads.
 //   latent_gather    the latent rows a prefill step can see, out of their pages into one matrix (operand of the key / value
 //                    up-projection).
 //
 // Page layout of a layer with n_kv heads of key size D and value size DV: [n_kv][16][D] then [n_kv][16][DV]; of a latent
-// layer: [16][rank]. The convolution ring is the one of recurrent.cuh. Only the first tile of a sequence reads the ring (a
+// layer: [16][rank + rotated part]. The convolution ring is the one of recurrent.cuh. Only the first tile of a sequence reads the ring (a
 // tile has at least taps - 1 tokens) and the same warp then writes it, so the entries need no ordering across CTAs.
 #include "recurrent.cuh"
 
@@ -447,6 +449,119 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const T* proj, long lo
   }
 }
 
+// Latent attention with a rotated part: [T, ld] holds n_q heads of D + RD query columns at column 0 and, at column kv_col, the
+// latent (rank columns) and one key part (RD columns) for all heads. RoPE on the first `rot` of the RD columns. The first
+// blocks handle the key / value rows (one warp per token), the others the queries, VEC channels (pairs) per thread.
+struct LatentRopeParams {
+  const void* proj;
+  long long ld;
+  int T, heads, D, RD, rot, rank, kv_col;
+  const float* kv_w;
+  float eps;
+  const int *positions, *slot_mapping;
+  const float *cos_t, *sin_t;
+  int max_pos;
+  void* q_out;               // head h of token t at t * q_tok + h * q_head: [D | RD] columns (copy) or the RD rotated ones
+  long long q_tok, q_head;
+  int copy;
+  void* cache;               // [num_pages * 16][rank + RD]
+  int num_pages;
+  int* err;
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) latent_rope_prep_kernel(const LatentRopeParams p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int half = p.rot / 2, kv_blocks = (p.T + 3) / 4, lane = threadIdx.x & 31;
+  auto position = [&](int t) {
+    int pos = p.positions[t];
+    if (pos < 0 || pos >= p.max_pos) {
+      if (p.err) atomicCAS(p.err, 0, ERR_BAD_ARG);
+      pos = 0;
+    }
+    return static_cast<long long>(pos) * half;
+  };
+  if (static_cast<int>(blockIdx.x) < kv_blocks) {
+    const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (t >= p.T) return;
+    const int slot = p.slot_mapping ? p.slot_mapping[t] : -1;
+    if (slot < 0) return;
+    if (slot / 16 >= p.num_pages) {
+      if (p.err && lane == 0) atomicCAS(p.err, 0, ERR_BAD_PAGE);
+      return;
+    }
+    const T* row = static_cast<const T*>(p.proj) + t * p.ld + p.kv_col;
+    T* dst = static_cast<T*>(p.cache) + static_cast<long long>(slot) * (p.rank + p.RD);
+    float ss = 0.f;
+    if constexpr (VEC == 8) {
+      for (int i = lane * 4; i < p.rank; i += 128) {
+        const float4 v = load4(row + i);
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      }
+    } else {
+      for (int i = lane; i < p.rank; i += 32) ss += to_f(row[i]) * to_f(row[i]);
+    }
+    const float r = 1.f / sqrtf(warp_sum(ss) / p.rank + p.eps);
+    if constexpr (VEC == 8) {
+      for (int i = lane * 4; i < p.rank; i += 128) {
+        const float4 v = load4(row + i), g = load4(p.kv_w + i);
+        store4(dst + i, make_float4(v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w));
+      }
+    } else {
+      for (int i = lane; i < p.rank; i += 32) dst[i] = from_f<T>(to_f(row[i]) * r * p.kv_w[i]);
+    }
+    row += p.rank;
+    dst += p.rank;
+    const long long at = position(t);
+    for (int i = lane; i < half; i += 32) {
+      const float u = to_f(row[i]), v = to_f(row[i + half]), c = p.cos_t[at + i], s = p.sin_t[at + i];
+      dst[i] = from_f<T>(u * c - v * s);
+      dst[i + half] = from_f<T>(v * c + u * s);
+    }
+    for (int i = p.rot + lane; i < p.RD; i += 32) dst[i] = row[i];
+    return;
+  }
+  const int pairs = half / VEC, rest = (p.RD - p.rot) / VEC, units = pairs + rest + (p.copy ? p.D / VEC : 0);
+  const long long id = static_cast<long long>(blockIdx.x - kv_blocks) * 128 + threadIdx.x;
+  const long long th = id / units;
+  if (th >= static_cast<long long>(p.T) * p.heads) return;
+  const int unit = static_cast<int>(id - th * units), t = static_cast<int>(th / p.heads), h = static_cast<int>(th % p.heads);
+  const T* src = static_cast<const T*>(p.proj) + t * p.ld + static_cast<long long>(h) * (p.D + p.RD) + p.D;
+  T* dst = static_cast<T*>(p.q_out) + t * p.q_tok + h * p.q_head + (p.copy ? p.D : 0);
+  if (unit >= pairs) {         // columns that stay as they are
+    const int c = unit < pairs + rest ? p.rot + (unit - pairs) * VEC : (unit - pairs - rest) * VEC - p.D;
+    if constexpr (VEC == 8) {
+      float v[8];
+      load8(src + c, v);
+      store8(dst + c, v);
+    } else {
+      dst[c] = src[c];
+    }
+    return;
+  }
+  const long long at = position(t) + unit * VEC;
+  if constexpr (VEC == 8) {
+    float u[8], v[8], c[8], s[8];
+    load8(src + unit * 8, u);
+    load8(src + half + unit * 8, v);
+    load8(p.cos_t + at, c);
+    load8(p.sin_t + at, s);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const float a = u[e] * c[e] - v[e] * s[e];
+      v[e] = v[e] * c[e] + u[e] * s[e];
+      u[e] = a;
+    }
+    store8(dst + unit * 8, u);
+    store8(dst + half + unit * 8, v);
+  } else {
+    const float u = to_f(src[unit]), v = to_f(src[unit + half]), c = p.cos_t[at], s = p.sin_t[at];
+    dst[unit] = from_f<T>(u * c - v * s);
+    dst[unit + half] = from_f<T>(v * c + u * s);
+  }
+}
+
 // Latent pages of each sequence from first_page[s] to its end -> rows of `out`, page i at page_base[s] + i.
 __global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* cache, int vecs, const int* block_tables, int max_blocks,
                                                             const int* ctx_lens, const int* first_page, const int* page_base,
@@ -524,6 +639,39 @@ GLLM_API int gllm_latent_prep(const void* proj, long long ld, int is_f32, int M,
   else { if (vec) LATENT(bf16_t, true); else LATENT(bf16_t, false); }
 #undef LATENT
   return prep_done(e, "latent_prep");
+}
+
+// strides: {ld, q_tok, q_head}. copy: q_out takes whole heads [D | RD], else their rotated parts only.
+GLLM_API int gllm_latent_rope_prep(const void* proj, const long long* strides, int is_f32, int T, int heads, int D, int RD, int rot,
+                                   int rank, int kv_col, const float* kv_w, float eps, const int* positions,
+                                   const int* slot_mapping, const float* cos_t, const float* sin_t, int max_pos, void* q_out,
+                                   int copy, void* cache, int num_pages, void* stream) {
+  if (T <= 0) return 0;
+  if (heads <= 0 || D < 0 || RD < 0 || rot < 0 || rot > RD || (rot & 1) || (rot > 0 && (!cos_t || !sin_t)) || rank <= 0) {
+    set_last_error("latent_rope_prep: %d heads of %d + %d (%d rotated), rank %d", heads, D, RD, rot, rank);
+    return -1;
+  }
+  LatentRopeParams p = {};
+  p.proj = proj; p.ld = strides[0]; p.T = T; p.heads = heads; p.D = D; p.RD = RD; p.rot = rot; p.rank = rank; p.kv_col = kv_col;
+  p.kv_w = kv_w; p.eps = eps; p.positions = positions; p.slot_mapping = slot_mapping; p.cos_t = cos_t; p.sin_t = sin_t;
+  p.max_pos = max_pos; p.q_out = q_out; p.q_tok = strides[1]; p.q_head = strides[2]; p.copy = copy; p.cache = cache;
+  p.num_pages = num_pages; p.err = gllm_error_word();
+  const auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = D % 8 == 0 && RD % 8 == 0 && rot % 16 == 0 && rank % 8 == 0 && kv_col % 8 == 0 &&
+                   ((strides[0] | strides[1] | strides[2]) & 7) == 0 && al(proj) && al(q_out) && al(cache) && al(kv_w) &&
+                   al(cos_t) && al(sin_t);
+  const int per = vec ? 8 : 1;
+  const long long units = static_cast<long long>(T) * heads * (rot / 2 / per + (RD - rot) / per + (copy ? D / per : 0));
+  const dim3 grid(static_cast<unsigned>((T + 3) / 4 + (units + 127) / 128));
+  auto s = static_cast<cudaStream_t>(stream);
+  cudaError_t e;
+  if (is_f32)
+    e = vec ? launch_kernel(latent_rope_prep_kernel<float, 8>, grid, dim3(128), 0, s, true, 0, p)
+            : launch_kernel(latent_rope_prep_kernel<float, 1>, grid, dim3(128), 0, s, true, 0, p);
+  else
+    e = vec ? launch_kernel(latent_rope_prep_kernel<bf16_t, 8>, grid, dim3(128), 0, s, true, 0, p)
+            : launch_kernel(latent_rope_prep_kernel<bf16_t, 1>, grid, dim3(128), 0, s, true, 0, p);
+  return prep_done(e, "latent_rope_prep");
 }
 
 // cache [num_pages, 16, R] and out [out_pages, 16, R] bf16 (R a multiple of 8).

@@ -18,7 +18,7 @@ constexpr int kMoeBlockRows = 128;
 
 // One warp per token. E <= 512.
 __global__ void moe_route_kernel(const float* logits, long long ld, int T, int E, int k, int norm_topk, int scoring,
-                                 const float* sel_bias, float scale, int* out_ids, float* out_w, int* err) {
+                                 const float* sel_bias, float scale, int groups, int keep, int* out_ids, float* out_w, int* err) {
   const int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (t >= T) return;
@@ -38,7 +38,7 @@ __global__ void moe_route_kernel(const float* logits, long long ld, int T, int E
     float z = 0.f;
     for (int i = 0; i < per; ++i) {
       const int e = lane + 32 * i;
-      score[i] = e < E ? __expf(score[i] - mx) : 0.f;
+      score[i] = e < E ? expf(score[i] - mx) : 0.f;
       z += score[i];
     }
     z = warp_sum(z);
@@ -53,16 +53,14 @@ __global__ void moe_route_kernel(const float* logits, long long ld, int T, int E
     const int e = lane + 32 * i;
     sel[i] = e < E ? score[i] + (sel_bias ? sel_bias[e] : 0.f) : -INFINITY;
   }
-  float wsum = 0.f;
-  float my_w = 0.f;   // lane j keeps the j-th pick
-  int my_id = 0;
-  for (int j = 0; j < k; ++j) {
-    float bv = -INFINITY;
-    int bi = 0x7fffffff;
+  // The best expert of lanes' candidates, lowest index on equal scores; every lane gets it.
+  auto best_of = [&](const float (&cand)[kPer], float& bv, int& bi) {
+    bv = -INFINITY;
+    bi = 0x7fffffff;
     for (int i = 0; i < per; ++i) {
       const int e = lane + 32 * i;
-      if (e < E && (sel[i] > bv || (sel[i] == bv && e < bi))) {
-        bv = sel[i];
+      if (e < E && (cand[i] > bv || (cand[i] == bv && e < bi))) {
+        bv = cand[i];
         bi = e;
       }
     }
@@ -75,6 +73,33 @@ __global__ void moe_route_kernel(const float* logits, long long ld, int T, int E
         bi = oi;
       }
     }
+  };
+  if (groups > 0) {
+    // the best expert among the groups not kept yet belongs to the next best group
+    const int size = E / groups;
+    float rest[kPer];
+    unsigned kept = 0;   // bit i: this lane's expert i is in a kept group
+    for (int i = 0; i < per; ++i) rest[i] = sel[i];
+    for (int j = 0; j < keep; ++j) {
+      float bv;
+      int bi;
+      best_of(rest, bv, bi);
+      for (int i = 0; i < per; ++i)
+        if ((lane + 32 * i) / size == bi / size) {
+          kept |= 1u << i;
+          rest[i] = -INFINITY;
+        }
+    }
+    for (int i = 0; i < per; ++i)
+      if (!(kept >> i & 1u)) sel[i] = -INFINITY;
+  }
+  float wsum = 0.f;
+  float my_w = 0.f;   // lane j keeps the j-th pick
+  int my_id = 0;
+  for (int j = 0; j < k; ++j) {
+    float bv;
+    int bi;
+    best_of(sel, bv, bi);
     // weight = the (unbiased) score of the winner
     const int owner = bi & 31, slot = bi >> 5;
     float w = 0.f;
@@ -242,15 +267,19 @@ extern "C" int* gllm_error_word();
   } while (0)
 
 GLLM_API int gllm_moe_route(const float* logits, long long ld, int T, int E, int k, int norm_topk, int scoring,
-                            const float* sel_bias, float scale, int* out_ids, float* out_w, void* stream) {
+                            const float* sel_bias, float scale, int groups, int keep, int* out_ids, float* out_w, void* stream) {
   if (E > 512 || k > 32 || k > E) {
     set_last_error("moe_route: E=%d (max 512) / k=%d (max 32) unsupported", E, k);
+    return -1;
+  }
+  if (groups > 0 && (E % groups != 0 || keep <= 0 || keep > groups)) {
+    set_last_error("moe_route: %d experts in %d groups, %d kept", E, groups, keep);
     return -1;
   }
   const int threads = 256;
   const int blocks = (T * 32 + threads - 1) / threads;
   moe_route_kernel<<<blocks, threads, 0, (cudaStream_t)stream>>>(logits, ld, T, E, k, norm_topk, scoring, sel_bias,
-                                                                 scale, out_ids, out_w, gllm_error_word());
+                                                                 scale, groups, keep, out_ids, out_w, gllm_error_word());
   MOE_CHECK("moe_route");
   return 0;
 }

@@ -1,6 +1,7 @@
-// The step between two sublayers of a sandwich-norm block over a residual stream kept in fp32, one pass per row:
+// The step between two sublayers of a pre-norm or sandwich-norm block over a residual stream kept in fp32, one pass per row:
 //
-//   s = sublayer output (a projection's row, or the sum of the row's routed expert outputs)
+//   s = sublayer output (a projection's row, or the weighted sum of the row's routed expert outputs)
+//       (+ the row of a sublayer that ran beside it) (+ sigmoid(gate) * the row of a shared expert)
 //   x += norm(s) * post_w;   x += add;   xb = norm(x) * pre_w      (each part optional)
 //
 // Norms are RMS or layer norms without bias, statistics in fp32; a layer norm takes its variance from the deviations. One
@@ -16,6 +17,13 @@ struct ResidualNormParams {
   long long ldy;
   const int* dest;        // [M, top] rows of y to sum (null: row m)
   int top;
+  const float* row_w;     // [M, top] weights of those rows (null: ones)
+  const float* plus;      // fp32 rows that join s, or null
+  long long ldp;
+  const float* gated;     // fp32 rows that join s times sigmoid(gate[m]), or null
+  long long ldg;
+  const float* gate;
+  long long ldgate;
   const float *post_w, *add, *pre_w;
   void* xb;
   long long ldb;
@@ -95,17 +103,31 @@ __global__ void __launch_bounds__(THREADS) residual_norm_kernel(const ResidualNo
       const long long r = p.dest ? p.dest[m * p.top + j] : m;
       if (r < 0) continue;
       const TY* yr = y + r * p.ldy;
+      const float w = p.row_w ? p.row_w[m * p.top + j] : 1.f;
 #pragma unroll
       for (int n = 0; n < N; ++n)
         if (idx(n) < H) {
           if constexpr (V == 4) {
             const float4 f = load4(yr + idx(n));
-            h[n * 4] += f.x; h[n * 4 + 1] += f.y; h[n * 4 + 2] += f.z; h[n * 4 + 3] += f.w;
+            h[n * 4] = fmaf(w, f.x, h[n * 4]); h[n * 4 + 1] = fmaf(w, f.y, h[n * 4 + 1]);
+            h[n * 4 + 2] = fmaf(w, f.z, h[n * 4 + 2]); h[n * 4 + 3] = fmaf(w, f.w, h[n * 4 + 3]);
           } else {
-            h[n] += to_f(yr[idx(n)]);
+            h[n] = fmaf(w, to_f(yr[idx(n)]), h[n]);
           }
         }
     }
+    auto join = [&](const float* row, float w) {
+#pragma unroll
+      for (int n = 0; n < N; ++n)
+        if (idx(n) < H) {
+          float f[V];
+          load_f(row, idx(n), f);
+#pragma unroll
+          for (int e = 0; e < V; ++e) h[n * V + e] = fmaf(w, f[e], h[n * V + e]);
+        }
+    };
+    if (p.plus) join(p.plus + m * p.ldp, 1.f);
+    if (p.gated) join(p.gated + m * p.ldg, p.gate ? sigmoid_f(p.gate[m * p.ldgate]) : 1.f);
     if (p.post_w) normalise(p.post_w, 0);
   } else {
 #pragma unroll
@@ -159,19 +181,21 @@ static cudaError_t residual_norm_launch(const ResidualNormParams& p, int M, bool
 using namespace gllm;
 
 GLLM_API int gllm_residual_norm(float* x, long long ldx, const void* y, long long ldy, int y_f32, const int* dest, int top,
-                                const float* post_w, const float* add, const float* pre_w, void* xb, int xb_f32, int M,
+                                const float* row_w, const float* plus, long long ldp, const float* gated, long long ldg,
+                                const float* gate, long long ldgate, const float* post_w, const float* add, const float* pre_w, void* xb, int xb_f32, int M,
                                 int hidden, int layer, float eps, const int* rows, int ldb, void* stream) {
   if (M <= 0) return 0;
-  if (hidden <= 0 || hidden > 16384 || (rows && y) || (pre_w && !xb) || (dest && top <= 0)) {
+  if (hidden <= 0 || hidden > 16384 || (rows && y) || ((plus || gated) && !y) || (pre_w && !xb) || (dest && top <= 0)) {
     set_last_error("residual_norm: hidden %d (at most 16384), rows with y, or a missing output", hidden);
     return -1;
   }
   ResidualNormParams p = {};
-  p.x = x; p.ldx = ldx; p.y = y; p.ldy = ldy; p.dest = dest; p.top = top;
+  p.x = x; p.ldx = ldx; p.y = y; p.ldy = ldy; p.dest = dest; p.top = top; p.row_w = row_w;
+  p.plus = plus; p.ldp = ldp; p.gated = gated; p.ldg = ldg; p.gate = gate; p.ldgate = ldgate;
   p.post_w = post_w; p.add = add; p.pre_w = pre_w; p.xb = xb; p.ldb = ldb;
   p.hidden = hidden; p.layer = layer; p.eps = eps; p.rows = rows;
   const auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
-  const bool vec = hidden % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && ldb % 4 == 0 && aligned(x) && aligned(y) &&
+  const bool vec = hidden % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && ldb % 4 == 0 && ldp % 4 == 0 && ldg % 4 == 0 && aligned(plus) && aligned(gated) && aligned(x) && aligned(y) &&
                    aligned(xb) && aligned(post_w) && aligned(add) && aligned(pre_w);
   auto s = static_cast<cudaStream_t>(stream);
   cudaError_t e;

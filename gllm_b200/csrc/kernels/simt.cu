@@ -22,14 +22,15 @@ __device__ __forceinline__ float block_reduce_sum(float v, float* red) {
 }
 
 // ---------------------------------------------------------------------------------------------
-// C[M, N] = A[M, K] B[N, K]^T (+ bias, soft cap): 64 x 64 tiles, 4 x 4 outputs per thread, fp32 FMAs. With `groups`, the 128-row
+// C[M, N] = A[M, K] B[N, K]^T (+ bias, soft cap, activation): 64 x 64 tiles, 4 x 4 outputs per thread, fp32 FMAs. With `groups`, the 128-row
 // block i of A multiplies the groups[i]-th [N, K] matrix of the stack B (negative: nothing), and only its first
 // block_rows[i] rows are there.
 // ---------------------------------------------------------------------------------------------
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const TI* A, long long lda, const TI* B, long long ldb, TO* C,
                                                         long long ldc, int M, int N, int K, const float* bias,
-                                                        float softcap, const int* groups, const int* block_rows) {
+                                                        float softcap, int act, int act_cols, const int* groups,
+                                                        const int* block_rows) {
   constexpr int BK = 16;
   __shared__ float As[BK][68], Bs[BK][68];
   const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
@@ -79,17 +80,18 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TI* A, long long l
       if (n >= N) continue;
       float v = acc[i][j] + (bias ? bias[n] : 0.f);
       if (softcap > 0.f) v = softcap * tanhf(v / softcap);
+      if (act && n < act_cols) v = act == 1 ? silu_exact(v) : store_act(v, act);
       C[static_cast<long long>(m) * ldc + n] = from_f<TO>(v);
     }
   }
 }
 
 // ---------------------------------------------------------------------------------------------
-// Embedding rows: x[m] = table[ids[m]] in fp32 (the residual stream), xb[m] the same row in the compute type.
+// Embedding rows: x[m] = table[ids[m]] * scale in fp32 (the residual stream), xb[m] the unscaled row in the compute type.
 // ---------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void __launch_bounds__(128) embed_rows_kernel(const int* ids, const T* table, int vocab, int hidden, float* x,
-                                                         T* xb, int* err) {
+__global__ void __launch_bounds__(128) embed_rows_kernel(const int* ids, const T* table, int vocab, int hidden, float scale,
+                                                         float* x, T* xb, int* err) {
   const long long m = blockIdx.x;
   int id = ids[m];
   if (id < 0 || id >= vocab) {
@@ -99,7 +101,7 @@ __global__ void __launch_bounds__(128) embed_rows_kernel(const int* ids, const T
   const T* src = table + static_cast<long long>(id) * hidden;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     const T v = src[i];
-    x[m * hidden + i] = to_f(v);
+    x[m * hidden + i] = to_f(v) * scale;
     if (xb) xb[m * hidden + i] = v;
   }
 }
@@ -290,8 +292,8 @@ extern "C" int* gllm_error_word();
 using bf16_t = __nv_bfloat16;
 
 static int gemm_simt(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M, int N, int K,
-                     int in_f32, int out_f32, const float* bias, float softcap, const int* groups, const int* block_rows,
-                     void* stream) {
+                     int in_f32, int out_f32, const float* bias, float softcap, int act, int act_cols, const int* groups,
+                     const int* block_rows, void* stream) {
   if (M <= 0 || N <= 0 || K <= 0 || (M + 63) / 64 > 65535) {
     set_last_error("gemm_simt: bad problem M=%d N=%d K=%d", M, N, K);
     return -1;
@@ -302,7 +304,7 @@ static int gemm_simt(const void* A, long long lda, const void* B, long long ldb,
     using TI = decltype(in);
     using TO = decltype(out);
     gemm_simt_kernel<TI, TO><<<grid, 256, 0, s>>>(static_cast<const TI*>(A), lda, static_cast<const TI*>(B), ldb,
-                                                  static_cast<TO*>(C), ldc, M, N, K, bias, softcap, groups, block_rows);
+                                                  static_cast<TO*>(C), ldc, M, N, K, bias, softcap, act, act_cols, groups, block_rows);
   };
   if (in_f32 && out_f32) run(float{}, float{});
   else if (in_f32) run(float{}, bf16_t{});
@@ -313,26 +315,27 @@ static int gemm_simt(const void* A, long long lda, const void* B, long long ldb,
 
 // in_f32 / out_f32: element types of A and B / of C (bf16 otherwise).
 GLLM_API int gllm_gemm_simt(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M,
-                            int N, int K, int in_f32, int out_f32, const float* bias, float softcap, void* stream) {
-  return gemm_simt(A, lda, B, ldb, C, ldc, M, N, K, in_f32, out_f32, bias, softcap, nullptr, nullptr, stream);
+                            int N, int K, int in_f32, int out_f32, const float* bias, float softcap, int act, int act_cols,
+                            void* stream) {
+  return gemm_simt(A, lda, B, ldb, C, ldc, M, N, K, in_f32, out_f32, bias, softcap, act, act_cols, nullptr, nullptr, stream);
 }
 
 // Grouped form: groups [M / 128] int32, block_rows [M / 128] int32 or null.
 GLLM_API int gllm_gemm_simt_grouped(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M,
                                     int N, int K, int in_f32, int out_f32, const int* groups, const int* block_rows,
                                     void* stream) {
-  return gemm_simt(A, lda, B, ldb, C, ldc, M, N, K, in_f32, out_f32, nullptr, 0.f, groups, block_rows, stream);
+  return gemm_simt(A, lda, B, ldb, C, ldc, M, N, K, in_f32, out_f32, nullptr, 0.f, 0, 0, groups, block_rows, stream);
 }
 
-GLLM_API int gllm_embed_rows(const int* ids, const void* table, int vocab, int hidden, int is_f32, float* x, void* xb,
+GLLM_API int gllm_embed_rows(const int* ids, const void* table, int vocab, int hidden, int is_f32, float scale, float* x, void* xb,
                              int M, void* stream) {
   if (M <= 0) return 0;
   auto s = static_cast<cudaStream_t>(stream);
   if (is_f32)
-    embed_rows_kernel<float><<<M, 128, 0, s>>>(ids, static_cast<const float*>(table), vocab, hidden, x,
+    embed_rows_kernel<float><<<M, 128, 0, s>>>(ids, static_cast<const float*>(table), vocab, hidden, scale, x,
                                                static_cast<float*>(xb), gllm_error_word());
   else
-    embed_rows_kernel<bf16_t><<<M, 128, 0, s>>>(ids, static_cast<const bf16_t*>(table), vocab, hidden, x,
+    embed_rows_kernel<bf16_t><<<M, 128, 0, s>>>(ids, static_cast<const bf16_t*>(table), vocab, hidden, scale, x,
                                                 static_cast<bf16_t*>(xb), gllm_error_word());
   SIMT_CHECK("embed_rows");
 }

@@ -32,6 +32,14 @@ class RopeScaling:
     attention_factor: Optional[float] = None
 
 
+def _yarn(s: Optional[Dict[str, Any]]) -> RopeScaling:
+    """YaRN parameters (factor, original, fast, slow); cos and sin are stretched by 0.1 ln(factor) + 1."""
+    if not s:
+        return RopeScaling()
+    return RopeScaling("yarn", factor=float(s["factor"]), original_max_position=int(s["original"]), beta_fast=float(s["fast"]),
+                       beta_slow=float(s["slow"]), attention_factor=0.1 * math.log(float(s["factor"])) + 1.0)
+
+
 @dataclass
 class MixerSpec:
     """Token mixer of one layer of a heterogeneous model (``ModelConfig.layer_specs``).
@@ -41,14 +49,21 @@ class MixerSpec:
                ``window`` > 0 = the last ``window`` keys and the first ``keep_first`` of the sequence; ``row_qk_norm`` = RMS
                norm over the whole q / k projection, ``head_qk_norm`` = over each head; ``v_from_k`` = values are the
                projected keys; ``taps`` > 0 = causal convolution over time on q, k and v (before norm and rotation);
-               ``o_bias`` = the output projection has a bias (q, k and v always do).
-    latent:    attention over a shared latent of ``kv_rank`` channels per token, no positions: ``heads`` heads of ``dim`` query /
-               key and ``vdim`` value dimensions, queries of rank ``q_rank``, sliding ``window``, ``sink`` = a learned extra
-               logit per head in the softmax denominator.
+               ``qkv_bias`` / ``o_bias`` = the projections have biases; ``softcap`` > 0: scores are cap * tanh(score / cap);
+               ``bias_max`` > 0 = a learned bias per head and distance is added to the (capped) scores, from a table of
+               ``bias_rows`` rows (0: taken from the weight) that ends at that distance (``ops.distance_rows``);
+               ``sink`` = a learned extra logit per head in the softmax denominator.
+    latent:    attention over a shared latent of ``kv_rank`` channels per token: ``heads`` heads of ``dim`` query / key and
+               ``vdim`` value dimensions, queries of rank ``q_rank`` (0: projected directly), sliding ``window``, ``sink`` as
+               above; ``rope_part`` > 0 = that many further query / key dimensions per head, the key part shared by all heads,
+               rotary (``rot_dim``, ``rot_base``, ``rot_scaling``); ``gate`` = the heads' outputs are multiplied by
+               sigmoid(W_g h).
     rglru:     real-gated linear recurrent unit over ``width`` channels, gates in ``blocks`` diagonal blocks, behind a
                causal convolution of ``taps`` taps.
     gla:       gated linear attention, ``heads`` x (``dim`` key, ``vdim`` value) channels, decay sigmoid(z)^(1 / tau)
-               with z of rank ``decay_rank`` (0: taken from the weight)."""
+               with z of rank ``decay_rank`` (0: taken from the weight).
+    lightning: linear attention with a fixed decay per head (``decay``), ``heads`` x (``dim`` key, ``vdim`` value) channels,
+               silu on q, k and v, one RMS norm over all heads and the gate sigmoid(W_g h) in front of the output."""
     kind: str = "attention"
     heads: int = 0
     kv_heads: int = 0
@@ -72,6 +87,14 @@ class MixerSpec:
     q_rank: int = 0
     kv_rank: int = 0
     sink: bool = False
+    qkv_bias: bool = True
+    softcap: float = 0.0
+    bias_max: int = 0
+    bias_rows: int = 0
+    rope_part: int = 0
+    rot_scaling: RopeScaling = field(default_factory=RopeScaling)
+    gate: bool = False
+    decay: tuple = ()
 
     @property
     def value_dim(self) -> int:
@@ -83,14 +106,14 @@ class MixerSpec:
             return self.taps * ((self.heads + self.kv_heads) * self.dim + self.kv_heads * self.value_dim)
         if self.kind == "rglru":
             return self.width * (self.taps + 1)
-        if self.kind == "gla":
+        if self.kind in ("gla", "lightning"):
             return self.heads * self.dim * self.vdim
         return 0
 
     def kv_elems(self) -> int:
         """KV cache elements per token."""
         if self.kind == "latent":
-            return self.kv_rank
+            return self.kv_rank + self.rope_part
         return self.kv_heads * (self.dim + self.value_dim) if self.kind == "attention" else 0
 
 
@@ -98,20 +121,29 @@ class MixerSpec:
 class MoeSpec:
     """Mixture-of-experts feed-forward of one layer: ``top`` of ``experts`` gated feed-forwards of intermediate size ``ff``.
     ``scoring``: sigmoid or softmax over the router logits; ``norm_topk``: the chosen scores are renormalised to sum 1;
-    ``scale_input``: the score multiplies the expert's input instead of its output."""
+    ``scale_input``: the score multiplies the expert's input instead of its output; ``scale``: factor of the weights.
+    ``groups`` > 0: only experts of the ``keep_groups`` groups (neighbours, equal sizes) with the largest best score are
+    chosen. ``shared_ff`` > 0: one more feed-forward of that size runs for every token, multiplied by a sigmoid gate of the
+    token when ``shared_gate``."""
     experts: int
     top: int
     ff: int
     scoring: str = "softmax"
     norm_topk: bool = True
     scale_input: bool = False
+    scale: float = 1.0
+    groups: int = 0
+    keep_groups: int = 0
+    shared_ff: int = 0
+    shared_gate: bool = False
 
 
 @dataclass
 class LayerSpec:
     mixer: MixerSpec
-    ff: int = 0             # intermediate size of the gated feed-forward, 0 = none
+    ff: int = 0             # intermediate size of the feed-forward, 0 = none
     act: str = "gelu_tanh"
+    gated: bool = True      # W_down(act(W_gate h) * W_up h), else W_down act(W_up h)
     moe: Optional[MoeSpec] = None
 
 
@@ -156,7 +188,8 @@ class ModelConfig:
     attn_scale: float = 0.0  # 0 -> 1/sqrt(head_dim)
     post_norm: bool = False  # encoder-style post-LN residual blocks
     # Heterogeneous decoders (models/hybrid.py): one spec per layer. ``block``: "post" = post-norm blocks
-    # x = norm(postln_alpha * x + f(x)), "sandwich" = x = x + norm_b(f(norm_a(x))); ``norm_type`` rms or layer (no bias).
+    # x = norm(postln_alpha * x + f(x)), "sandwich" = x = x + norm_b(f(norm_a(x))), "parallel" = h = norm(x),
+    # x = x + (mixer(h) + ff(h)); ``norm_type`` rms or layer (no bias), ``norm_one_plus_w``: weights stored around zero.
     # ``loop`` = (start, stop, times): that range of layers runs ``times`` times in a row with the same weights, a learned
     # vector added to the stream before each pass; every pass has its own cache and state.
     layer_specs: Optional[List[LayerSpec]] = None
@@ -305,15 +338,16 @@ class ModelConfig:
                 if m.kind == "attention":
                     total += h * ((m.heads + m.kv_heads) * m.dim + (m.heads + (0 if m.v_from_k else m.kv_heads)) * m.value_dim)
                 elif m.kind == "latent":
-                    total += h * (m.q_rank + m.kv_rank + m.heads * m.vdim) + m.heads * (
-                        m.q_rank * m.dim + m.kv_rank * (m.dim + m.vdim))
+                    qd = m.heads * (m.dim + m.rope_part)
+                    total += h * (m.q_rank + m.kv_rank + m.rope_part + m.heads * m.vdim * (2 if m.gate else 1)) + (
+                        (m.q_rank or h) * qd + m.heads * m.kv_rank * (m.dim + m.vdim))
                 elif m.kind == "rglru":
                     total += 3 * h * m.width + 2 * m.width * m.width // m.blocks
                 else:
                     total += h * m.heads * (2 * m.dim + 3 * m.vdim) + m.decay_rank * (h + m.heads * m.dim)
-                total += 3 * h * l.ff
+                total += (3 if l.gated else 2) * h * l.ff
                 if l.moe:
-                    total += h * l.moe.experts * (3 * l.moe.ff + 1)
+                    total += h * (l.moe.experts * (3 * l.moe.ff + 1) + 3 * l.moe.shared_ff + l.moe.shared_gate)
             return total
         attn = h * (self.q_size + 2 * self.kv_size) + self.q_size * h
         if self.is_mla:
@@ -352,6 +386,8 @@ class ModelConfig:
             return ModelConfig.from_zenevik_dict(d)
         if d.get("architecture") == "Gorulorn":
             return ModelConfig.from_gorulorn_dict(d)
+        if d.get("architecture") == "Ritirax":
+            return ModelConfig.from_ritirax_dict(d)
         tc = d.get("text_config") or d
         arch = (d.get("model_type") or tc.get("model_type") or "llama").lower()
         g = lambda *keys, default=None: next((tc[k] for k in keys if k in tc and tc[k] is not None), default)
@@ -505,6 +541,48 @@ class ModelConfig:
         cfg.set_hybrid_dims()
         return cfg
 
+    @staticmethod
+    def from_ritirax_dict(d: Dict[str, Any]) -> "ModelConfig":
+        """Ritirax ``config.json``: parallel blocks of attention with capped scores, distance biases and sinks, gated latent
+        attention with a rotated key part, or lightning attention, beside a dense or a sparse feed-forward."""
+        specs = []
+        for i, l in enumerate(d["layers"]):
+            m, kind, mlp = l["mixer"], l["type"], l.get("mlp")
+            size = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]))
+            if kind == "attention":
+                mixer = MixerSpec("attention", kv_heads=int(m["kv_heads"]), scale=float(m["scale"]), head_qk_norm=True, qkv_bias=False,
+                                  o_bias=False, softcap=float(m.get("softcap") or 0.0), bias_max=int(m.get("bias_max") or 0),
+                                  sink=True, **size)
+            elif kind == "latent_attention":
+                rot = m.get("rot") or {}
+                mixer = MixerSpec("latent", kv_rank=int(m["kv_rank"]), rope_part=int(m.get("rot_dim") or 0),
+                                  rot_dim=int(rot.get("dims") or 0), rot_base=float(rot.get("base", 10000.0)),
+                                  rot_scaling=_yarn(rot.get("scaling")), scale=float(m["scale"]), gate=True, **size)
+            elif kind == "lightning":
+                mixer = MixerSpec("lightning", decay=tuple(float(x) for x in m["decay"]), **size)
+                if len(mixer.decay) != mixer.heads:
+                    raise ValueError(f"layer {i}: {len(mixer.decay)} decays for {mixer.heads} heads")
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            spec = LayerSpec(mixer, act="silu")
+            if mlp is not None and mlp["kind"] == "dense":
+                spec.ff, spec.act, spec.gated = int(mlp["ff"]), "relu2", False
+            elif mlp is not None and mlp["kind"] == "moe":
+                r, groups, shared = mlp["router"], mlp["router"].get("groups") or {}, mlp.get("shared") or {}
+                spec.moe = MoeSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]), scoring="softmax",
+                                   norm_topk=False, scale=float(r.get("scale", 1.0)), groups=int(groups.get("count") or 0),
+                                   keep_groups=int(groups.get("keep") or 0), shared_ff=int(shared.get("ff") or 0),
+                                   shared_gate=bool(shared))
+            elif mlp is not None:
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            specs.append(spec)
+        cfg = ModelConfig(arch="ritirax", hidden_size=int(d["width"]), num_layers=len(specs), vocab_size=int(d["vocab"]),
+                          rms_norm_eps=float(d["norm"]["eps"]), norm_one_plus_w=True, block="parallel", hidden_act="silu",
+                          embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
+                          max_position_embeddings=int(d.get("max_positions", 1 << 20)), layer_specs=specs)
+        cfg.set_hybrid_dims()
+        return cfg
+
     def set_hybrid_dims(self):
         """The scalar head / feed-forward sizes of a heterogeneous model: the largest over its layers (they size shared
         buffers; the layers use their specs). ``head_dim`` is 128 when any layer can use the head_dim-128 kernels."""
@@ -513,7 +591,7 @@ class ModelConfig:
         self.num_kv_heads = max([m.kv_heads for m in att], default=1)
         dims = [m.dim for m in att if m.value_dim == m.dim] or [64]
         self.head_dim = 128 if 128 in dims else max(dims)
-        self.intermediate_size = max([max(l.ff, l.moe.ff if l.moe else 0) for l in self.layer_specs] + [0])
+        self.intermediate_size = max([max(l.ff, max(l.moe.ff, l.moe.shared_ff) if l.moe else 0) for l in self.layer_specs] + [0])
 
     @staticmethod
     def from_json_file(path) -> "ModelConfig":
@@ -636,6 +714,19 @@ def preset(name: str) -> ModelConfig:
                           block="sandwich", loop=(1, 3, 2), hidden_act="silu", max_position_embeddings=2048,
                           layer_specs=[LayerSpec(att, act="silu", moe=moe), LayerSpec(lat, act="silu", moe=moe),
                                        LayerSpec(att, act="silu")], eos_token_ids=[2])
+        cfg.set_hybrid_dims()
+        return cfg
+    if n in ("tiny-ritirax",):
+        att = MixerSpec("attention", heads=4, kv_heads=2, dim=128, vdim=128, scale=0.09, head_qk_norm=True, qkv_bias=False, o_bias=False,
+                        softcap=20.0, bias_max=90, bias_rows=20, sink=True)
+        lat = MixerSpec("latent", heads=3, dim=64, vdim=128, kv_rank=160, rope_part=64, rot_dim=64, rot_base=5000.0, scale=0.1,
+                        gate=True, rot_scaling=RopeScaling("yarn", factor=3.0, original_max_position=256, attention_factor=1.1))
+        lig = MixerSpec("lightning", heads=3, dim=48, vdim=64, decay=(0.5, 0.9, 0.99))
+        moe = MoeSpec(experts=12, top=3, ff=96, norm_topk=False, scale=1.5, groups=4, keep_groups=2, shared_ff=128, shared_gate=True)
+        cfg = ModelConfig(arch="ritirax", hidden_size=256, num_layers=3, vocab_size=1024, rms_norm_eps=1e-6, norm_one_plus_w=True,
+                          block="parallel", hidden_act="silu", embedding_scale=16.0, max_position_embeddings=2048,
+                          layer_specs=[LayerSpec(att, ff=384, act="relu2", gated=False), LayerSpec(lat, act="silu", moe=moe),
+                                       LayerSpec(lig, act="silu", moe=moe)], eos_token_ids=[2])
         cfg.set_hybrid_dims()
         return cfg
     if n in ("tiny-bert",):

@@ -1,8 +1,9 @@
-"""Heterogeneous decoders: every layer has its own token mixer (``models/mixers.py``) and an optional feed-forward (gated, or
-a mixture of experts: ``models/moe.py::ExpertFF``), over a residual stream kept in fp32. Two kinds of block:
+"""Heterogeneous decoders: every layer has its own token mixer (``models/mixers.py``) and an optional feed-forward
+(``models/moe.py``: gated, plain, or a mixture of experts), over a residual stream kept in fp32. Three kinds of block:
 
     post      x = norm1(alpha * x + mixer(x));         x = norm2(alpha * x + ff(x))
     sandwich  x = x + norm1b(mixer(norm1(x)));         x = x + norm2b(ff(norm2(x)))
+    parallel  h = norm1(x);                            x = x + (mixer(h) + ff(h))
 
 A range of layers may run several times in a row with the same weights; a learned vector joins the stream before each pass,
 and each pass has its own cache and state (``ModelConfig.layer_runs``: "run" below is one execution of a layer).
@@ -10,7 +11,7 @@ and each pass has its own cache and state (``ModelConfig.layer_runs``: "run" bel
 The model plugs into the engine like ``DecoderModel``: same ``ForwardBatch``, paged KV cache for its attention layers, and
 recurrent state in the batcher's sequence slots (``kv_cache/recurrent_state.py``) for the others. The workspace holds the
 stream ``x`` in fp32 (the residual sum and its norms) and ``xb``, the next GEMM's operand in the compute dtype: the stream
-itself in post-norm blocks, its normalised rows in sandwich blocks.
+itself in post-norm blocks, its normalised rows in the others.
 
 dtype bfloat16: tensor-core GEMMs with fp32 accumulation; positions, attention scores and weights, norms, gates, decays
 and states in fp32. dtype float32: every operation in true 32-bit arithmetic.
@@ -22,15 +23,14 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from .. import ops
 from ..engine.batch import ForwardBatch
 from ..ops import linear as L
 from ..ops import recurrent as R
 from ..ops.residual import residual_norm
 from .config import ModelConfig
-from .mixers import MIXERS, ROW_PAD, mixer_shapes, rope_table
-from .moe import ExpertFF
-from .weights import glu_tile_width, layer_prefix
+from .mixers import MIXERS, mixer_shapes, rope_table
+from .moe import ExpertFF, GatedFF, PlainFF
+from .weights import layer_prefix
 
 
 def is_norm_weight(name: str) -> bool:
@@ -52,12 +52,18 @@ def tensor_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:
         s.update({f"{p}norm1{b}": (H,) for b in norms})
         for n, shape in mixer_shapes(l.mixer, H).items():
             s[f"{p}mix.{n}"] = shape
-        if l.ff or l.moe:
+        if (l.ff or l.moe) and cfg.block != "parallel":
             s.update({f"{p}norm2{b}": (H,) for b in norms})
         gated = lambda q, ff: {q + "gate": (ff, H), q + "up": (ff, H), q + "down": (H, ff)}
         if l.ff:
             s.update(gated(p + "mlp.", l.ff))
+            if not l.gated:
+                del s[p + "mlp.gate"]
         if l.moe:
+            if l.moe.shared_ff:
+                s.update(gated(p + "mlp.shared.", l.moe.shared_ff))
+            if l.moe.shared_gate:
+                s[p + "mlp.shared.sg"] = (1, H)
             s[p + "mlp.router"] = (l.moe.experts, H)
             for e in range(l.moe.experts):
                 s.update(gated(f"{p}mlp.e{e}.", l.moe.ff))
@@ -70,11 +76,7 @@ class HybridLayer:
     mixer: object
     norm1: torch.Tensor
     norm2: Optional[torch.Tensor] = None
-    w_gate_up: Optional[torch.Tensor] = None
-    w_down: Optional[torch.Tensor] = None
-    glu_fused: bool = False
-    glu_bn: int = 128
-    act: int = 1
+    ff: Optional[object] = None            # GatedFF | PlainFF
     moe: Optional[object] = None           # None: what the engine asks of other models' layers (expert balancing)
     experts: Optional[ExpertFF] = None
     norm1b: Optional[torch.Tensor] = None  # sandwich blocks: the norms behind the sublayers
@@ -87,22 +89,25 @@ class HybridWorkspace:
     """Static activation buffers (CUDA graphs replay over them). ``take`` hands out a contiguous [T, n] view of a named
     buffer; ``f32`` buffers are fp32 whatever the compute dtype."""
 
-    F32 = ("f32", "f32b", "y")
+    F32 = ("f32", "f32b", "y", "y2")       # y, y2: what the mixer and a feed-forward beside it put out
 
     def __init__(self, model: "HybridDecoder", tokens: int):
         dev, dt, H = model.device, model.dtype, model.cfg.hidden_size
         self.max_tokens = tokens
         self.x = torch.zeros((tokens, H), dtype=torch.float32, device=dev)
-        self.xb = self.x if dt == torch.float32 and not model.sandwich else torch.zeros((tokens, H), dtype=dt, device=dev)
+        self.xb = self.x if dt == torch.float32 and model.post else torch.zeros((tokens, H), dtype=dt, device=dev)
         need: Dict[str, int] = {}
         for l in model.layers:
             sizes = dict(l.mixer.workspace())
             sizes["y"] = l.mixer.w["wo"].shape[0]
-            if l.w_down is not None:
-                sizes["y"] = max(sizes["y"], l.w_down.shape[0])
-                sizes["act"] = l.w_down.shape[1]
-                if not l.glu_fused:
-                    sizes["gu"] = l.w_gate_up.shape[0]
+            if l.ff is not None:
+                ff = l.ff.workspace()
+                out = ff.pop("y")
+                sizes.update(ff)
+                if model.parallel:
+                    sizes["y2"] = out
+                else:
+                    sizes["y"] = max(sizes["y"], out)
             for k, v in sizes.items():
                 need[k] = max(need.get(k, 0), v)
         self.buf = {k: torch.zeros(tokens * n, dtype=torch.float32 if k in self.F32 else dt, device=dev)
@@ -137,10 +142,13 @@ class HybridDecoder:
             raise ValueError(f"not available for heterogeneous decoders: {', '.join(sorted(bad))}")
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError(f"compute dtype {dtype}: bfloat16 or float32")
-        self.sandwich = cfg.block == "sandwich"
-        if cfg.block not in ("post", "sandwich") or (not self.sandwich and (
-                cfg.norm_type != "rms" or cfg.loop or any(l.moe for l in cfg.layer_specs))):
-            raise ValueError("heterogeneous decoder: looped layers, layer norms and experts are built for sandwich blocks")
+        self.post, self.parallel = cfg.block == "post", cfg.block == "parallel"
+        if cfg.block not in ("post", "sandwich", "parallel") or (self.post and (
+                cfg.norm_type != "rms" or cfg.loop or cfg.embedding_scale != 1.0 or any(l.moe for l in cfg.layer_specs))):
+            raise ValueError("heterogeneous decoder: looped layers, layer norms, a scaled embedding and experts are not built for "
+                             "post-norm blocks")
+        if any(l.moe and not l.moe.scale_input for l in cfg.layer_specs) and not self.parallel:
+            raise ValueError("heterogeneous decoder: weighted expert outputs are built for parallel blocks")
         self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
         self.layer_ids = list(range(cfg.num_layers))
         self.kv_dtype, self.kv_scale = dtype, 1.0
@@ -157,42 +165,30 @@ class HybridDecoder:
         dev = self.device
         to = lambda n: src.get(n).to(dev, dtype).contiguous()
         f32 = lambda n: src.get(n).float().to(dev).contiguous()
+        norm = (lambda n: f32(n) + 1.0) if cfg.norm_one_plus_w else f32
         self.embed = to("embed_tokens")
-        self.final_norm = f32("final_norm")
+        self.final_norm = norm("final_norm")
         self.lm_head = L.pad_rows(to("lm_head"), 256).contiguous()
         self.layers: List[HybridLayer] = []
         for i, spec in enumerate(cfg.layer_specs):
             p = layer_prefix(i)
             lw = HybridLayer(MIXERS[spec.mixer.kind](spec.mixer, src, p, cfg.hidden_size, cfg.rms_norm_eps, dev, dtype),
-                             norm1=f32(p + "norm1"), act=L.ACT_IDS[spec.act])
-            if spec.ff or spec.moe:
-                lw.norm2 = f32(p + "norm2")
-            if self.sandwich:
-                lw.norm1b = f32(p + "norm1b")
-                lw.norm2b = f32(p + "norm2b") if spec.ff or spec.moe else None
-            if spec.ff:
-                self._pack_ff(lw, to(p + "mlp.gate"), to(p + "mlp.up"), to(p + "mlp.down"))
+                             norm1=norm(p + "norm1"))
+            if (spec.ff or spec.moe) and not self.parallel:
+                lw.norm2 = norm(p + "norm2")
+            if cfg.block == "sandwich":
+                lw.norm1b = norm(p + "norm1b")
+                lw.norm2b = norm(p + "norm2b") if spec.ff or spec.moe else None
+            if spec.ff and spec.gated:
+                lw.ff = GatedFF(to(p + "mlp.gate"), to(p + "mlp.up"), to(p + "mlp.down"), L.ACT_IDS[spec.act], dtype)
+            elif spec.ff:
+                lw.ff = PlainFF(to(p + "mlp.up"), to(p + "mlp.down"), spec.act, dtype)
             if spec.moe:
-                lw.experts = ExpertFF(spec.moe, lw.act, src, p, cfg.hidden_size, dev, dtype)
+                lw.experts = ExpertFF(spec.moe, L.ACT_IDS[spec.act], src, p, cfg.hidden_size, dev, dtype)
             self.layers.append(lw)
         self.runs = cfg.layer_runs()
         steps = f32("loop_step") if any(t is not None for _, t in self.runs) else None
         self.run_step = [None if t is None else steps[t] for _, t in self.runs]
-
-    def _pack_ff(self, lw: HybridLayer, gate, up, down):
-        inter, hidden = gate.shape
-        lw.glu_fused = self.dtype == torch.bfloat16 and hidden % 8 == 0
-        if lw.glu_fused:
-            pad = -inter % 64         # zero gate / up rows and down columns: whole 128-column tiles, nothing added to the sums
-            z = lambda w: torch.nn.functional.pad(w, (0, 0, 0, pad))
-            lw.glu_bn = glu_tile_width(inter + pad)
-            lw.w_gate_up = L.interleave_gate_up(z(gate), z(up), lw.glu_bn)
-            down = torch.nn.functional.pad(down, (0, pad))
-        else:
-            lw.w_gate_up = torch.cat([gate, up], 0).contiguous()
-            if self.dtype == torch.bfloat16:
-                lw.w_gate_up = L.pad_rows(lw.w_gate_up, 1).contiguous()
-        lw.w_down = L.pad_rows(down, ROW_PAD).contiguous()
 
     # ------------------------------------------------------------------------------------------
     def mark(self, name: str):
@@ -200,17 +196,17 @@ class HybridDecoder:
         if tm is not None:
             tm.mark(name)
 
-    def rope_tables(self, rot_dim: int, base: float):
-        key = (rot_dim, base)
+    def rope_tables(self, rot_dim: int, base: float, scaling=None):
+        key = (rot_dim, base, repr(scaling))
         if key not in self._rope:
-            self._rope[key] = rope_table(rot_dim, base, self.max_positions, self.device)
+            self._rope[key] = rope_table(rot_dim, base, self.max_positions, self.device, scaling)
         return self._rope[key]
 
     def weight_bytes(self) -> int:
         ts = [self.embed, self.lm_head, self.final_norm]
         for l in self.layers:
-            ts += [t for t in list(l.mixer.w.values()) + [l.norm1, l.norm2, l.norm1b, l.norm2b, l.w_gate_up, l.w_down]
-                   + (l.experts.tensors() if l.experts else []) if t is not None]
+            ts += [t for t in list(l.mixer.w.values()) + [l.norm1, l.norm2, l.norm1b, l.norm2b]
+                   + (l.ff.tensors() if l.ff else []) + (l.experts.tensors() if l.experts else []) if t is not None]
         return sum(t.numel() * t.element_size() for t in ts)
 
     def page_bytes(self) -> int:
@@ -240,10 +236,10 @@ class HybridDecoder:
         ws = self.workspace(T)
         ws.decode_ws = decode_ws
         x, xb = ws.x[:T], ws.xb[:T]
-        copy = xb if ws.xb is not ws.x and not self.sandwich else None
+        copy = xb if ws.xb is not ws.x and self.post else None
         self.mark("begin")
         if hidden_in is None:
-            R.embed_rows(batch.token_ids, self.embed, x, copy)
+            R.embed_rows(batch.token_ids, self.embed, x, copy, scale=self.cfg.embedding_scale)
             self.mark("embed")
         else:
             x.copy_(hidden_in.float())
@@ -251,7 +247,7 @@ class HybridDecoder:
                 copy.copy_(hidden_in)
         self.callback_action, self.callback_info = None, {}
         self.captured = {}
-        layers = self._sandwich_layers if self.sandwich else self._post_layers
+        layers = self._post_layers if self.post else self._parallel_layers if self.parallel else self._sandwich_layers
         layers(x, xb, ws, batch, kv_caches, T, capture_layers or (), callbacks)
         if return_hidden:
             return x
@@ -273,8 +269,8 @@ class HybridDecoder:
             self.mark("out_gemm")
             R.scaled_add_norm(x, y, lw.norm1, c.postln_alpha, c.rms_norm_eps, x_out=x, xb=copy)
             self.mark("norm")
-            if lw.w_down is not None:
-                y = self._feed_forward(lw, ws, T)
+            if lw.ff is not None:
+                y = lw.ff.forward(self, xb, T, ws.take, "y")
                 R.scaled_add_norm(x, y, lw.norm2, c.postln_alpha, c.rms_norm_eps, x_out=x, xb=copy)
                 self.mark("norm")
             if r in capture:
@@ -309,10 +305,9 @@ class HybridDecoder:
                 residual_norm(x, y, post_w=lw.norm1b, pre_w=lw.norm2, xb=xb, **norm)
                 self.mark("norm")
                 if lw.experts is not None:
-                    y, dest = lw.experts.forward(self, xb, T)
-                    routed = dict(dest=dest, top=lw.experts.spec.top)
+                    y, routed = lw.experts.forward(self, xb, T)
                 else:
-                    y = self._feed_forward(lw, ws, T)
+                    y = lw.ff.forward(self, xb, T, ws.take, "y")
             residual_norm(x, y, post_w=lw.norm1b if lw.norm2 is None else lw.norm2b, **routed, **ahead, **norm)
             self.mark("norm")
             if r in capture:
@@ -320,23 +315,40 @@ class HybridDecoder:
             if callbacks is not None and self._run_callbacks(callbacks, "post", r, x, None):
                 break
 
-    def _feed_forward(self, lw: HybridLayer, ws, T: int):
-        xb = ws.xb[:T]
-        if lw.glu_fused:
-            bn = 256 if (T > 1024 and lw.w_gate_up.shape[0] % 256 == 0) else lw.glu_bn
-            act = ops.gemm_glu(xb, lw.w_gate_up, act=lw.act, out=ws.take("act", T, lw.w_down.shape[1]), bn=bn)
-        else:
-            gu = L.gemm(xb, lw.w_gate_up, out=ws.take("gu", T, lw.w_gate_up.shape[0]))
-            act = ops.glu(gu, lw.act, out=ws.take("act", T, lw.w_down.shape[1]))
-        self.mark("gate_up_gemm")
-        y = L.gemm(act, lw.w_down, out=ws.take("y", T, lw.w_down.shape[0]))
-        self.mark("down_gemm")
-        return y
+    def _parallel_layers(self, x, xb, ws, batch, kv_caches, T, capture, callbacks):
+        """One fused pass between two layers: both sublayers' outputs join the residual sum, norm in front of the next layer."""
+        norm = dict(kind=self.cfg.norm_type, eps=self.cfg.rms_norm_eps)
+        for r, (i, _) in enumerate(self.runs):
+            lw = self.layers[i]
+            if r == 0 or callbacks is not None or r - 1 in capture:      # not done by the pass behind the layer before
+                if self.run_step[r] is not None:
+                    residual_norm(x, add=self.run_step[r], **norm)
+                if callbacks is not None and self._run_callbacks(callbacks, "pre", r, x, None):
+                    break
+                residual_norm(x, pre_w=lw.norm1, xb=xb, **norm)
+                self.mark("norm")
+            ahead = {}
+            if not (r + 1 == len(self.runs) or callbacks is not None or r in capture):
+                ahead = dict(add=self.run_step[r + 1], pre_w=self.layers[self.runs[r + 1][0]].norm1, xb=xb)
+            y, parts = lw.mixer.forward(self, ws, batch, kv_caches[r], T), {}
+            self.mark("out_gemm")
+            if lw.experts is not None:
+                mixed = y
+                y, parts = lw.experts.forward(self, xb, T)
+                parts["plus"] = mixed
+            elif lw.ff is not None:
+                parts["plus"] = lw.ff.forward(self, xb, T, ws.take, "y2")
+            residual_norm(x, y, **parts, **ahead, **norm)
+            self.mark("norm")
+            if r in capture:
+                self.captured[r] = x.clone()
+            if callbacks is not None and self._run_callbacks(callbacks, "post", r, x, None):
+                break
 
     def _final_norm(self, x, rows=None):
         n = x.shape[0] if rows is None else rows.shape[0]
         hn = torch.empty((n, self.cfg.hidden_size), dtype=self.dtype, device=self.device)
-        if self.sandwich:
+        if not self.post:
             residual_norm(x, pre_w=self.final_norm, xb=hn, rows=rows, kind=self.cfg.norm_type, eps=self.cfg.rms_norm_eps)
         else:
             R.scaled_add_norm(x, None, self.final_norm, 1.0, self.cfg.rms_norm_eps, rows=rows, xb=hn)

@@ -1,5 +1,6 @@
 """Token mixers of heterogeneous decoders: attention (chunked, windowed with kept first tokens or full; query / key norm over
-the row or per head; optional short convolution), windowed latent attention, RG-LRU and gated linear attention. Each class
+the row or per head; optional short convolution, soft-capped scores, distance biases, sinks), latent attention (windowed or
+full, with or without a rotated part and an output gate), RG-LRU, gated linear and lightning attention. Each class
 packs its layer's weights into the layouts of the ops and runs a step's tokens:
 ``forward(model, ws, batch, cache, T) -> y [T, >= hidden]``, reading the layer input from ``ws.xb``.
 
@@ -65,7 +66,14 @@ class AttentionMixer(_Mixer):
         self.nq, self.nk, self.nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * self.dv
         names = ("q", "k") if m.v_from_k else ("q", "k", "v")
         self.w["wqk"] = self.mat(*names)
-        self.w["bqk"] = _pad_bias([self._src.get(self._p + n + ".b") for n in names], self.w["wqk"].shape[0], self.device)
+        self.w["bqk"] = (_pad_bias([self._src.get(self._p + n + ".b") for n in names], self.w["wqk"].shape[0], self.device)
+                         if m.qkv_bias else None)
+        self.w["sink"] = self.vec("sink") if m.sink else None
+        self.w["rel"] = None
+        if m.bias_max:            # the learned table, one entry per distance
+            table = self.vec("rel")
+            rows = torch.tensor(ops.distance_rows(table.shape[0], m.bias_max), device=self.device)
+            self.w["rel"] = table[rows].t().contiguous()
         self.w["wo"] = self.mat("o")
         self.w["bo"] = _pad_bias([self._src.get(self._p + "o.b")], self.w["wo"].shape[0], self.device) if m.o_bias else None
         norm = m.row_qk_norm or m.head_qk_norm
@@ -103,7 +111,8 @@ class AttentionMixer(_Mixer):
                             ring=cache.state["conv"] if m.taps else None, **common)
         model.mark("qk_prep")
         o = ws.take("mix", T, m.heads * self.dv)
-        mask = dict(window=ops.chunk_window(m.chunk) if m.chunk > 0 else m.window, keep_first=m.keep_first, dim=m.dim)
+        mask = dict(window=ops.chunk_window(m.chunk) if m.chunk > 0 else m.window, keep_first=m.keep_first, dim=m.dim,
+                    sinks=self.w["sink"], softcap=m.softcap, rel_bias=self.w["rel"])
         if batch.is_decode:
             ops.paged_decode(q, kv, batch.block_tables, batch.ctx_lens, n_q=m.heads, n_kv=m.kv_heads, scale=m.scale, out=o,
                              workspace=ws.decode_ws, pages_per_split=getattr(ws.decode_ws, "pages_per_split", 32),
@@ -117,10 +126,11 @@ class AttentionMixer(_Mixer):
 
 
 class LatentMixer(_Mixer):
-    """Latent attention without positions. Absorbed form: the key up-projection moves into the query, the value up-projection
-    behind the attention, and every head attends over the same cached latent rows (decode steps, and any sizes). Prefill
-    steps with head sizes of 128 expand the keys and values of the rows they can see instead: a third of the products, on
-    the tcgen05 attention kernel."""
+    """Latent attention. Absorbed form: the key up-projection moves into the query, the value up-projection behind the
+    attention, and every head attends over the same cached rows (decode steps, and any sizes). Prefill steps with head sizes
+    of 128 expand the keys and values of the rows they can see instead: a third of the products, on the tcgen05 attention
+    kernel. A rotated part is ``rope_part`` further columns of queries and cached rows; the expansion copies the key part
+    into every head's key by an identity block of its weight."""
 
     def pack(self):
         m = self.spec
@@ -128,26 +138,41 @@ class LatentMixer(_Mixer):
         torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
         if self.dtype == torch.float32:
             torch.backends.cuda.matmul.allow_tf32 = False
-        self.w["wdown"] = self.mat("dq", "dkv")
-        self.w["q_norm"], self.w["kv_norm"] = self.vec("dq.norm"), self.vec("dkv.norm")
-        self.w["wuq"] = self.mat("uq")
+        self.direct = m.q_rank == 0              # queries straight from the layer input
+        if self.direct:
+            self.w["wdown"] = self.mat("q", "dkv", *(["g"] if m.gate else []))
+            self.w["q_norm"] = self.w["wuq"] = None
+            # queries | latent and key part | gate, every slice on a 16-byte boundary where the sizes allow it
+            self.kv_col = m.heads * (m.dim + m.rope_part)
+            self.g_col = self.kv_col + m.kv_rank + m.rope_part
+        else:
+            if m.gate or m.rope_part:
+                raise ValueError("latent mixer: a gate or a rotated part goes with directly projected queries")
+            self.w["wdown"] = self.mat("dq", "dkv")
+            self.w["q_norm"] = self.vec("dq.norm")
+            self.w["wuq"] = self.mat("uq")
+        self.w["kv_norm"] = self.vec("dkv.norm")
         up = lambda n, d: self._src.get(self._p + n).to(self.device, self.dtype).reshape(m.heads, d, m.kv_rank)
         self.w["wuk"] = up("uk", m.dim).contiguous()                           # [heads, dim, rank]
         self.w["wuv"] = up("uv", m.vdim).transpose(1, 2).contiguous()          # [heads, rank, vdim]
-        self.expand = (self.dtype == torch.bfloat16 and self.device.type == "cuda" and m.dim == m.vdim == 128
-                       and m.kv_rank % 8 == 0)
+        self.expand = (self.dtype == torch.bfloat16 and self.device.type == "cuda" and m.dim + m.rope_part == m.vdim == 128
+                       and m.kv_rank % 8 == 0 and m.rope_part % 8 == 0)
         if self.expand:
-            self.w["wukv"] = torch.stack([up("uk", 128), up("uv", 128)], 1).reshape(m.heads * 256, m.kv_rank).contiguous()
+            n, r = m.rope_part, m.kv_rank
+            k, v = torch.nn.functional.pad(up("uk", m.dim), (0, n)), torch.nn.functional.pad(up("uv", 128), (0, n))
+            part = torch.eye(r + n, device=self.device, dtype=self.dtype)[r:].expand(m.heads, n, r + n)
+            self.w["wukv"] = torch.cat([k, part, v], 1).reshape(m.heads * 256, r + n).contiguous()
         self.w["sink"] = self.vec("sink") if m.sink else None
         self.w["wo"] = self.mat("o")
 
     def workspace(self):
         m = self.spec
-        return {"proj": self.w["wdown"].shape[0], "cq": m.q_rank, "q": self.w["wuq"].shape[0], "qlat": m.heads * m.kv_rank,
+        q = {"q": m.heads * (m.dim + m.rope_part)} if self.direct else {"cq": m.q_rank, "q": self.w["wuq"].shape[0]}
+        return {"proj": self.w["wdown"].shape[0], **q, "qlat": m.heads * (m.kv_rank + m.rope_part),
                 "olat": m.heads * m.kv_rank, "mix": m.heads * m.vdim}
 
     def alloc(self, num_pages, slots):
-        return torch.zeros((num_pages, PAGE, self.spec.kv_rank), dtype=self.dtype, device=self.device)
+        return torch.zeros((num_pages, PAGE, self.spec.kv_elems()), dtype=self.dtype, device=self.device)
 
     def _span(self, batch, T: int):
         """The expanded form's rows, or None when the step takes the absorbed form: decode steps, and portions so short that
@@ -164,14 +189,26 @@ class LatentMixer(_Mixer):
         m, w = self.spec, self.w
         p = L.gemm(ws.xb[:T], w["wdown"], out=ws.take("proj", T, w["wdown"].shape[0]))
         model.mark("in_gemm")
-        cq = ws.take("cq", T, m.q_rank)
-        MLA.latent_prep(p, m.q_rank, m.kv_rank, w["q_norm"], w["kv_norm"], self.eps, batch.slot_mapping, cq, cache)
-        model.mark("latent_prep")
-        q = L.gemm(cq, w["wuq"], out=ws.take("q", T, w["wuq"].shape[0]))
-        model.mark("uq_gemm")
-        span = self._span(batch, T)
+        span, RK = self._span(batch, T), m.kv_elems()
+        ql = ws.take("qlat", m.heads * T, RK).view(m.heads, T, RK)
+        if self.direct:
+            cos, sin = model.rope_tables(m.rot_dim, m.rot_base, m.rot_scaling)
+            whole = span is not None or m.rope_part == 0       # whole heads, or the rotated parts behind the absorbed queries
+            q = ws.take("q", T, m.heads * (m.dim + m.rope_part))
+            MLA.latent_rope_prep(p, heads=m.heads, dim=m.dim, part=m.rope_part, rot=m.rot_dim, rank=m.kv_rank, kv_col=self.kv_col,
+                                 kv_w=w["kv_norm"], eps=self.eps, positions=batch.positions, slot_mapping=batch.slot_mapping,
+                                 cos_t=cos, sin_t=sin, copy=whole, cache=cache,
+                                 q_out=q.unflatten(1, (m.heads, -1)) if whole else ql[:, :, m.kv_rank:].transpose(0, 1))
+            q = q if whole else p
+            model.mark("latent_prep")
+        else:
+            cq = ws.take("cq", T, m.q_rank)
+            MLA.latent_prep(p, m.q_rank, m.kv_rank, w["q_norm"], w["kv_norm"], self.eps, batch.slot_mapping, cq, cache)
+            model.mark("latent_prep")
+            q = L.gemm(cq, w["wuq"], out=ws.take("q", T, w["wuq"].shape[0]))
+            model.mark("uq_gemm")
         if span is not None:
-            lat = ws.spare("latent_rows", span.pages * PAGE, m.kv_rank)
+            lat = ws.spare("latent_rows", span.pages * PAGE, RK)
             MLA.latent_gather(cache, batch.block_tables, batch.ctx_lens, span, lat)
             kv = L.gemm(lat, w["wukv"], out=ws.spare("latent_kv", span.pages * PAGE, m.heads * 256))
             model.mark("ukv_gemm")
@@ -179,9 +216,9 @@ class LatentMixer(_Mixer):
                                      heads=m.heads, scale=m.scale, window=m.window, sinks=w["sink"],
                                      out=ws.take("mix", T, m.heads * 128))
             model.mark("latent_prefill")
-            return L.gemm(o, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
-        ql = ws.take("qlat", m.heads * T, m.kv_rank).view(m.heads, T, m.kv_rank)
-        torch.bmm(q[:, :m.heads * m.dim].unflatten(1, (m.heads, m.dim)).transpose(0, 1), w["wuk"], out=ql)
+            return self._output(model, ws, p, o, T)
+        plain = q[:, :m.heads * (m.dim + m.rope_part)].unflatten(1, (m.heads, -1))[:, :, :m.dim].transpose(0, 1)
+        torch.bmm(plain, w["wuk"], out=ql[:, :, :m.kv_rank])
         model.mark("uk_gemm")
         ol = ws.take("olat", m.heads * T, m.kv_rank).view(m.heads, T, m.kv_rank)
         rows = (None, None) if batch.is_decode else (batch.q_start, batch.q_len)
@@ -192,7 +229,13 @@ class LatentMixer(_Mixer):
         o = ws.take("mix", T, m.heads * m.vdim)
         torch.bmm(ol, w["wuv"], out=o.unflatten(1, (m.heads, m.vdim)).transpose(0, 1))
         model.mark("uv_gemm")
-        return L.gemm(o, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
+        return self._output(model, ws, p, o, T)
+
+    def _output(self, model, ws, p, o, T):
+        if self.spec.gate:
+            R.sigmoid_gate(o, p[:, self.g_col:self.g_col + o.shape[1]])
+            model.mark("out_gate")
+        return L.gemm(o, self.w["wo"], out=ws.take("y", T, self.w["wo"].shape[0]))
 
 
 class RgLruMixer(_Mixer):
@@ -287,18 +330,54 @@ class GlaMixer(_Mixer):
         return L.gemm(out, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
 
 
-MIXERS = {"attention": AttentionMixer, "latent": LatentMixer, "rglru": RgLruMixer, "gla": GlaMixer}
+class LightningMixer(_Mixer):
+    def pack(self):
+        m = self.spec
+        self.nk, self.nv = m.heads * m.dim, m.heads * m.vdim
+        self.w["wqkvg"] = self.mat("q", "k", "v", "g")
+        self.w["norm"] = self.vec("norm")
+        self.w["wo"] = self.mat("o")
+        self.w["forget"], self.w["powers"] = R.lightning_tables(m.decay, self.device)
+
+    def workspace(self):
+        return {"proj": self.w["wqkvg"].shape[0], "mix": self.nv, "f32": self.nv}
+
+    def state_shapes(self):
+        m = self.spec
+        return {"rec": (m.heads, m.dim, m.vdim)}
+
+    def forward(self, model, ws, batch, st, T):
+        m, w, nk, nv = self.spec, self.w, self.nk, self.nv
+        p = L.gemm(ws.xb[:T], w["wqkvg"], out=ws.take("proj", T, w["wqkvg"].shape[0]), act="silu", act_cols=2 * nk + nv)
+        model.mark("in_gemm")
+        acc = ws.take("f32", T, nv)
+        R.lightning(SeqView.of(batch), p[:, :nk], p[:, nk:2 * nk], p[:, 2 * nk:2 * nk + nv], heads=m.heads, dim=m.dim, vdim=m.vdim,
+                    tables=(w["forget"], w["powers"]), state=st["rec"], out=acc)
+        model.mark("lightning")
+        out = ws.take("mix", T, nv)
+        R.row_norm_gate(acc, p[:, 2 * nk + nv:2 * (nk + nv)], w["norm"], self.eps, out)
+        model.mark("lightning_gate")
+        return L.gemm(out, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
+
+
+MIXERS = {"attention": AttentionMixer, "latent": LatentMixer, "rglru": RgLruMixer, "gla": GlaMixer, "lightning": LightningMixer}
 
 
 def mixer_shapes(m: MixerSpec, hidden: int) -> Dict[str, Tuple[int, ...]]:
     """Checkpoint tensors of a mixer (names behind ``mix.``) and their shapes."""
     if m.kind == "attention":
         nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.value_dim
-        s = {"q": (nq, hidden), "q.b": (nq,), "k": (nk, hidden), "k.b": (nk,), "o": (hidden, m.heads * m.value_dim)}
+        s = {"q": (nq, hidden), "k": (nk, hidden), "o": (hidden, m.heads * m.value_dim)}
+        if not m.v_from_k:
+            s["v"] = (nv, hidden)
+        if m.qkv_bias:
+            s.update({n + ".b": s[n][:1] for n in ("q", "k", "v") if n in s})
         if m.o_bias:
             s["o.b"] = (hidden,)
-        if not m.v_from_k:
-            s.update({"v": (nv, hidden), "v.b": (nv,)})
+        if m.sink:
+            s["sink"] = (m.heads,)
+        if m.bias_max:
+            s["rel"] = (m.bias_rows or 32, m.heads)
         if m.row_qk_norm:
             s.update({"q.norm": (nq,), "k.norm": (nk,)})
         if m.head_qk_norm:
@@ -307,7 +386,11 @@ def mixer_shapes(m: MixerSpec, hidden: int) -> Dict[str, Tuple[int, ...]]:
             s.update({n + ".conv": (s[n][0], m.taps) for n in ("q", "k", "v") if n in s})
         return s
     if m.kind == "latent":
-        s = {"dq": (m.q_rank, hidden), "dq.norm": (m.q_rank,), "uq": (m.heads * m.dim, m.q_rank), "dkv": (m.kv_rank, hidden),
+        qd = m.heads * (m.dim + m.rope_part)
+        s = {"dq": (m.q_rank, hidden), "dq.norm": (m.q_rank,), "uq": (qd, m.q_rank)} if m.q_rank else {"q": (qd, hidden)}
+        if m.gate:
+            s["g"] = (m.heads * m.vdim, hidden)
+        s = {**s, "dkv": (m.kv_rank + m.rope_part, hidden),
              "dkv.norm": (m.kv_rank,), "uk": (m.heads * m.dim, m.kv_rank), "uv": (m.heads * m.vdim, m.kv_rank),
              "o": (hidden, m.heads * m.vdim)}
         if m.sink:
@@ -319,13 +402,15 @@ def mixer_shapes(m: MixerSpec, hidden: int) -> Dict[str, Tuple[int, ...]]:
         return {"y": (w, hidden), "y.b": (w,), "x": (w, hidden), "x.b": (w,), "conv": (w, m.taps), "conv.b": (w,),
                 "ra": (nb, bs, bs), "ra.b": (nb, bs), "ri": (nb, bs, bs), "ri.b": (nb, bs), "lam": (w,), "o": (hidden, w)}
     nk, nv, r = m.heads * m.dim, m.heads * m.vdim, m.decay_rank or 16
+    if m.kind == "lightning":
+        return {"q": (nk, hidden), "k": (nk, hidden), "v": (nv, hidden), "g": (nv, hidden), "o": (hidden, nv), "norm": (nv,)}
     return {"q": (nk, hidden), "k": (nk, hidden), "v": (nv, hidden), "g": (nv, hidden), "o": (hidden, nv), "norm": (m.vdim,),
             "a1": (r, hidden), "a2": (nk, r), "a2.b": (nk,)}
 
 
-def rope_table(rot_dim: int, base: float, max_positions: int, device):
+def rope_table(rot_dim: int, base: float, max_positions: int, device, scaling: Optional[RopeScaling] = None):
     if rot_dim == 0:
         return None, None
-    inv, _ = rope.inv_frequencies(rot_dim, base, RopeScaling(), max_positions)
+    inv, stretch = rope.inv_frequencies(rot_dim, base, scaling or RopeScaling(), max_positions)
     ang = torch.arange(max_positions, dtype=torch.float64)[:, None] * inv[None, :]
-    return ang.cos().float().contiguous().to(device), ang.sin().float().contiguous().to(device)
+    return (ang.cos() * stretch).float().contiguous().to(device), (ang.sin() * stretch).float().contiguous().to(device)

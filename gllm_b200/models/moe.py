@@ -20,7 +20,9 @@ from .. import ops
 from ..ops import linear as L
 from ..ops import moe as M
 from .config import ModelConfig, MoeSpec
-from .weights import _fold, layer_prefix, shard_range
+from .weights import _fold, glu_tile_width, layer_prefix, shard_range
+
+FF_ROW_PAD = 32       # out-features of packed feed-forward matrices are padded to this many rows (the GEMM's column granularity)
 
 
 @dataclass
@@ -516,17 +518,80 @@ class ExpertPager:
 # --------------------------------------------------------------------------------------------------------------------
 # mixture of experts of a heterogeneous decoder's layer (models/hybrid.py)
 # --------------------------------------------------------------------------------------------------------------------
+class GatedFF:
+    """W_down(act(W_gate h) * W_up h), bf16 (the activation in the epilogue of one GEMM) or true fp32."""
+
+    def __init__(self, gate, up, down, act: int, dtype):
+        inter, hidden = gate.shape
+        self.act = act
+        self.fused = dtype == torch.bfloat16 and hidden % 8 == 0
+        if self.fused:
+            pad = -inter % 64         # zero gate / up rows and down columns: whole 128-column tiles, nothing added to the sums
+            z = lambda w: torch.nn.functional.pad(w, (0, 0, 0, pad))
+            self.bn = glu_tile_width(inter + pad)
+            self.w_in = L.interleave_gate_up(z(gate), z(up), self.bn)
+            down = torch.nn.functional.pad(down, (0, pad))
+        else:
+            self.w_in = torch.cat([gate, up], 0).contiguous()
+        self.w_down = L.pad_rows(down, FF_ROW_PAD).contiguous()
+
+    def tensors(self):
+        return [self.w_in, self.w_down]
+
+    def workspace(self):
+        return {"act": self.w_down.shape[1], "y": self.w_down.shape[0], **({} if self.fused else {"gu": self.w_in.shape[0]})}
+
+    def forward(self, model, h, T: int, take, y: str, marks=("gate_up_gemm", "down_gemm")):
+        """``take(name, rows, columns)``: a workspace buffer; the result goes to the fp32 buffer ``y``."""
+        act = take("act", T, self.w_down.shape[1])
+        if self.fused:
+            bn = 256 if (T > 1024 and self.w_in.shape[0] % 256 == 0) else self.bn
+            ops.gemm_glu(h, self.w_in, act=self.act, out=act, bn=bn)
+        else:
+            ops.glu(L.gemm(h, self.w_in, out=take("gu", T, self.w_in.shape[0])), self.act, out=act)
+        model.mark(marks[0])
+        out = L.gemm(act, self.w_down, out=take(y, T, self.w_down.shape[0]))
+        model.mark(marks[1])
+        return out
+
+
+class PlainFF:
+    """W_down act(W_up h), the activation (``ops.linear.STORE_ACTS``) in the epilogue of the first GEMM."""
+
+    def __init__(self, up, down, act: str, dtype):
+        self.act = act
+        pad = -up.shape[0] % FF_ROW_PAD if dtype == torch.bfloat16 else 0
+        self.w_in = torch.nn.functional.pad(up, (0, 0, 0, pad)).contiguous()
+        self.w_down = L.pad_rows(torch.nn.functional.pad(down, (0, pad)), FF_ROW_PAD).contiguous()
+
+    def tensors(self):
+        return [self.w_in, self.w_down]
+
+    def workspace(self):
+        return {"act": self.w_in.shape[0], "y": self.w_down.shape[0]}
+
+    def forward(self, model, h, T: int, take, y: str, marks=("up_gemm", "down_gemm")):
+        act = L.gemm(h, self.w_in, out=take("act", T, self.w_in.shape[0]), act=self.act)
+        model.mark(marks[0])
+        out = L.gemm(act, self.w_down, out=take(y, T, self.w_down.shape[0]))
+        model.mark(marks[1])
+        return out
+
+
 class ExpertFF:
     """One layer's experts, bf16 or true fp32: router -> top-k -> routed rows in per-expert blocks -> grouped gate / up and
-    down projections. ``forward`` returns the experts' rows and the place of each (token, pick) among them; the caller sums
-    them (``ops.residual.residual_norm`` does it together with the norm behind the sublayer)."""
+    down projections; beside them a shared expert (its gate is one more row of the router's projection). ``forward`` returns
+    what the caller sums with ``ops.residual.residual_norm`` (together with the norms around the sublayer): the experts' rows
+    and, by keyword, the place of each (token, pick) among them, the picks' weights (unless the spec scales the experts'
+    inputs), the shared expert's rows and gate."""
 
     def __init__(self, spec: MoeSpec, act: int, src, prefix: str, hidden: int, device, dtype):
-        if not spec.scale_input:
-            raise ValueError("expert outputs are summed unweighted: the spec must scale the experts' inputs")
         self.spec, self.act, self.hidden = spec, act, hidden
         get = lambda n: src.get(prefix + "mlp." + n).to(device, dtype)
-        self.router = L.pad_rows(get("router"), 32).contiguous()
+        self.router = get("router")
+        if spec.shared_gate:
+            self.router = torch.cat([self.router, get("shared.sg")], 0)
+        self.router = L.pad_rows(self.router, 32).contiguous()
         self.fused = dtype == torch.bfloat16 and hidden % 8 == 0
         pad = -spec.ff % 64 if self.fused else 0       # zero gate / up rows and down columns add nothing to the sums
         self.inter = spec.ff + pad
@@ -538,20 +603,24 @@ class ExpertFF:
             downs.append(L.pad_rows(d, 128))
         self.w_gate_up, self.w_down = torch.cat(gus).contiguous(), torch.cat(downs).contiguous()
         self.glu_bn = 256 if self.inter % 128 == 0 else 128
+        self.shared = GatedFF(get("shared.gate"), get("shared.up"), get("shared.down"), act, dtype) if spec.shared_ff else None
 
     def tensors(self):
-        return [self.router, self.w_gate_up, self.w_down]
+        return [self.router, self.w_gate_up, self.w_down] + (self.shared.tensors() if self.shared else [])
 
     def workspace(self, model, T: int) -> M.MoeWorkspace:
         holder = model.__dict__.setdefault("_expert_ws", {})
         s = self.spec
-        key = (s.experts, s.top, self.inter)
+        key = (s.experts, s.top, self.inter, s.shared_ff)
         ws = holder.get(key)
         if ws is None or ws.ids.shape[0] < T:
             n = max(T, 256)
             ws = M.MoeWorkspace(n, s.top, self.hidden, self.inter, s.experts, model.device, model.dtype,
                                 out_cols=self.w_down.shape[0] // s.experts)
             ws.logits = torch.zeros((n, self.router.shape[0]), dtype=torch.float32, device=model.device)
+            if self.shared is not None:
+                ws.shared = {k: torch.zeros((n, c), dtype=torch.float32 if k == "y" else model.dtype, device=model.device)
+                             for k, c in self.shared.workspace().items()}
             ws.gu = None if self.fused else torch.zeros((ws.max_rows, 2 * self.inter), dtype=model.dtype, device=model.device)
             holder[key] = ws
         return ws
@@ -561,9 +630,10 @@ class ExpertFF:
         ws = self.workspace(model, T)
         logits = L.gemm(h, self.router, out=ws.logits[:T])
         on_gpu = dict(out_ids=ws.ids[:T], out_w=ws.w[:T]) if h.is_cuda else {}
-        ids, w = M.route(logits[:, :s.experts], s.top, norm_topk=s.norm_topk, scoring=s.scoring, **on_gpu)
+        ids, w = M.route(logits[:, :s.experts], s.top, norm_topk=s.norm_topk, scoring=s.scoring, scale=s.scale, groups=s.groups,
+                         keep_groups=s.keep_groups, **on_gpu)
         model.mark("moe_route")
-        M.permute(h, None, ids, ws, 0, s.experts, row_w=w)
+        M.permute(h, None, ids, ws, 0, s.experts, row_w=w if s.scale_input else None)
         model.mark("moe_permute")
         if self.fused:
             L.set_block_rows(ws.blk_rows if h.is_cuda else None)
@@ -575,4 +645,9 @@ class ExpertFF:
         model.mark("moe_gate_up")
         L.gemm_grouped(ws.act, self.w_down, ws.blk_group, s.experts, out=ws.y_perm, block_rows=ws.blk_rows)
         model.mark("moe_down")
-        return ws.y_perm, ws.dest
+        out = dict(dest=ws.dest, top=s.top, row_w=None if s.scale_input else w)
+        if self.shared is not None:
+            take = lambda k, rows, cols: ws.shared[k][:rows]
+            out["gated"] = self.shared.forward(model, h, T, take, "y", ("shared_gate_up", "shared_down"))
+            out["gate"] = logits[:, s.experts] if s.shared_gate else None
+        return ws.y_perm, out

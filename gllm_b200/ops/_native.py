@@ -26,6 +26,7 @@ _SIGNATURES = {
     "gllm_kernels_abi_version": (I, []),
     "gllm_gemm_bf16": (I, [P, L, P, L, P, L, I, I, I, I, P, P, I, F, F, I, P, I, I]),
     "gllm_gemm_bf16_softcap": (I, [P, L, P, L, P, L, I, I, I, I, P, P, I, F, F, I, P, F]),
+    "gllm_gemm_bf16_act": (I, [P, L, P, L, P, L, I, I, I, I, P, I, I, I, P]),
     "gllm_gemm_set_splitk_workspace": (I, [P, L, P, I]),
     "gllm_gemm_set_splitk_workspace_stream": (I, [P, P, L, P, I]),
     "gllm_gemm_bf16_residual": (I, [P, L, P, L, P, L, P, L, P, I, I, I, P, I, P, I, I]),
@@ -46,9 +47,9 @@ _SIGNATURES = {
     "gllm_gemm_bf16_qkv_fp8kv": (I, [P, L, P, L, I, I, I, I, P, P, I, P, P, P, P, I, P, P, F, P, I, F, F, P, F, P, I, I]),
     "gllm_gemm_fp8": (I, [P, L, P, L, P, L, I, I, I, I, P, P, I, P, I, I]),
     "gllm_decode_scratch_floats": (L, [I, I, I]),
-    "gllm_paged_decode": (I, [P, P, P, I, P, I, P, I, I, I, F, I, I, P, P, I, I, P, I, P]),
+    "gllm_paged_decode": (I, [P, P, P, I, P, I, P, I, I, I, F, I, I, P, P, I, I, P, I, F, P, I, P]),
     "gllm_paged_prefill": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, F, I, I, P, P]),
-    "gllm_paged_prefill_tc": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, F, I, I, I, P, I, P]),
+    "gllm_paged_prefill_tc": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, F, I, I, I, P, I, F, P, I, P]),
     "gllm_paged_decode_fp8": (I, [P, P, P, I, P, I, P, I, I, I, F, I, I, P, P, I, P, F, P]),
     "gllm_paged_prefill_fp8": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, F, I, I, P, F, P]),
     "gllm_embed_gather": (I, [P, P, I, I, F, P, P, I, P]),
@@ -56,10 +57,10 @@ _SIGNATURES = {
     "gllm_layernorm": (I, [P, P, P, P, I, I, F, P, P]),
     "gllm_glu": (I, [P, L, I, I, I, P, P]),
     "gllm_rope_kv_write": (I, [P, L, I, I, I, I, I, P, P, P, P, I, P, P, F, P, P, I, P]),
-    "gllm_attention_any": (I, [P, P, P, P, I, I, P, I, P, P, P, I, I, I, I, I, I, F, I, I, I, P, P]),
-    "gllm_attention_mma": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, F, I, I, I, P, P]),
+    "gllm_attention_any": (I, [P, P, P, P, I, I, P, I, P, P, P, I, I, I, I, I, I, F, I, I, I, P, F, P, I, P]),
+    "gllm_attention_mma": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, F, I, I, I, P, F, P, I, P]),
     "gllm_gemm_simt_grouped": (I, [P, L, P, L, P, L, I, I, I, I, I, P, P, P]),
-    "gllm_gemm_simt": (I, [P, L, P, L, P, L, I, I, I, I, I, P, F, P]),
+    "gllm_gemm_simt": (I, [P, L, P, L, P, L, I, I, I, I, I, P, F, I, I, P]),
     "gllm_paged_attention_fp8kv": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, F, I, I, F, P]),
     "gllm_rope_kv_write_fp8": (I, [P, L, I, I, I, I, I, P, P, P, P, I, P, P, F, P, P, I, F, P]),
     "gllm_pool": (I, [P, P, P, I, I, I, P, P]),

@@ -6,7 +6,8 @@ CUDA path: ``csrc/kernels/attention.cu`` / ``fa_prefill_sm100.cu`` (head size 12
 ``attention_mma.cu`` (other multiples of 8 up to 256, warp-level tensor cores), ``attention_any.cu`` (any size, bf16 or fp32)
 or the fp8 kernel in ``misc.cu``. CPU path / oracle: plain fp32 softmax attention with the
 reference's semantics (src/compat/scalar_ops.rs:196-278,316-378): scale 1/sqrt(d), GQA head mapping
-``kv_h = h // (Hq/Hkv)``, causal mask, max-subtracted softmax, optional sliding window (with kept first tokens) and sinks.
+``kv_h = h // (Hq/Hkv)``, causal mask, max-subtracted softmax, optional sliding window (with kept first tokens) and sinks, soft-capped scores and
+biases by distance.
 """
 from __future__ import annotations
 
@@ -53,10 +54,27 @@ def chunk_window(chunk: int) -> int:
     return -int(chunk)
 
 
+def distance_rows(rows: int, far: int):
+    """Which row of a learned table of ``rows`` rows belongs to a key n tokens back, for n = 0, 1, ... up to the first distance
+    of the last row (every longer one has it too): one row per distance up to half the table, then logarithmic steps that
+    end at distance ``far``."""
+    half, out = rows // 2, []
+    while not out or out[-1] < rows - 1:
+        n = len(out)
+        if n < half:
+            out.append(n)
+        elif half == 0 or far <= half:
+            out.append(rows - 1)
+        else:
+            out.append(min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half))))
+    return out
+
+
 def attention_ref(q, kv_cache, block_tables, q_start, q_len, ctx_lens, n_q, n_kv, scale, causal=True, window=0,
-                  sinks=None, keep_first=0, dim=None):
+                  sinks=None, keep_first=0, dim=None, softcap=0.0, rel_bias=None):
     """q: [T, n_q*D]. Returns [T, n_q*DV] in q.dtype. Works on any device (used as the oracle). ``window`` > 0: sliding
-    window, the first ``keep_first`` tokens stay visible; < 0: chunks of -window positions (``chunk_window``)."""
+    window, the first ``keep_first`` tokens stay visible; < 0: chunks of -window positions (``chunk_window``). ``softcap``: scores
+    become cap * tanh(score / cap); ``rel_bias`` [n_q, n] joins the capped scores, by distance (the last entry: n - 1 and more)."""
     D, DV = head_sizes(kv_cache, n_kv, dim)
     out = q.new_zeros((q.shape[0], n_q * DV))
     group = n_q // n_kv
@@ -71,6 +89,10 @@ def attention_ref(q, kv_cache, block_tables, q_start, q_len, ctx_lens, n_q, n_kv
         scores = torch.einsum("qhd,khd->hqk", qs, kk) * scale
         pos_q = torch.arange(ctx - ql, ctx, device=q.device)[:, None]
         pos_k = torch.arange(ctx, device=q.device)[None, :]
+        if softcap:
+            scores = softcap * torch.tanh(scores / softcap)
+        if rel_bias is not None:
+            scores = scores + rel_bias[:, (pos_q - pos_k).clamp(0, rel_bias.shape[1] - 1)]
         mask = torch.ones((ql, ctx), dtype=torch.bool, device=q.device)
         if causal:
             mask &= pos_k <= pos_q
@@ -107,18 +129,26 @@ def _mma_head(q, kv_cache, D, DV) -> bool:
             and max(D, DV) <= 256 and q.is_contiguous())
 
 
+def _bias_args(rel_bias, n_q):
+    if rel_bias is None:
+        return None, 0
+    assert rel_bias.dtype == torch.float32 and rel_bias.is_contiguous() and rel_bias.shape[0] == n_q
+    return rel_bias.data_ptr(), rel_bias.shape[1]
+
+
 def _attention_mma(q, out, kv_cache, block_tables, q_start, q_len, ctx_lens, n_seqs, max_q_len, n_q, n_kv, D, DV, scale, causal,
-                   window, keep_first, sinks):
+                   window, keep_first, sinks, softcap, rel_bias):
     rc = nv.lib().gllm_attention_mma(q.data_ptr(), out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
                                      block_tables.data_ptr(), block_tables.shape[1], nv.ptr(q_start), nv.ptr(q_len),
                                      ctx_lens.data_ptr(), n_seqs, max_q_len, n_q, n_kv, D, DV, scale,
-                                     1 if causal else 0, window, keep_first, nv.ptr(sinks), nv.stream_ptr())
+                                     1 if causal else 0, window, keep_first, nv.ptr(sinks), softcap, *_bias_args(rel_bias, n_q),
+                                     nv.stream_ptr())
     nv.check(rc, "attention_mma")
     return out
 
 
 def attention_any(q, out, kv_cache, strides, block_tables, q_start, q_len, ctx_lens, n_seqs, max_q_len, n_q, n_kv, D, DV, scale,
-                  causal=True, window=0, keep_first=0, sinks=None):
+                  causal=True, window=0, keep_first=0, sinks=None, softcap=0.0, rel_bias=None):
     """The CUDA-core kernel for any sizes, bf16 or fp32. ``strides``: q token, q head, out token, out head, page, key head,
     key token, first value, value head, value token (elements)."""
     if q.dtype != kv_cache.dtype or q.dtype not in (torch.bfloat16, torch.float32):
@@ -127,7 +157,7 @@ def attention_any(q, out, kv_cache, strides, block_tables, q_start, q_len, ctx_l
                                      1 if q.dtype == torch.float32 else 0, kv_cache.shape[0], block_tables.data_ptr(),
                                      block_tables.shape[1], nv.ptr(q_start), nv.ptr(q_len), ctx_lens.data_ptr(), n_seqs,
                                      max_q_len, n_q, n_kv, D, DV, float(scale), 1 if causal else 0, window, keep_first,
-                                     nv.ptr(sinks), nv.stream_ptr())
+                                     nv.ptr(sinks), float(softcap), *_bias_args(rel_bias, n_q), nv.stream_ptr())
     nv.check(rc, "attention_any")
     return out
 
@@ -138,10 +168,13 @@ def _kv_strides(n_q, n_kv, D, DV):
 
 def paged_decode(q, kv_cache, block_tables, ctx_lens, *, n_q, n_kv, scale=None, out=None, workspace=None,
                  pages_per_split=32, window=0, sinks=None, kv_scale: float = 1.0, full_weights: bool = False,
-                 keep_first: int = 0, dim=None):
+                 keep_first: int = 0, dim=None, softcap: float = 0.0, rel_bias=None):
     """One query token per sequence. q: [B, n_q*D]; ctx_lens includes the token just written. ``full_weights``: the softmax
     weights enter the second product as a bf16 pair (value + remainder, 16 bits of mantissa) instead of one bf16.
-    ``keep_first``: with a sliding window, the first tokens stay visible."""
+    ``keep_first``: with a sliding window, the first tokens stay visible. ``softcap``, ``rel_bias`` [n_q, n] fp32: see
+    ``attention_ref``."""
+    softcap = float(softcap or 0.0)
+    _no_fp8_scores(kv_cache, softcap, rel_bias)
     B = q.shape[0]
     D, DV = head_sizes(kv_cache, n_kv, dim)
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -151,7 +184,7 @@ def paged_decode(q, kv_cache, block_tables, ctx_lens, *, n_q, n_kv, scale=None, 
         ar = torch.arange(B, dtype=torch.int32)
         ones = (ctx_lens > 0).to(torch.int32)
         out.copy_(attention_ref(q, _dequant_cache(kv_cache, kv_scale), block_tables, ar, ones, ctx_lens, n_q, n_kv, scale,
-                                True, window, sinks, keep_first, dim))
+                                True, window, sinks, keep_first, dim, softcap, rel_bias))
         return out
     if D == DV == 128 and n_q // n_kv <= 16 and q.dtype == torch.bfloat16:
         max_blocks = block_tables.shape[1]
@@ -170,34 +203,43 @@ def paged_decode(q, kv_cache, block_tables, ctx_lens, *, n_q, n_kv, scale=None, 
                                         block_tables.data_ptr(), max_blocks, ctx_lens.data_ptr(), B, n_q, n_kv,
                                         scale, pages_per_split, workspace.max_splits, workspace.scratch.data_ptr(),
                                         workspace.counters.data_ptr(), window, keep_first, nv.ptr(sinks),
-                                        1 if full_weights else 0, nv.stream_ptr())
+                                        1 if full_weights or softcap or rel_bias is not None else 0, softcap,
+                                        *_bias_args(rel_bias, n_q), nv.stream_ptr())
         nv.check(rc, "paged_decode")
         return out
     if _mma_head(q, kv_cache, D, DV) and out.is_contiguous():
         return _attention_mma(q, out, kv_cache, block_tables, None, None, ctx_lens, B, 1, n_q, n_kv, D, DV, scale, True, window,
-                              keep_first, sinks)
+                              keep_first, sinks, softcap, rel_bias)
     if kv_cache.dtype == q.dtype:
         return attention_any(q, out, kv_cache, _kv_strides(n_q, n_kv, D, DV), block_tables, None, None, ctx_lens, B, 1, n_q, n_kv,
-                             D, DV, scale, True, window, keep_first, sinks)
+                             D, DV, scale, True, window, keep_first, sinks, softcap, rel_bias)
     ar = torch.arange(B, dtype=torch.int32, device=q.device)
     ones = (ctx_lens > 0).to(torch.int32)
     return paged_prefill(q, kv_cache, block_tables, ar, ones, ctx_lens, max_q_len=1, n_q=n_q, n_kv=n_kv, scale=scale,
                          out=out, window=window, sinks=sinks, kv_scale=kv_scale, full_weights=full_weights,
-                         keep_first=keep_first, dim=dim)
+                         keep_first=keep_first, dim=dim, softcap=softcap, rel_bias=rel_bias)
+
+
+def _no_fp8_scores(kv_cache, softcap, rel_bias):
+    if kv_cache.dtype == torch.float8_e4m3fn and (softcap or rel_bias is not None):
+        raise NotImplementedError("capped or biased scores with an fp8 KV cache")
 
 
 def paged_prefill(q, kv_cache, block_tables, q_start, q_len, ctx_lens, *, max_q_len, n_q, n_kv, scale=None,
                   out=None, causal=True, window=0, sinks=None, kv_scale: float = 1.0, full_weights: bool = False,
-                  keep_first: int = 0, dim=None):
+                  keep_first: int = 0, dim=None, softcap: float = 0.0, rel_bias=None):
     """Variable-length (chunked) prefill. q: [T, n_q*D] flat tokens; sequence i owns rows
     [q_start[i], q_start[i]+q_len[i]) which are the last q_len[i] of its ctx_lens[i] cached tokens."""
+    softcap = float(softcap or 0.0)
+    scored = bool(softcap) or rel_bias is not None
+    _no_fp8_scores(kv_cache, softcap, rel_bias)
     D, DV = head_sizes(kv_cache, n_kv, dim)
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     if out is None:
         out = q.new_empty((q.shape[0], n_q * DV))
     if not q.is_cuda:
         out.copy_(attention_ref(q, _dequant_cache(kv_cache, kv_scale), block_tables, q_start, q_len, ctx_lens, n_q, n_kv, scale,
-                                causal, window, sinks, keep_first, dim))
+                                causal, window, sinks, keep_first, dim, softcap, rel_bias))
         return out
     S = q_len.shape[0]
     if keep_first and kv_cache.dtype == torch.float8_e4m3fn:
@@ -218,15 +260,16 @@ def paged_prefill(q, kv_cache, block_tables, q_start, q_len, ctx_lens, *, max_q_
                                                  1 if causal else 0, window, float(kv_scale), nv.stream_ptr())
         nv.check(rc, "paged_attention_fp8kv")
         return out
-    if D == DV == 128 and q.dtype == torch.bfloat16 and (nv.get_option("prefill_tc") != 0 or full_weights or keep_first) and q.is_contiguous() and out.is_contiguous():
+    if D == DV == 128 and q.dtype == torch.bfloat16 and (nv.get_option("prefill_tc") != 0 or full_weights or keep_first or scored) and q.is_contiguous() and out.is_contiguous():
         # tcgen05 flash attention (S and O accumulators in tensor memory)
         rc = nv.lib().gllm_paged_prefill_tc(q.data_ptr(), out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
                                             block_tables.data_ptr(), block_tables.shape[1], q_start.data_ptr(),
                                             q_len.data_ptr(), ctx_lens.data_ptr(), S, max_q_len, q.shape[0], n_q, n_kv,
                                             scale, 1 if causal else 0, window, keep_first, nv.ptr(sinks),
-                                            1 if full_weights else 0, nv.stream_ptr())
+                                            1 if full_weights or scored else 0, softcap, *_bias_args(rel_bias, n_q),
+                                            nv.stream_ptr())
         nv.check(rc, "paged_prefill_tc")
-    elif D == DV == 128 and q.dtype == torch.bfloat16 and not keep_first:
+    elif D == DV == 128 and q.dtype == torch.bfloat16 and not keep_first and not scored:
         rc = nv.lib().gllm_paged_prefill(q.data_ptr(), out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
                                          block_tables.data_ptr(), block_tables.shape[1], q_start.data_ptr(),
                                          q_len.data_ptr(), ctx_lens.data_ptr(), S, max_q_len, n_q, n_kv, scale,
@@ -234,8 +277,8 @@ def paged_prefill(q, kv_cache, block_tables, q_start, q_len, ctx_lens, *, max_q_
         nv.check(rc, "paged_prefill")
     elif _mma_head(q, kv_cache, D, DV) and out.is_contiguous():
         _attention_mma(q, out, kv_cache, block_tables, q_start, q_len, ctx_lens, S, max_q_len, n_q, n_kv, D, DV, scale, causal,
-                       window, keep_first, sinks)
+                       window, keep_first, sinks, softcap, rel_bias)
     else:
         attention_any(q, out, kv_cache, _kv_strides(n_q, n_kv, D, DV), block_tables, q_start, q_len, ctx_lens, S, max_q_len, n_q,
-                      n_kv, D, DV, scale, causal, window, keep_first, sinks)
+                      n_kv, D, DV, scale, causal, window, keep_first, sinks, softcap, rel_bias)
     return out

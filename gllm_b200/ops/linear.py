@@ -84,11 +84,15 @@ def tensor_core_shape(a, w) -> bool:
 # plain GEMM (+ RMSNorm-as-row-scale prologue, + bias)
 # --------------------------------------------------------------------------------------------
 def gemm(a, w, *, out=None, out_dtype=torch.bfloat16, bias=None, row_ss=None, norm_dim=0, eps=0.0,
-         bn=None, max_ctas=0, splits=0, softcap: float = 0.0):
+         bn=None, max_ctas=0, splits=0, softcap: float = 0.0, act=None, act_cols=None):
     """out[M,N] = rowscale(a) @ w.T (+ bias). ``row_ss`` [M, parts] are partial sums of squares of ``a``'s
     rows; when given, each output row is scaled by rsqrt(sum/norm_dim + eps) (the norm weight must
     already be folded into ``w``). ``softcap`` > 0 applies cap * tanh(x / cap) to the result (final-logit soft
-    capping) in the GEMM epilogue."""
+    capping) in the GEMM epilogue. ``act``: activation (``STORE_ACTS``) of the first ``act_cols`` output columns (all by
+    default), without a row scale or a cap."""
+    act_id, act_cols = (STORE_ACTS[act], w.shape[0] if act_cols is None else int(act_cols)) if act else (0, 0)
+    if act and (row_ss is not None or softcap):
+        raise ValueError("gemm: an activation goes with neither a row scale nor a cap")
     from .quant_gemm import QuantWeight, qgemm
     if isinstance(w, QuantWeight):      # quantised weight: dequantisation fused into the GEMM main loop
         y = qgemm(a, w, row_ss=row_ss, norm_dim=norm_dim, eps=eps)
@@ -112,6 +116,8 @@ def gemm(a, w, *, out=None, out_dtype=torch.bfloat16, bias=None, row_ss=None, no
             acc = acc + bias.float()
         if softcap:
             acc = torch.tanh(acc / softcap) * softcap
+        if act:
+            acc[:, :act_cols] = _store_act_ref(acc[:, :act_cols], act_id)
         res = acc.to(out.dtype if out is not None else out_dtype)
         if out is not None:
             out.copy_(res)
@@ -128,11 +134,17 @@ def gemm(a, w, *, out=None, out_dtype=torch.bfloat16, bias=None, row_ss=None, no
             raise ValueError("gemm: the row-scale prologue needs the tensor-core kernel (bf16, rows of 16-byte multiples)")
         rc = nv.lib().gllm_gemm_simt(a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M,
                                      N, K, 1 if a.dtype == torch.float32 else 0, 1 if out.dtype == torch.float32 else 0,
-                                     nv.ptr(bias), float(softcap), nv.stream_ptr())
+                                     nv.ptr(bias), float(softcap), act_id, act_cols, nv.stream_ptr())
         nv.check(rc, "gemm_simt")
         return out
     bn = bn or _bn_for(N, M)
     nv.ensure_splitk_workspace(a.device)
+    if act:
+        rc = nv.lib().gllm_gemm_bf16_act(a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N,
+                                         K, 1 if out.dtype == torch.float32 else 0, nv.ptr(bias), bn, act_id, act_cols,
+                                         nv.stream_ptr())
+        nv.check(rc, "gemm_bf16_act")
+        return out
     parts = 0 if row_ss is None else (row_ss.shape[1] if row_ss.dim() > 1 else 1)
     if softcap:
         rc = nv.lib().gllm_gemm_bf16_softcap(a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(),
@@ -214,6 +226,13 @@ def set_pair_max_m(max_m: int, epi_mask: int = 0xF):
 def set_pair_big_m(big_m: int) -> int:
     """256-wide GEMMs with M >= ``big_m`` run on CTA pairs (0 = never). Returns the previous threshold."""
     return int(nv.lib().gllm_gemm_set_pair_big_m(int(big_m)))
+
+
+STORE_ACTS = {"silu": 1, "relu2": 2}       # activations of a plain projection's output columns
+
+
+def _store_act_ref(x, act_id):
+    return torch.nn.functional.silu(x) if act_id == 1 else torch.relu(x).square()
 
 
 ACT_IDS = {"silu": 0, "swiglu": 0, "gelu_tanh": 1, "gelu_new": 1, "gelu_pytorch_tanh": 1, "geglu": 1, "gelu": 1}

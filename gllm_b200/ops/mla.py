@@ -1,7 +1,7 @@
 """Multi-head latent attention ops: latent cache write and attention over the latent cache.
 
-CUDA path: ``csrc/kernels/mla.cu`` and ``mla_decode.cu`` (latent with a rotated key part), ``mixer_prep.cu``,
-``latent_attention.cu`` and ``attention_any.cu`` (windowed latent attention without positions). CPU path / oracle: plain fp32
+CUDA path: ``csrc/kernels/mla.cu`` and ``mla_decode.cu`` (the MLA models), ``mixer_prep.cu``, ``latent_attention.cu`` and
+``attention_any.cu`` (latent layers of heterogeneous decoders: windows, sinks, with or without a rotated key part). CPU path / oracle: plain fp32
 PyTorch of the same math.
 Reference parity: MlaKvCompress / MlaQAbsorb / MlaAttention
 (src/arch/auto_graph_fragments/build_graph.inc.rs:1486-1578).
@@ -21,10 +21,11 @@ nv.register("gllm_mla_attention", I, [P, P, P, I, P, I, P, P, P, P, I, I, I, I, 
 nv.register("gllm_mla_decode_scratch_floats", L, [I, I, I])
 nv.register("gllm_mla_decode", I, [P, P, P, I, P, I, P, I, I, I, F, I, P, L, P])
 
-nv.register("gllm_latent_attention_scratch", L, [I, I, I, I, P])
-nv.register("gllm_latent_attention", I, [P, L, L, P, L, L, P, I, P, I, P, P, P, I, I, I, I, F, I, P, I, P, P, P])
+nv.register("gllm_latent_attention_scratch", L, [I, I, I, I, I, P])
+nv.register("gllm_latent_attention", I, [P, L, L, P, L, L, P, I, P, I, P, P, P, I, I, I, I, I, F, I, P, I, P, P, P])
 nv.register("gllm_latent_gather", I, [P, I, I, P, I, P, P, P, I, I, P, I, P])
 nv.register("gllm_rows_prefill_tc", I, [P, P, P, I, P, P, P, P, I, I, I, I, I, F, I, P, I, P])
+nv.register("gllm_latent_rope_prep", I, [P, P, I, I, I, I, I, I, I, I, P, F, P, P, P, P, I, P, I, P, I, P])
 nv.register("gllm_latent_prep", I, [P, L, I, I, I, I, P, P, F, P, P, P, I, P])
 
 PAGE = 16
@@ -147,7 +148,8 @@ def latent_prefill(q, cache, block_tables, row_seq, positions, ctx_lens, *, n_he
 
 
 # ------------------------------------------------------------------------------------------------------------------------------
-# windowed latent attention without positions: one normalised latent row per token is key and value of every head
+# latent layers of heterogeneous decoders: one normalised latent per token is key and value of every head; a rotated key part,
+# shared by the heads, may follow it in the cached row
 # ------------------------------------------------------------------------------------------------------------------------------
 def latent_prep(proj, q_rank, kv_rank, q_w, kv_w, eps, slot_mapping, cq, cache):
     """proj [T, >= q_rank + kv_rank] = query latent | key / value latent; each RMS-normed with its weight: into ``cq``
@@ -166,10 +168,45 @@ def latent_prep(proj, q_rank, kv_rank, q_w, kv_w, eps, slot_mapping, cq, cache):
                                        cache.data_ptr(), cache.shape[0], nv.stream_ptr()), "latent_prep")
 
 
+def latent_rope_prep(proj, *, heads, dim, part, rot, rank, kv_col, kv_w, eps, positions, slot_mapping, cos_t, sin_t, q_out, copy,
+                     cache):
+    """proj [T, ...] = queries (``heads`` x (dim + part) columns) and, from column ``kv_col``, latent (rank) | key part (part).
+    RMS norm of the latent, RoPE on the first ``rot`` of the part columns of queries and key part; latent and key part go to
+    the token's row of ``cache`` [pages, 16, rank + part]. ``q_out`` [T, heads, width]: whole heads, the part rotated
+    (``copy``), or the rotated parts alone."""
+    T = proj.shape[0]
+    if not proj.is_cuda:
+        half = rot // 2
+
+        def turn(x):               # [T, ..., part]
+            shape = [T] + [1] * (x.dim() - 2) + [half]
+            if rot == 0:
+                return x
+            c, s = cos_t[positions.long()].reshape(shape), sin_t[positions.long()].reshape(shape)
+            return torch.cat([rope_half(x[..., :rot], c, s), x[..., rot:]], -1)
+        q = proj[:, :heads * (dim + part)].float().reshape(T, heads, dim + part)
+        r = turn(q[..., dim:])
+        q_out.copy_((torch.cat([q[..., :dim], r], -1) if copy else r).to(q_out.dtype))
+        c = proj[:, kv_col:kv_col + rank].float()
+        c = c / torch.sqrt(c.pow(2).mean(-1, keepdim=True) + eps) * kv_w
+        row = torch.cat([c, turn(proj[:, kv_col + rank:kv_col + rank + part].float())], -1)
+        if slot_mapping is not None:
+            ok = slot_mapping >= 0
+            cache.view(-1, rank + part)[slot_mapping[ok].long()] = row[ok].to(cache.dtype)
+        return
+    assert q_out.stride(2) == 1
+    strides = (ctypes.c_longlong * 3)(proj.stride(0), q_out.stride(0), q_out.stride(1))
+    nv.check(nv.lib().gllm_latent_rope_prep(
+        proj.data_ptr(), strides, 1 if proj.dtype == torch.float32 else 0, T, heads, dim, part, rot, rank, kv_col, kv_w.data_ptr(),
+        float(eps), positions.data_ptr(), nv.ptr(slot_mapping), nv.ptr(cos_t), nv.ptr(sin_t),
+        cos_t.shape[0] if cos_t is not None else 1, q_out.data_ptr(), 1 if copy else 0, cache.data_ptr(), cache.shape[0],
+        nv.stream_ptr()), "latent_rope_prep")
+
+
 def latent_splits(n_seqs: int, heads: int, rank: int, keys: int) -> int:
-    """Into how many parts a decode step cuts the ``keys`` of each sequence: one wave of CTAs, at least two 64-token blocks
+    """Into how many parts a decode step cuts the ``keys`` (of ``rank`` channels) of each sequence: one wave of CTAs, at least two 64-token blocks
     each."""
-    rows = 16 if heads <= 16 else 32 if heads <= 32 else 64
+    rows = 16 if heads <= 16 else 32 if heads <= 32 or rank > 512 else 64
     units = n_seqs * -(-heads // rows)
     wave = 148 * (1 if rank > 256 else 2)
     return max(1, min(wave // units, -(-keys // 128), 16))
@@ -177,11 +214,12 @@ def latent_splits(n_seqs: int, heads: int, rank: int, keys: int) -> int:
 
 def window_latent_attention(q, cache, block_tables, q_start, q_len, ctx_lens, *, max_q_len, scale, window=0, sinks=None, out,
                             scratch: Optional[dict] = None):
-    """q [heads, T, rank] (the query with the key up-projection absorbed); cache [pages, 16, rank]; out [heads, T, rank]: the
-    weighted latent of each head, causal with a sliding ``window`` (0: everything), ``sinks`` [heads] fp32 in the denominator.
+    """q [heads, T, rank (+ part)] (the query with the key up-projection absorbed, then its rotated part); cache [pages, 16,
+    rank (+ part)]; out [heads, T, rank]: the weighted latent of each head, causal with a sliding ``window`` (0: everything), ``sinks`` [heads] fp32 in the denominator.
     ``q_start`` None: a decode step (row = sequence). ``scratch``: a dict that keeps the buffers of split decode steps from
     call to call (no splitting without it)."""
-    H, T, R = q.shape
+    H, T, RK = q.shape
+    R = out.shape[2]
     S = ctx_lens.shape[0]
     if not q.is_cuda:
         if q_start is None:
@@ -190,7 +228,7 @@ def window_latent_attention(q, cache, block_tables, q_start, q_len, ctx_lens, *,
             ql, ctx, st = int(q_len[s]), int(ctx_lens[s]), int(q_start[s])
             if ql <= 0 or ctx <= 0:
                 continue
-            rows = cache[block_tables[s, :(ctx + PAGE - 1) // PAGE].long()].reshape(-1, R)[:ctx].float()
+            rows = cache[block_tables[s, :(ctx + PAGE - 1) // PAGE].long()].reshape(-1, RK)[:ctx].float()
             sc = torch.einsum("hqd,kd->hqk", q[:, st:st + ql].float(), rows) * scale
             pq, pk = torch.arange(ctx - ql, ctx)[:, None], torch.arange(ctx)[None, :]
             ok = (pk <= pq) & ((pk > pq - window) if window > 0 else True)
@@ -198,30 +236,30 @@ def window_latent_attention(q, cache, block_tables, q_start, q_len, ctx_lens, *,
             if sinks is not None:
                 sc = torch.cat([sc, sinks.float().reshape(H, 1, 1).expand(H, ql, 1)], -1)
             p = torch.softmax(sc, -1)[..., :ctx]
-            out[:, st:st + ql] = torch.einsum("hqk,kd->hqd", p, rows).to(out.dtype)
+            out[:, st:st + ql] = torch.einsum("hqk,kd->hqd", p, rows[:, :R]).to(out.dtype)
         return out
-    if (q.dtype == torch.bfloat16 and cache.dtype == q.dtype and R % 8 == 0 and R <= 512
+    if (q.dtype == torch.bfloat16 and cache.dtype == q.dtype and R % 8 == 0 and R <= 512 and RK % 8 == 0 and RK <= 576
             and not (q.stride(0) | q.stride(1) | out.stride(0) | out.stride(1)) & 7):
         splits, buf, cnt = 1, None, None
         if q_start is None and scratch is not None:
             keys = block_tables.shape[1] * PAGE
-            splits = latent_splits(S, H, R, min(keys, window + 64) if window > 0 else keys)
+            splits = latent_splits(S, H, RK, min(keys, window + 64) if window > 0 else keys)
         if splits > 1:
-            key = (S, H, R, splits)
+            key = (S, H, R, RK, splits)
             if key not in scratch:
                 n_cnt = ctypes.c_int()
-                n = nv.lib().gllm_latent_attention_scratch(S, H, R, splits, ctypes.byref(n_cnt))
+                n = nv.lib().gllm_latent_attention_scratch(S, H, R, RK, splits, ctypes.byref(n_cnt))
                 scratch[key] = (torch.empty(int(n), dtype=torch.float32, device=q.device),
                                 torch.zeros(n_cnt.value, dtype=torch.int32, device=q.device))
             buf, cnt = scratch[key]
         nv.check(nv.lib().gllm_latent_attention(
             q.data_ptr(), q.stride(0), q.stride(1), out.data_ptr(), out.stride(0), out.stride(1), cache.data_ptr(), cache.shape[0],
-            block_tables.data_ptr(), block_tables.shape[1], nv.ptr(q_start), nv.ptr(q_len), ctx_lens.data_ptr(), S, max_q_len, H, R,
+            block_tables.data_ptr(), block_tables.shape[1], nv.ptr(q_start), nv.ptr(q_len), ctx_lens.data_ptr(), S, max_q_len, H, R, RK,
             float(scale), window, nv.ptr(sinks), splits, nv.ptr(buf), nv.ptr(cnt), nv.stream_ptr()), "latent_attention")
         return out
     from .attention import attention_any
-    strides = (q.stride(1), q.stride(0), out.stride(1), out.stride(0), PAGE * R, 0, R, 0, 0, R)
-    return attention_any(q, out, cache, strides, block_tables, q_start, q_len, ctx_lens, S, max_q_len, H, 1, R, R, scale, True,
+    strides = (q.stride(1), q.stride(0), out.stride(1), out.stride(0), PAGE * RK, 0, RK, 0, 0, RK)
+    return attention_any(q, out, cache, strides, block_tables, q_start, q_len, ctx_lens, S, max_q_len, H, 1, RK, R, scale, True,
                          window, 0, sinks)
 
 

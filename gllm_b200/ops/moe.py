@@ -10,17 +10,21 @@ import torch
 from . import _native as nv
 from ._native import F, I, L, P
 
-nv.register("gllm_moe_route", I, [P, L, I, I, I, I, I, P, F, P, P, P])
+nv.register("gllm_moe_route", I, [P, L, I, I, I, I, I, P, F, I, I, P, P, P])
 nv.register("gllm_moe_permute", I, [P, I, P, I, P, P, I, I, I, I, I, P, P, P, P, I, P, P, P, P, P])
 nv.register("gllm_moe_combine", I, [P, P, P, I, I, I, P, P, P, P])
 
 BLOCK = 128
 
 
-def route_ref(logits, k, norm_topk=True, scoring="softmax", sel_bias=None, scale=1.0):
+def route_ref(logits, k, norm_topk=True, scoring="softmax", sel_bias=None, scale=1.0, groups=0, keep_groups=0):
     lg = logits.float()
     score = torch.softmax(lg, -1) if scoring == "softmax" else torch.sigmoid(lg)
     sel = score if sel_bias is None else score + sel_bias.float()
+    if groups > 0:
+        best = sel.unflatten(-1, (groups, -1)).amax(-1)
+        kept = torch.zeros_like(best).scatter_(-1, torch.topk(best, keep_groups, dim=-1).indices, 1.0) > 0
+        sel = sel.masked_fill(~kept.repeat_interleave(sel.shape[-1] // groups, -1), float("-inf"))
     _, ids = torch.topk(sel, k, dim=-1, sorted=True)
     w = torch.gather(score, 1, ids)
     if norm_topk:
@@ -28,16 +32,20 @@ def route_ref(logits, k, norm_topk=True, scoring="softmax", sel_bias=None, scale
     return ids.to(torch.int32), w * scale
 
 
-def route(logits, k, *, norm_topk=True, scoring="softmax", sel_bias=None, scale=1.0, out_ids=None, out_w=None):
-    """logits [T,E] fp32 -> (ids [T,k] int32, weights [T,k] fp32)."""
+def route(logits, k, *, norm_topk=True, scoring="softmax", sel_bias=None, scale=1.0, groups=0, keep_groups=0, out_ids=None,
+          out_w=None):
+    """logits [T,E] fp32 -> (ids [T,k] int32, weights [T,k] fp32). ``groups`` > 0: the experts form that many groups of
+    neighbours; only those of the ``keep_groups`` groups with the largest best score are chosen."""
     T, E = logits.shape
+    if groups > 0 and (E % groups or not 0 < keep_groups <= groups or keep_groups * (E // groups) < k):
+        raise ValueError(f"route: {E} experts in {groups} groups, {keep_groups} kept, top {k}")
     if not logits.is_cuda:
-        return route_ref(logits, k, norm_topk, scoring, sel_bias, scale)
+        return route_ref(logits, k, norm_topk, scoring, sel_bias, scale, groups, keep_groups)
     if out_ids is None:
         out_ids = torch.empty((T, k), dtype=torch.int32, device=logits.device)
         out_w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
     rc = nv.lib().gllm_moe_route(logits.data_ptr(), logits.stride(0), T, E, k, 1 if norm_topk else 0,
-                                 0 if scoring == "softmax" else 1, nv.ptr(sel_bias), float(scale), out_ids.data_ptr(),
+                                 0 if scoring == "softmax" else 1, nv.ptr(sel_bias), float(scale), groups, keep_groups, out_ids.data_ptr(),
                                  out_w.data_ptr(), nv.stream_ptr())
     nv.check(rc, "moe_route")
     return out_ids, out_w

@@ -1,7 +1,7 @@
-"""Recurrent token mixers (short convolution, RG-LRU, gated linear attention) and the ops of a residual stream kept in
+"""Recurrent token mixers (short convolution, RG-LRU, gated linear attention, lightning attention) and the ops of a residual stream kept in
 fp32: embedding rows, scaled post-norm, query / key preparation with a norm over the whole projection.
 
-CUDA path: ``csrc/kernels/recurrent.cu`` and ``csrc/kernels/simt.cu`` (bf16 or fp32 tensors, fp32 states). CPU path: an
+CUDA path: ``csrc/kernels/recurrent.cu``, ``lightning.cu`` and ``csrc/kernels/simt.cu`` (bf16 or fp32 tensors, fp32 states). CPU path: an
 fp32 restatement of each op.
 
 The sequences of a step come as a ``SeqView``: sequence i owns rows [q_start, q_start + q_len) of the flat batch, the
@@ -19,7 +19,7 @@ import torch
 from . import _native as nv
 
 P, I, L, F = c_void_p, c_int, c_longlong, c_float
-nv.register("gllm_embed_rows", I, [P, P, I, I, I, P, P, I, P])
+nv.register("gllm_embed_rows", I, [P, P, I, I, I, F, P, P, I, P])
 nv.register("gllm_scaled_add_norm", I, [P, L, P, L, I, P, I, I, F, F, P, P, P, I, P])
 nv.register("gllm_glu_f32", I, [P, L, I, I, I, P, P])
 nv.register("gllm_qk_row_norm_rope", I, [P, L, I, I, I, I, I, I, I, P, P, P, P, I, P, P, F, P, P, I, P])
@@ -33,6 +33,9 @@ nv.register("gllm_gla_tile_ok", I, [I, I, I, L])
 nv.register("gllm_gla_decode", I, [P, I, P, P, P, P, P, L, P, P, P, I, I, I, I, F, F, F, P, P, P])
 nv.register("gllm_gla_prefill", I, [P, P, P, P, I, I, P, P, P, P, L, P, P, I, I, I, I, F, F, P, P, P, P])
 nv.register("gllm_conv_qkv_prep", I, [P, P, P, P, I, I, P, L, I, I, I, I, I, I, I, P, P, P, F, P, P, P, P, I, P, P, P, I, P])
+nv.register("gllm_lightning", I, [P, P, P, P, I, P, P, P, L, I, I, I, I, P, P, P, P, I, P])
+nv.register("gllm_row_norm_gate", I, [P, P, L, I, P, I, I, F, P, P])
+nv.register("gllm_sigmoid_gate", I, [P, P, L, I, L, I, P])
 nv.register("gllm_head_norm_gate", I, [P, P, L, I, P, L, I, I, F, P, P])
 
 RGLRU_C = 8.0        # exponent of the RG-LRU decay: log a = -8 r softplus(lam)
@@ -79,16 +82,16 @@ def _f32(t) -> int:
     return 1 if t.dtype == torch.float32 else 0
 
 
-def embed_rows(ids, table, x, xb=None):
-    """x[m] = table[ids[m]] in fp32; ``xb`` (optional) the same rows in the table's dtype."""
+def embed_rows(ids, table, x, xb=None, scale=1.0):
+    """x[m] = table[ids[m]] * scale in fp32; ``xb`` (optional) the unscaled rows in the table's dtype."""
     M = ids.shape[0]
     if not table.is_cuda:
         rows = table[ids.long()]
-        x.copy_(rows.float())
+        x.copy_(rows.float() * scale)
         if xb is not None:
             xb.copy_(rows)
         return x
-    nv.check(nv.lib().gllm_embed_rows(ids.data_ptr(), table.data_ptr(), table.shape[0], table.shape[1], _f32(table),
+    nv.check(nv.lib().gllm_embed_rows(ids.data_ptr(), table.data_ptr(), table.shape[0], table.shape[1], _f32(table), float(scale),
                                       x.data_ptr(), nv.ptr(xb), M, nv.stream_ptr()), "embed_rows")
     return x
 
@@ -358,3 +361,59 @@ def head_norm_gate(o, g, w, *, heads, vdim, eps, out):
     nv.check(nv.lib().gllm_head_norm_gate(o.data_ptr(), g.data_ptr(), g.stride(0), _f32(g), w.data_ptr(), T, heads, vdim,
                                           float(eps), out.data_ptr(), nv.stream_ptr()), "head_norm_gate")
     return out
+
+
+# --------------------------------------------------------------------------------------------
+# lightning attention: linear attention with a fixed decay per head
+# --------------------------------------------------------------------------------------------
+LIGHTNING_CHUNK = 64
+
+
+def lightning_tables(decay, device):
+    """(1 - a [heads], a^0 .. a^64 [heads, 65]) in fp32, from the decays in double precision."""
+    a = torch.tensor(decay, dtype=torch.float64)
+    powers = a[:, None] ** torch.arange(LIGHTNING_CHUNK + 1, dtype=torch.float64)
+    return (1 - a).float().contiguous().to(device), powers.float().contiguous().to(device)
+
+
+def lightning(sv: SeqView, q, k, v, *, heads, dim, vdim, tables, state, out, general=False):
+    """S = a S + k v^T, o = S^T q per head. q, k, v: column slices of one buffer (same row pitch), activated; out
+    [T, heads * vdim] fp32; state [slots, heads, dim, vdim] fp32. ``general``: the token-by-token kernel whatever the sizes."""
+    forget, powers = tables
+    if not q.is_cuda:
+        for r0, n, start, slot in sv.rows():
+            S = state[slot].clone() if start > 0 else torch.zeros_like(state[slot])
+            qq, kk = q[r0:r0 + n].float().reshape(n, heads, dim), k[r0:r0 + n].float().reshape(n, heads, dim)
+            vv = v[r0:r0 + n].float().reshape(n, heads, vdim)
+            for i in range(n):
+                S = S - forget[:, None, None] * S + kk[i][:, :, None] * vv[i][:, None, :]
+                out[r0 + i] = torch.einsum("hdv,hd->hv", S, qq[i]).reshape(-1)
+            state[slot].copy_(S)
+        return out
+    assert q.stride(0) == k.stride(0) == v.stride(0)
+    nv.check(nv.lib().gllm_lightning(*sv.ptrs(), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), _f32(q), heads, dim, vdim,
+                                     forget.data_ptr(), powers.data_ptr(), state.data_ptr(), out.data_ptr(), 1 if general else 0,
+                                     nv.stream_ptr()), "lightning")
+    return out
+
+
+def row_norm_gate(o, g, w, eps, out):
+    """RMS norm of the whole rows of o [T, n] (fp32) with the weight w, times sigmoid(g)."""
+    T, n = o.shape
+    if not o.is_cuda:
+        h = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w
+        out.copy_((h * torch.sigmoid(g.float())).to(out.dtype))
+        return out
+    nv.check(nv.lib().gllm_row_norm_gate(o.data_ptr(), g.data_ptr(), g.stride(0), _f32(g), w.data_ptr(), T, n, float(eps),
+                                         out.data_ptr(), nv.stream_ptr()), "row_norm_gate")
+    return out
+
+
+def sigmoid_gate(x, g):
+    """x [T, n] *= sigmoid(g [T, n]) in place (g may be a column slice)."""
+    if not x.is_cuda:
+        x.copy_((x.float() * torch.sigmoid(g.float())).to(x.dtype))
+        return x
+    nv.check(nv.lib().gllm_sigmoid_gate(x.data_ptr(), g.data_ptr(), g.stride(0), _f32(x), x.shape[0], x.shape[1], nv.stream_ptr()),
+             "sigmoid_gate")
+    return x

@@ -1,9 +1,9 @@
-"""The step between two sublayers of a sandwich-norm block, over a residual stream kept in fp32:
+"""The step between two sublayers of a pre-norm or sandwich-norm block, over a residual stream kept in fp32:
 
     x = x + post_norm(y) (+ vector);   operand of the next sublayer = pre_norm(x)
 
-``y`` is the sublayer's output, either rows of a projection or, behind a mixture of experts, the sum of each token's routed
-rows. CUDA path: ``csrc/kernels/residual.cu``; CPU path: an fp32 restatement.
+``y`` is the sublayer's output, either rows of a projection or, behind a mixture of experts, the (weighted) sum of each token's
+routed rows; ``plus`` and ``gated`` join it where sublayers run side by side. CUDA path: ``csrc/kernels/residual.cu``; CPU path: an fp32 restatement.
 """
 from __future__ import annotations
 
@@ -14,7 +14,7 @@ import torch
 from . import _native as nv
 
 P, I, L, F = c_void_p, c_int, c_longlong, c_float
-nv.register("gllm_residual_norm", I, [P, L, P, L, I, P, I, P, P, P, P, I, I, I, I, F, P, I, P])
+nv.register("gllm_residual_norm", I, [P, L, P, L, I, P, I, P, P, L, P, L, P, L, P, P, P, P, I, I, I, I, F, P, I, P])
 
 KINDS = {"rms": 0, "layer": 1}
 
@@ -27,11 +27,12 @@ def norm_ref(h, w, kind: str, eps: float):
 
 
 def residual_norm(x, y=None, *, kind: str, eps: float, post_w=None, add=None, pre_w=None, xb=None, rows=None, dest=None,
-                  top: int = 0):
-    """x (fp32 [T, H], in place) += norm(y) * post_w, then += ``add`` [H]; xb = norm(x) * pre_w in xb's dtype. ``kind``: rms
-    or layer (no bias). Everything but x is optional. With ``dest`` (int32 [T * top]) the sublayer output of token t is
-    sum_j y[dest[t * top + j]] (negative entries: nothing). ``rows`` (int32): only those rows of x are normalised, into
-    xb[0..], and x stays as it is (no y)."""
+                  top: int = 0, row_w=None, plus=None, gated=None, gate=None):
+    """x (fp32 [T, H], in place) += norm(s) * post_w, then += ``add`` [H]; xb = norm(x) * pre_w in xb's dtype. ``kind``: rms
+    or layer (no bias). Everything but x is optional. s, the sublayer output, is y; with ``dest`` (int32 [T * top]) that of
+    token t is sum_j row_w[t, j] * y[dest[t * top + j]] (negative entries: nothing; no ``row_w``: ones). With y: ``plus`` (fp32
+    [T, >= H]) joins s, and so does sigmoid(``gate``) * ``gated`` (fp32 [T, >= H]; gate: one fp32 number per token).
+    ``rows`` (int32): only those rows of x are normalised, into xb[0..], and x stays as it is (no y)."""
     M = x.shape[0] if rows is None else rows.shape[0]
     H = x.shape[1]
     if not x.is_cuda:
@@ -41,9 +42,14 @@ def residual_norm(x, y=None, *, kind: str, eps: float, post_w=None, add=None, pr
         if y is not None:
             if dest is not None:
                 d = dest[:M * top].reshape(M, top).long()
-                s = (y[d.clamp_min(0)][..., :H].float() * (d >= 0)[..., None]).sum(1)
+                s = y[d.clamp_min(0)][..., :H].float() * (d >= 0)[..., None]
+                s = (s if row_w is None else s * row_w[:M, :, None]).sum(1)
             else:
                 s = y[:M, :H].float()
+            if plus is not None:
+                s = s + plus[:M, :H]
+            if gated is not None:
+                s = s + gated[:M, :H] * (1.0 if gate is None else torch.sigmoid(gate[:M])[:, None])
             x += s if post_w is None else norm_ref(s, post_w, kind, eps)
         if add is not None:
             x += add
@@ -52,6 +58,7 @@ def residual_norm(x, y=None, *, kind: str, eps: float, post_w=None, add=None, pr
         return
     nv.check(nv.lib().gllm_residual_norm(
         x.data_ptr(), x.stride(0), nv.ptr(y), 0 if y is None else y.stride(0), 1 if y is None or y.dtype == torch.float32 else 0,
-        nv.ptr(dest), int(top), nv.ptr(post_w), nv.ptr(add), nv.ptr(pre_w), nv.ptr(xb),
+        nv.ptr(dest), int(top), nv.ptr(row_w), nv.ptr(plus), 0 if plus is None else plus.stride(0), nv.ptr(gated),
+        0 if gated is None else gated.stride(0), nv.ptr(gate), 0 if gate is None else gate.stride(0), nv.ptr(post_w), nv.ptr(add), nv.ptr(pre_w), nv.ptr(xb),
         1 if xb is None or xb.dtype == torch.float32 else 0, M, H, KINDS[kind], float(eps), nv.ptr(rows),
         0 if xb is None else xb.stride(0), nv.stream_ptr()), "residual_norm")

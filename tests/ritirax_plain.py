@@ -1,0 +1,197 @@
+"""A plain, slow statement of the Ritirax decoder for the tests: one function per mechanism, float64 tensors, whole sequences,
+no cache, no batch; nothing from the package is used. Also the tests' own configurations and random weights."""
+import json
+import math
+import struct
+
+import torch
+
+D = torch.float64
+ROUND = None        # set while ``rounded_forward`` runs: what a 16-bit projection does to its input and output
+
+
+def lin(x, w):
+    if ROUND is None:
+        return x @ w.T
+    return ROUND(ROUND(x) @ w.T)
+
+
+def rms_norm(x, w, eps):
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * w
+
+
+def zero_norm(x, w, eps):
+    """The norm whose weight is stored around zero."""
+    return rms_norm(x, 1 + w, eps)
+
+
+def silu(z):
+    return z / (1 + torch.exp(-z))
+
+
+def sigmoid(z):
+    return 1 / (1 + torch.exp(-z))
+
+
+def bucket(n, rows, far):
+    """Row of the distance table for a key ``n`` tokens back: one row per distance up to half the table, then logarithmic
+    steps that reach the table's end at distance ``far``."""
+    half = rows // 2
+    if n < half:
+        return n
+    return min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half)))
+
+
+def distance_bias(T, table, far):
+    """[heads, query, key] from a table [rows, heads]."""
+    rows = torch.tensor([bucket(n, table.shape[0], far) for n in range(T)])
+    n = torch.arange(T)[:, None] - torch.arange(T)[None, :]
+    return table[rows[n.clamp_min(0)]].permute(2, 0, 1)
+
+
+def causal(T):
+    return torch.arange(T)[None, :] <= torch.arange(T)[:, None]
+
+
+def softmax(score, ok, sink=None):
+    """Weights over the visible keys of each row; ``sink`` is one more logit of the denominator without a key."""
+    score = score.masked_fill(~ok, -math.inf)
+    m = score.max(-1, keepdim=True).values
+    if sink is not None:
+        m = m.clamp_min(float(sink))
+    e = torch.exp(score - m)
+    z = e.sum(-1, keepdim=True)
+    if sink is not None:
+        z = z + torch.exp(sink - m)
+    return e / z
+
+
+def attention(h, w, m, eps):
+    T, H, G, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    q = rms_norm(lin(h, w["q"]).reshape(T, H, d), w["q.norm"], eps)
+    k = rms_norm(lin(h, w["k"]).reshape(T, G, d), w["k.norm"], eps)
+    v = lin(h, w["v"]).reshape(T, G, dv)
+    bias, ok, cap = distance_bias(T, w["rel"], m["bias_max"]), causal(T), m["softcap"]
+    out = []
+    for a in range(H):
+        b = a // (H // G)
+        score = cap * torch.tanh((q[:, a] @ k[:, b].T) * m["scale"] / cap) + bias[a]
+        out.append(softmax(score, ok, w["sink"][a]) @ v[:, b])
+    return lin(torch.cat(out, -1), w["o"])
+
+
+def yarn(rot):
+    """(angular speed of every pair, factor of cos and sin)."""
+    dims, base, s = rot["dims"], rot["base"], rot.get("scaling")
+    f = [base ** (-2.0 * i / dims) for i in range(dims // 2)]
+    if not s:
+        return f, 1.0
+    at = lambda turns: dims * math.log(s["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
+    lo, hi = max(math.floor(at(s["fast"])), 0), min(math.ceil(at(s["slow"])), dims - 1)
+    ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(dims // 2)]
+    return [x / s["factor"] * r + x * (1 - r) for x, r in zip(f, ramp)], 0.1 * math.log(s["factor"]) + 1
+
+
+def rotate(x, rot):
+    """x [T, ..., d]: pairs (i, i + dims / 2) of the first ``dims`` dimensions turned by position * speed, and stretched."""
+    y, half = x.clone(), rot["dims"] // 2
+    speed, stretch = yarn(rot)
+    for i in range(half):
+        a = torch.arange(x.shape[0], dtype=D).reshape([-1] + [1] * (x.dim() - 2)) * speed[i]
+        c, s = torch.cos(a) * stretch, torch.sin(a) * stretch
+        u, v = x[..., i], x[..., i + half]
+        y[..., i] = u * c - v * s
+        y[..., i + half] = v * c + u * s
+    return y
+
+
+def latent_attention(h, w, m, eps):
+    T, H, d, r, dv, rank = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    q = lin(h, w["q"]).reshape(T, H, d + r)
+    down = lin(h, w["dkv"])
+    c = rms_norm(down[:, :rank], w["dkv.norm"], eps)
+    kr = rotate(down[:, rank:], m["rot"])
+    k, v = lin(c, w["uk"]).reshape(T, H, d), lin(c, w["uv"]).reshape(T, H, dv)
+    ok, out = causal(T), []
+    for a in range(H):
+        score = (q[:, a, :d] @ k[:, a].T + rotate(q[:, a, d:], m["rot"]) @ kr.T) * m["scale"]
+        out.append(softmax(score, ok) @ v[:, a])
+    return lin(torch.cat(out, -1) * sigmoid(lin(h, w["g"])), w["o"])
+
+
+def lightning(h, w, m, eps):
+    T, H, d, dv = h.shape[0], m["heads"], m["dim"], m["vdim"]
+    q, k, v = (silu(lin(h, w[n])).reshape(T, H, -1) for n in ("q", "k", "v"))
+    decay = torch.tensor(m["decay"], dtype=D)[:, None, None]
+    S, out = torch.zeros(H, d, dv, dtype=D), torch.zeros(T, H, dv, dtype=D)
+    for t in range(T):
+        S = decay * S + k[t][:, :, None] * v[t][:, None, :]
+        out[t] = torch.einsum("hdv,hd->hv", S, q[t])
+    o = rms_norm(out.reshape(T, H * dv), w["norm"], eps)
+    return lin(o * sigmoid(lin(h, w["g"])), w["o"])
+
+
+def dense(h, w, m):
+    return lin(torch.relu(lin(h, w["up"])) ** 2, w["down"])
+
+
+def expert(h, w, p):
+    return lin(silu(lin(h, w[p + "gate"])) * lin(h, w[p + "up"]), w[p + "down"])
+
+
+def choose(score, top, groups, keep):
+    """The ``top`` best experts among those of the ``keep`` groups whose best expert is best."""
+    E = len(score)
+    size = E // groups
+    best = sorted(range(groups), key=lambda g: -max(score[g * size:(g + 1) * size]))[:keep]
+    return sorted((e for e in range(E) if e // size in best), key=lambda e: -score[e])[:top]
+
+
+def experts(h, w, m):
+    r = m["router"]
+    score = torch.softmax(h @ w["router"].T, -1)
+    out = sigmoid(h @ w["shared.sg"].T) * expert(h, w, "shared.")
+    for t in range(h.shape[0]):
+        for e in choose(score[t].tolist(), r["top"], r["groups"]["count"], r["groups"]["keep"]):
+            out[t] += r["scale"] * score[t, e] * expert(h[t:t + 1], w, f"e{e}.")[0]
+    return out
+
+
+MIX = {"attention": attention, "latent_attention": latent_attention, "lightning": lightning}
+FF = {"dense": dense, "moe": experts}
+
+
+def forward(cfg, weights, tokens, stream=False):
+    """Logits [T, vocab] (and the residual stream after every layer)."""
+    W = {k: v.to(D) for k, v in weights.items()}
+    sub = lambda p: {k[len(p):]: v for k, v in W.items() if k.startswith(p)}
+    eps = cfg["norm"]["eps"]
+    x = W["embed"][torch.as_tensor(tokens)] * cfg["embedding"]["scale"]
+    layers = []
+    for n, layer in enumerate(cfg["layers"]):
+        p = f"l{n}."
+        h = zero_norm(x, W[p + "norm1"], eps)
+        y = MIX[layer["type"]](h, sub(p + "mix."), layer["mixer"], eps)
+        if layer["mlp"]:
+            y = y + FF[layer["mlp"]["kind"]](h, sub(p + "mlp."), layer["mlp"])
+        x = x + y
+        layers.append(x)
+    logits = lin(zero_norm(x, W["final.norm"], eps), W["head"])
+    return (logits, layers) if stream else logits
+
+
+def rounded_forward(cfg, weights, tokens):
+    """The same with every projection's input and output rounded to bf16: how far rounding alone moves the logits."""
+    global ROUND
+    ROUND = lambda t: t.to(torch.bfloat16).to(D)
+    try:
+        return forward(cfg, weights, tokens)
+    finally:
+        ROUND = None
+
+
+def greedy(cfg, weights, prompt, n):
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(forward(cfg, weights, toks)[-1].argmax()))
+    return toks[len(prompt):]
