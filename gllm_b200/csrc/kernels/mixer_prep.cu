@@ -474,7 +474,8 @@ __global__ void __launch_bounds__(128) latent_rope_prep_kernel(const LatentRopeP
   pdl_wait();
   pdl_launch_dependents();
   const int half = p.rot / 2, kv_blocks = (p.T + 3) / 4, lane = threadIdx.x & 31;
-  auto position = [&](int t) {
+  auto position = [&](int t) -> long long {
+    if (half == 0) return 0;
     int pos = p.positions[t];
     if (pos < 0 || pos >= p.max_pos) {
       if (p.err) atomicCAS(p.err, 0, ERR_BAD_ARG);

@@ -195,3 +195,122 @@ def greedy(cfg, weights, prompt, n):
     for _ in range(n):
         toks.append(int(forward(cfg, weights, toks)[-1].argmax()))
     return toks[len(prompt):]
+
+
+# ------------------------------------------------------------------------------------------------
+# configurations and weights of the tests
+# ------------------------------------------------------------------------------------------------
+def dense_ff(ff=72):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(ff=24, experts=6, top=2, groups=3, keep=2, scale=1.7, shared=40):
+    return {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": shared},
+            "router": {"experts": experts, "top": top, "scale": scale, "groups": {"count": groups, "keep": keep}}}
+
+
+def att(heads=4, kv_heads=2, dim=16, vdim=24, softcap=9.0, far=50, scale=None, mlp=None):
+    return {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim,
+                                                       "scale": scale or dim ** -0.5, "softcap": softcap, "bias_max": far}}
+
+
+def lat(heads=3, dim=16, rot_dim=8, vdim=24, kv_rank=40, scale=None, base=300.0, scaling=(3.0, 64, 8.0, 1.0), mlp=None):
+    rot = {"dims": rot_dim, "base": base}
+    if scaling:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim,
+                                                              "kv_rank": kv_rank, "scale": scale or (dim + rot_dim) ** -0.5, "rot": rot}}
+
+
+def lig(heads=3, dim=16, vdim=24, decay=None, mlp=None):
+    decay = decay or [1 - 0.6 * 0.3 ** i for i in range(heads)]
+    return {"type": "lightning", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay}}
+
+
+def config(layers, width=64, vocab=96, eps=1e-6, embed=6.5):
+    return {"architecture": "Ritirax", "layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps},
+            "embedding": {"scale": embed}}
+
+
+def weights(cfg, seed=0, sharp=2.0, rows=12):
+    """Random weights, rounded to bf16. ``sharp`` scales the queries (one key then stands out in a softmax), ``rows`` is the
+    length of the distance tables. With experts every token id has one of four kinds, a strong direction of its embedding,
+    and the router separates the chosen experts of each kind from the others, so that 16-bit rounding does not decide who
+    is chosen; among the others one expert of every group that is not kept would come before some of the chosen."""
+    gen = torch.Generator().manual_seed(seed)
+    rn = lambda *shape, s=1.0: torch.randn(shape, generator=gen) * s
+    lin = lambda o, i, s=1.0: rn(o, i, s=s / math.sqrt(i))
+    one = lambda n, s=1.0: s * (1 + 0.2 * rn(n))
+    zero = lambda n: 0.2 * rn(n)
+    Wd, V, scale = cfg["width"], cfg["vocab"], cfg["embedding"]["scale"]
+    w = {"embed": rn(V, Wd), "head": lin(V, Wd, 2.0), "final.norm": zero(Wd)}
+    kinds = torch.linalg.qr(rn(Wd, 4)).Q.T
+    if any(l["mlp"] and l["mlp"]["kind"] == "moe" for l in cfg["layers"]):
+        w["embed"] += 3 * math.sqrt(Wd) * kinds[torch.arange(V) % 4]
+    w["embed"] /= scale
+
+    def router(r):
+        E, n, keep = r["experts"], r["groups"]["count"], r["groups"]["keep"]
+        size, z = E // n, -2 - rn(4, E).abs()
+        for k in range(4):
+            kept = torch.randperm(n, generator=gen)
+            inside = torch.cat([torch.arange(size) + g * size for g in kept[:keep].tolist()])
+            lead = [int(g) * size for g in kept[:keep]]               # the best expert of every kept group
+            rest = [e for e in inside.tolist() if e not in lead]
+            chosen = (lead + rest)[:r["top"]]
+            z[k, lead] = 2.0 + torch.rand(len(lead), generator=gen)   # kept groups lead, also where they are not chosen
+            for e in chosen:
+                if e not in lead:
+                    z[k, e] = 0.2 + 0.3 * float(torch.rand(1, generator=gen))
+            for g in kept[keep:].tolist():                            # better than those, in a group that is not kept
+                z[k, g * size] = 1.2
+        return z.T @ kinds / math.sqrt(Wd) + lin(E, Wd, 0.1)
+    for n, layer in enumerate(cfg["layers"]):
+        m, p = layer["mixer"], f"l{n}.mix."
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "attention":
+            G = m["kv_heads"]
+            t = {"q": lin(H * d, Wd), "k": lin(G * d, Wd), "v": lin(G * dv, Wd), "q.norm": one(d, sharp), "k.norm": one(d),
+                 "rel": 1.5 * rn(rows, H), "sink": 1.5 * rn(H)}
+        elif layer["type"] == "latent_attention":
+            r, rd = m["kv_rank"], m["rot_dim"]
+            t = {"q": lin(H * (d + rd), Wd, sharp), "dkv": lin(r + rd, Wd), "dkv.norm": one(r), "uk": lin(H * d, r),
+                 "uv": lin(H * dv, r), "g": lin(H * dv, Wd, 1.5)}
+        else:
+            t = {"q": lin(H * d, Wd), "k": lin(H * d, Wd), "v": lin(H * dv, Wd), "g": lin(H * dv, Wd, 1.5), "norm": one(H * dv)}
+        t["o"] = lin(Wd, H * dv)
+        w.update({p + k: v for k, v in t.items()})
+        w[f"l{n}.norm1"] = zero(Wd)
+        mlp, q = layer["mlp"], f"l{n}.mlp."
+        if mlp and mlp["kind"] == "dense":
+            w.update({q + "up": lin(mlp["ff"], Wd), q + "down": lin(Wd, mlp["ff"])})
+        elif mlp:
+            w[q + "router"], w[q + "shared.sg"] = router(mlp["router"]), lin(1, Wd, 1.5)
+            w[f"l{n}.norm1"] = 0.05 * rn(Wd)
+            for e, f in [(f"e{e}", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])] + [("shared", mlp["shared"]["ff"])]:
+                w.update({f"{q}{e}.gate": lin(f, Wd, 1.5), f"{q}{e}.up": lin(f, Wd, 1.5), f"{q}{e}.down": lin(Wd, f)})
+    return {k: v.to(torch.bfloat16) for k, v in w.items()}
+
+
+def tokens(cfg, n, seed=0):
+    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(1000 + seed)).tolist()
+
+
+def save(folder, cfg, w):
+    """config.json and model.safetensors (bf16)."""
+    (folder / "config.json").write_text(json.dumps(cfg))
+    head, data = {}, b""
+    for k, v in w.items():
+        raw = v.contiguous().view(torch.int16).numpy().tobytes()
+        head[k] = {"dtype": "BF16", "shape": list(v.shape), "data_offsets": [len(data), len(data) + len(raw)]}
+        data += raw
+    h = json.dumps(head).encode()
+    (folder / "model.safetensors").write_bytes(struct.pack("<Q", len(h)) + h + data)
+    return folder
+
+
+def error(got, want):
+    """Largest over the rows of rms(difference of centred logits) / rms(centred logits)."""
+    c = lambda t: t.to(D) - t.to(D).mean(-1, keepdim=True)
+    g, w = c(torch.as_tensor(got)), c(torch.as_tensor(want))
+    return float(((g - w).pow(2).mean(-1).sqrt() / w.pow(2).mean(-1).sqrt()).max())
