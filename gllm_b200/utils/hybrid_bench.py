@@ -1,6 +1,8 @@
 """Throughput of the heterogeneous decoders beside the closest other decoder of equal size: Zenevik beside a dense decoder
 (``bench.py --hybrid``), Gorulorn beside a mixture-of-experts decoder with the same sliding window (``bench.py --gorulorn``; its
-latent attention also beside the latent kernel of the MLA models, at the same heads, rank and number of keys).
+latent attention also beside the latent kernel of the MLA models, at the same heads, rank and number of keys), Ritirax beside a
+mixture-of-experts decoder (``bench.py --ritirax``; its latent layers also beside Gorulorn's and the MLA kernel, its lightning
+layers beside gated linear attention, all at equal sizes).
 
 Both models have random weights, the same width, depth, attention heads, feed-forward and vocabulary. Prefill: one forward
 over 4 prompts of 2048 tokens. Decode: one captured step of B sequences at context 2048. Whole steps are timed with CUDA
@@ -33,6 +35,12 @@ GORULORN_SIZES = {
     "1024": dict(hidden=1024, heads=16, kv=4, lat=8, q_rank=512, kv_rank=256, experts=32, top=4, ff=512),
     "2048": dict(hidden=2048, heads=32, kv=4, lat=16, q_rank=768, kv_rank=512, experts=64, top=8, ff=768),
     "4096": dict(hidden=4096, heads=32, kv=8, lat=32, q_rank=1536, kv_rank=512, experts=64, top=8, ff=1536),
+}
+# width, query / kv heads, heads and rank of the latent layers, heads of the linear layers, experts
+RITIRAX_SIZES = {
+    "1024": dict(hidden=1024, heads=16, kv=4, lat=8, kv_rank=256, lin=8, experts=32, top=4, ff=512, dense=4096),
+    "2048": dict(hidden=2048, heads=32, kv=4, lat=16, kv_rank=512, lin=16, experts=64, top=8, ff=768, dense=6144),
+    "4096": dict(hidden=4096, heads=32, kv=8, lat=32, kv_rank=512, lin=32, experts=64, top=8, ff=1536, dense=12288),
 }
 VOCAB, CHUNK, PROMPT, PROMPTS = 32768, 2048, 2048, 4
 WINDOW, KEEP = 1024, 64
@@ -71,9 +79,46 @@ def gorulorn_config(s: dict) -> ModelConfig:
     return cfg
 
 
-def moe_config(s: dict) -> ModelConfig:
-    return ModelConfig(arch="qwen3_moe", hidden_size=s["hidden"], num_layers=8, num_heads=s["heads"], num_kv_heads=s["kv"],
-                       head_dim=128, intermediate_size=s["ff"], vocab_size=VOCAB, qk_norm=True, sliding_window=WINDOW,
+def ritirax_config(s: dict) -> ModelConfig:
+    att = MixerSpec("attention", heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5, head_qk_norm=True,
+                    qkv_bias=False, o_bias=False, softcap=30.0, bias_max=256, sink=True)
+    lat = MixerSpec("latent", heads=s["lat"], dim=64, vdim=128, kv_rank=s["kv_rank"], rope_part=64, rot_dim=64, scale=128 ** -0.5,
+                    gate=True)
+    lin = MixerSpec("lightning", heads=s["lin"], dim=128, vdim=128, decay=tuple(1 - 2.0 ** -(1 + 8 * h / s["lin"]) for h in range(s["lin"])))
+    moe = MoeSpec(experts=s["experts"], top=s["top"], ff=s["ff"], norm_topk=False, scale=2.5, groups=8, keep_groups=4,
+                  shared_ff=s["ff"], shared_gate=True)
+    specs = [LayerSpec(att, ff=s["dense"], act="relu2", gated=False)] + [LayerSpec(m, act="silu", moe=moe) for m in (lat, lin, att, lin, lat)]
+    cfg = ModelConfig(arch="ritirax", hidden_size=s["hidden"], num_layers=6, vocab_size=VOCAB, rms_norm_eps=1e-5, norm_one_plus_w=True,
+                      block="parallel", hidden_act="silu", embedding_scale=s["hidden"] ** 0.5, max_position_embeddings=1 << 16,
+                      layer_specs=specs)
+    cfg.set_hybrid_dims()
+    return cfg
+
+
+def gla_config(s: dict) -> ModelConfig:
+    """Gated linear attention layers with the heads of ``ritirax_config``'s lightning layers."""
+    gla = MixerSpec("gla", heads=s["lin"], dim=128, vdim=128, tau=16.0, decay_rank=16)
+    cfg = ModelConfig(arch="zenevik", hidden_size=s["hidden"], num_layers=2, vocab_size=VOCAB, rms_norm_eps=1e-5, postln_alpha=2.0,
+                      hidden_act="gelu_tanh", max_position_embeddings=1 << 16, layer_specs=[LayerSpec(gla), LayerSpec(gla)])
+    cfg.set_hybrid_dims()
+    return cfg
+
+
+def latent_config(s: dict) -> ModelConfig:
+    """Latent layers without positions or windows, with the heads of ``ritirax_config``'s, and plain attention beside them."""
+    att = MixerSpec("attention", heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5, rot_dim=64, taps=4,
+                    head_qk_norm=True, o_bias=False)
+    lat = MixerSpec("latent", heads=s["lat"], dim=128, vdim=128, q_rank=512, kv_rank=s["kv_rank"], scale=128 ** -0.5, sink=True)
+    cfg = ModelConfig(arch="gorulorn", hidden_size=s["hidden"], num_layers=2, vocab_size=VOCAB, rms_norm_eps=1e-5, norm_type="layer",
+                      block="sandwich", hidden_act="silu", max_position_embeddings=1 << 16,
+                      layer_specs=[LayerSpec(att, act="silu"), LayerSpec(lat, act="silu")])
+    cfg.set_hybrid_dims()
+    return cfg
+
+
+def moe_config(s: dict, layers: int = 8, window: int = WINDOW) -> ModelConfig:
+    return ModelConfig(arch="qwen3_moe", hidden_size=s["hidden"], num_layers=layers, num_heads=s["heads"], num_kv_heads=s["kv"],
+                       head_dim=128, intermediate_size=s["ff"], vocab_size=VOCAB, qk_norm=True, sliding_window=window,
                        num_experts=s["experts"], num_experts_per_tok=s["top"], moe_intermediate_size=s["ff"],
                        max_position_embeddings=1 << 16)
 
@@ -136,7 +181,46 @@ def work(cfg: ModelConfig, T: int, decode: bool, rows: int) -> Dict[str, tuple]:
         add("moe_permute", ((T + rows) * H * 2, 0))
         add("moe_gate_up", (rows * (H + ff) * 2 + used * 2 * ff * H * 2, 4 * rows * ff * H))
         add("moe_down", (rows * (H + ff) * 2 + used * ff * H * 2, 2 * rows * ff * H))
-    if cfg.block == "sandwich":
+    if cfg.block == "parallel":
+        for l in cfg.layer_specs:
+            m, moe = l.mixer, l.moe
+            if m.kind == "attention":
+                nq, nk, out_rows = m.heads * m.dim, m.kv_heads * m.dim, m.heads * m.value_dim
+                add("in_gemm", _gemm(T, nq + 2 * nk, H))
+                add("qk_prep", (T * (2 * nq + 4 * nk) * 2, 0))
+                attend(m.heads, m.kv_heads, m.dim)
+            elif m.kind == "latent":
+                r, p, n, hq, out_rows = m.kv_rank, m.rope_part, keys(), m.heads * (m.dim + m.rope_part), m.heads * m.vdim
+                add("in_gemm", _gemm(T, hq + r + p + out_rows, H))
+                add("latent_prep", (T * ((m.heads * p if decode else hq) + r + p) * 4, 0))
+                if decode:
+                    for name, d in (("uk_gemm", m.dim), ("uv_gemm", m.vdim)):
+                        add(name, (T * m.heads * (d + r) * 2 + m.heads * d * r * 2, 2 * T * m.heads * d * r))
+                    add("latent_attention", (T * n * (r + p) * 2 + T * m.heads * (2 * r + p) * 2, 2 * T * n * m.heads * (2 * r + p)))
+                else:
+                    add("ukv_gemm", _gemm(T, m.heads * (m.dim + m.vdim), r))
+                    add("latent_prefill", (T * 4 * hq * 2, 4 * T * n * hq))
+                add("out_gate", (T * out_rows * 6, 0))
+            else:
+                nk, nv, out_rows = m.heads * m.dim, m.heads * m.vdim, m.heads * m.vdim
+                add("in_gemm", _gemm(T, 2 * nk + 2 * nv, H))
+                if decode:
+                    add("lightning", (T * m.heads * m.dim * m.vdim * 8 + T * (2 * nk + nv) * 2 + T * nv * 4, 0))
+                else:      # as for gated linear attention below
+                    add("lightning", (T * (2 * nk + nv) * 2 + T * nv * 4,
+                                      2 * T * m.heads * (2 * m.dim * m.vdim + 32 * (m.dim + m.vdim))))
+                add("lightning_gate", (T * nv * (4 + 2 + 2), 0))
+            add("out_gemm", _gemm(T, H, out_rows, 4))
+            if l.ff:
+                add("up_gemm", _gemm(T, l.ff, H))
+                add("down_gemm", _gemm(T, H, l.ff, 4))
+            else:
+                experts(moe.experts, moe.top, moe.ff)
+                add("shared_gate_up", (T * H * 2 + 2 * moe.shared_ff * H * 2 + T * moe.shared_ff * 2, 4 * T * moe.shared_ff * H))
+                add("shared_down", _gemm(T, H, moe.shared_ff, 4))
+            # the stream read and written, the next operand written, the sublayers' outputs read
+            add("norm", (T * H * (4 + 4 + 2 + 4 + (4 if l.ff else 4 + 2 * moe.top)), 0))
+    elif cfg.block == "sandwich":
         stream = T * H * (4 + 4 + 2)          # the residual sum read and written, the next operand written
         for i, _ in cfg.layer_runs():
             m, moe = cfg.layer_specs[i].mixer, cfg.layer_specs[i].moe
@@ -161,6 +245,8 @@ def work(cfg: ModelConfig, T: int, decode: bool, rows: int) -> Dict[str, tuple]:
                     add("latent_prefill", (T * 4 * hd * 2, 4 * T * n * hd))
                 add("out_gemm", _gemm(T, H, hd, 4))
             add("norm", (stream + T * H * 4, 0))
+            if not moe:
+                continue
             experts(moe.experts, moe.top, moe.ff)
             add("norm", (stream + T * H * 2 * moe.top, 0))
     elif cfg.is_hybrid:
@@ -288,13 +374,13 @@ def bench_model(model, steps: int, warmup: int, decode_sizes=(64, 256)) -> dict:
     return res
 
 
-def mla_kernel(heads: int, steps: int, warmup: int, decode_sizes=(64, 256)) -> dict:
-    """The latent kernel of the MLA models (rank 512 + 64 rotated dimensions, no window) over WINDOW keys per row in decoding
-    and over whole prompts in prefill: ms and share of the roofline."""
+def mla_kernel(heads: int, steps: int, warmup: int, decode_sizes=(64, 256), context: int = WINDOW) -> dict:
+    """The latent kernel of the MLA models (rank 512 + 64 rotated dimensions, no window) over ``context`` keys per row in
+    decoding and over whole prompts in prefill: ms and share of the roofline."""
     from ..ops import mla as MLA
     hbm, tf, _ = _peaks()
     res = {}
-    for name, rows, keys in [("prefill", PROMPT * PROMPTS, None)] + [(f"decode_{B}", B, WINDOW) for B in decode_sizes]:
+    for name, rows, keys in [("prefill", PROMPT * PROMPTS, None)] + [(f"decode_{B}", B, context) for B in decode_sizes]:
         seqs = PROMPTS if keys is None else rows
         per = PROMPT // 16
         cache = torch.randn(seqs * per, 16, 576, device="cuda").to(torch.bfloat16)
@@ -325,6 +411,21 @@ def gorulorn_main(sizes=tuple(GORULORN_SIZES), steps: int = 10, warmup: int = 3)
             del model, src
             torch.cuda.empty_cache()
         out[f"mla-kernel-{size}"] = mla_kernel(s["lat"], steps, warmup)
+    return out
+
+
+def ritirax_main(sizes=tuple(RITIRAX_SIZES), steps: int = 10, warmup: int = 3) -> dict:
+    out = {}
+    for size in sizes:
+        s = RITIRAX_SIZES[size]
+        for name, cls, cfg in (("ritirax", HybridDecoder, ritirax_config(s)), ("moe", DecoderModel, moe_config(s, 6, 0)),
+                               ("gla", HybridDecoder, gla_config(s)), ("latent", HybridDecoder, latent_config(s))):
+            src = RandomWeights(cfg, "cuda", torch.bfloat16, seed=0)
+            model = cls(cfg, src, device="cuda", dtype=torch.bfloat16, max_positions=PROMPT)
+            out[f"{name}-{size}"] = bench_model(model, steps, warmup)
+            del model, src
+            torch.cuda.empty_cache()
+        out[f"mla-kernel-{size}"] = mla_kernel(s["lat"], steps, warmup, context=PROMPT)
     return out
 
 
