@@ -1036,7 +1036,7 @@ static int paged_decode_impl(const void* q, void* out, const void* kv_cache, int
 }
 
 // full_weights: softmax weights as bf16 pairs in the second product. keep: the first `keep` tokens stay visible outside the
-// window. softcap, bias [n_q_heads][nb]: capped and biased scores (with full weights).
+// window. softcap, bias: capped and biased scores (score_mod.cuh; with full weights).
 GLLM_API int gllm_paged_decode(const void* q, void* out, const void* kv_cache, int num_pages,
                                const int* block_tables, int max_blocks, const int* ctx_lens, int batch,
                                int n_q_heads, int n_kv_heads, float scale, int pages_per_split, int max_splits,

@@ -25,7 +25,7 @@ struct AnyAttnParams {
   int causal, window, keep, num_pages;
   const float* sinks;
   float softcap;
-  const float* bias;                                    // [n_q][nb] by distance, the last entry for every longer one
+  const float* bias;                                    // by distance: score_mod.cuh
   int nb;
   int* err;
 };
@@ -83,7 +83,7 @@ __global__ void __launch_bounds__(128) attention_any_kernel(const AnyAttnParams 
     }
     s = warp_sum(s);
     if (p.softcap > 0.f) s = p.softcap * any_tanh<T>(s / p.softcap);
-    if (p.bias) s += p.bias[static_cast<long long>(head) * p.nb + min(max(hi - 1 - t, 0), p.nb - 1)];
+    if (p.bias) s += bias_row(p.bias, p.nb, head)[min(max(hi - 1 - t, 0), p.nb - 1)] * 0.6931471805599453f;
     const float mn = fmaxf(mx, s);
     const float c = any_exp<T>(mx - mn), w = any_exp<T>(s - mn);
     l = l * c + w;

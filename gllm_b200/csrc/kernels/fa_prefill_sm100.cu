@@ -11,12 +11,13 @@
 //               of the second product: it is used exactly as the pages store it (tokens x head_dim).
 //   warps 2-5   softmax of tile 0: each thread owns one query row = one TMEM lane. tcgen05.ld of the S row, online
 //   warps 6-9   softmax of tile 1   softmax in the exp2 domain, P written as bf16 into shared memory in the K-major
-//               128-byte-swizzled layout the second product reads; when a row maximum of the warp moved, the warp
-//               rescales its 32 lanes of the O accumulator in TMEM (tcgen05.ld / tcgen05.st).
+//               128-byte-swizzled layout the second product reads; when a row maximum of the warp moved far, the
+//               warp rescales its 32 lanes of the O accumulator in TMEM (tcgen05.ld / tcgen05.st).
 //
-// The issuer interleaves the tiles (PV_0(j), S_0(j+1), PV_1(j), S_1(j+1), ...), so the tensor core works on one tile
-// while the other tile's softmax runs. A commit after S_t(j+1) also covers PV_t(j): "S ready" tells the softmax
-// warps that the P buffer and the O accumulator of their tile are theirs again.
+// Each tile has two S accumulators: the issuer sends S_0(j+1) and S_1(j+1) before it waits for the weights of block j, so the
+// softmax of a tile goes on to the next block's scores while PV_t(j) runs; only its rescaling of O and its writing of P
+// wait for PV_t(j) (`pv_done`). S_t(j+2) may overwrite the scores of block j because the weights of block j, which the
+// issuer has waited for by then, are written after those scores were read.
 //
 // Semantics are those of paged_prefill_kernel (attention.cu): the queries of a sequence are the last q_len of its ctx
 // tokens, causal (or bidirectional) mask, optional sliding window and learnable sinks; scale 1/sqrt(d) folded into
@@ -44,8 +45,9 @@ constexpr int kFaOffP = kFaOffV + kFaStages * kFaKvTile;
 template <bool kFW> constexpr int kFaOffBarOf = kFaOffP + (kFW ? 4 : 2) * kFaPTile;
 template <bool kFW> constexpr int kFaSmemOf = kFaOffBarOf<kFW> + 256 + 1024;
 static_assert(kFaSmemOf<true> <= 227 * 1024, "shared memory of one CTA");
+constexpr float kFaLazy = 8.f;
 constexpr int kFaThreads = 320;
-constexpr int kFaTmemCols = 512;               // S_0, S_1: 64 columns each; O_0, O_1: 128 columns each (384 used)
+constexpr int kFaTmemCols = 512;               // S_0, S_1: two times 64 columns each; O_0, O_1: 128 columns each
 
 struct FaParams {
   __nv_bfloat16* out;        // [T, Hq, 128]
@@ -98,37 +100,69 @@ __device__ __forceinline__ uint64_t umma_desc_sw128_mn(uint32_t smem_addr, uint3
   return d;
 }
 
-// 64 raw scores of one row against tokens t0 ..: soft cap, then the bias by distance (`n0`: distance to t0, `far`: the bias
-// at the table's end). The choice between the forms of tanh is the warp's, so it costs one vote.
-__device__ __forceinline__ void modify_scores(const ScoreMod& m, int head, int n0, float far, uint32_t (&sr)[2][32]) {
-  float big = 0.f;
-#pragma unroll
-  for (int h = 0; h < 2; ++h)
-#pragma unroll
-    for (int i = 0; i < 32; ++i) {
-      const float z = __uint_as_float(sr[h][i]) * m.in;
-      sr[h][i] = __float_as_uint(z);
-      big = fmaxf(big, fabsf(z));
-    }
-  const bool is_far = n0 - (kFaKv - 1) >= m.nb - 1;
+__device__ __forceinline__ float max3(float a, float b, float c) {
+  float r;
+  asm("max.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c));
+  return r;
+}
+
+// 64 raw scores of one row against tokens t0 ..: soft cap, then the bias by distance (`n0`: distance to t0, `bias`: the
+// head's biases or null, `far`: the one at the table's end). Whether the tile lies behind the table's end and which form of
+// tanh it needs is the warp's choice, so the loops have no branches; two scores go through each instruction.
+__device__ __forceinline__ void modify_scores(const ScoreMod& m, const float* bias, int n0, float far, uint32_t (&sr)[2][32]) {
+  const bool near = bias && __any_sync(0xffffffffu, n0 - (kFaKv - 1) < m.nb - 1);
+  const uint64_t in2 = f2_pack(m.in, m.in), far2 = f2_pack(far, far);
+  // rows ahead of the tile and rows behind the table's end stay within the table's margins
+  const float* row = bias + max(min(n0, m.nb - 1 + kBiasBehind), kFaKv - 1 - kBiasBefore);
+  auto pair = [&](int h, int i) { return f2_pack(__uint_as_float(sr[h][i]), __uint_as_float(sr[h][i + 1])); };
+  auto put = [&](int h, int i, uint64_t v) {
+    float a, b;
+    f2_unpack(v, a, b);
+    sr[h][i] = __float_as_uint(a);
+    sr[h][i + 1] = __float_as_uint(b);
+  };
+  auto bias2 = [&](int h, int i) { return f2_pack(__ldg(row - h * 32 - i), __ldg(row - h * 32 - i - 1)); };
   auto each = [&](auto f) {
-    if (__all_sync(0xffffffffu, is_far)) {
+    if (near) {
 #pragma unroll
       for (int h = 0; h < 2; ++h)
 #pragma unroll
-        for (int i = 0; i < 32; ++i) sr[h][i] = __float_as_uint(f(__uint_as_float(sr[h][i])) + far);
+        for (int i = 0; i < 32; i += 2) put(h, i, f(pair(h, i), bias2(h, i)));
     } else {
 #pragma unroll
       for (int h = 0; h < 2; ++h)
 #pragma unroll
-        for (int i = 0; i < 32; ++i)
-          sr[h][i] = __float_as_uint(f(__uint_as_float(sr[h][i])) + score_bias(m, head, n0 - h * 32 - i));
+        for (int i = 0; i < 32; i += 2) put(h, i, f(pair(h, i), far2));
     }
   };
-  const float out = m.out;
-  if (out <= 0.f) each([](float z) { return z; });
-  else if (__all_sync(0xffffffffu, big <= kTanhSmall)) each([out](float z) { return out * tanh_small(z); });
-  else each([out](float z) { return out * tanh_score(z); });
+  if (m.out <= 0.f) {
+    each([in2](uint64_t s, uint64_t b) { return f2_fma(s, in2, b); });
+    return;
+  }
+  float lo = 0.f, hi = 0.f;
+#pragma unroll
+  for (int h = 0; h < 2; ++h)
+#pragma unroll
+    for (int i = 0; i < 32; i += 2) {
+      hi = max3(hi, __uint_as_float(sr[h][i]), __uint_as_float(sr[h][i + 1]));
+      lo = max3(lo, -__uint_as_float(sr[h][i]), -__uint_as_float(sr[h][i + 1]));
+    }
+  if (__all_sync(0xffffffffu, fmaxf(lo, hi) * m.in <= kTanhSmall)) {
+    const float o = m.out;
+    const uint64_t k0 = f2_pack(o, o), k1 = f2_pack(o * kTanh1, o * kTanh1), k2 = f2_pack(o * kTanh2, o * kTanh2),
+                   k3 = f2_pack(o * kTanh3, o * kTanh3), k4 = f2_pack(o * kTanh4, o * kTanh4);
+    each([&](uint64_t s, uint64_t b) {
+      const uint64_t z = f2_mul(s, in2), u = f2_mul(z, z);
+      return f2_fma(z, f2_fma(f2_fma(f2_fma(f2_fma(k4, u, k3), u, k2), u, k1), u, k0), b);
+    });
+  } else {
+    each([&](uint64_t s, uint64_t b) {
+      float x, y, bx, by;
+      f2_unpack(s, x, y);
+      f2_unpack(b, bx, by);
+      return f2_pack(fmaf(m.out, tanh_score(x * m.in), bx), fmaf(m.out, tanh_score(y * m.in), by));
+    });
+  }
 }
 
 // KV token range of one query tile: tiles [j0, j1) of 64 tokens, counted in visiting order (see `kv_tile_of`).
@@ -149,11 +183,11 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   uint64_t* k_empty = bars + 4;            // 3
   uint64_t* v_full = bars + 7;             // 3
   uint64_t* v_empty = bars + 10;           // 3
-  uint64_t* s_full = bars + 13;            // 2 (per tile)
-  uint64_t* p_full = bars + 15;            // 2
-  uint64_t* o_full = bars + 17;            // 2
-  uint32_t* tmem_base_ptr = reinterpret_cast<uint32_t*>(bars + 19);
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 20);
+  uint64_t* s_full = bars + 13;            // 4 (per tile and accumulator: 2 * tile + block & 1)
+  uint64_t* p_full = bars + 17;            // 2 (per tile)
+  uint64_t* pv_done = bars + 19;           // 2
+  uint32_t* tmem_base_ptr = reinterpret_cast<uint32_t*>(bars + 21);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(bars + 22);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = blockIdx.z;
@@ -222,9 +256,10 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       mbar_init(&v_empty[i], 1);
     }
     for (int t = 0; t < 2; ++t) {
-      mbar_init(&s_full[t], 1);
+      mbar_init(&s_full[2 * t], 1);
+      mbar_init(&s_full[2 * t + 1], 1);
       mbar_init(&p_full[t], 128);
-      mbar_init(&o_full[t], 1);
+      mbar_init(&pv_done[t], 1);
     }
     mbar_fence_init();
     fence_proxy_async_smem();
@@ -308,14 +343,14 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       bool ok = mbar_wait(q_full, 0, abort_flag, p.err, ERR_TIMEOUT_TMA_FULL, wait_ns);
       auto in_range = [&](int t, int j) { return tile[t].rows > 0 && j >= tile[t].j0 && j < tile[t].j1; };
       auto issue_s = [&](int t, int j) {
-        const int stg = (j - J0) % kFaStages;
+        const int stg = (j - J0) % kFaStages, buf = 2 * t + ((j - tile[t].j0) & 1);
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
           const uint64_t a = umma_desc_sw128(q_addr + t * kFaQTile + (k >> 2) * (kFaQTile / 2) + (k & 3) * 32);
           const uint64_t b = umma_desc_sw128(k_addr + stg * kFaKvTile + (k >> 2) * (kFaKvTile / 2) + (k & 3) * 32);
-          umma_f16(tmem_base + t * kFaKv, a, b, idesc_s, k > 0 ? 1u : 0u);
+          umma_f16(tmem_base + buf * kFaKv, a, b, idesc_s, k > 0 ? 1u : 0u);
         }
-        umma_commit(&s_full[t]);
+        umma_commit(&s_full[buf]);
       };
       auto issue_pv = [&](int t, int j) {
         const int stg = (j - J0) % kFaStages;
@@ -323,9 +358,9 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         for (int k = 0; k < 4; ++k) {
           const uint64_t a = umma_desc_sw128(p_addr + t * kFaPTile + k * 32);
           const uint64_t b = umma_desc_sw128_mn(v_addr + stg * kFaKvTile + k * 2048, kFaKvTile / 2);
-          umma_f16(tmem_base + 128 + t * kFaD, a, b, idesc_o, (j > tile[t].j0 || k > 0) ? 1u : 0u);
+          umma_f16(tmem_base + 4 * kFaKv + t * kFaD, a, b, idesc_o, (j > tile[t].j0 || k > 0) ? 1u : 0u);
           if constexpr (kFW)      // the remainders of the same 16 tokens
-            umma_f16(tmem_base + 128 + t * kFaD, umma_desc_sw128(p_addr + (2 + t) * kFaPTile + k * 32), b, idesc_o, 1u);
+            umma_f16(tmem_base + 4 * kFaKv + t * kFaD, umma_desc_sw128(p_addr + (2 + t) * kFaPTile + k * 32), b, idesc_o, 1u);
         }
       };
       // prologue: the first S of every tile whose range starts at J0
@@ -341,35 +376,27 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       int np[2] = {0, 0};   // P buffers consumed so far, per tile
       for (int j = J0; j < J1 && ok; ++j) {
         const int n = j - J0, stg = n % kFaStages;
-        const bool has_next = j + 1 < J1;
-        const int stg1 = (n + 1) % kFaStages;
-        bool k_ready = false;
+        if (j + 1 < J1) {
+          const int stg1 = (n + 1) % kFaStages;
+          ok = mbar_wait(&k_full[stg1], ((n + 1) / kFaStages) & 1, abort_flag, p.err, ERR_TIMEOUT_TMA_FULL, wait_ns);
+          if (!ok) break;
+          tc_fence_after();
+          for (int t = 0; t < 2; ++t)
+            if (in_range(t, j + 1)) issue_s(t, j + 1);
+          umma_commit(&k_empty[stg1]);
+        }
         ok = mbar_wait(&v_full[stg], (n / kFaStages) & 1, abort_flag, p.err, ERR_TIMEOUT_TMA_FULL, wait_ns);
         for (int t = 0; t < 2 && ok; ++t) {
-          if (in_range(t, j)) {
-            ok = mbar_wait(&p_full[t], np[t] & 1, abort_flag, p.err, ERR_TIMEOUT_TMEM_FULL, wait_ns);
-            if (!ok) break;
-            ++np[t];
-            tc_fence_after();
-            issue_pv(t, j);
-            if (j + 1 == tile[t].j1) umma_commit(&o_full[t]);
-          }
-          if (has_next && in_range(t, j + 1)) {
-            if (!k_ready) {
-              ok = mbar_wait(&k_full[stg1], ((n + 1) / kFaStages) & 1, abort_flag, p.err, ERR_TIMEOUT_TMA_FULL, wait_ns);
-              if (!ok) break;
-              k_ready = true;
-              tc_fence_after();
-            }
-            issue_s(t, j + 1);
-          }
+          if (!in_range(t, j)) continue;
+          ok = mbar_wait(&p_full[t], np[t] & 1, abort_flag, p.err, ERR_TIMEOUT_TMEM_FULL, wait_ns);
+          if (!ok) break;
+          ++np[t];
+          tc_fence_after();
+          issue_pv(t, j);
+          umma_commit(&pv_done[t]);
         }
         if (!ok) break;
         umma_commit(&v_empty[stg]);
-        if (has_next) {
-          if (!k_ready) ok = mbar_wait(&k_full[stg1], ((n + 1) / kFaStages) & 1, abort_flag, p.err, ERR_TIMEOUT_TMA_FULL, wait_ns);
-          umma_commit(&k_empty[stg1]);
-        }
       }
     }
   } else {
@@ -380,8 +407,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       const int quarter = warp & 3;                    // the TMEM lanes this warp may touch: 32 * (warp % 4) ...
       const int row = quarter * 32 + lane;
       const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16);
-      const uint32_t s_addr = lane_addr + t * kFaKv;
-      const uint32_t o_addr = lane_addr + 128 + t * kFaD;
+      const uint32_t o_addr = lane_addr + 4 * kFaKv + t * kFaD;
       const bool row_ok = row < ti.rows;
       const int pos = ctx - qlen + ti.row0 + (row_ok ? row : 0);
       const int hi = p.causal ? min(ctx - 1, pos) : ctx - 1;
@@ -389,10 +415,12 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       uint8_t* p_row = smem + kFaOffP + t * kFaPTile + (row >> 3) * 1024 + (row & 7) * 128;
       float m = -INFINITY, l = 0.f;
       [[maybe_unused]] const float far = MOD ? score_bias(p.mod, ti.head, p.mod.nb) : 0.f;
+      [[maybe_unused]] const float* bias = MOD && p.mod.bias ? bias_row(p.mod.bias, p.mod.nb, ti.head) : nullptr;
       bool ok = true;
       for (int j = ti.j0; j < ti.j1; ++j) {
         const int c = j - ti.j0;
-        ok = mbar_wait(&s_full[t], c & 1, abort_flag, p.err, ERR_TIMEOUT_TMEM_FULL, wait_ns);
+        const uint32_t s_addr = lane_addr + (2 * t + (c & 1)) * kFaKv;
+        ok = mbar_wait(&s_full[2 * t + (c & 1)], (c >> 1) & 1, abort_flag, p.err, ERR_TIMEOUT_TMEM_FULL, wait_ns);
         if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
         tc_fence_after();
         uint32_t sr[2][32];
@@ -402,23 +430,30 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         const int t0 = kv_tile_of(j) * kFaKv;
         const bool full_tile = t0 >= lo && t0 + kFaKv - 1 <= hi;
         float mx = -INFINITY;
-        if constexpr (MOD) modify_scores(p.mod, ti.head, pos - t0, far, sr);
+        if constexpr (MOD) modify_scores(p.mod, bias, pos - t0, far, sr);
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            float x = MOD ? __uint_as_float(sr[h][i]) : __uint_as_float(sr[h][i]) * p.scale_log2;
-            if (!full_tile) {
-              const int tk = t0 + h * 32 + i;
-              if ((tk < lo && tk >= p.keep) || tk > hi) x = -INFINITY;
+          for (int i = 0; i < 32; i += 2) {
+            float x[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              x[e] = MOD ? __uint_as_float(sr[h][i + e]) : __uint_as_float(sr[h][i + e]) * p.scale_log2;
+              if (!full_tile) {
+                const int tk = t0 + h * 32 + i + e;
+                if ((tk < lo && tk >= p.keep) || tk > hi) x[e] = -INFINITY;
+              }
+              sr[h][i + e] = __float_as_uint(x[e]);
             }
-            sr[h][i] = __float_as_uint(x);
-            mx = fmaxf(mx, x);
+            mx = max3(mx, x[0], x[1]);
           }
-        const float m_new = fmaxf(m, mx);
+        // the reference of the exponentials follows the row maximum only when that grew by more than a factor of 2^8: the
+        // weights stay below 2^8 and the accumulator is rarely rescaled
+        const bool moved = mx > m + kFaLazy;
+        const float m_new = moved ? mx : m;
         const float m_ref = (m_new == -INFINITY) ? 0.f : m_new;
         const float corr = ex2_approx(m - m_ref);        // m = -inf: 0
-        float sum = 0.f;
+        float sum = 0.f, sum2 = 0.f;
         uint32_t pk[32];
         [[maybe_unused]] uint32_t pr[kFW ? 32 : 1];
 #pragma unroll
@@ -427,14 +462,21 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
           for (int i = 0; i < 32; i += 2) {
             const float e0 = ex2_approx(__uint_as_float(sr[h][i]) - m_ref);
             const float e1 = ex2_approx(__uint_as_float(sr[h][i + 1]) - m_ref);
-            sum += e0 + e1;
-            pk[h * 16 + (i >> 1)] = pack_bf16x2(e0, e1);
-            if constexpr (kFW) pr[h * 16 + (i >> 1)] = pack_bf16x2(e0 - bf16_round(e0), e1 - bf16_round(e1));
+            sum += e0;
+            sum2 += e1;
+            const uint32_t w = pack_bf16x2(e0, e1);
+            pk[h * 16 + (i >> 1)] = w;
+            if constexpr (kFW)
+              pr[h * 16 + (i >> 1)] = pack_bf16x2(e0 - __uint_as_float(w << 16), e1 - __uint_as_float(w & 0xFFFF0000u));
           }
-        l = l * corr + sum;
-        // the O accumulator: rescaled by the warp when any of its rows moved its maximum (never on the first tile:
+        l = l * corr + (sum + sum2);
+        if (c > 0) {          // P and O of this tile are free again once the product of the block before is done
+          ok = mbar_wait(&pv_done[t], (c - 1) & 1, abort_flag, p.err, ERR_TIMEOUT_TMEM_FULL, wait_ns);
+          if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+          tc_fence_after();
+        }
+        // the O accumulator: rescaled by the warp when any of its rows moved its reference (never on the first tile:
         // the first product overwrites the accumulator)
-        const bool moved = m_new > m;
         m = m_new;
         if (c > 0 && __any_sync(0xffffffffu, moved)) {
 #pragma unroll 1
@@ -461,7 +503,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         tc_fence_before();
         mbar_arrive(&p_full[t]);
       }
-      if (ok) ok = mbar_wait(&o_full[t], 0, abort_flag, p.err, ERR_TIMEOUT_TMEM_FULL, wait_ns);
+      if (ok) ok = mbar_wait(&pv_done[t], (ti.j1 - ti.j0 - 1) & 1, abort_flag, p.err, ERR_TIMEOUT_TMEM_FULL, wait_ns);
       if (__all_sync(0xffffffffu, ok)) {
         tc_fence_after();
         if (p.sinks) l += ex2_approx(p.sinks[ti.head] * 1.4426950408889634f - m);

@@ -69,11 +69,12 @@ class AttentionMixer(_Mixer):
         self.w["bqk"] = (_pad_bias([self._src.get(self._p + n + ".b") for n in names], self.w["wqk"].shape[0], self.device)
                          if m.qkv_bias else None)
         self.w["sink"] = self.vec("sink") if m.sink else None
-        self.w["rel"] = None
+        self.rel = None
         if m.bias_max:            # the learned table, one entry per distance
             table = self.vec("rel")
             rows = torch.tensor(ops.distance_rows(table.shape[0], m.bias_max), device=self.device)
-            self.w["rel"] = table[rows].t().contiguous()
+            self.rel = ops.DistanceBias(table[rows].t())
+            self.w["rel"] = self.rel.table
         self.w["wo"] = self.mat("o")
         self.w["bo"] = _pad_bias([self._src.get(self._p + "o.b")], self.w["wo"].shape[0], self.device) if m.o_bias else None
         norm = m.row_qk_norm or m.head_qk_norm
@@ -112,7 +113,7 @@ class AttentionMixer(_Mixer):
         model.mark("qk_prep")
         o = ws.take("mix", T, m.heads * self.dv)
         mask = dict(window=ops.chunk_window(m.chunk) if m.chunk > 0 else m.window, keep_first=m.keep_first, dim=m.dim,
-                    sinks=self.w["sink"], softcap=m.softcap, rel_bias=self.w["rel"])
+                    sinks=self.w["sink"], softcap=m.softcap, rel_bias=self.rel)
         if batch.is_decode:
             ops.paged_decode(q, kv, batch.block_tables, batch.ctx_lens, n_q=m.heads, n_kv=m.kv_heads, scale=m.scale, out=o,
                              workspace=ws.decode_ws, pages_per_split=getattr(ws.decode_ws, "pages_per_split", 32),

@@ -70,11 +70,23 @@ def distance_rows(rows: int, far: int):
     return out
 
 
+class DistanceBias:
+    """A learned bias per head and distance, for the ``rel_bias`` argument of the attention ops. ``values`` [n_q, n] fp32: by
+    distance, the last entry for n - 1 and more. The kernels' table: in units of log2, with margins (csrc/kernels/score_mod.cuh)."""
+
+    BEFORE, BEHIND = 192, 96
+
+    def __init__(self, values):
+        self.values, self.n = values.float(), values.shape[1]
+        log2 = values.double() / math.log(2.0)
+        self.table = torch.cat([log2[:, :1].expand(-1, self.BEFORE), log2, log2[:, -1:].expand(-1, self.BEHIND)], 1).float().contiguous()
+
+
 def attention_ref(q, kv_cache, block_tables, q_start, q_len, ctx_lens, n_q, n_kv, scale, causal=True, window=0,
                   sinks=None, keep_first=0, dim=None, softcap=0.0, rel_bias=None):
     """q: [T, n_q*D]. Returns [T, n_q*DV] in q.dtype. Works on any device (used as the oracle). ``window`` > 0: sliding
     window, the first ``keep_first`` tokens stay visible; < 0: chunks of -window positions (``chunk_window``). ``softcap``: scores
-    become cap * tanh(score / cap); ``rel_bias`` [n_q, n] joins the capped scores, by distance (the last entry: n - 1 and more)."""
+    become cap * tanh(score / cap); ``rel_bias`` (``DistanceBias``) joins the capped scores."""
     D, DV = head_sizes(kv_cache, n_kv, dim)
     out = q.new_zeros((q.shape[0], n_q * DV))
     group = n_q // n_kv
@@ -92,7 +104,7 @@ def attention_ref(q, kv_cache, block_tables, q_start, q_len, ctx_lens, n_q, n_kv
         if softcap:
             scores = softcap * torch.tanh(scores / softcap)
         if rel_bias is not None:
-            scores = scores + rel_bias[:, (pos_q - pos_k).clamp(0, rel_bias.shape[1] - 1)]
+            scores = scores + rel_bias.values[:, (pos_q - pos_k).clamp(0, rel_bias.n - 1)]
         mask = torch.ones((ql, ctx), dtype=torch.bool, device=q.device)
         if causal:
             mask &= pos_k <= pos_q
@@ -132,8 +144,8 @@ def _mma_head(q, kv_cache, D, DV) -> bool:
 def _bias_args(rel_bias, n_q):
     if rel_bias is None:
         return None, 0
-    assert rel_bias.dtype == torch.float32 and rel_bias.is_contiguous() and rel_bias.shape[0] == n_q
-    return rel_bias.data_ptr(), rel_bias.shape[1]
+    assert rel_bias.table.is_cuda and rel_bias.table.shape[0] == n_q
+    return rel_bias.table.data_ptr(), rel_bias.n
 
 
 def _attention_mma(q, out, kv_cache, block_tables, q_start, q_len, ctx_lens, n_seqs, max_q_len, n_q, n_kv, D, DV, scale, causal,
@@ -171,7 +183,7 @@ def paged_decode(q, kv_cache, block_tables, ctx_lens, *, n_q, n_kv, scale=None, 
                  keep_first: int = 0, dim=None, softcap: float = 0.0, rel_bias=None):
     """One query token per sequence. q: [B, n_q*D]; ctx_lens includes the token just written. ``full_weights``: the softmax
     weights enter the second product as a bf16 pair (value + remainder, 16 bits of mantissa) instead of one bf16.
-    ``keep_first``: with a sliding window, the first tokens stay visible. ``softcap``, ``rel_bias`` [n_q, n] fp32: see
+    ``keep_first``: with a sliding window, the first tokens stay visible. ``softcap``, ``rel_bias``: see
     ``attention_ref``."""
     softcap = float(softcap or 0.0)
     _no_fp8_scores(kv_cache, softcap, rel_bias)

@@ -109,18 +109,19 @@ def test_capped_and_biased_attention(D, DV, nq, nkv, dt, softcap, far, spread):
     rel = None
     if far:
         rows = ops.distance_rows(32, far)
-        rel = rnd(32, nq, seed=3, s=1.5)[torch.tensor(rows)].t().contiguous()
-    kw = dict(n_q=nq, n_kv=nkv, scale=D ** -0.5, sinks=rnd(nq, seed=4, s=2.0), softcap=softcap, rel_bias=rel, dim=D, full_weights=True)
+        rel = rnd(32, nq, seed=3, s=1.5)[torch.tensor(rows)].t()
+    kw = dict(n_q=nq, n_kv=nkv, scale=D ** -0.5, sinks=rnd(nq, seed=4, s=2.0), softcap=softcap, dim=D, full_weights=True)
+    bias = {dev: dict(rel_bias=ops.DistanceBias(rel.to(dev)) if far else None) for dev in ("cpu", "cuda")}
     tol = 3e-6 if dt == F32 else 6e-3
     args = (bt, i32(start), i32(ql), i32(ctx))
-    want = ops.paged_prefill(q, kv, *args, max_q_len=300, **kw)
-    got = ops.paged_prefill(q.cuda(), kv.cuda(), *[t.cuda() for t in args], max_q_len=300, **cuda(kw))
+    want = ops.paged_prefill(q, kv, *args, max_q_len=300, **kw, **bias["cpu"])
+    got = ops.paged_prefill(q.cuda(), kv.cuda(), *[t.cuda() for t in args], max_q_len=300, **cuda(kw), **bias["cuda"])
     close(got, want, tol)
     q1, dctx = rnd(len(ctx) + 1, nq * D, seed=5, s=spread, dt=dt), i32([*ctx, 0])
     bt1 = torch.cat([bt, torch.zeros_like(bt[:1])])
-    want = ops.paged_decode(q1, kv, bt1, dctx, **kw)[:-1]
+    want = ops.paged_decode(q1, kv, bt1, dctx, **kw, **bias["cpu"])[:-1]
     for per in (32, 8):                      # one part, several parts
-        got = ops.paged_decode(q1.cuda(), kv.cuda(), bt1.cuda(), dctx.cuda(), pages_per_split=per, **cuda(kw))[:-1]
+        got = ops.paged_decode(q1.cuda(), kv.cuda(), bt1.cuda(), dctx.cuda(), pages_per_split=per, **cuda(kw), **bias["cuda"])[:-1]
         close(got, want, tol)
 
 
