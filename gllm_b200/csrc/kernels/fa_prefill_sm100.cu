@@ -430,46 +430,67 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         const int t0 = kv_tile_of(j) * kFaKv;
         const bool full_tile = t0 >= lo && t0 + kFaKv - 1 <= hi;
         float mx = -INFINITY;
-        if constexpr (MOD) modify_scores(p.mod, bias, pos - t0, far, sr);
+        if constexpr (MOD) {
+          modify_scores(p.mod, bias, pos - t0, far, sr);
+        } else {
+          const uint64_t scale2 = f2_pack(p.scale_log2, p.scale_log2);
+#pragma unroll
+          for (int h = 0; h < 2; ++h)
+#pragma unroll
+            for (int i = 0; i < 32; i += 2) {
+              float a, b;
+              f2_unpack(f2_mul(f2_pack(__uint_as_float(sr[h][i]), __uint_as_float(sr[h][i + 1])), scale2), a, b);
+              sr[h][i] = __float_as_uint(a);
+              sr[h][i + 1] = __float_as_uint(b);
+            }
+        }
+        if (!__all_sync(0xffffffffu, full_tile)) {       // the warp's choice: most tiles need no mask
+#pragma unroll
+          for (int h = 0; h < 2; ++h)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const int tk = t0 + h * 32 + i;
+              if ((tk < lo && tk >= p.keep) || tk > hi) sr[h][i] = 0xFF800000u;
+            }
+        }
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
-          for (int i = 0; i < 32; i += 2) {
-            float x[2];
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-              x[e] = MOD ? __uint_as_float(sr[h][i + e]) : __uint_as_float(sr[h][i + e]) * p.scale_log2;
-              if (!full_tile) {
-                const int tk = t0 + h * 32 + i + e;
-                if ((tk < lo && tk >= p.keep) || tk > hi) x[e] = -INFINITY;
-              }
-              sr[h][i + e] = __float_as_uint(x[e]);
-            }
-            mx = max3(mx, x[0], x[1]);
-          }
+          for (int i = 0; i < 32; i += 2) mx = max3(mx, __uint_as_float(sr[h][i]), __uint_as_float(sr[h][i + 1]));
         // the reference of the exponentials follows the row maximum only when that grew by more than a factor of 2^8: the
         // weights stay below 2^8 and the accumulator is rarely rescaled
         const bool moved = mx > m + kFaLazy;
         const float m_new = moved ? mx : m;
         const float m_ref = (m_new == -INFINITY) ? 0.f : m_new;
         const float corr = ex2_approx(m - m_ref);        // m = -inf: 0
-        float sum = 0.f, sum2 = 0.f;
+        const uint64_t ref2 = f2_pack(-m_ref, -m_ref);
+        [[maybe_unused]] const uint64_t minus2 = f2_pack(-1.f, -1.f);
+        uint64_t sum2 = f2_pack(0.f, 0.f);
         uint32_t pk[32];
         [[maybe_unused]] uint32_t pr[kFW ? 32 : 1];
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
-            const float e0 = ex2_approx(__uint_as_float(sr[h][i]) - m_ref);
-            const float e1 = ex2_approx(__uint_as_float(sr[h][i + 1]) - m_ref);
-            sum += e0;
-            sum2 += e1;
+            float e0, e1;
+            f2_unpack(f2_add(f2_pack(__uint_as_float(sr[h][i]), __uint_as_float(sr[h][i + 1])), ref2), e0, e1);
+            e0 = ex2_approx(e0);
+            e1 = ex2_approx(e1);
+            const uint64_t e2 = f2_pack(e0, e1);
+            sum2 = f2_add(sum2, e2);
             const uint32_t w = pack_bf16x2(e0, e1);
             pk[h * 16 + (i >> 1)] = w;
-            if constexpr (kFW)
-              pr[h * 16 + (i >> 1)] = pack_bf16x2(e0 - __uint_as_float(w << 16), e1 - __uint_as_float(w & 0xFFFF0000u));
+            if constexpr (kFW) {
+              float r0, r1;
+              f2_unpack(f2_fma(f2_pack(__uint_as_float(w << 16), __uint_as_float(w & 0xFFFF0000u)), minus2, e2), r0, r1);
+              pr[h * 16 + (i >> 1)] = pack_bf16x2(r0, r1);
+            }
           }
-        l = l * corr + (sum + sum2);
+        {
+          float s0, s1;
+          f2_unpack(sum2, s0, s1);
+          l = l * corr + (s0 + s1);
+        }
         if (c > 0) {          // P and O of this tile are free again once the product of the block before is done
           ok = mbar_wait(&pv_done[t], (c - 1) & 1, abort_flag, p.err, ERR_TIMEOUT_TMEM_FULL, wait_ns);
           if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
