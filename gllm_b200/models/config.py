@@ -189,7 +189,7 @@ class ModelConfig:
     post_norm: bool = False  # encoder-style post-LN residual blocks
     # Heterogeneous decoders (models/hybrid.py): one spec per layer. ``block``: "post" = post-norm blocks
     # x = norm(postln_alpha * x + f(x)), "sandwich" = x = x + norm_b(f(norm_a(x))), "parallel" = h = norm(x),
-    # x = x + (mixer(h) + ff(h)); ``norm_type`` rms or layer (no bias), ``norm_one_plus_w``: weights stored around zero.
+    # x = x + (mixer(h) + ff(h)); ``norm_type`` rms or layer (no bias), ``norm_one_plus_w``: weights enter as 1 + w.
     # ``loop`` = (start, stop, times): that range of layers runs ``times`` times in a row with the same weights, a learned
     # vector added to the stream before each pass; every pass has its own cache and state.
     layer_specs: Optional[List[LayerSpec]] = None

@@ -85,7 +85,7 @@ def ritirax_config(s: dict) -> ModelConfig:
     lat = MixerSpec("latent", heads=s["lat"], dim=64, vdim=128, kv_rank=s["kv_rank"], rope_part=64, rot_dim=64, scale=128 ** -0.5,
                     gate=True)
     lin = MixerSpec("lightning", heads=s["lin"], dim=128, vdim=128, decay=tuple(1 - 2.0 ** -(1 + 8 * h / s["lin"]) for h in range(s["lin"])))
-    moe = MoeSpec(experts=s["experts"], top=s["top"], ff=s["ff"], norm_topk=False, scale=2.5, groups=8, keep_groups=4,
+    moe = MoeSpec(experts=s["experts"], top=s["top"], ff=s["ff"], norm_topk=False, scale=2.0, groups=8, keep_groups=4,
                   shared_ff=s["ff"], shared_gate=True)
     specs = [LayerSpec(att, ff=s["dense"], act="relu2", gated=False)] + [LayerSpec(m, act="silu", moe=moe) for m in (lat, lin, att, lin, lat)]
     cfg = ModelConfig(arch="ritirax", hidden_size=s["hidden"], num_layers=6, vocab_size=VOCAB, rms_norm_eps=1e-5, norm_one_plus_w=True,

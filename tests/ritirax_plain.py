@@ -21,7 +21,7 @@ def rms_norm(x, w, eps):
 
 
 def zero_norm(x, w, eps):
-    """The norm whose weight is stored around zero."""
+    """The norm whose weight enters as 1 + w."""
     return rms_norm(x, 1 + w, eps)
 
 

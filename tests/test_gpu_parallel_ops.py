@@ -64,7 +64,7 @@ def test_residual_norm_of_sublayers_side_by_side(H, dt):
             close(ob, oa, 2e-6 if dt == F32 else 4e-3)
 
 
-@pytest.mark.parametrize("E,k,groups,keep", [(16, 4, 4, 3), (64, 8, 8, 4), (512, 32, 16, 2), (72, 6, 12, 3), (40, 3, 40, 7), (24, 5, 2, 1),
+@pytest.mark.parametrize("E,k,groups,keep", [(20, 4, 5, 3), (64, 8, 8, 4), (512, 32, 16, 2), (72, 6, 12, 3), (40, 3, 40, 7), (24, 5, 2, 1),
                                              (9, 2, 1, 1), (100, 4, 0, 0)])
 def test_routing_among_the_best_groups(E, k, groups, keep):
     z = rnd(301, E + 3, s=2.0)
@@ -90,12 +90,12 @@ def test_projection_with_an_activation(M_, N, K, act, cols, dt):
         close(L.gemm(a.cuda(), w.cuda(), act=act, act_cols=cols), want, 4e-3)
 
 
-SCORES = [(128, 128, 32, 8, BF), (128, 128, 16, 1, BF), (128, 128, 6, 6, BF), (96, 64, 16, 4, BF), (64, 64, 32, 4, BF), (192, 128, 8, 8, BF),
+SCORES = [(128, 128, 32, 8, BF), (128, 128, 16, 1, BF), (128, 128, 6, 6, BF), (96, 80, 16, 4, BF), (64, 64, 32, 4, BF), (192, 128, 8, 8, BF),
           (36, 20, 4, 2, BF), (30, 14, 4, 2, BF), (48, 64, 6, 2, F32), (128, 128, 8, 2, F32)]
 
 
 @pytest.mark.parametrize("D,DV,nq,nkv,dt", SCORES)
-@pytest.mark.parametrize("softcap,far,spread", [(30.0, 240, 1.0), (2.0, 33, 6.0), (0.0, 600, 1.0), (20.0, 0, 8.0)])
+@pytest.mark.parametrize("softcap,far,spread", [(25.0, 260, 1.0), (2.0, 33, 6.0), (0.0, 600, 1.0), (20.0, 0, 8.0)])
 def test_capped_and_biased_attention(D, DV, nq, nkv, dt, softcap, far, spread):
     """Prompts (whole, and portions behind a cached context) and decode steps, with sinks; scores inside the cap's linear
     range and far outside."""
@@ -125,7 +125,7 @@ def test_capped_and_biased_attention(D, DV, nq, nkv, dt, softcap, far, spread):
         close(got, want, tol)
 
 
-LATENT = [(16, 512, 64, BF), (64, 512, 64, BF), (8, 256, 64, BF), (33, 128, 64, BF), (5, 96, 32, BF), (20, 200, 56, BF), (3, 448, 64, BF),
+LATENT = [(16, 512, 64, BF), (64, 512, 64, BF), (8, 256, 64, BF), (33, 128, 64, BF), (5, 104, 32, BF), (20, 200, 56, BF), (3, 448, 64, BF),
           (4, 512, 128, BF), (3, 20, 6, BF), (4, 64, 32, F32)]
 
 

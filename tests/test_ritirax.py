@@ -240,7 +240,7 @@ def test_every_step_of_the_distance_bias(name, be):
 
 
 def test_rows_of_the_distance_table():
-    for rows, far in ((12, 50), (32, 240), (32, 128), (2, 10), (1, 5), (7, 33), (20, 11), (16, 100000)):
+    for rows, far in ((12, 50), (32, 300), (32, 128), (2, 10), (1, 5), (7, 33), (20, 11), (16, 100000)):
         got = ops.distance_rows(rows, far)
         assert got[-1] == rows - 1 and got.count(rows - 1) == 1
         if far > rows // 2 > 0:
