@@ -3203,13 +3203,15 @@ GLLM_API int gllm_gemm_bf16_glu(const void* A, long long lda, const void* B, lon
   return dispatch_gemm<EPI_GLU, false>(A, lda, B, ldb, b_rows, p, bn, (cudaStream_t)stream, max_ctas, force_splits);
 }
 
-// Grouped plain GEMM (MoE down projection): m-block i multiplies group mblk_group[i]'s [N,K] weight.
+// Grouped plain GEMM (expert projections without a gate): m-block i multiplies group mblk_group[i]'s [N,K] weight; act as in
+// gllm_gemm_bf16_act, on every column.
 GLLM_API int gllm_gemm_bf16_grouped(const void* A, long long lda, const void* B, long long ldb, void* out,
                                     long long ldo, int M, int N, int K, const int* mblk_group, int num_groups,
-                                    int bn, void* stream, int max_ctas) {
+                                    int bn, int act, void* stream, int max_ctas) {
   GemmParams p = {};
   p.M = M; p.N = N; p.K = K;
   p.out = out; p.ldo = ldo;
+  p.act = act; p.act_cols = act ? N : 0;
   p.mblk_group = mblk_group; p.group_rows = N;
   p.err = gllm_error_word();
   const long long b_rows = static_cast<long long>(num_groups) * N;

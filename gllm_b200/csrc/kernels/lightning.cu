@@ -1,4 +1,9 @@
-// Linear attention with a fixed decay per head (lightning attention), per head S_t = a S_{t-1} + k_t v_t^T, o_t = S_t^T q_t:
+// Linear attention with one decay per head and token, S_t = a_t S_{t-1} + d_t k_t v_t^T, o_t = S_t^T q_t (+ D v_t), in two forms:
+//
+//   lightning attention    a fixed per head, d = 1, no D
+//   state-space duality    (Dao and Gu, "Transformers are SSMs: Generalized Models and Efficient Algorithms Through Structured
+//                          State Space Duality"; template argument SSD) d = softplus(step + bias), a = exp(neg_a d), the step
+//                          projected from the token; q and k (C and B there) are shared by a group of heads
 //
 //   lightning_chunk_kernel    bf16 prompts in chunks of 64 tokens on tensor cores; a CTA owns one (sequence, head, 64 value
 //                             columns) and keeps its slice of the state in fp32 registers from chunk to chunk
@@ -11,7 +16,8 @@
 //   o_i = a^(i+1) S^T q_i + sum_{j <= i} a^(i-j) (q_i . k_j) v_j,   S' = a^n S + sum_j a^(n-1-j) k_j v_j^T
 // q, k and v are bf16; what carries decays or is a state (the scores, the scaled values, S) is fp32 and meets the bf16 tensor
 // core as a (value, remainder) pair. The powers a^0 .. a^64 of every head come from a table, 1 - a as a number of its own: a
-// state remembers 1 / (1 - a) tokens, so the distance of a decay to 1 has to keep its relative accuracy.
+// state remembers 1 / (1 - a) tokens, so the distance of a decay to 1 has to keep its relative accuracy. With decays per token
+// a^(i-j) becomes the exponential of a difference of running sums, and the values are scaled by d_j.
 #include "mma.cuh"
 #include "recurrent.cuh"
 
@@ -30,7 +36,22 @@ struct LightningParams {
   const float* powers;     // [heads][kLiC + 1] decay^n
   float* state;            // [slots][heads][dim][vdim]
   float* out;              // [rows, heads * vdim]
+  // SSD: the steps [rows, heads] (type and rows of q, pitch ldt), [heads] each of the others, heads per q / k head
+  const void* dt;
+  long long ldt;
+  const float *dt_bias, *neg_a, *skip;
+  int group;
 };
+
+template <typename T> __device__ __forceinline__ float ssd_step(const LightningParams& p, long long row, int head) {
+  return softplus_f(to_f(static_cast<const T*>(p.dt)[row * p.ldt + head]) + p.dt_bias[head]);
+}
+__device__ __forceinline__ float li_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float kLiLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ void li_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(x, y);
@@ -47,10 +68,11 @@ __device__ __forceinline__ void li_cp16(void* dst, const void* src, bool there) 
 template <int NSL, int ST> struct LiShape {
   static constexpr int KP = NSL * kLiSlice + 8;
   static constexpr int kK = kLiC * KP * 2, kV = kLiC * kLiVP * 2, kS = NSL * kLiSlice * kLiV * 2, kA = kLiC * kLiAP * 2;
-  static constexpr int kSmem = ST * (2 * kK + kV) + 2 * kV + 2 * kS + 2 * kA + (kLiC + 8) * 4;
+  static constexpr int kTab = 2 * kLiC + 8;        // floats of a table: powers of the decay, or running sums and steps
+  static constexpr int kSmem = ST * (2 * kK + kV) + 2 * kV + 2 * kS + 2 * kA + 2 * kTab * 4;
 };
 
-template <int NSL, int ST>
+template <int NSL, int ST, bool SSD>
 __global__ void __launch_bounds__(kLiThreads, 1) lightning_chunk_kernel(const LightningParams p) {
   using Sh = LiShape<NSL, ST>;
   constexpr int KP = Sh::KP;
@@ -64,17 +86,26 @@ __global__ void __launch_bounds__(kLiThreads, 1) lightning_chunk_kernel(const Li
   bf16_t* s_lo = s_hi + NSL * kLiSlice * kLiV;
   bf16_t* a_hi = s_lo + NSL * kLiSlice * kLiV;                      // [64][kLiAP] decayed scores
   bf16_t* a_lo = a_hi + kLiC * kLiAP;
-  float* pw = reinterpret_cast<float*>(a_lo + kLiC * kLiAP);        // [65]
+  float* const tab = reinterpret_cast<float*>(a_lo + kLiC * kLiAP);   // [2][kTab]
+  float* pw = tab;          // decays a^n; SSD: log2 of the decays from the chunk's start to before token n, then the 64 steps
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int v0 = blockIdx.x * kLiV, head = blockIdx.y;
-  for (int i = tid; i <= kLiC; i += kLiThreads) pw[i] = p.powers[head * (kLiC + 1) + i];
+  const int qk_head = SSD ? head / p.group : head;
+  float step_bias = 0.f, neg_a = 0.f, skip = 0.f;
+  if constexpr (SSD) {
+    step_bias = p.dt_bias[head];
+    neg_a = p.neg_a[head] * kLiLog2e;
+    skip = p.skip[head];
+  } else {
+    for (int i = tid; i <= kLiC; i += kLiThreads) pw[i] = p.powers[head * (kLiC + 1) + i];
+  }
   pdl_wait();
   pdl_launch_dependents();
   const SeqRows s = seq_rows(p.sv, blockIdx.z);
   if (s.len <= 0) return;
   const int nv = p.heads * p.vdim, kvec = p.dim / 8, vvec = min(kLiV, p.vdim - v0) / 8;
-  const bf16_t* qg = static_cast<const bf16_t*>(p.q) + static_cast<long long>(s.row0) * p.ld + head * p.dim;
-  const bf16_t* kg = static_cast<const bf16_t*>(p.k) + static_cast<long long>(s.row0) * p.ld + head * p.dim;
+  const bf16_t* qg = static_cast<const bf16_t*>(p.q) + static_cast<long long>(s.row0) * p.ld + qk_head * p.dim;
+  const bf16_t* kg = static_cast<const bf16_t*>(p.k) + static_cast<long long>(s.row0) * p.ld + qk_head * p.dim;
   const bf16_t* vg = static_cast<const bf16_t*>(p.v) + static_cast<long long>(s.row0) * p.ld + head * p.vdim + v0;
   float* st = p.state + (static_cast<long long>(s.slot) * p.heads + head) * p.dim * p.vdim;
   // query rows (block I of 16) x 32 columns (half h); every scheduler gets as many long rows as short ones
@@ -124,10 +155,49 @@ __global__ void __launch_bounds__(kLiThreads, 1) lightning_chunk_kernel(const Li
   };
   publish_state();
 
+  // SSD: the first warp turns the next chunk's steps into its table while the chunk's tiles arrive; lane l has tokens 2l, 2l + 1
+  float raw[2] = {};
+  auto fetch_steps = [&](int c0) {
+    if (SSD && warp == 0)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = c0 + lane * 2 + e;
+        raw[e] = t < s.len ? to_f(static_cast<const bf16_t*>(p.dt)[(s.row0 + t) * p.ldt + head]) : 0.f;
+      }
+  };
+  auto make_table = [&](int c0, float* at) {
+    if (SSD && warp == 0) {
+      float d[2], sum[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) d[e] = c0 + lane * 2 + e < s.len ? softplus_f(raw[e] + step_bias) : 0.f;
+      sum[0] = neg_a * d[0];
+      sum[1] = fmaf(neg_a, d[1], sum[0]);
+      float run = sum[1];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, run, o);
+        if (lane >= o) run += up;
+      }
+      const float before = run - sum[1];
+      if (lane == 0) at[0] = 0.f;
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        at[lane * 2 + e + 1] = before + sum[e];
+        at[kLiC + 4 + lane * 2 + e] = d[e];
+      }
+    }
+  };
+  fetch_steps(0);
   if constexpr (ST == 2) load(0, 0);
-  int stage = 0;
-  for (int c0 = 0; c0 < s.len; c0 += kLiC, stage ^= ST - 1) {
+  int stage = 0, parity = 0;
+  for (int c0 = 0; c0 < s.len; c0 += kLiC, stage ^= ST - 1, parity ^= 1) {
     const int n = min(kLiC, s.len - c0);
+    if constexpr (SSD) {
+      pw = tab + parity * Sh::kTab;      // the chunk before may still be using the other one
+      make_table(c0, pw);
+      fetch_steps(c0 + kLiC);
+    }
+    const float* step = pw + kLiC + 4;
     if constexpr (ST == 1) {
       __syncthreads();                 // the readers of the chunk before are done
       load(c0, 0);
@@ -142,7 +212,8 @@ __global__ void __launch_bounds__(kLiThreads, 1) lightning_chunk_kernel(const Li
     const bf16_t* vt = v_s + stage * kLiC * kLiVP;
     {                                  // values times a^(n-1-j), as pairs
       const int r = tid >> 2, c = (tid & 3) * 16;
-      const float f = r < n ? pw[n - 1 - r] : 0.f;
+      float f = 0.f;
+      if (r < n) f = SSD ? li_exp2(pw[n] - pw[r + 1]) * step[r] : pw[n - 1 - r];
 #pragma unroll
       for (int i = 0; i < 16; i += 2) {
         const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vt + r * kLiVP + c + i));
@@ -187,13 +258,19 @@ __global__ void __launch_bounds__(kLiThreads, 1) lightning_chunk_kernel(const Li
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
         const int i = i0 + r * 8, j = h * 32 + nt * 8 + t4 * 2;
-        const float x = j <= i ? A[nt][r * 2] * pw[i - j] : 0.f;
-        const float y = j + 1 <= i ? A[nt][r * 2 + 1] * pw[i - j - 1] : 0.f;
+        float x = 0.f, y = 0.f;
+        if constexpr (SSD) {
+          if (j <= i) x = A[nt][r * 2] * (li_exp2(pw[i + 1] - pw[j + 1]) * step[j]);
+          if (j + 1 <= i) y = A[nt][r * 2 + 1] * (li_exp2(pw[i + 1] - pw[j + 2]) * step[j + 1]);
+        } else {
+          x = j <= i ? A[nt][r * 2] * pw[i - j] : 0.f;
+          y = j + 1 <= i ? A[nt][r * 2 + 1] * pw[i - j - 1] : 0.f;
+        }
         uint32_t hi, lo;
         li_split2(x, y, hi, lo);
         *reinterpret_cast<uint32_t*>(a_hi + i * kLiAP + j) = hi;
         *reinterpret_cast<uint32_t*>(a_lo + i * kLiAP + j) = lo;
-        const float f = pw[i + 1];
+        const float f = SSD ? li_exp2(pw[i + 1]) : pw[i + 1];
         O[nt][r * 2] *= f;
         O[nt][r * 2 + 1] *= f;
       }
@@ -220,12 +297,17 @@ __global__ void __launch_bounds__(kLiThreads, 1) lightning_chunk_kernel(const Li
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
         const int i = i0 + r * 8, c = v0 + h * 32 + nt * 8 + t4 * 2;
-        if (i < n && c < p.vdim)
-          *reinterpret_cast<float2*>(p.out + (s.row0 + c0 + i) * static_cast<long long>(nv) + head * p.vdim + c) =
-              make_float2(O[nt][r * 2], O[nt][r * 2 + 1]);
+        if (i < n && c < p.vdim) {
+          float2 o = make_float2(O[nt][r * 2], O[nt][r * 2 + 1]);
+          if constexpr (SSD) {
+            const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vt + i * kLiVP + c - v0));
+            o = make_float2(fmaf(skip, x.x, o.x), fmaf(skip, x.y, o.y));
+          }
+          *reinterpret_cast<float2*>(p.out + (s.row0 + c0 + i) * static_cast<long long>(nv) + head * p.vdim + c) = o;
+        }
       }
     // ---- state ----
-    const float f = pw[n];
+    const float f = SSD ? li_exp2(pw[n]) : pw[n];
 #pragma unroll
     for (int sl = 0; sl < NSL; ++sl) {
       const int d0 = sl * kLiSlice + warp * 16;
@@ -265,7 +347,7 @@ __global__ void __launch_bounds__(kLiThreads, 1) lightning_chunk_kernel(const Li
 // S = a S + x, with the decay as its distance to 1
 __device__ __forceinline__ float li_decay(float S, float forget, float x) { return fmaf(-forget, S, S) + x; }
 
-template <typename T>
+template <typename T, bool SSD>
 __global__ void __launch_bounds__(256) lightning_decode_kernel(const LightningParams p) {
   extern __shared__ __align__(16) float ld_s[];
   const int head = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
@@ -273,15 +355,20 @@ __global__ void __launch_bounds__(256) lightning_decode_kernel(const LightningPa
   float* qs = ld_s;
   float* ks = qs + ((p.dim + 3) & ~3);
   float* red = ks + ((p.dim + 3) & ~3);      // [groups][vdim]
-  const float forget = p.forget[head];
+  float forget = SSD ? 0.f : p.forget[head], step = 1.f;
+  const int qk_head = SSD ? head / p.group : head;
   pdl_wait();
   pdl_launch_dependents();
   const int ctx = p.sv.ctx_lens[b];
   if (ctx <= 0) return;
   const long long row = static_cast<long long>(b) * p.ld;
+  if constexpr (SSD) {
+    step = ssd_step<T>(p, b, head);
+    forget = -expm1f(p.neg_a[head] * step);
+  }
   for (int d = tid; d < p.dim; d += 256) {
-    qs[d] = to_f(static_cast<const T*>(p.q)[row + head * p.dim + d]);
-    ks[d] = to_f(static_cast<const T*>(p.k)[row + head * p.dim + d]);
+    qs[d] = to_f(static_cast<const T*>(p.q)[row + qk_head * p.dim + d]);
+    ks[d] = to_f(static_cast<const T*>(p.k)[row + qk_head * p.dim + d]) * step;
   }
   __syncthreads();
   const int c = (tid % vq) * 4, rg = tid / vq;
@@ -308,6 +395,11 @@ __global__ void __launch_bounds__(256) lightning_decode_kernel(const LightningPa
       const float4 t = *reinterpret_cast<const float4*>(red + h * p.vdim + c);
       o.x += t.x; o.y += t.y; o.z += t.z; o.w += t.w;
     }
+    if constexpr (SSD) {
+      const float4 x = load4(static_cast<const T*>(p.v) + row + head * p.vdim + c);
+      const float skip = p.skip[head];
+      o.x = fmaf(skip, x.x, o.x); o.y = fmaf(skip, x.y, o.y); o.z = fmaf(skip, x.z, o.z); o.w = fmaf(skip, x.w, o.w);
+    }
     *reinterpret_cast<float4*>(p.out + (static_cast<long long>(b) * p.heads + head) * p.vdim + c) = o;
   }
 }
@@ -315,13 +407,15 @@ __global__ void __launch_bounds__(256) lightning_decode_kernel(const LightningPa
 // Any sizes, token by token: a CTA owns 32 value columns of one (sequence, head); eight threads of a warp share a column's
 // rows (row d belongs to thread d % 8).
 constexpr int kLsCols = 32, kLsG = 8, kLsTok = 8;
-template <typename T, int R>
+template <typename T, int R, bool SSD>
 __global__ void __launch_bounds__(kLsCols * kLsG) lightning_step_kernel(const LightningParams p) {
   extern __shared__ float ls_s[];            // [kLsTok][dim] queries, then keys
+  __shared__ float forget_s[kLsTok];
   float* qs = ls_s;
   float* ks = qs + kLsTok * p.dim;
   const int head = blockIdx.y, lane = threadIdx.x & 31, g = lane & 7, col = blockIdx.x * kLsCols + (threadIdx.x >> 5) * 4 + (lane >> 3);
-  const float forget = p.forget[head];
+  const int qk_head = SSD ? head / p.group : head;
+  float forget = SSD ? 0.f : p.forget[head];
   pdl_wait();
   pdl_launch_dependents();
   const SeqRows s = seq_rows(p.sv, blockIdx.z);
@@ -339,15 +433,18 @@ __global__ void __launch_bounds__(kLsCols * kLsG) lightning_step_kernel(const Li
     __syncthreads();
     for (int i = threadIdx.x; i < n * p.dim; i += blockDim.x) {
       const int t = i / p.dim, d = i - t * p.dim;
-      const long long at = static_cast<long long>(s.row0 + t0 + t) * p.ld + head * p.dim + d;
+      const long long at = static_cast<long long>(s.row0 + t0 + t) * p.ld + qk_head * p.dim + d;
       qs[i] = to_f(static_cast<const T*>(p.q)[at]);
-      ks[i] = to_f(static_cast<const T*>(p.k)[at]);
+      ks[i] = to_f(static_cast<const T*>(p.k)[at]) * (SSD ? ssd_step<T>(p, s.row0 + t0 + t, head) : 1.f);
     }
+    if (SSD && static_cast<int>(threadIdx.x) < n)
+      forget_s[threadIdx.x] = -expm1f(p.neg_a[head] * ssd_step<T>(p, s.row0 + t0 + threadIdx.x, head));
     __syncthreads();
     for (int t = 0; t < n; ++t) {
       const long long m = s.row0 + t0 + t;
       const float v = live ? to_f(static_cast<const T*>(p.v)[m * p.ld + head * p.vdim + col]) : 0.f;
       float o = 0.f;
+      if constexpr (SSD) forget = forget_s[t];
 #pragma unroll
       for (int r = 0; r < R; ++r) {
         const int d = g + kLsG * r;
@@ -358,7 +455,7 @@ __global__ void __launch_bounds__(kLsCols * kLsG) lightning_step_kernel(const Li
       }
 #pragma unroll
       for (int x = 1; x < kLsG; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
-      if (live && g == 0) p.out[(m * p.heads + head) * p.vdim + col] = o;
+      if (live && g == 0) p.out[(m * p.heads + head) * p.vdim + col] = SSD ? fmaf(p.skip[head], v, o) : o;
     }
   }
 #pragma unroll
@@ -443,7 +540,7 @@ static int li_done(cudaError_t e, const char* what) {
 }
 static bool li_al16(const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; }
 
-template <int NSL, int ST>
+template <int NSL, int ST, bool SSD>
 static int li_chunks(const LightningParams& p, cudaStream_t s) {
   constexpr int smem = LiShape<NSL, ST>::kSmem;
   static_assert(smem <= 227 * 1024, "shared memory of one CTA");
@@ -451,12 +548,45 @@ static int li_chunks(const LightningParams& p, cudaStream_t s) {
   int dev = 0;
   cudaGetDevice(&dev);
   if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(lightning_chunk_kernel<NSL, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(lightning_chunk_kernel<NSL, ST, SSD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return li_done(e, "attributes");
     attr_set[dev & 63] = true;
   }
-  return li_done(launch_kernel(lightning_chunk_kernel<NSL, ST>, dim3((p.vdim + kLiV - 1) / kLiV, p.heads, p.sv.n), dim3(kLiThreads),
+  return li_done(launch_kernel(lightning_chunk_kernel<NSL, ST, SSD>, dim3((p.vdim + kLiV - 1) / kLiV, p.heads, p.sv.n), dim3(kLiThreads),
                                smem, s, true, 0, p), "chunks");
+}
+
+template <typename T, bool SSD>
+static int li_steps(const LightningParams& p, cudaStream_t s) {
+  const dim3 grid((p.vdim + kLsCols - 1) / kLsCols, p.heads, p.sv.n);
+  const size_t smem = sizeof(float) * 2 * kLsTok * p.dim;
+  const int rows = (p.dim + kLsG - 1) / kLsG;
+#define LI_STEP(R) \
+  return li_done(launch_kernel(lightning_step_kernel<T, R, SSD>, grid, dim3(kLsCols * kLsG), smem, s, true, 0, p), "steps")
+  if (rows <= 8) LI_STEP(8);
+  if (rows <= 16) LI_STEP(16);
+  LI_STEP(64);
+#undef LI_STEP
+}
+
+template <bool SSD>
+static int li_run(const LightningParams& p, int is_f32, int general, cudaStream_t s) {
+  const int dim = p.dim, vdim = p.vdim, heads = p.heads, n_seqs = p.sv.n;
+  if (dim <= 0 || dim > 512 || vdim <= 0 || heads <= 0 || n_seqs > 65535 || heads > 65535) {
+    set_last_error("lightning: %d heads of %d (at most 512) x %d, %d sequences", heads, dim, vdim, n_seqs);
+    return -1;
+  }
+  const size_t decode_smem = sizeof(float) * (2 * ((dim + 3) & ~3) + (vdim >= 4 ? 256 / (vdim / 4) * vdim : 0));
+  if (!general && !p.sv.q_start && vdim % 4 == 0 && vdim <= 1024 && p.ld % 4 == 0 && decode_smem <= 48 * 1024 && li_al16(p.state) &&
+      li_al16(p.out) && (reinterpret_cast<uintptr_t>(p.v) & (is_f32 ? 15 : 7)) == 0) {
+    const dim3 grid(heads, n_seqs);
+    return li_done(is_f32 ? launch_kernel(lightning_decode_kernel<float, SSD>, grid, dim3(256), decode_smem, s, true, 0, p)
+                          : launch_kernel(lightning_decode_kernel<bf16_t, SSD>, grid, dim3(256), decode_smem, s, true, 0, p), "decode");
+  }
+  if (!general && p.sv.q_start && !is_f32 && dim % 16 == 0 && dim <= 2 * kLiSlice && vdim % 8 == 0 && p.ld % 8 == 0 && li_al16(p.q) &&
+      li_al16(p.k) && li_al16(p.v))
+    return dim <= kLiSlice ? li_chunks<1, 2, SSD>(p, s) : li_chunks<2, 1, SSD>(p, s);
+  return is_f32 ? li_steps<float, SSD>(p, s) : li_steps<bf16_t, SSD>(p, s);
 }
 
 // q, k [rows, heads * dim] and v [rows, heads * vdim] share the row pitch ld; out [rows, heads * vdim] fp32; state [slots,
@@ -465,39 +595,30 @@ GLLM_API int gllm_lightning(const int* q_start, const int* q_len, const int* ctx
                             const void* k, const void* v, long long ld, int is_f32, int heads, int dim, int vdim,
                             const float* forget, const float* powers, float* state, float* out, int general, void* stream) {
   if (n_seqs <= 0) return 0;
-  if (dim <= 0 || dim > 512 || vdim <= 0 || heads <= 0 || n_seqs > 65535 || heads > 65535) {
-    set_last_error("lightning: %d heads of %d (at most 512) x %d, %d sequences", heads, dim, vdim, n_seqs);
-    return -1;
-  }
   LightningParams p = {};
   p.sv.q_start = q_start; p.sv.q_len = q_len; p.sv.ctx_lens = ctx_lens; p.sv.slots = slots; p.sv.n = n_seqs;
   p.q = q; p.k = k; p.v = v; p.ld = ld; p.heads = heads; p.dim = dim; p.vdim = vdim;
   p.forget = forget; p.powers = powers; p.state = state; p.out = out;
-  auto s = static_cast<cudaStream_t>(stream);
-  const size_t decode_smem = sizeof(float) * (2 * ((dim + 3) & ~3) + (vdim >= 4 ? 256 / (vdim / 4) * vdim : 0));
-  if (!general && !q_start && vdim % 4 == 0 && vdim <= 1024 && ld % 4 == 0 && decode_smem <= 48 * 1024 && li_al16(state) &&
-      li_al16(out) && (reinterpret_cast<uintptr_t>(v) & (is_f32 ? 15 : 7)) == 0) {
-    const dim3 grid(heads, n_seqs);
-    return li_done(is_f32 ? launch_kernel(lightning_decode_kernel<float>, grid, dim3(256), decode_smem, s, true, 0, p)
-                          : launch_kernel(lightning_decode_kernel<bf16_t>, grid, dim3(256), decode_smem, s, true, 0, p), "decode");
+  return li_run<false>(p, is_f32, general, static_cast<cudaStream_t>(stream));
+}
+
+// State-space duality: C, B [rows, groups * N] and x [rows, heads * P] share the row pitch ld; dt [rows, >= heads] with pitch ldt;
+// dt_bias, neg_a (= -exp(A_log)), skip [heads] fp32; state [slots, heads, N, P] fp32, out [rows, heads * P] fp32.
+GLLM_API int gllm_ssd(const int* q_start, const int* q_len, const int* ctx_lens, const int* slots, int n_seqs, const void* C,
+                      const void* B, const void* x, long long ld, const void* dt, long long ldt, int is_f32, int heads, int groups,
+                      int N, int P, const float* dt_bias, const float* neg_a, const float* skip, float* state, float* out, int general,
+                      void* stream) {
+  if (n_seqs <= 0) return 0;
+  if (groups <= 0 || heads % groups != 0) {
+    set_last_error("ssd: %d heads in %d groups", heads, groups);
+    return -1;
   }
-  if (!general && q_start && !is_f32 && dim % 16 == 0 && dim <= 2 * kLiSlice && vdim % 8 == 0 && ld % 8 == 0 && li_al16(q) &&
-      li_al16(k) && li_al16(v))
-    return dim <= kLiSlice ? li_chunks<1, 2>(p, s) : li_chunks<2, 1>(p, s);
-  const dim3 grid((vdim + kLsCols - 1) / kLsCols, heads, n_seqs);
-  const size_t smem = sizeof(float) * 2 * kLsTok * dim;
-  const int rows = (dim + kLsG - 1) / kLsG;
-#define LI_STEP(T, R) \
-  return li_done(launch_kernel(lightning_step_kernel<T, R>, grid, dim3(kLsCols * kLsG), smem, s, true, 0, p), "steps")
-  if (is_f32) {
-    if (rows <= 8) LI_STEP(float, 8);
-    if (rows <= 16) LI_STEP(float, 16);
-    LI_STEP(float, 64);
-  }
-  if (rows <= 8) LI_STEP(bf16_t, 8);
-  if (rows <= 16) LI_STEP(bf16_t, 16);
-  LI_STEP(bf16_t, 64);
-#undef LI_STEP
+  LightningParams p = {};
+  p.sv.q_start = q_start; p.sv.q_len = q_len; p.sv.ctx_lens = ctx_lens; p.sv.slots = slots; p.sv.n = n_seqs;
+  p.q = C; p.k = B; p.v = x; p.ld = ld; p.heads = heads; p.dim = N; p.vdim = P;
+  p.dt = dt; p.ldt = ldt; p.dt_bias = dt_bias; p.neg_a = neg_a; p.skip = skip; p.group = heads / groups;
+  p.state = state; p.out = out;
+  return li_run<true>(p, is_f32, general, static_cast<cudaStream_t>(stream));
 }
 
 // o [rows, n] fp32, g [rows, >= n] with pitch ldg, out [rows, n] in g's type.

@@ -2,7 +2,8 @@
 //
 //   conv_qkv_prep    causal convolution over time on the projected q, k and v -> RMS norm of each q / k head -> RoPE on the
 //                    first dimensions of q and k -> q buffer, K page, V page; the last projected values enter the ring
-//                    of the sequence's slot. One pass: a warp owns one head's channels over a tile of tokens.
+//                    of the sequence's slot. One pass: a warp owns one head's channels over a tile of tokens. Options: values
+//                    divided by their own root mean square, queries times a factor that grows with the position.
 //   latent_prep      RMS norm of the query latent (operand of the query up-projection) and of the key / value latent
 //                    (written to its page), one warp per token and part.
 //   latent_rope_prep the same for latent layers with a rotated key part and directly projected queries: latent norm and
@@ -25,6 +26,9 @@ struct ConvPrepParams {
   const float* conv;         // [channels, taps] (taps 0: no convolution)
   const float *q_w, *k_w;    // [D] or null
   float eps;
+  int v_norm;                // values are divided by their root mean square
+  float temp_coef;           // queries: times 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1) (temp_every 0: no factor)
+  int temp_every;
   const int *positions, *slot_mapping;
   const float *cos_t, *sin_t;
   int max_pos;
@@ -35,6 +39,10 @@ struct ConvPrepParams {
 };
 
 constexpr int kPrepWarps = 4;
+
+__device__ __forceinline__ float query_temperature(const ConvPrepParams& p, int pos) {
+  return fmaf(p.temp_coef, logf(static_cast<float>((pos + 1) / p.temp_every + 1)), 1.f);
+}
 
 // VEC consecutive elements per lane and step, N steps; TAPS -1: any number (0: none), weights re-read per token.
 template <typename T, int VEC, int N, int TAPS>
@@ -58,6 +66,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32) conv_qkv_prep_kernel(const Co
   const int taps = TAPS >= 0 ? TAPS : p.taps;
   float* stage = prep_smem + warp * max(p.D, p.DV);
   const float* norm_w = kind == 0 ? p.q_w : kind == 1 ? p.k_w : nullptr;
+  const bool scaled = kind == 2 ? p.v_norm != 0 : kind == 0 && p.temp_every > 0;      // a factor without a weight
   const int rot = kind == 2 ? 0 : p.rot_dim, half = rot / 2;
   auto el = [&](int j) { return (j * 32 + lane) * VEC; };
   auto load = [&](const T* row, int j, float (&v)[VEC]) {
@@ -137,13 +146,14 @@ __global__ void __launch_bounds__(kPrepWarps * 32) conv_qkv_prep_kernel(const Co
         ss += a * a;
       }
     }
-    if (norm_w) {
-      const float r = 1.f / sqrtf(warp_sum(ss) / D + p.eps);
+    if (norm_w || scaled) {
+      float r = norm_w || kind == 2 ? 1.f / sqrtf(warp_sum(ss) / D + p.eps) : 1.f;
+      if (kind == 0 && p.temp_every > 0) r *= query_temperature(p, p.positions[m]);
 #pragma unroll
       for (int j = 0; j < N; ++j)
         if (el(j) < D)
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) y[j * VEC + e] *= r * norm_w[el(j) + e];
+          for (int e = 0; e < VEC; ++e) y[j * VEC + e] *= norm_w ? r * norm_w[el(j) + e] : r;
     }
     if (rot > 0) {
       int pos = p.positions[m];
@@ -206,31 +216,6 @@ __global__ void __launch_bounds__(kPrepWarps * 32) conv_qkv_prep_kernel(const Co
 
 // The same for heads of 32, 64, 128 or 256 channels (keys and values alike), up to four taps, rotary halves of whole 8-channel
 // groups: a lane owns 8 consecutive channels of one head, 32 / LPH heads share a warp, the rotary partner is a shuffle away.
-template <typename T> __device__ __forceinline__ void load8(const T* p, float (&v)[8]) {
-  if constexpr (sizeof(T) == 2) {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
-    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      v[2 * i] = __uint_as_float(w[i] << 16);
-      v[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
-    }
-  } else {
-    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-  }
-}
-template <typename T> __device__ __forceinline__ void store8(T* p, const float (&v)[8]) {
-  if constexpr (sizeof(T) == 2) {
-    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
-                                              pack_bf16x2(v[6], v[7]));
-  } else {
-    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
-  }
-}
-
 template <typename T, int LPH, int TAPS>
 __global__ void __launch_bounds__(kPrepWarps * 32) conv_qkv_prep8_kernel(const ConvPrepParams p) {
   constexpr int D = LPH * 8, HPW = 32 / LPH, H = TAPS > 1 ? TAPS - 1 : 1;
@@ -282,6 +267,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32) conv_qkv_prep8_kernel(const C
 #pragma unroll
     for (int e = 0; e < 8; ++e) g[e] = 1.f;
   }
+  const bool v_norm = kind == 2 && p.v_norm, temp = kind == 0 && p.temp_every > 0;
   const int half = p.rot_dim / 2, hl = half / 8;
   const bool rot = kind != 2 && d0 < p.rot_dim, upper = d0 >= half;
   const int partner = rot ? (upper ? lane - hl : lane + hl) : lane, fi = upper ? d0 - half : d0;
@@ -309,8 +295,9 @@ __global__ void __launch_bounds__(kPrepWarps * 32) conv_qkv_prep8_kernel(const C
     for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
 #pragma unroll
     for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if (norm_w) {
-      const float r = 1.f / sqrtf(ss * (1.f / D) + p.eps);
+    if (norm_w || v_norm || temp) {
+      float r = norm_w || v_norm ? 1.f / sqrtf(ss * (1.f / D) + p.eps) : 1.f;
+      if (temp) r *= query_temperature(p, p.positions[m]);
 #pragma unroll
       for (int e = 0; e < 8; ++e) y[e] *= r * g[e];
     }
@@ -597,11 +584,11 @@ static int prep_done(cudaError_t e, const char* name) {
 GLLM_API int gllm_conv_qkv_prep(const int* q_start, const int* q_len, const int* ctx_lens, const int* slots, int n_seqs,
                                 int max_q_len, const void* proj, long long ld, int is_f32, int n_q, int n_kv, int D, int DV,
                                 int rot_dim, int taps, const float* conv, const float* q_w, const float* k_w, float eps,
-                                const int* positions, const int* slot_mapping, const float* cos_t, const float* sin_t,
+                                int v_norm, float temp_coef, int temp_every, const int* positions, const int* slot_mapping, const float* cos_t, const float* sin_t,
                                 int max_pos, float* ring, void* q_out, void* kv, int num_pages, void* stream) {
   if (n_seqs <= 0 || max_q_len <= 0) return 0;
   if (D <= 0 || DV <= 0 || D > 1024 || DV > 1024 || rot_dim > D || (rot_dim & 1) || (rot_dim > 0 && (!cos_t || !sin_t)) ||
-      taps < 0 || (taps > 0 && !conv) || (taps > 1 && !ring) || n_seqs > 65535) {
+      taps < 0 || (taps > 0 && !conv) || (taps > 1 && !ring) || n_seqs > 65535 || temp_every < 0) {
     set_last_error("conv_qkv_prep: sizes %d / %d, rot_dim %d, taps %d, %d sequences", D, DV, rot_dim, taps, n_seqs);
     return -1;
   }
@@ -612,6 +599,7 @@ GLLM_API int gllm_conv_qkv_prep(const int* q_start, const int* q_len, const int*
   p.tile = rows >= 1024 ? 32 : rows >= 128 ? 16 : 8;
   if (p.tile < taps - 1) p.tile = taps - 1;
   p.conv = conv; p.q_w = q_w; p.k_w = k_w; p.eps = eps; p.positions = positions; p.slot_mapping = slot_mapping;
+  p.v_norm = v_norm; p.temp_coef = temp_coef; p.temp_every = temp_every;
   p.cos_t = cos_t; p.sin_t = sin_t; p.max_pos = max_pos; p.ring = ring; p.q_out = q_out; p.kv = kv;
   p.num_pages = num_pages; p.err = gllm_error_word();
   dim3 grid((n_q + 2 * n_kv + kPrepWarps - 1) / kPrepWarps, (rows + p.tile - 1) / p.tile, n_seqs);

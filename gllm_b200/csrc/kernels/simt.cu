@@ -87,11 +87,12 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TI* A, long long l
 }
 
 // ---------------------------------------------------------------------------------------------
-// Embedding rows: x[m] = table[ids[m]] * scale in fp32 (the residual stream), xb[m] the unscaled row in the compute type.
+// Embedding rows: x[m] = table[ids[m]] * scale in fp32 (the residual stream, or `streams` equal ones side by side), xb[m] the
+// unscaled row in the compute type.
 // ---------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(128) embed_rows_kernel(const int* ids, const T* table, int vocab, int hidden, float scale,
-                                                         float* x, T* xb, int* err) {
+                                                         int streams, float* x, T* xb, int* err) {
   const long long m = blockIdx.x;
   int id = ids[m];
   if (id < 0 || id >= vocab) {
@@ -101,7 +102,7 @@ __global__ void __launch_bounds__(128) embed_rows_kernel(const int* ids, const T
   const T* src = table + static_cast<long long>(id) * hidden;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     const T v = src[i];
-    x[m * hidden + i] = to_f(v) * scale;
+    for (int s = 0; s < streams; ++s) x[(m * streams + s) * hidden + i] = to_f(v) * scale;
     if (xb) xb[m * hidden + i] = v;
   }
 }
@@ -320,22 +321,22 @@ GLLM_API int gllm_gemm_simt(const void* A, long long lda, const void* B, long lo
   return gemm_simt(A, lda, B, ldb, C, ldc, M, N, K, in_f32, out_f32, bias, softcap, act, act_cols, nullptr, nullptr, stream);
 }
 
-// Grouped form: groups [M / 128] int32, block_rows [M / 128] int32 or null.
+// Grouped form: groups [M / 128] int32, block_rows [M / 128] int32 or null, act on every column.
 GLLM_API int gllm_gemm_simt_grouped(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M,
-                                    int N, int K, int in_f32, int out_f32, const int* groups, const int* block_rows,
+                                    int N, int K, int in_f32, int out_f32, const int* groups, const int* block_rows, int act,
                                     void* stream) {
-  return gemm_simt(A, lda, B, ldb, C, ldc, M, N, K, in_f32, out_f32, nullptr, 0.f, 0, 0, groups, block_rows, stream);
+  return gemm_simt(A, lda, B, ldb, C, ldc, M, N, K, in_f32, out_f32, nullptr, 0.f, act, act ? N : 0, groups, block_rows, stream);
 }
 
-GLLM_API int gllm_embed_rows(const int* ids, const void* table, int vocab, int hidden, int is_f32, float scale, float* x, void* xb,
-                             int M, void* stream) {
+GLLM_API int gllm_embed_rows(const int* ids, const void* table, int vocab, int hidden, int is_f32, float scale, int streams,
+                             float* x, void* xb, int M, void* stream) {
   if (M <= 0) return 0;
   auto s = static_cast<cudaStream_t>(stream);
   if (is_f32)
-    embed_rows_kernel<float><<<M, 128, 0, s>>>(ids, static_cast<const float*>(table), vocab, hidden, scale, x,
+    embed_rows_kernel<float><<<M, 128, 0, s>>>(ids, static_cast<const float*>(table), vocab, hidden, scale, streams, x,
                                                static_cast<float*>(xb), gllm_error_word());
   else
-    embed_rows_kernel<bf16_t><<<M, 128, 0, s>>>(ids, static_cast<const bf16_t*>(table), vocab, hidden, scale, x,
+    embed_rows_kernel<bf16_t><<<M, 128, 0, s>>>(ids, static_cast<const bf16_t*>(table), vocab, hidden, scale, streams, x,
                                                 static_cast<bf16_t*>(xb), gllm_error_word());
   SIMT_CHECK("embed_rows");
 }

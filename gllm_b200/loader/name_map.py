@@ -51,6 +51,7 @@ class TensorRole(str, Enum):
     MOE_SHARED_DOWN = "moe_shared_down"
     MIXER = "mixer"                # tensor of a token mixer (heterogeneous models: models/hybrid.py)
     MIXER_NORM = "mixer_norm"
+    STREAM_WEIGHTS = "stream_weights"   # hyper-connections: weights into, out of and between the residual streams
     LOOP_STEP = "loop_step"        # vector added to the residual stream before each pass of a looped range of layers
     CLASSIFIER = "classifier"
     POOLER = "pooler"
@@ -111,11 +112,12 @@ _GLOBAL_RULES = [
 _GLOBAL_RULES = [(re.compile(p), c, r) for p, c, r in _GLOBAL_RULES]
 
 # Heterogeneous models: ``l<i>.mix.<name>``, ``l<i>.mlp.<name>`` (``mlp.e<j>.<name>``, ``mlp.shared.<name>``, ``mlp.router`` with experts),
-# ``l<i>.norm1|2`` (and ``norm1b|2b`` behind the sublayers), ``embed``, ``head``, ``final.norm``, ``loop.step``
-_HYBRID_LAYER = re.compile(r"^l(\d+)\.(mix\.[\w.]+|mlp\.(?:gate|up|down|router)|mlp\.(?:e\d+|shared)\.(?:gate|up|down)|mlp\.shared\.sg|norm[12]b?)$")
+# ``l<i>.norm1|2`` (and ``norm1b|2b`` behind the sublayers), ``l<i>.hc1|2.in|out|mix``, ``embed``, ``head``, ``final.norm``, ``loop.step``
+_HYBRID_LAYER = re.compile(r"^l(\d+)\.(mix\.[\w.]+|mlp\.(?:gate|up|down|router|correction)|mlp\.(?:e\d+|shared)\.(?:gate|up|down)|mlp\.shared\.sg|norm[12]b?|hc[12]\.(?:in|out|mix))$")
 _HYBRID_GLOBAL = {"embed": ("embed_tokens", TensorRole.EMBEDDING), "head": ("lm_head", TensorRole.OUTPUT_HEAD),
                   "final.norm": ("final_norm", TensorRole.FINAL_NORM), "loop.step": ("loop_step", TensorRole.LOOP_STEP)}
-_HYBRID_MLP = {"gate": TensorRole.FFN_GATE, "up": TensorRole.FFN_UP, "down": TensorRole.FFN_DOWN, "router": TensorRole.MOE_ROUTER}
+_HYBRID_MLP = {"gate": TensorRole.FFN_GATE, "up": TensorRole.FFN_UP, "down": TensorRole.FFN_DOWN, "router": TensorRole.MOE_ROUTER,
+               "correction": TensorRole.MOE_ROUTER_BIAS}
 _HYBRID_EXPERT = {"gate": TensorRole.MOE_EXPERT_GATE, "up": TensorRole.MOE_EXPERT_UP, "down": TensorRole.MOE_EXPERT_DOWN}
 _HYBRID_SHARED = {"gate": TensorRole.MOE_SHARED_GATE, "up": TensorRole.MOE_SHARED_UP, "down": TensorRole.MOE_SHARED_DOWN,
                   "sg": TensorRole.MOE_ROUTER}
@@ -148,6 +150,7 @@ def match_tensor_role(name: str) -> Tuple[TensorRole, Optional[int], Optional[st
     if m:
         rest = m.group(2)
         role = TensorRole.MIXER if rest.startswith("mix.") else TensorRole.MIXER_NORM if rest.startswith("norm") else \
+            TensorRole.STREAM_WEIGHTS if rest.startswith("hc") else \
             (_HYBRID_SHARED if rest.startswith("mlp.shared.") else _HYBRID_EXPERT if rest.count(".") == 2 else
              _HYBRID_MLP)[rest.rsplit(".", 1)[1]]
         return role, int(m.group(1)), f"L{m.group(1)}.{rest}", ""

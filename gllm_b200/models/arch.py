@@ -22,7 +22,7 @@ ARCH_ALIASES = {
     "gpt_oss": "gpt_oss", "gptoss": "gpt_oss", "gpt-oss": "gpt_oss", "mixtral": "mixtral",
     "bert": "bert", "xlm-roberta": "bert", "xlmr": "bert", "roberta": "bert", "bge": "bert", "e5": "bert",
     "modernbert": "modernbert", "siglip": "siglip", "usm": "usm", "gpt2": "gpt2",
-    "zenevik": "zenevik", "gorulorn": "gorulorn", "ritirax": "ritirax",
+    "zenevik": "zenevik", "gorulorn": "gorulorn", "ritirax": "ritirax", "tomopel": "tomopel",
 }
 
 

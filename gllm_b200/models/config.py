@@ -52,7 +52,9 @@ class MixerSpec:
                ``qkv_bias`` / ``o_bias`` = the projections have biases; ``softcap`` > 0: scores are cap * tanh(score / cap);
                ``bias_max`` > 0 = a learned bias per head and distance is added to the (capped) scores, from a table of
                ``bias_rows`` rows (0: taken from the weight) that ends at that distance (``ops.distance_rows``);
-               ``sink`` = a learned extra logit per head in the softmax denominator.
+               ``sink`` = a learned extra logit per head in the softmax denominator; ``v_norm`` = each value head is divided by its
+               root mean square; ``q_temp`` = (coef, every): queries are multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at
+               position p; ``head_gate`` = each head's output is multiplied by sigmoid of one number projected from the token.
     latent:    attention over a shared latent of ``kv_rank`` channels per token: ``heads`` heads of ``dim`` query / key and
                ``vdim`` value dimensions, queries of rank ``q_rank`` (0: projected directly), sliding ``window``, ``sink`` as
                above; ``rope_part`` > 0 = that many further query / key dimensions per head, the key part shared by all heads,
@@ -63,7 +65,13 @@ class MixerSpec:
     gla:       gated linear attention, ``heads`` x (``dim`` key, ``vdim`` value) channels, decay sigmoid(z)^(1 / tau)
                with z of rank ``decay_rank`` (0: taken from the weight).
     lightning: linear attention with a fixed decay per head (``decay``), ``heads`` x (``dim`` key, ``vdim`` value) channels,
-               silu on q, k and v, one RMS norm over all heads and the gate sigmoid(W_g h) in front of the output."""
+               silu on q, k and v, one RMS norm over all heads and the gate sigmoid(W_g h) in front of the output.
+    ssd:       state-space duality (Mamba-2): ``heads`` x (``dim`` state, ``vdim`` value) channels, input and output maps shared by the
+               heads of each of ``groups`` groups, decay and step size per token and head, a convolution of ``taps`` taps with silu in
+               front; its output times silu(z) is normed in ``norm_groups`` equal parts.
+    mingru:    gated recurrence over ``width`` channels whose gates read only the current token.
+    parallel:  ``left`` and ``right`` side by side over the same input, left_scale * left + right_scale * right (``left``: attention,
+               ``right``: ssd)."""
     kind: str = "attention"
     heads: int = 0
     kv_heads: int = 0
@@ -95,10 +103,29 @@ class MixerSpec:
     rot_scaling: RopeScaling = field(default_factory=RopeScaling)
     gate: bool = False
     decay: tuple = ()
+    v_norm: bool = False
+    q_temp: tuple = ()
+    head_gate: bool = False
+    groups: int = 1
+    norm_groups: int = 1
+    left: Optional["MixerSpec"] = None
+    right: Optional["MixerSpec"] = None
+    left_scale: float = 1.0
+    right_scale: float = 1.0
 
     @property
     def value_dim(self) -> int:
         return self.vdim or self.dim
+
+    @property
+    def parts(self) -> tuple:
+        """The mixers this one consists of (itself unless it sets two side by side)."""
+        return (self.left, self.right) if self.kind == "parallel" else (self,)
+
+    @property
+    def conv_channels(self) -> int:
+        """Channels of an ssd layer's convolution: values, input maps, output maps."""
+        return self.heads * self.vdim + 2 * self.groups * self.dim
 
     def state_floats(self) -> int:
         """fp32 words of recurrent state per sequence."""
@@ -108,19 +135,28 @@ class MixerSpec:
             return self.width * (self.taps + 1)
         if self.kind in ("gla", "lightning"):
             return self.heads * self.dim * self.vdim
+        if self.kind == "ssd":
+            return self.heads * self.dim * self.vdim + self.taps * self.conv_channels
+        if self.kind == "mingru":
+            return self.width
+        if self.kind == "parallel":
+            return sum(m.state_floats() for m in self.parts)
         return 0
 
     def kv_elems(self) -> int:
         """KV cache elements per token."""
         if self.kind == "latent":
             return self.kv_rank + self.rope_part
+        if self.kind == "parallel":
+            return sum(m.kv_elems() for m in self.parts)
         return self.kv_heads * (self.dim + self.value_dim) if self.kind == "attention" else 0
 
 
 @dataclass
 class MoeSpec:
-    """Mixture-of-experts feed-forward of one layer: ``top`` of ``experts`` gated feed-forwards of intermediate size ``ff``.
-    ``scoring``: sigmoid or softmax over the router logits; ``norm_topk``: the chosen scores are renormalised to sum 1;
+    """Mixture-of-experts feed-forward of one layer: ``top`` of ``experts`` feed-forwards of intermediate size ``ff``, W_down(act(W_gate
+    h) * W_up h) or, not ``gated``, W_down act(W_up h). ``scoring``: sigmoid or softmax over the router logits; ``correction``: a learned
+    number per expert joins the scores for the choice only; ``norm_topk``: the chosen scores are renormalised to sum 1;
     ``scale_input``: the score multiplies the expert's input instead of its output; ``scale``: factor of the weights.
     ``groups`` > 0: only experts of the ``keep_groups`` groups (neighbours, equal sizes) with the largest best score are
     chosen. ``shared_ff`` > 0: one more feed-forward of that size runs for every token, multiplied by a sigmoid gate of the
@@ -136,6 +172,8 @@ class MoeSpec:
     keep_groups: int = 0
     shared_ff: int = 0
     shared_gate: bool = False
+    gated: bool = True
+    correction: bool = False
 
 
 @dataclass
@@ -189,13 +227,17 @@ class ModelConfig:
     post_norm: bool = False  # encoder-style post-LN residual blocks
     # Heterogeneous decoders (models/hybrid.py): one spec per layer. ``block``: "post" = post-norm blocks
     # x = norm(postln_alpha * x + f(x)), "sandwich" = x = x + norm_b(f(norm_a(x))), "parallel" = h = norm(x),
-    # x = x + (mixer(h) + ff(h)); ``norm_type`` rms or layer (no bias), ``norm_one_plus_w``: weights enter as 1 + w.
+    # x = x + (mixer(h) + ff(h)), "pre" = x = x + residual_mult * f(norm(x)); ``norm_type`` rms or layer (no bias),
+    # ``norm_one_plus_w``: weights enter as 1 + w. ``streams`` > 0 (pre-norm blocks): hyper-connections, that many residual streams
+    # with learned weights into, out of and between the streams at every sublayer.
     # ``loop`` = (start, stop, times): that range of layers runs ``times`` times in a row with the same weights, a learned
     # vector added to the stream before each pass; every pass has its own cache and state.
     layer_specs: Optional[List[LayerSpec]] = None
     postln_alpha: float = 1.0
     block: str = "post"
     loop: Optional[tuple] = None
+    residual_mult: float = 1.0
+    streams: int = 0
     causal: bool = True
     # MoE
     num_experts: int = 0
@@ -333,21 +375,29 @@ class ModelConfig:
         h, L = self.hidden_size, self.num_layers
         if self.is_hybrid:
             total = 2 * self.vocab_size * h
-            for l in self.layer_specs:
-                m = l.mixer
+            for l, m in [(l, m) for l in self.layer_specs for m in l.mixer.parts]:
                 if m.kind == "attention":
-                    total += h * ((m.heads + m.kv_heads) * m.dim + (m.heads + (0 if m.v_from_k else m.kv_heads)) * m.value_dim)
+                    total += h * ((m.heads + m.kv_heads) * m.dim + (m.heads + (0 if m.v_from_k else m.kv_heads)) * m.value_dim
+                                  + (m.heads if m.head_gate else 0))
                 elif m.kind == "latent":
                     qd = m.heads * (m.dim + m.rope_part)
                     total += h * (m.q_rank + m.kv_rank + m.rope_part + m.heads * m.vdim * (2 if m.gate else 1)) + (
                         (m.q_rank or h) * qd + m.heads * m.kv_rank * (m.dim + m.vdim))
                 elif m.kind == "rglru":
                     total += 3 * h * m.width + 2 * m.width * m.width // m.blocks
+                elif m.kind == "mingru":
+                    total += 4 * h * m.width
+                elif m.kind == "ssd":
+                    total += h * (2 * m.heads * m.vdim + m.conv_channels + m.heads) + m.taps * m.conv_channels
                 else:
                     total += h * m.heads * (2 * m.dim + 3 * m.vdim) + m.decay_rank * (h + m.heads * m.dim)
+            for l in self.layer_specs:
                 total += (3 if l.gated else 2) * h * l.ff
                 if l.moe:
-                    total += h * (l.moe.experts * (3 * l.moe.ff + 1) + 3 * l.moe.shared_ff + l.moe.shared_gate)
+                    n = 3 if l.moe.gated else 2
+                    total += h * (l.moe.experts * (n * l.moe.ff + 1) + n * l.moe.shared_ff + l.moe.shared_gate)
+                if self.streams:
+                    total += self.streams * self.streams * (2 if l.ff or l.moe else 1)
             return total
         attn = h * (self.q_size + 2 * self.kv_size) + self.q_size * h
         if self.is_mla:
@@ -388,6 +438,8 @@ class ModelConfig:
             return ModelConfig.from_gorulorn_dict(d)
         if d.get("architecture") == "Ritirax":
             return ModelConfig.from_ritirax_dict(d)
+        if d.get("architecture") == "Tomopel":
+            return ModelConfig.from_tomopel_dict(d)
         tc = d.get("text_config") or d
         arch = (d.get("model_type") or tc.get("model_type") or "llama").lower()
         g = lambda *keys, default=None: next((tc[k] for k in keys if k in tc and tc[k] is not None), default)
@@ -583,10 +635,54 @@ class ModelConfig:
         cfg.set_hybrid_dims()
         return cfg
 
+    @staticmethod
+    def from_tomopel_dict(d: Dict[str, Any]) -> "ModelConfig":
+        """Tomopel ``config.json``: pre-norm layers over hyper-connected residual streams; mixers are a minGRU, or attention (distance
+        biases, query temperature, normed values, a gate per head) and a state-space layer side by side; feed-forwards are dense, or
+        squared-ReLU experts beside a shared one."""
+        specs = []
+        for i, l in enumerate(d["layers"]):
+            m, kind, mlp = l["mixer"], l["type"], l.get("mlp")
+            if kind == "mingru":
+                mixer = MixerSpec("mingru", width=int(m["width"]))
+            elif kind == "parallel":
+                a, r = m["left"], m["right"]
+                temp = a.get("q_temp") or {}
+                left = MixerSpec("attention", heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), dim=int(a["dim"]),
+                                 vdim=int(a["vdim"]), scale=float(a["scale"]), bias_max=int(a["bias_max"]), head_qk_norm=True,
+                                 qkv_bias=False, o_bias=False, v_norm=True, head_gate=True,
+                                 q_temp=(float(temp["coef"]), int(temp["every"])) if temp else ())
+                right = MixerSpec("ssd", heads=int(r["heads"]), vdim=int(r["vdim"]), dim=int(r["state"]),
+                                  groups=int(r.get("groups") or 1), taps=int(r["conv"]), norm_groups=int(r.get("norm_groups") or 1))
+                if right.heads % right.groups or right.heads * right.vdim % right.norm_groups or left.heads % left.kv_heads:
+                    raise ValueError(f"layer {i}: {right.heads} heads of {right.vdim} in {right.groups} groups, {right.norm_groups} parts "
+                                     f"of the norm, {left.heads} query heads on {left.kv_heads}: nothing may be left over")
+                mixer = MixerSpec("parallel", left=left, right=right, left_scale=float(m["left_scale"]),
+                                  right_scale=float(m["right_scale"]))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            spec = LayerSpec(mixer, act="silu")
+            if mlp is not None and mlp["kind"] == "dense":
+                spec.ff = int(mlp["ff"])
+            elif mlp is not None and mlp["kind"] == "moe":
+                spec.act = "relu2"
+                spec.moe = MoeSpec(experts=int(mlp["router"]["experts"]), top=int(mlp["router"]["top"]), ff=int(mlp["expert"]["ff"]),
+                                   gated=False, correction=True, shared_ff=int((mlp.get("shared") or {}).get("ff") or 0))
+            elif mlp is not None:
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            specs.append(spec)
+        cfg = ModelConfig(arch="tomopel", hidden_size=int(d["width"]), num_layers=len(specs), vocab_size=int(d["vocab"]),
+                          rms_norm_eps=float(d["norm"]["eps"]), norm_one_plus_w=True, block="pre", hidden_act="silu",
+                          embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
+                          residual_mult=float(d.get("residual_mult", 1.0)), streams=int(d.get("streams") or 0),
+                          max_position_embeddings=int(d.get("max_positions", 1 << 20)), layer_specs=specs)
+        cfg.set_hybrid_dims()
+        return cfg
+
     def set_hybrid_dims(self):
         """The scalar head / feed-forward sizes of a heterogeneous model: the largest over its layers (they size shared
         buffers; the layers use their specs). ``head_dim`` is 128 when any layer can use the head_dim-128 kernels."""
-        att = [l.mixer for l in self.layer_specs if l.mixer.kind == "attention"]
+        att = [m for l in self.layer_specs for m in l.mixer.parts if m.kind == "attention"]
         self.num_heads = max([m.heads for m in att], default=1)
         self.num_kv_heads = max([m.kv_heads for m in att], default=1)
         dims = [m.dim for m in att if m.value_dim == m.dim] or [64]
@@ -727,6 +823,20 @@ def preset(name: str) -> ModelConfig:
                           block="parallel", hidden_act="silu", embedding_scale=16.0, max_position_embeddings=2048,
                           layer_specs=[LayerSpec(att, ff=384, act="relu2", gated=False), LayerSpec(lat, act="silu", moe=moe),
                                        LayerSpec(lig, act="silu", moe=moe)], eos_token_ids=[2])
+        cfg.set_hybrid_dims()
+        return cfg
+    if n in ("tiny-tomopel",):
+        att = MixerSpec("attention", heads=4, kv_heads=2, dim=128, vdim=128, scale=0.09, head_qk_norm=True, qkv_bias=False, o_bias=False,
+                        bias_max=90, bias_rows=20, v_norm=True, q_temp=(0.3, 48), head_gate=True)
+        ssd = MixerSpec("ssd", heads=6, vdim=64, dim=32, groups=2, taps=4, norm_groups=3)
+        both = MixerSpec("parallel", left=att, right=ssd, left_scale=0.8, right_scale=1.1)
+        gru = MixerSpec("mingru", width=320)
+        moe = MoeSpec(experts=12, top=3, ff=96, gated=False, correction=True, shared_ff=128)
+        cfg = ModelConfig(arch="tomopel", hidden_size=256, num_layers=3, vocab_size=1024, rms_norm_eps=1e-6, norm_one_plus_w=True,
+                          block="pre", streams=3, residual_mult=0.9, hidden_act="silu", embedding_scale=16.0,
+                          max_position_embeddings=2048, eos_token_ids=[2],
+                          layer_specs=[LayerSpec(both, ff=384, act="silu"), LayerSpec(gru, act="relu2", moe=moe),
+                                       LayerSpec(both, act="relu2", moe=moe)])
         cfg.set_hybrid_dims()
         return cfg
     if n in ("tiny-bert",):

@@ -1,12 +1,17 @@
 """Heterogeneous decoders: every layer has its own token mixer (``models/mixers.py``) and an optional feed-forward
-(``models/moe.py``: gated, plain, or a mixture of experts), over a residual stream kept in fp32. Three kinds of block:
+(``models/moe.py``: gated, plain, or a mixture of experts), over a residual stream kept in fp32. Four kinds of block:
 
+    pre       x = x + mult * mixer(norm1(x));          x = x + mult * ff(norm2(x))
     post      x = norm1(alpha * x + mixer(x));         x = norm2(alpha * x + ff(x))
     sandwich  x = x + norm1b(mixer(norm1(x)));         x = x + norm2b(ff(norm2(x)))
     parallel  h = norm1(x);                            x = x + (mixer(h) + ff(h))
 
 A range of layers may run several times in a row with the same weights; a learned vector joins the stream before each pass,
 and each pass has its own cache and state (``ModelConfig.layer_runs``: "run" below is one execution of a layer).
+
+Pre-norm blocks may keep several residual streams per token (hyper-connections; Zhu et al., "Hyper-Connections"): a sublayer reads
+a weighted sum of them and its output joins each with a weight, while the streams are mixed with one another. What the outside sees as
+the stream (callbacks, captures, hidden states) is then their sum.
 
 The model plugs into the engine like ``DecoderModel``: same ``ForwardBatch``, paged KV cache for its attention layers, and
 recurrent state in the batcher's sequence slots (``kv_cache/recurrent_state.py``) for the others. The workspace holds the
@@ -26,7 +31,7 @@ import torch
 from ..engine.batch import ForwardBatch
 from ..ops import linear as L
 from ..ops import recurrent as R
-from ..ops.residual import residual_norm
+from ..ops.residual import hyper_norm, residual_norm
 from .config import ModelConfig
 from .mixers import MIXERS, mixer_shapes, rope_table
 from .moe import ExpertFF, GatedFF, PlainFF
@@ -45,6 +50,10 @@ def tensor_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:
     H = cfg.hidden_size
     s = {"embed_tokens": (cfg.vocab_size, H), "lm_head": (cfg.vocab_size, H), "final_norm": (H,)}
     norms = ("", "b") if cfg.block == "sandwich" else ("",)
+    def streams(p, sub):
+        if cfg.streams:
+            n = cfg.streams
+            s.update({f"{p}hc{sub}.in": (n,), f"{p}hc{sub}.out": (n,), f"{p}hc{sub}.mix": (n, n)})
     if cfg.loop:
         s["loop_step"] = (cfg.loop[2], H)
     for i, l in enumerate(cfg.layer_specs):
@@ -52,23 +61,40 @@ def tensor_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:
         s.update({f"{p}norm1{b}": (H,) for b in norms})
         for n, shape in mixer_shapes(l.mixer, H).items():
             s[f"{p}mix.{n}"] = shape
+        streams(p, 1)
         if (l.ff or l.moe) and cfg.block != "parallel":
             s.update({f"{p}norm2{b}": (H,) for b in norms})
+            streams(p, 2)
         gated = lambda q, ff: {q + "gate": (ff, H), q + "up": (ff, H), q + "down": (H, ff)}
         if l.ff:
             s.update(gated(p + "mlp.", l.ff))
             if not l.gated:
                 del s[p + "mlp.gate"]
         if l.moe:
+            expert = lambda q, ff: {k: v for k, v in gated(q, ff).items() if l.moe.gated or not k.endswith("gate")}
             if l.moe.shared_ff:
-                s.update(gated(p + "mlp.shared.", l.moe.shared_ff))
+                s.update(expert(p + "mlp.shared.", l.moe.shared_ff))
             if l.moe.shared_gate:
                 s[p + "mlp.shared.sg"] = (1, H)
             s[p + "mlp.router"] = (l.moe.experts, H)
+            if l.moe.correction:
+                s[p + "mlp.correction"] = (l.moe.experts,)
             for e in range(l.moe.experts):
-                s.update(gated(f"{p}mlp.e{e}.", l.moe.ff))
+                s.update(expert(f"{p}mlp.e{e}.", l.moe.ff))
     cfg.__dict__["_tensor_shapes"] = s
     return s
+
+
+class StreamWeights:
+    """Hyper-connection weights of one sublayer in fp32: ``read`` [S] into it, ``out`` [S] (times the residual factor) behind it, ``mix``
+    [S, S] (from, to). Without hyper-connections: one stream, all of them 1."""
+
+    def __init__(self, streams: int, get, mult: float, device):
+        if streams:
+            self.read, out, self.mix = (get(n).float().to(device).contiguous() for n in ("in", "out", "mix"))
+        else:
+            self.read, out, self.mix = (torch.ones(n, device=device) for n in ((1,), (1,), (1, 1)))
+        self.out = (out * mult).contiguous()
 
 
 @dataclass
@@ -81,6 +107,8 @@ class HybridLayer:
     experts: Optional[ExpertFF] = None
     norm1b: Optional[torch.Tensor] = None  # sandwich blocks: the norms behind the sublayers
     norm2b: Optional[torch.Tensor] = None
+    hc1: Optional[StreamWeights] = None    # pre-norm blocks
+    hc2: Optional[StreamWeights] = None
     kv_donor: Optional[int] = None
     extra: Dict[str, torch.Tensor] = field(default_factory=dict)
 
@@ -94,7 +122,7 @@ class HybridWorkspace:
     def __init__(self, model: "HybridDecoder", tokens: int):
         dev, dt, H = model.device, model.dtype, model.cfg.hidden_size
         self.max_tokens = tokens
-        self.x = torch.zeros((tokens, H), dtype=torch.float32, device=dev)
+        self.x = torch.zeros((tokens, H * model.streams), dtype=torch.float32, device=dev)
         self.xb = self.x if dt == torch.float32 and model.post else torch.zeros((tokens, H), dtype=dt, device=dev)
         need: Dict[str, int] = {}
         for l in model.layers:
@@ -142,13 +170,18 @@ class HybridDecoder:
             raise ValueError(f"not available for heterogeneous decoders: {', '.join(sorted(bad))}")
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError(f"compute dtype {dtype}: bfloat16 or float32")
-        self.post, self.parallel = cfg.block == "post", cfg.block == "parallel"
-        if cfg.block not in ("post", "sandwich", "parallel") or (self.post and (
+        self.post, self.parallel, self.pre = (cfg.block == b for b in ("post", "parallel", "pre"))
+        self.streams = max(cfg.streams, 1)
+        if (cfg.streams or cfg.residual_mult != 1.0) and not self.pre or self.pre and (
+                cfg.norm_type != "rms" or cfg.loop or any(l.moe and (l.moe.scale_input or l.moe.shared_gate) for l in cfg.layer_specs)):
+            raise ValueError("heterogeneous decoder: residual factors and several streams are built for pre-norm blocks, and these without "
+                             "loops, layer norms, weighted expert inputs and gated shared experts")
+        if cfg.block not in ("post", "sandwich", "parallel", "pre") or (self.post and (
                 cfg.norm_type != "rms" or cfg.loop or cfg.embedding_scale != 1.0 or any(l.moe for l in cfg.layer_specs))):
             raise ValueError("heterogeneous decoder: looped layers, layer norms, a scaled embedding and experts are not built for "
                              "post-norm blocks")
-        if any(l.moe and not l.moe.scale_input for l in cfg.layer_specs) and not self.parallel:
-            raise ValueError("heterogeneous decoder: weighted expert outputs are built for parallel blocks")
+        if any(l.moe and not l.moe.scale_input for l in cfg.layer_specs) and not (self.parallel or self.pre):
+            raise ValueError("heterogeneous decoder: weighted expert outputs are built for parallel and pre-norm blocks")
         self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
         self.layer_ids = list(range(cfg.num_layers))
         self.kv_dtype, self.kv_scale = dtype, 1.0
@@ -179,13 +212,18 @@ class HybridDecoder:
             if cfg.block == "sandwich":
                 lw.norm1b = norm(p + "norm1b")
                 lw.norm2b = norm(p + "norm2b") if spec.ff or spec.moe else None
+            if self.pre:
+                hc = lambda sub: StreamWeights(cfg.streams, lambda n: src.get(f"{p}hc{sub}.{n}"), cfg.residual_mult, dev)
+                lw.hc1 = hc(1)
+                lw.hc2 = hc(2) if lw.norm2 is not None else None
             if spec.ff and spec.gated:
                 lw.ff = GatedFF(to(p + "mlp.gate"), to(p + "mlp.up"), to(p + "mlp.down"), L.ACT_IDS[spec.act], dtype)
             elif spec.ff:
                 lw.ff = PlainFF(to(p + "mlp.up"), to(p + "mlp.down"), spec.act, dtype)
             if spec.moe:
-                lw.experts = ExpertFF(spec.moe, L.ACT_IDS[spec.act], src, p, cfg.hidden_size, dev, dtype)
+                lw.experts = ExpertFF(spec.moe, spec.act, src, p, cfg.hidden_size, dev, dtype)
             self.layers.append(lw)
+        self.sum_streams = torch.ones(self.streams, device=dev)
         self.runs = cfg.layer_runs()
         steps = f32("loop_step") if any(t is not None for _, t in self.runs) else None
         self.run_step = [None if t is None else steps[t] for _, t in self.runs]
@@ -205,6 +243,8 @@ class HybridDecoder:
     def weight_bytes(self) -> int:
         ts = [self.embed, self.lm_head, self.final_norm]
         for l in self.layers:
+            for hc in (l.hc1, l.hc2):
+                ts += [hc.read, hc.out, hc.mix] if hc is not None else []
             ts += [t for t in list(l.mixer.w.values()) + [l.norm1, l.norm2, l.norm1b, l.norm2b]
                    + (l.ff.tensors() if l.ff else []) + (l.experts.tensors() if l.experts else []) if t is not None]
         return sum(t.numel() * t.element_size() for t in ts)
@@ -235,22 +275,23 @@ class HybridDecoder:
         T = batch.num_tokens
         ws = self.workspace(T)
         ws.decode_ws = decode_ws
-        x, xb = ws.x[:T], ws.xb[:T]
+        x, xb = ws.x[:T], ws.xb[:T]              # x: [T, hidden], or all streams of a token side by side
         copy = xb if ws.xb is not ws.x and self.post else None
         self.mark("begin")
         if hidden_in is None:
-            R.embed_rows(batch.token_ids, self.embed, x, copy, scale=self.cfg.embedding_scale)
+            R.embed_rows(batch.token_ids, self.embed, x, copy, scale=self.cfg.embedding_scale, streams=self.streams)
             self.mark("embed")
         else:
-            x.copy_(hidden_in.float())
+            x.copy_(hidden_in.float().repeat(1, self.streams))
             if copy is not None:
                 copy.copy_(hidden_in)
         self.callback_action, self.callback_info = None, {}
         self.captured = {}
-        layers = self._post_layers if self.post else self._parallel_layers if self.parallel else self._sandwich_layers
+        layers = (self._post_layers if self.post else self._parallel_layers if self.parallel else self._pre_layers if self.pre
+                  else self._sandwich_layers)
         layers(x, xb, ws, batch, kv_caches, T, capture_layers or (), callbacks)
         if return_hidden:
-            return x
+            return self._stream(x)
         rows = batch.logits_rows
         if rows is not None and rows.dtype != torch.int32:
             rows = rows.to(torch.int32)
@@ -345,10 +386,59 @@ class HybridDecoder:
             if callbacks is not None and self._run_callbacks(callbacks, "post", r, x, None):
                 break
 
+    def _pre_layers(self, x, xb, ws, batch, kv_caches, T, capture, callbacks):
+        """One fused pass between two sublayers: the output joins the streams, the streams are mixed, weighted sum and norm in front of
+        the next sublayer. It is split where somebody looks at the stream between two layers."""
+        step = dict(streams=self.streams, eps=self.cfg.rms_norm_eps)
+        for r, (i, _) in enumerate(self.runs):
+            lw = self.layers[i]
+            if r == 0 or callbacks is not None or r - 1 in capture:      # not done by the pass behind the layer before
+                if callbacks is not None and self._stream_callbacks(callbacks, "pre", r, x):
+                    break
+                hyper_norm(x, in_w=lw.hc1.read, pre_w=lw.norm1, xb=xb, **step)
+                self.mark("norm")
+            ahead = {}
+            if not (r + 1 == len(self.runs) or callbacks is not None or r in capture):
+                nxt = self.layers[self.runs[r + 1][0]]
+                ahead = dict(in_w=nxt.hc1.read, pre_w=nxt.norm1, xb=xb)
+            y, hc, routed = lw.mixer.forward(self, ws, batch, kv_caches[r], T), lw.hc1, {}
+            self.mark("out_gemm")
+            if lw.norm2 is not None:
+                hyper_norm(x, y, mix=hc.mix, out_w=hc.out, in_w=lw.hc2.read, pre_w=lw.norm2, xb=xb, **step)
+                self.mark("norm")
+                hc = lw.hc2
+                if lw.experts is not None:
+                    y, routed = lw.experts.forward(self, xb, T)
+                else:
+                    y = lw.ff.forward(self, xb, T, ws.take, "y")
+            hyper_norm(x, y, mix=hc.mix, out_w=hc.out, **routed, **ahead, **step)
+            self.mark("norm")
+            if r in capture:
+                self.captured[r] = self._stream(x).clone()
+            if callbacks is not None and self._stream_callbacks(callbacks, "post", r, x):
+                break
+
+    def _stream(self, x):
+        """The residual stream as the outside sees it: the sum of the streams."""
+        return x if self.streams == 1 else x.unflatten(1, (self.streams, -1)).sum(1)
+
+    def _stream_callbacks(self, callbacks, when: str, i: int, x) -> bool:
+        """``_run_callbacks`` on the sum of the streams; a change of it is shared out equally among them."""
+        if self.streams == 1 or i not in callbacks.layers_of_interest(len(self.runs)):
+            return self._run_callbacks(callbacks, when, i, x, None)
+        before = self._stream(x)
+        after = before.clone()
+        stop = self._run_callbacks(callbacks, when, i, after, None)
+        x.unflatten(1, (self.streams, -1)).add_(((after - before) / self.streams)[:, None])
+        return stop
+
     def _final_norm(self, x, rows=None):
         n = x.shape[0] if rows is None else rows.shape[0]
         hn = torch.empty((n, self.cfg.hidden_size), dtype=self.dtype, device=self.device)
-        if not self.post:
+        if self.pre:                  # x: the streams of a step, or rows of their sum
+            n = x.shape[1] // self.cfg.hidden_size
+            hyper_norm(x, streams=n, eps=self.cfg.rms_norm_eps, in_w=self.sum_streams[:n], pre_w=self.final_norm, xb=hn, rows=rows)
+        elif not self.post:
             residual_norm(x, pre_w=self.final_norm, xb=hn, rows=rows, kind=self.cfg.norm_type, eps=self.cfg.rms_norm_eps)
         else:
             R.scaled_add_norm(x, None, self.final_norm, 1.0, self.cfg.rms_norm_eps, rows=rows, xb=hn)

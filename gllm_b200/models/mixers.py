@@ -1,12 +1,13 @@
 """Token mixers of heterogeneous decoders: attention (chunked, windowed with kept first tokens or full; query / key norm over
-the row or per head; optional short convolution, soft-capped scores, distance biases, sinks), latent attention (windowed or
-full, with or without a rotated part and an output gate), RG-LRU, gated linear and lightning attention. Each class
-packs its layer's weights into the layouts of the ops and runs a step's tokens:
-``forward(model, ws, batch, cache, T) -> y [T, >= hidden]``, reading the layer input from ``ws.xb``.
+the row or per head; optional short convolution, soft-capped scores, distance biases, sinks, normed values, query temperature, a
+gate per head), latent attention (windowed or full, with or without a rotated part and an output gate), RG-LRU, gated linear and
+lightning attention, state-space duality, minGRU, and two mixers side by side. Each class packs its layer's weights into the layouts
+of the ops and runs a step's tokens: ``forward(model, ws, batch, cache, T) -> y [T, >= hidden]``, reading the layer input from
+``ws.xb``.
 
 ``cache`` is what ``alloc`` returned for the layer: paged K / V (or latent rows) for attention, a ``RecurrentState`` for the
-recurrent mixers, both (``PagedWithState``) for attention behind a convolution. All constants come from the layer's
-``MixerSpec``, so other designs can combine the same mixers differently.
+recurrent mixers, both (``PagedWithState``) for attention behind a convolution or beside a recurrent mixer. All constants come from
+the layer's ``MixerSpec``, so other designs can combine the same mixers differently.
 """
 from __future__ import annotations
 
@@ -33,17 +34,31 @@ def _pad_bias(parts, total: int, device) -> torch.Tensor:
 
 
 class _Mixer:
-    def __init__(self, spec: MixerSpec, src, prefix: str, hidden: int, eps: float, device, dtype):
+    """``part`` ("left.", "right."): the mixer is one of two over the same input (``ParallelMixer``). Its input and output projections
+    are then parts of theirs, and its ``core`` leaves the operand of the output projection, times ``factor``, where it is told."""
+
+    def __init__(self, spec: MixerSpec, src, prefix: str, hidden: int, eps: float, device, dtype, part: str = "", factor: float = 1.0):
         self.spec, self.eps, self.device, self.dtype = spec, eps, torch.device(device), dtype
         self.w: Dict[str, torch.Tensor] = {}
-        self._src, self._p, self._hidden = src, prefix + "mix.", hidden
+        self.part, self.factor = part, factor
+        self._src, self._p, self._hidden = src, prefix + "mix." + part, hidden
         self.pack()
         del self._src
 
+    def rows(self, *names) -> torch.Tensor:
+        """The named matrices stacked along the out-features, in the compute dtype."""
+        return torch.cat([self._src.get(self._p + n).to(self.device, self.dtype) for n in names], 0)
+
     def mat(self, *names) -> torch.Tensor:
-        """The named matrices stacked along the out-features, padded, in the compute dtype."""
-        w = torch.cat([self._src.get(self._p + n).to(self.device, self.dtype) for n in names], 0)
-        return L.pad_rows(w, ROW_PAD).contiguous()
+        """``rows``, padded."""
+        return L.pad_rows(self.rows(*names), ROW_PAD).contiguous()
+
+    def pack_ends(self, key: str, *names):
+        """Input projection ``w[key]`` and output projection, or, of a part, the rows and columns the pair's are made of."""
+        if self.part:
+            self.in_rows, self.out_cols = self.rows(*names), self.rows("o")
+        else:
+            self.w[key], self.w["wo"] = self.mat(*names), self.mat("o")
 
     def vec(self, name) -> torch.Tensor:
         return self._src.get(self._p + name).float().to(self.device).contiguous()
@@ -65,7 +80,7 @@ class AttentionMixer(_Mixer):
         self.dv = m.value_dim
         self.nq, self.nk, self.nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * self.dv
         names = ("q", "k") if m.v_from_k else ("q", "k", "v")
-        self.w["wqk"] = self.mat(*names)
+        self.pack_ends("wqk", *names, *(("g",) if m.head_gate else ()))
         self.w["bqk"] = (_pad_bias([self._src.get(self._p + n + ".b") for n in names], self.w["wqk"].shape[0], self.device)
                          if m.qkv_bias else None)
         self.w["sink"] = self.vec("sink") if m.sink else None
@@ -75,17 +90,19 @@ class AttentionMixer(_Mixer):
             rows = torch.tensor(ops.distance_rows(table.shape[0], m.bias_max), device=self.device)
             self.rel = ops.DistanceBias(table[rows].t())
             self.w["rel"] = self.rel.table
-        self.w["wo"] = self.mat("o")
         self.w["bo"] = _pad_bias([self._src.get(self._p + "o.b")], self.w["wo"].shape[0], self.device) if m.o_bias else None
         norm = m.row_qk_norm or m.head_qk_norm
         self.w["q_norm"] = self.vec("q.norm") if norm else None
         self.w["k_norm"] = self.vec("k.norm") if norm else None
         self.w["conv"] = torch.cat([self.vec(n + ".conv") for n in names]).contiguous() if m.taps else None
-        if m.row_qk_norm and (m.taps or self.dv != m.dim) or m.v_from_k and not m.row_qk_norm or (m.keep_first and m.chunk):
+        if (m.row_qk_norm and (m.taps or self.dv != m.dim or m.v_norm or m.q_temp) or m.v_from_k and (not m.row_qk_norm or m.head_gate)
+                or (m.keep_first and m.chunk) or (self.part and (m.taps or m.qkv_bias or m.o_bias))):
             raise ValueError("attention mixer: this combination of norm, values, convolution and mask is not built")
 
     def workspace(self):
-        return {"proj": self.w["wqk"].shape[0], "q": self.nq, "mix": self.spec.heads * self.dv}
+        n = self.spec.heads * self.dv
+        own = {} if self.part else {"proj": self.w["wqk"].shape[0], **({"gated": n} if self.spec.head_gate else {})}
+        return {"q": self.nq, "mix": n, **own}
 
     def state_shapes(self):
         return {"conv": (self.spec.taps, self.nq + self.nk + self.nv)} if self.spec.taps else None
@@ -97,10 +114,15 @@ class AttentionMixer(_Mixer):
         return PagedWithState(kv, RecurrentState(slots, self.state_shapes(), self.device)) if m.taps else kv
 
     def forward(self, model, ws, batch, cache, T):
-        m = self.spec
-        kv = cache.pages if m.taps else cache
         qk = L.gemm(ws.xb[:T], self.w["wqk"], out=ws.take("proj", T, self.w["wqk"].shape[0]), bias=self.w["bqk"])
         model.mark("in_gemm")
+        o = self.core(model, ws, batch, cache, T, qk, ws.take("gated", T, self.spec.heads * self.dv) if self.spec.head_gate else None)
+        return L.gemm(o, self.w["wo"], out=ws.take("y", T, self.w["wo"].shape[0]), bias=self.w["bo"])
+
+    def core(self, model, ws, batch, cache, T, qk, out):
+        """From the projected rows to the operand of the output projection; ``out`` None: a buffer of its own."""
+        m = self.spec
+        kv = cache.pages if m.taps else cache
         cos, sin = model.rope_tables(m.rot_dim, m.rot_base)
         q = ws.take("q", T, self.nq)
         common = dict(rot_dim=m.rot_dim, positions=batch.positions, slot_mapping=batch.slot_mapping, cos_t=cos, sin_t=sin,
@@ -109,7 +131,7 @@ class AttentionMixer(_Mixer):
             R.qk_row_norm_rope(qk, n_q=m.heads, n_kv=m.kv_heads, head_dim=m.dim, v_from_k=m.v_from_k, **common)
         else:
             R.conv_qkv_prep(SeqView.of(batch), qk, n_q=m.heads, n_kv=m.kv_heads, dim=m.dim, vdim=self.dv, conv=self.w["conv"],
-                            ring=cache.state["conv"] if m.taps else None, **common)
+                            ring=cache.state["conv"] if m.taps else None, v_norm=m.v_norm, q_temp=m.q_temp, **common)
         model.mark("qk_prep")
         o = ws.take("mix", T, m.heads * self.dv)
         mask = dict(window=ops.chunk_window(m.chunk) if m.chunk > 0 else m.window, keep_first=m.keep_first, dim=m.dim,
@@ -123,7 +145,12 @@ class AttentionMixer(_Mixer):
                               max_q_len=batch.max_q_len, n_q=m.heads, n_kv=m.kv_heads, scale=m.scale, out=o,
                               full_weights=True, **mask)
         model.mark("attention")
-        return L.gemm(o, self.w["wo"], out=ws.take("y", T, self.w["wo"].shape[0]), bias=self.w["bo"])
+        if out is None:
+            return o
+        g = self.nq + self.nk + self.nv
+        R.head_gate(o, qk[:, g:g + m.heads] if m.head_gate else None, self.factor, heads=m.heads, vdim=self.dv, out=out)
+        model.mark("head_gate")
+        return out
 
 
 class LatentMixer(_Mixer):
@@ -361,7 +388,101 @@ class LightningMixer(_Mixer):
         return L.gemm(out, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
 
 
-MIXERS = {"attention": AttentionMixer, "latent": LatentMixer, "rglru": RgLruMixer, "gla": GlaMixer, "lightning": LightningMixer}
+class SsdMixer(_Mixer):
+    def pack(self):
+        m = self.spec
+        self.inner, self.channels = m.heads * m.vdim, m.conv_channels
+        self.pack_ends("win", "in")
+        self.w["conv"], self.w["conv_b"], self.w["dt_bias"], self.w["skip"] = (self.vec(n) for n in ("conv", "conv.b", "dt_bias", "D"))
+        self.w["neg_a"] = -torch.exp(self.vec("A_log").double()).float()
+        self.w["norm"] = self.vec("norm") * self.factor
+
+    def workspace(self):
+        own = {} if self.part else {"proj": self.w["win"].shape[0], "mix": self.inner}
+        return {"conv": self.channels, "f32": self.inner, **own}
+
+    def state_shapes(self):
+        m = self.spec
+        return {"rec": (m.heads, m.dim, m.vdim), "conv": (m.taps, self.channels)}
+
+    def forward(self, model, ws, batch, st, T):
+        p = L.gemm(ws.xb[:T], self.w["win"], out=ws.take("proj", T, self.w["win"].shape[0]))
+        model.mark("in_gemm")
+        o = self.core(model, ws, batch, st, T, p, ws.take("mix", T, self.inner))
+        return L.gemm(o, self.w["wo"], out=ws.take("y", T, self.w["wo"].shape[0]))
+
+    def core(self, model, ws, batch, st, T, p, out):
+        m, w, inner = self.spec, self.w, self.inner
+        sv, at = SeqView.of(batch), inner + self.channels
+        u = R.conv_act(sv, p[:, inner:at], w["conv"], w["conv_b"], st["conv"], ws.take("conv", T, self.channels))
+        model.mark("ssd_conv")
+        acc, n = ws.take("f32", T, inner), m.groups * m.dim
+        R.ssd(sv, u[:, inner + n:], u[:, inner:inner + n], u[:, :inner], p[:, at:at + m.heads], heads=m.heads, groups=m.groups, N=m.dim,
+              P=m.vdim, dt_bias=w["dt_bias"], neg_a=w["neg_a"], skip=w["skip"], state=st["rec"], out=acc)
+        model.mark("ssd")
+        R.gate_norm(acc, p[:, :inner], w["norm"], groups=m.norm_groups, eps=self.eps, out=out)
+        model.mark("ssd_gate")
+        return out
+
+
+class MinGruMixer(_Mixer):
+    def pack(self):
+        self.w["wzxg"] = self.mat("z", "x", "g")
+        self.w["bz"], self.w["bx"] = self.vec("z.b"), self.vec("x.b")      # fp32, added in the recurrence: gates next to 0 stay exact
+        self.w["wo"] = self.mat("o")
+
+    def workspace(self):
+        return {"proj": self.w["wzxg"].shape[0], "mix": self.spec.width}
+
+    def state_shapes(self):
+        return {"rec": (self.spec.width,)}
+
+    def forward(self, model, ws, batch, st, T):
+        w, n = self.w, self.spec.width
+        p = L.gemm(ws.xb[:T], w["wzxg"], out=ws.take("proj", T, w["wzxg"].shape[0]))
+        model.mark("in_gemm")
+        out = R.mingru(SeqView.of(batch), p[:, :n], p[:, n:2 * n], p[:, 2 * n:3 * n], w["bz"], w["bx"], st["rec"], ws.take("mix", T, n))
+        model.mark("mingru")
+        return L.gemm(out, w["wo"], out=ws.take("y", T, w["wo"].shape[0]))
+
+
+class ParallelMixer(_Mixer):
+    """Two mixers over the same input: one input projection for both, one output projection that also sums them (their factors are
+    in its operand, where they are applied in fp32)."""
+
+    def pack(self):
+        m = self.spec
+        if (m.left.kind, m.right.kind) != ("attention", "ssd"):
+            raise ValueError(f"mixers side by side: attention and ssd are built, not {m.left.kind} and {m.right.kind}")
+        prefix = self._p[:-len("mix.")]
+        make = lambda spec, part, factor: MIXERS[spec.kind](spec, self._src, prefix, self._hidden, self.eps, self.device, self.dtype, part,
+                                                            factor)
+        self.left, self.right = make(m.left, "left.", m.left_scale), make(m.right, "right.", m.right_scale)
+        first = L.pad_rows(self.left.in_rows, 8)           # the right part's columns start on a 16-byte boundary
+        self.col, self.out_col = first.shape[0], self.left.out_cols.shape[1]
+        self.w["win"] = L.pad_rows(torch.cat([first, self.right.in_rows]), ROW_PAD).contiguous()
+        self.w["wo"] = L.pad_rows(torch.cat([self.left.out_cols, self.right.out_cols], 1), ROW_PAD).contiguous()
+        for side in (self.left, self.right):
+            del side.in_rows, side.out_cols
+            self.w.update({side.part + k: v for k, v in side.w.items() if v is not None})
+
+    def workspace(self):
+        return {"proj": self.w["win"].shape[0], "both": self.w["wo"].shape[1], **self.left.workspace(), **self.right.workspace()}
+
+    def alloc(self, num_pages, slots):
+        return PagedWithState(self.left.alloc(num_pages, slots), self.right.alloc(num_pages, slots))
+
+    def forward(self, model, ws, batch, cache, T):
+        p = L.gemm(ws.xb[:T], self.w["win"], out=ws.take("proj", T, self.w["win"].shape[0]))
+        model.mark("in_gemm")
+        both = ws.take("both", T, self.w["wo"].shape[1])
+        self.left.core(model, ws, batch, cache.pages, T, p[:, :self.col], both[:, :self.out_col])
+        self.right.core(model, ws, batch, cache.state, T, p[:, self.col:], both[:, self.out_col:])
+        return L.gemm(both, self.w["wo"], out=ws.take("y", T, self.w["wo"].shape[0]))
+
+
+MIXERS = {"attention": AttentionMixer, "latent": LatentMixer, "rglru": RgLruMixer, "gla": GlaMixer, "lightning": LightningMixer,
+          "ssd": SsdMixer, "mingru": MinGruMixer, "parallel": ParallelMixer}
 
 
 def mixer_shapes(m: MixerSpec, hidden: int) -> Dict[str, Tuple[int, ...]]:
@@ -377,6 +498,8 @@ def mixer_shapes(m: MixerSpec, hidden: int) -> Dict[str, Tuple[int, ...]]:
             s["o.b"] = (hidden,)
         if m.sink:
             s["sink"] = (m.heads,)
+        if m.head_gate:
+            s["g"] = (m.heads, hidden)
         if m.bias_max:
             s["rel"] = (m.bias_rows or 32, m.heads)
         if m.row_qk_norm:
@@ -402,6 +525,16 @@ def mixer_shapes(m: MixerSpec, hidden: int) -> Dict[str, Tuple[int, ...]]:
         bs = w // nb
         return {"y": (w, hidden), "y.b": (w,), "x": (w, hidden), "x.b": (w,), "conv": (w, m.taps), "conv.b": (w,),
                 "ra": (nb, bs, bs), "ra.b": (nb, bs), "ri": (nb, bs, bs), "ri.b": (nb, bs), "lam": (w,), "o": (hidden, w)}
+    if m.kind == "mingru":
+        return {"z": (m.width, hidden), "z.b": (m.width,), "x": (m.width, hidden), "x.b": (m.width,), "g": (m.width, hidden),
+                "o": (hidden, m.width)}
+    if m.kind == "ssd":
+        inner, ch = m.heads * m.vdim, m.conv_channels
+        return {"in": (inner + ch + m.heads, hidden), "conv": (ch, m.taps), "conv.b": (ch,), "dt_bias": (m.heads,),
+                "A_log": (m.heads,), "D": (m.heads,), "norm": (inner,), "o": (hidden, inner)}
+    if m.kind == "parallel":
+        return {f"{side}.{n}": shape for side, part in (("left", m.left), ("right", m.right))
+                for n, shape in mixer_shapes(part, hidden).items()}
     nk, nv, r = m.heads * m.dim, m.heads * m.vdim, m.decay_rank or 16
     if m.kind == "lightning":
         return {"q": (nk, hidden), "k": (nk, hidden), "v": (nv, hidden), "g": (nv, hidden), "o": (hidden, nv), "norm": (nv,)}

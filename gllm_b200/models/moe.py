@@ -579,39 +579,48 @@ class PlainFF:
 
 
 class ExpertFF:
-    """One layer's experts, bf16 or true fp32: router -> top-k -> routed rows in per-expert blocks -> grouped gate / up and
-    down projections; beside them a shared expert (its gate is one more row of the router's projection). ``forward`` returns
+    """One layer's experts, gated or plain, bf16 or true fp32: router -> top-k -> routed rows in per-expert blocks -> grouped (gate and)
+    up and down projections; beside them a shared expert (its gate is one more row of the router's projection). ``forward`` returns
     what the caller sums with ``ops.residual.residual_norm`` (together with the norms around the sublayer): the experts' rows
     and, by keyword, the place of each (token, pick) among them, the picks' weights (unless the spec scales the experts'
     inputs), the shared expert's rows and gate."""
 
-    def __init__(self, spec: MoeSpec, act: int, src, prefix: str, hidden: int, device, dtype):
-        self.spec, self.act, self.hidden = spec, act, hidden
+    def __init__(self, spec: MoeSpec, act: str, src, prefix: str, hidden: int, device, dtype):
+        self.spec, self.hidden = spec, hidden
+        self.act = L.ACT_IDS[act] if spec.gated else act
         get = lambda n: src.get(prefix + "mlp." + n).to(device, dtype)
         self.router = get("router")
         if spec.shared_gate:
             self.router = torch.cat([self.router, get("shared.sg")], 0)
         self.router = L.pad_rows(self.router, 32).contiguous()
+        self.correction = src.get(prefix + "mlp.correction").float().to(device).contiguous() if spec.correction else None
         self.fused = dtype == torch.bfloat16 and hidden % 8 == 0
         pad = -spec.ff % 64 if self.fused else 0       # zero gate / up rows and down columns add nothing to the sums
         self.inter = spec.ff + pad
         rows = lambda w: torch.nn.functional.pad(w, (0, 0, 0, pad))
-        gus, downs = [], []
+        ins, downs = [], []
         for e in range(spec.experts):
-            g, u, d = rows(get(f"e{e}.gate")), rows(get(f"e{e}.up")), torch.nn.functional.pad(get(f"e{e}.down"), (0, pad))
-            gus.append(L.interleave_gate_up(g, u) if self.fused else torch.cat([g, u], 0))
+            u, d = rows(get(f"e{e}.up")), torch.nn.functional.pad(get(f"e{e}.down"), (0, pad))
+            if spec.gated:
+                g = rows(get(f"e{e}.gate"))
+                u = L.interleave_gate_up(g, u) if self.fused else torch.cat([g, u], 0)
+            ins.append(u)
             downs.append(L.pad_rows(d, 128))
-        self.w_gate_up, self.w_down = torch.cat(gus).contiguous(), torch.cat(downs).contiguous()
+        self.w_in, self.w_down = torch.cat(ins).contiguous(), torch.cat(downs).contiguous()
         self.glu_bn = 256 if self.inter % 128 == 0 else 128
-        self.shared = GatedFF(get("shared.gate"), get("shared.up"), get("shared.down"), act, dtype) if spec.shared_ff else None
+        self.shared = None
+        if spec.shared_ff and spec.gated:
+            self.shared = GatedFF(get("shared.gate"), get("shared.up"), get("shared.down"), self.act, dtype)
+        elif spec.shared_ff:
+            self.shared = PlainFF(get("shared.up"), get("shared.down"), act, dtype)
 
     def tensors(self):
-        return [self.router, self.w_gate_up, self.w_down] + (self.shared.tensors() if self.shared else [])
+        return [self.router, self.w_in, self.w_down] + (self.shared.tensors() if self.shared else [])
 
     def workspace(self, model, T: int) -> M.MoeWorkspace:
         holder = model.__dict__.setdefault("_expert_ws", {})
         s = self.spec
-        key = (s.experts, s.top, self.inter, s.shared_ff)
+        key = (s.experts, s.top, self.inter, s.shared_ff, s.gated)
         ws = holder.get(key)
         if ws is None or ws.ids.shape[0] < T:
             n = max(T, 256)
@@ -621,7 +630,7 @@ class ExpertFF:
             if self.shared is not None:
                 ws.shared = {k: torch.zeros((n, c), dtype=torch.float32 if k == "y" else model.dtype, device=model.device)
                              for k, c in self.shared.workspace().items()}
-            ws.gu = None if self.fused else torch.zeros((ws.max_rows, 2 * self.inter), dtype=model.dtype, device=model.device)
+            ws.gu = None if self.fused or not s.gated else torch.zeros((ws.max_rows, 2 * self.inter), dtype=model.dtype, device=model.device)
             holder[key] = ws
         return ws
 
@@ -630,24 +639,26 @@ class ExpertFF:
         ws = self.workspace(model, T)
         logits = L.gemm(h, self.router, out=ws.logits[:T])
         on_gpu = dict(out_ids=ws.ids[:T], out_w=ws.w[:T]) if h.is_cuda else {}
-        ids, w = M.route(logits[:, :s.experts], s.top, norm_topk=s.norm_topk, scoring=s.scoring, scale=s.scale, groups=s.groups,
-                         keep_groups=s.keep_groups, **on_gpu)
+        ids, w = M.route(logits[:, :s.experts], s.top, norm_topk=s.norm_topk, scoring=s.scoring, sel_bias=self.correction, scale=s.scale,
+                         groups=s.groups, keep_groups=s.keep_groups, **on_gpu)
         model.mark("moe_route")
         M.permute(h, None, ids, ws, 0, s.experts, row_w=w if s.scale_input else None)
         model.mark("moe_permute")
-        if self.fused:
+        if not s.gated:
+            L.gemm_grouped(ws.a_perm, self.w_in, ws.blk_group, s.experts, out=ws.act, block_rows=ws.blk_rows, act=self.act)
+        elif self.fused:
             L.set_block_rows(ws.blk_rows if h.is_cuda else None)
-            L.gemm_glu(ws.a_perm, self.w_gate_up, act=self.act, out=ws.act, bn=self.glu_bn, mblk_group=ws.blk_group,
+            L.gemm_glu(ws.a_perm, self.w_in, act=self.act, out=ws.act, bn=self.glu_bn, mblk_group=ws.blk_group,
                        num_groups=s.experts)
         else:
-            L.gemm_grouped(ws.a_perm, self.w_gate_up, ws.blk_group, s.experts, out=ws.gu, block_rows=ws.blk_rows)
+            L.gemm_grouped(ws.a_perm, self.w_in, ws.blk_group, s.experts, out=ws.gu, block_rows=ws.blk_rows)
             ops.glu(ws.gu, self.act, out=ws.act)
-        model.mark("moe_gate_up")
+        model.mark("moe_gate_up" if s.gated else "moe_up")
         L.gemm_grouped(ws.act, self.w_down, ws.blk_group, s.experts, out=ws.y_perm, block_rows=ws.blk_rows)
         model.mark("moe_down")
         out = dict(dest=ws.dest, top=s.top, row_w=None if s.scale_input else w)
         if self.shared is not None:
             take = lambda k, rows, cols: ws.shared[k][:rows]
-            out["gated"] = self.shared.forward(model, h, T, take, "y", ("shared_gate_up", "shared_down"))
+            out["gated"] = self.shared.forward(model, h, T, take, "y", ("shared_gate_up" if s.gated else "shared_up", "shared_down"))
             out["gate"] = logits[:, s.experts] if s.shared_gate else None
         return ws.y_perm, out

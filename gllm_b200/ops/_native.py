@@ -42,7 +42,7 @@ _SIGNATURES = {
     "gllm_get_option": (L, [ctypes.c_char_p]),
     "gllm_gemm_trace_enabled": (I, []),
     "gllm_gemm_bf16_glu": (I, [P, L, P, L, P, L, I, I, I, I, P, I, F, F, I, P, I, P, I, I]),
-    "gllm_gemm_bf16_grouped": (I, [P, L, P, L, P, L, I, I, I, P, I, I, P, I]),
+    "gllm_gemm_bf16_grouped": (I, [P, L, P, L, P, L, I, I, I, P, I, I, I, P, I]),
     "gllm_gemm_bf16_qkv": (I, [P, L, P, L, I, I, I, I, P, P, I, P, P, P, P, I, P, P, F, P, I, F, F, P, P, I, I]),
     "gllm_gemm_bf16_qkv_fp8kv": (I, [P, L, P, L, I, I, I, I, P, P, I, P, P, P, P, I, P, P, F, P, I, F, F, P, F, P, I, I]),
     "gllm_gemm_fp8": (I, [P, L, P, L, P, L, I, I, I, I, P, P, I, P, I, I]),
@@ -59,7 +59,7 @@ _SIGNATURES = {
     "gllm_rope_kv_write": (I, [P, L, I, I, I, I, I, P, P, P, P, I, P, P, F, P, P, I, P]),
     "gllm_attention_any": (I, [P, P, P, P, I, I, P, I, P, P, P, I, I, I, I, I, I, F, I, I, I, P, F, P, I, P]),
     "gllm_attention_mma": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, F, I, I, I, P, F, P, I, P]),
-    "gllm_gemm_simt_grouped": (I, [P, L, P, L, P, L, I, I, I, I, I, P, P, P]),
+    "gllm_gemm_simt_grouped": (I, [P, L, P, L, P, L, I, I, I, I, I, P, P, I, P]),
     "gllm_gemm_simt": (I, [P, L, P, L, P, L, I, I, I, I, I, P, F, I, I, P]),
     "gllm_paged_attention_fp8kv": (I, [P, P, P, I, P, I, P, P, P, I, I, I, I, I, F, I, I, F, P]),
     "gllm_rope_kv_write_fp8": (I, [P, L, I, I, I, I, I, P, P, P, P, I, P, P, F, P, P, I, F, P]),

@@ -292,10 +292,11 @@ def set_block_rows(rows):
         nv.check(nv.lib().gllm_gemm_set_block_rows(rows.data_ptr()), "gemm_set_block_rows")
 
 
-def gemm_grouped(a, w_stack, mblk_group, num_groups, *, out=None, bn=128, max_ctas=0, block_rows=None):
+def gemm_grouped(a, w_stack, mblk_group, num_groups, *, out=None, bn=128, max_ctas=0, block_rows=None, act=None):
     """Grouped GEMM: rows [128i, 128i+128) of ``a`` multiply expert ``mblk_group[i]``'s [N,K] weight; with ``block_rows``
-    only the first ``block_rows[i]`` of them exist. fp32 operands, and bf16 ones the tensor-core kernel cannot address, run
-    on CUDA cores."""
+    only the first ``block_rows[i]`` of them exist. ``act``: activation (``STORE_ACTS``) of the result. fp32 operands, and bf16
+    ones the tensor-core kernel cannot address, run on CUDA cores."""
+    act_id = STORE_ACTS[act] if act else 0
     M, K = a.shape
     N = w_stack.shape[0] // num_groups
     if not a.is_cuda:
@@ -304,7 +305,8 @@ def gemm_grouped(a, w_stack, mblk_group, num_groups, *, out=None, bn=128, max_ct
             g = int(mblk_group[i])
             if g < 0:
                 continue
-            res[i * 128:(i + 1) * 128] = (a[i * 128:(i + 1) * 128].float() @ w_stack[g * N:(g + 1) * N].float().t()).to(a.dtype)
+            acc = a[i * 128:(i + 1) * 128].float() @ w_stack[g * N:(g + 1) * N].float().t()
+            res[i * 128:(i + 1) * 128] = (_store_act_ref(acc, act_id) if act else acc).to(a.dtype)
         if out is not None:
             out.copy_(res)
             return out
@@ -316,13 +318,13 @@ def gemm_grouped(a, w_stack, mblk_group, num_groups, *, out=None, bn=128, max_ct
         rc = nv.lib().gllm_gemm_simt_grouped(a.data_ptr(), a.stride(0), w_stack.data_ptr(), w_stack.stride(0), out.data_ptr(),
                                              out.stride(0), M, N, K, 1 if a.dtype == torch.float32 else 0,
                                              1 if out.dtype == torch.float32 else 0, mblk_group.data_ptr(),
-                                             nv.ptr(block_rows), nv.stream_ptr())
+                                             nv.ptr(block_rows), act_id, nv.stream_ptr())
         nv.check(rc, "gemm_simt_grouped")
         return out
     set_block_rows(block_rows)
     rc = nv.lib().gllm_gemm_bf16_grouped(a.data_ptr(), a.stride(0), w_stack.data_ptr(), w_stack.stride(0),
                                          out.data_ptr(), out.stride(0), M, N, K, mblk_group.data_ptr(), num_groups,
-                                         bn, nv.stream_ptr(), max_ctas)
+                                         bn, act_id, nv.stream_ptr(), max_ctas)
     nv.check(rc, "gemm_bf16_grouped")
     return out
 

@@ -1,8 +1,8 @@
-"""Recurrent token mixers (short convolution, RG-LRU, gated linear attention, lightning attention) and the ops of a residual stream kept in
-fp32: embedding rows, scaled post-norm, query / key preparation with a norm over the whole projection.
+"""Recurrent token mixers (short convolution, RG-LRU, gated linear attention, lightning attention, state-space duality, minGRU) and
+the ops of a residual stream kept in fp32: embedding rows, scaled post-norm, query / key preparation.
 
-CUDA path: ``csrc/kernels/recurrent.cu``, ``lightning.cu`` and ``csrc/kernels/simt.cu`` (bf16 or fp32 tensors, fp32 states). CPU path: an
-fp32 restatement of each op.
+CUDA path: ``csrc/kernels/recurrent.cu``, ``lightning.cu``, ``state_space.cu``, ``mingru.cu``, ``mixer_prep.cu`` and ``simt.cu`` (bf16 or
+fp32 tensors, fp32 states). CPU path: an fp32 restatement of each op.
 
 The sequences of a step come as a ``SeqView``: sequence i owns rows [q_start, q_start + q_len) of the flat batch, the
 last q_len of its ctx tokens, and the state slot slots[i]; a decode view has one row per slot (row = slot, live where
@@ -19,7 +19,7 @@ import torch
 from . import _native as nv
 
 P, I, L, F = c_void_p, c_int, c_longlong, c_float
-nv.register("gllm_embed_rows", I, [P, P, I, I, I, F, P, P, I, P])
+nv.register("gllm_embed_rows", I, [P, P, I, I, I, F, I, P, P, I, P])
 nv.register("gllm_scaled_add_norm", I, [P, L, P, L, I, P, I, I, F, F, P, P, P, I, P])
 nv.register("gllm_glu_f32", I, [P, L, I, I, I, P, P])
 nv.register("gllm_qk_row_norm_rope", I, [P, L, I, I, I, I, I, I, I, P, P, P, P, I, P, P, F, P, P, I, P])
@@ -32,10 +32,15 @@ nv.register("gllm_gla_step", I, [P, P, P, P, I, P, P, P, P, L, I, P, P, I, I, I,
 nv.register("gllm_gla_tile_ok", I, [I, I, I, L])
 nv.register("gllm_gla_decode", I, [P, I, P, P, P, P, P, L, P, P, P, I, I, I, I, F, F, F, P, P, P])
 nv.register("gllm_gla_prefill", I, [P, P, P, P, I, I, P, P, P, P, L, P, P, I, I, I, I, F, F, P, P, P, P])
-nv.register("gllm_conv_qkv_prep", I, [P, P, P, P, I, I, P, L, I, I, I, I, I, I, I, P, P, P, F, P, P, P, P, I, P, P, P, I, P])
+nv.register("gllm_conv_qkv_prep", I, [P, P, P, P, I, I, P, L, I, I, I, I, I, I, I, P, P, P, F, I, F, I, P, P, P, P, I, P, P, P, I, P])
 nv.register("gllm_lightning", I, [P, P, P, P, I, P, P, P, L, I, I, I, I, P, P, P, P, I, P])
 nv.register("gllm_row_norm_gate", I, [P, P, L, I, P, I, I, F, P, P])
 nv.register("gllm_sigmoid_gate", I, [P, P, L, I, L, I, P])
+nv.register("gllm_ssd", I, [P, P, P, P, I, P, P, P, L, P, L, I, I, I, I, I, P, P, P, P, P, I, P])
+nv.register("gllm_conv_act", I, [P, P, P, P, I, I, P, L, I, P, P, P, I, I, P, P])
+nv.register("gllm_gate_norm", I, [P, P, L, I, P, I, I, I, F, P, L, P])
+nv.register("gllm_head_gate", I, [P, P, L, I, I, I, F, L, P, L, P])
+nv.register("gllm_mingru", I, [P, P, P, P, I, I, P, P, P, L, I, P, P, I, P, P, I, P, I, P])
 nv.register("gllm_head_norm_gate", I, [P, P, L, I, P, L, I, I, F, P, P])
 
 RGLRU_C = 8.0        # exponent of the RG-LRU decay: log a = -8 r softplus(lam)
@@ -82,17 +87,18 @@ def _f32(t) -> int:
     return 1 if t.dtype == torch.float32 else 0
 
 
-def embed_rows(ids, table, x, xb=None, scale=1.0):
-    """x[m] = table[ids[m]] * scale in fp32; ``xb`` (optional) the unscaled rows in the table's dtype."""
+def embed_rows(ids, table, x, xb=None, scale=1.0, streams=1):
+    """x[m] = table[ids[m]] * scale in fp32, ``streams`` times side by side; ``xb`` (optional) the unscaled rows in the table's
+    dtype."""
     M = ids.shape[0]
     if not table.is_cuda:
         rows = table[ids.long()]
-        x.copy_(rows.float() * scale)
+        x.copy_((rows.float() * scale).repeat(1, streams))
         if xb is not None:
             xb.copy_(rows)
         return x
     nv.check(nv.lib().gllm_embed_rows(ids.data_ptr(), table.data_ptr(), table.shape[0], table.shape[1], _f32(table), float(scale),
-                                      x.data_ptr(), nv.ptr(xb), M, nv.stream_ptr()), "embed_rows")
+                                      int(streams), x.data_ptr(), nv.ptr(xb), M, nv.stream_ptr()), "embed_rows")
     return x
 
 
@@ -155,11 +161,12 @@ def qk_row_norm_rope(qk, *, n_q, n_kv, head_dim, rot_dim, v_from_k, positions, s
 
 
 def conv_qkv_prep(sv: "SeqView", qkv, *, n_q, n_kv, dim, vdim, rot_dim, conv, q_w, k_w, eps, positions, slot_mapping, cos_t, sin_t,
-                  ring, q_out, kv_cache):
-    """Attention layers with a short convolution: causal convolution per channel of the projected q | k | v rows (``conv``
+                  ring, q_out, kv_cache, v_norm=False, q_temp=None):
+    """Attention layers with or without a short convolution: causal convolution per channel of the projected q | k | v rows (``conv``
     [channels, taps] fp32, or None) -> RMS norm of each q / k head (weights [dim] shared by the heads, or None) -> RoPE on
     the first ``rot_dim`` dimensions of q and k -> q buffer, K and V pages. ``ring`` [slots, taps, channels] fp32 keeps the
-    last projected values of each sequence: the one of position p in entry p % taps."""
+    last projected values of each sequence: the one of position p in entry p % taps. ``v_norm``: each value head is divided by
+    its root mean square. ``q_temp`` (coef, every): queries are multiplied by 1 + coef ln(floor((position + 1) / every) + 1)."""
     M = qkv.shape[0]
     nq, nk, nv_ = n_q * dim, n_kv * dim, n_kv * vdim
     taps = 0 if conv is None else conv.shape[1]
@@ -184,18 +191,26 @@ def conv_qkv_prep(sv: "SeqView", qkv, *, n_q, n_kv, dim, vdim, rot_dim, conv, q_
             c, s = cos_t[positions.long()][:, None], sin_t[positions.long()][:, None]
             a, b = t[..., :half], t[..., half:rot_dim]
             return torch.cat([a * c - b * s, b * c + a * s, t[..., rot_dim:]], -1)
-        q_out[:M].copy_(prep(y[:, :nq], n_q, q_w).reshape(M, nq).to(q_out.dtype))
+        q = prep(y[:, :nq], n_q, q_w)
+        if q_temp:
+            p = torch.div(positions.long() + 1, int(q_temp[1]), rounding_mode="floor")
+            q = q * (1 + q_temp[0] * torch.log((p + 1).float()))[:, None, None]
+        q_out[:M].copy_(q.reshape(M, nq).to(q_out.dtype))
+        v = y[:, nq + nk:].reshape(M, n_kv, vdim)
+        if v_norm:
+            v = v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)
         if slot_mapping is not None:
             from .attention import kv_views
             kc, vc = kv_views(kv_cache, n_kv, dim)
             ok = slot_mapping >= 0
             sl = slot_mapping[ok].long()
             kc[sl // 16, :, sl % 16] = prep(y[:, nq:nq + nk], n_kv, k_w)[ok].to(kv_cache.dtype)
-            vc[sl // 16, :, sl % 16] = y[:, nq + nk:].reshape(M, n_kv, vdim)[ok].to(kv_cache.dtype)
+            vc[sl // 16, :, sl % 16] = v[ok].to(kv_cache.dtype)
         return q_out
     nv.check(nv.lib().gllm_conv_qkv_prep(
         *sv.ptrs(), sv.max_q_len, qkv.data_ptr(), qkv.stride(0), _f32(qkv), n_q, n_kv, dim, vdim, rot_dim, taps, nv.ptr(conv),
-        nv.ptr(q_w), nv.ptr(k_w), float(eps), positions.data_ptr(), nv.ptr(slot_mapping), nv.ptr(cos_t), nv.ptr(sin_t),
+        nv.ptr(q_w), nv.ptr(k_w), float(eps), 1 if v_norm else 0, float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 0,
+        positions.data_ptr(), nv.ptr(slot_mapping), nv.ptr(cos_t), nv.ptr(sin_t),
         cos_t.shape[0] if cos_t is not None else 1, nv.ptr(ring), q_out.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
         nv.stream_ptr()), "conv_qkv_prep")
     return q_out
@@ -417,3 +432,111 @@ def sigmoid_gate(x, g):
     nv.check(nv.lib().gllm_sigmoid_gate(x.data_ptr(), g.data_ptr(), g.stride(0), _f32(x), x.shape[0], x.shape[1], nv.stream_ptr()),
              "sigmoid_gate")
     return x
+
+
+def head_gate(o, g, scale, *, heads, vdim, out):
+    """out = scale * sigmoid(g[:, head]) * o per head; g None: scale * o. o [T, heads * vdim]; g and out may be column slices."""
+    T = o.shape[0]
+    if not o.is_cuda:
+        f = scale if g is None else scale * torch.sigmoid(g[:, :heads].float())[:, :, None]
+        out.copy_((o.float().reshape(T, heads, vdim) * f).reshape(T, heads * vdim).to(out.dtype))
+        return out
+    nv.check(nv.lib().gllm_head_gate(o.data_ptr(), nv.ptr(g), 0 if g is None else g.stride(0), _f32(o), heads, vdim, float(scale), T,
+                                     out.data_ptr(), out.stride(0), nv.stream_ptr()), "head_gate")
+    return out
+
+
+# --------------------------------------------------------------------------------------------
+# state-space duality (Mamba-2)
+# --------------------------------------------------------------------------------------------
+def conv_act(sv: SeqView, x, w, b, ring, out):
+    """silu(causal convolution per channel + b): x [T, channels] (a column slice is fine), w [channels, taps], b [channels] fp32,
+    ring [slots, taps, channels] fp32 (the input of position p in entry p % taps, moved forward), out [T, channels]."""
+    channels, taps = w.shape
+    if not x.is_cuda:
+        for r0, n, start, slot in sv.rows():
+            u = x[r0:r0 + n, :channels].float()
+            z = torch.cat([_conv_history(ring[slot], start, taps), u])
+            a = sum(z[j:j + n] * w[:, j] for j in range(taps)) + b
+            out[r0:r0 + n].copy_(torch.nn.functional.silu(a).to(out.dtype))
+            for i in range(max(0, n - taps), n):
+                ring[slot, (start + i) % taps] = u[i]
+        return out
+    nv.check(nv.lib().gllm_conv_act(*sv.ptrs(), sv.max_q_len, x.data_ptr(), x.stride(0), _f32(x), w.data_ptr(), b.data_ptr(),
+                                    ring.data_ptr(), channels, taps, out.data_ptr(), nv.stream_ptr()), "conv_act")
+    return out
+
+
+def ssd(sv: SeqView, C, B, x, dt, *, heads, groups, N, P, dt_bias, neg_a, skip, state, out, general=False):
+    """Per head, with d = softplus(dt + dt_bias): S = exp(neg_a d) S + d B x^T, out = S^T C + skip x. C, B [T, groups * N] (head h
+    uses group h // (heads // groups)) and x [T, heads * P] are column slices of one buffer, dt [T, heads] one of any; out
+    [T, heads * P] fp32; state [slots, heads, N, P] fp32. ``general``: the token-by-token kernel whatever the sizes."""
+    if not x.is_cuda:
+        for r0, n, start, slot in sv.rows():
+            S = state[slot].clone() if start > 0 else torch.zeros_like(state[slot])
+            per = lambda t: t[r0:r0 + n].float().reshape(n, groups, N).repeat_interleave(heads // groups, 1)
+            cc, bb, xx = per(C), per(B), x[r0:r0 + n].float().reshape(n, heads, P)
+            d = torch.nn.functional.softplus(dt[r0:r0 + n, :heads].float() + dt_bias)
+            forget = -torch.expm1(neg_a * d)
+            for i in range(n):
+                S = S - forget[i][:, None, None] * S + (d[i][:, None] * bb[i])[:, :, None] * xx[i][:, None, :]
+                out[r0 + i] = (torch.einsum("hnp,hn->hp", S, cc[i]) + skip[:, None] * xx[i]).reshape(-1)
+            state[slot].copy_(S)
+        return out
+    assert C.stride(0) == B.stride(0) == x.stride(0) and dt.dtype == x.dtype
+    nv.check(nv.lib().gllm_ssd(*sv.ptrs(), C.data_ptr(), B.data_ptr(), x.data_ptr(), x.stride(0), dt.data_ptr(), dt.stride(0), _f32(x),
+                               heads, groups, N, P, dt_bias.data_ptr(), neg_a.data_ptr(), skip.data_ptr(), state.data_ptr(),
+                               out.data_ptr(), 1 if general else 0, nv.stream_ptr()), "ssd")
+    return out
+
+
+def gate_norm(y, z, w, *, groups, eps, out):
+    """y * silu(z), then an RMS norm over each of ``groups`` equal parts of the row, times w. y [T, n] fp32; z and out may be
+    column slices."""
+    T, n = y.shape
+    if not y.is_cuda:
+        h = (y * torch.nn.functional.silu(z[:, :n].float())).reshape(T, groups, -1)
+        h = (h / torch.sqrt(h.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, n) * w
+        out.copy_(h.to(out.dtype))
+        return out
+    nv.check(nv.lib().gllm_gate_norm(y.data_ptr(), z.data_ptr(), z.stride(0), _f32(z), w.data_ptr(), T, n, groups, float(eps),
+                                     out.data_ptr(), out.stride(0), nv.stream_ptr()), "gate_norm")
+    return out
+
+
+# --------------------------------------------------------------------------------------------
+# minGRU
+# --------------------------------------------------------------------------------------------
+def mingru_segments(width: int, n_seqs: int, max_q_len: int) -> int:
+    """Into how many time segments a prefill step is cut: enough CTAs for every SM twice, not under four 128-token tiles each (a
+    segmented step reads its gates twice)."""
+    want = 296 // max(-(-width // 32) * n_seqs, 1)
+    return max(1, min(want, max_q_len // 512, 16))
+
+
+def mingru(sv: SeqView, zx, cx, g, b_z, b_x, state, out, *, segments=None, general=False):
+    """z = sigmoid(zx + b_z), c = u + 1/2 where u = cx + b_x >= 0, else sigmoid(u); S = (1 - z) S + z c; out = S * silu(g). zx, cx,
+    g [T, width]: column slices of one projection; b_z, b_x [width] and state [slots, width] fp32; out [T, width]."""
+    width = state.shape[1]
+    if not zx.is_cuda:
+        for r0, n, start, slot in sv.rows():
+            S = state[slot].clone() if start > 0 else torch.zeros_like(state[slot])
+            z = torch.sigmoid(zx[r0:r0 + n, :width].float() + b_z)
+            u = cx[r0:r0 + n, :width].float() + b_x
+            c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+            gate = torch.nn.functional.silu(g[r0:r0 + n, :width].float())
+            for i in range(n):
+                S = S - z[i] * S + z[i] * c[i]
+                out[r0 + i].copy_((S * gate[i]).to(out.dtype))
+            state[slot].copy_(S)
+        return out
+    assert zx.stride(0) == cx.stride(0) == g.stride(0)
+    n_seg, scratch = 1, None
+    if sv.q_start is not None and not general:
+        n_seg = segments or mingru_segments(width, sv.n, sv.max_q_len)
+        if n_seg > 1:
+            scratch = torch.empty(3 * sv.n * n_seg * width, dtype=torch.float32, device=zx.device)
+    nv.check(nv.lib().gllm_mingru(*sv.ptrs(), sv.max_q_len, zx.data_ptr(), cx.data_ptr(), g.data_ptr(), zx.stride(0), _f32(zx),
+                                  b_z.data_ptr(), b_x.data_ptr(), width, state.data_ptr(), out.data_ptr(), n_seg, nv.ptr(scratch),
+                                  1 if general else 0, nv.stream_ptr()), "mingru")
+    return out
