@@ -60,6 +60,9 @@ def parse_args():
     ap.add_argument("--ritirax", nargs="?", const="1024,2048,4096", default=None, metavar="SIZES",
                     help="instead of the headline workload: prefill and decode throughput of the parallel-block decoder (Ritirax) "
                          "beside a mixture-of-experts decoder of equal size, per-op times against the roofline (one GPU)")
+    ap.add_argument("--tomopel", nargs="?", const="1024,2048,4096", default=None, metavar="SIZES",
+                    help="instead of the headline workload: prefill and decode throughput of the hyper-connected decoder (Tomopel) "
+                         "beside a mixture-of-experts decoder of equal size, per-op times against the roofline (one GPU)")
     ap.add_argument("--layers", type=int, default=0, help="debug only: a value other than 0 marks the result invalid")
     ap.add_argument("--no-baseline", action="store_true",
                     help="skip the NCCL baseline arm (unfused GEMM + ncclAllReduce) that vs_baseline is measured against")
@@ -140,12 +143,13 @@ def main():
         print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}))
         return 0
 
-    if args.hybrid or args.gorulorn or args.ritirax:
+    if args.hybrid or args.gorulorn or args.ritirax or args.tomopel:
         from gllm_b200.utils import hybrid_bench
         clocks = ClockSampler(0)
         clocks.start()
-        run = (hybrid_bench.main if args.hybrid else hybrid_bench.gorulorn_main if args.gorulorn else hybrid_bench.ritirax_main)
-        res = run((args.hybrid or args.gorulorn or args.ritirax).split(","), max(args.steps, 3), max(args.warmup, 3))
+        run = (hybrid_bench.main if args.hybrid else hybrid_bench.gorulorn_main if args.gorulorn else
+               hybrid_bench.ritirax_main if args.ritirax else hybrid_bench.tomopel_main)
+        res = run((args.hybrid or args.gorulorn or args.ritirax or args.tomopel).split(","), max(args.steps, 3), max(args.warmup, 3))
         print(json.dumps({"metric": "hybrid_decoder_tokens_per_s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
                           "dtype": "bf16", "data": "synthetic", "clocks": clocks.stop(), "results": res}))
         return 0

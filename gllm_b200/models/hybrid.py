@@ -39,6 +39,9 @@ from .weights import layer_prefix
 
 
 def is_norm_weight(name: str) -> bool:
+    """Tensors around 1: norm weights, and the weights in front of and behind a sublayer of hyper-connected streams."""
+    if name.endswith((".hc1.in", ".hc1.out", ".hc2.in", ".hc2.out")):
+        return True
     return name.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2", "norm1b", "norm2b", "final_norm")
 
 

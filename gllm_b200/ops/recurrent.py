@@ -459,7 +459,7 @@ def conv_act(sv: SeqView, x, w, b, ring, out):
             z = torch.cat([_conv_history(ring[slot], start, taps), u])
             a = sum(z[j:j + n] * w[:, j] for j in range(taps)) + b
             out[r0:r0 + n].copy_(torch.nn.functional.silu(a).to(out.dtype))
-            for i in range(max(0, n - taps), n):
+            for i in range(max(0, n - taps) if taps > 1 else n, n):
                 ring[slot, (start + i) % taps] = u[i]
         return out
     nv.check(nv.lib().gllm_conv_act(*sv.ptrs(), sv.max_q_len, x.data_ptr(), x.stride(0), _f32(x), w.data_ptr(), b.data_ptr(),

@@ -2,7 +2,8 @@
 (``bench.py --hybrid``), Gorulorn beside a mixture-of-experts decoder with the same sliding window (``bench.py --gorulorn``; its
 latent attention also beside the latent kernel of the MLA models, at the same heads, rank and number of keys), Ritirax beside a
 mixture-of-experts decoder (``bench.py --ritirax``; its latent layers also beside Gorulorn's and the MLA kernel, its lightning
-layers beside gated linear attention, all at equal sizes).
+layers beside gated linear attention, all at equal sizes), Tomopel beside a mixture-of-experts decoder (``bench.py --tomopel``; its
+attention and state-space layers also beside Ritirax's attention and lightning layers, its minGRU beside the RG-LRU).
 
 Both models have random weights, the same width, depth, attention heads, feed-forward and vocabulary. Prefill: one forward
 over 4 prompts of 2048 tokens. Decode: one captured step of B sequences at context 2048. Whole steps are timed with CUDA
@@ -41,6 +42,12 @@ RITIRAX_SIZES = {
     "1024": dict(hidden=1024, heads=16, kv=4, lat=8, kv_rank=256, lin=8, experts=32, top=4, ff=512, dense=4096),
     "2048": dict(hidden=2048, heads=32, kv=4, lat=16, kv_rank=512, lin=16, experts=64, top=8, ff=768, dense=6144),
     "4096": dict(hidden=4096, heads=32, kv=8, lat=32, kv_rank=512, lin=32, experts=64, top=8, ff=1536, dense=12288),
+}
+# width, query / kv heads, heads of 64 and groups of the state-space layers, width of the minGRU, experts
+TOMOPEL_SIZES = {
+    "1024": dict(hidden=1024, heads=16, kv=4, ssd=32, groups=1, gru=1536, experts=32, top=4, ff=512, dense=3072),
+    "2048": dict(hidden=2048, heads=32, kv=4, ssd=64, groups=1, gru=3072, experts=64, top=8, ff=768, dense=6144),
+    "4096": dict(hidden=4096, heads=32, kv=8, ssd=128, groups=8, gru=4096, experts=64, top=8, ff=1536, dense=12288),
 }
 VOCAB, CHUNK, PROMPT, PROMPTS = 32768, 2048, 2048, 4
 WINDOW, KEEP = 1024, 64
@@ -91,6 +98,43 @@ def ritirax_config(s: dict) -> ModelConfig:
     cfg = ModelConfig(arch="ritirax", hidden_size=s["hidden"], num_layers=6, vocab_size=VOCAB, rms_norm_eps=1e-5, norm_one_plus_w=True,
                       block="parallel", hidden_act="silu", embedding_scale=s["hidden"] ** 0.5, max_position_embeddings=1 << 16,
                       layer_specs=specs)
+    cfg.set_hybrid_dims()
+    return cfg
+
+
+def tomopel_config(s: dict, streams: int = 4) -> ModelConfig:
+    att = MixerSpec("attention", heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5, head_qk_norm=True,
+                    qkv_bias=False, o_bias=False, bias_max=256, v_norm=True, q_temp=(0.1, 512), head_gate=True)
+    ssd = MixerSpec("ssd", heads=s["ssd"], vdim=64, dim=128, groups=s["groups"], taps=4, norm_groups=s["groups"])
+    both = MixerSpec("parallel", left=att, right=ssd, left_scale=0.8, right_scale=1.1)
+    gru = MixerSpec("mingru", width=s["gru"])
+    moe = MoeSpec(experts=s["experts"], top=s["top"], ff=s["ff"], gated=False, correction=True, shared_ff=s["ff"])
+    specs = [LayerSpec(both, ff=s["dense"], act="silu")] + [LayerSpec(m, act="relu2", moe=moe) for m in (gru, both, both, gru, both)]
+    cfg = ModelConfig(arch="tomopel", hidden_size=s["hidden"], num_layers=6, vocab_size=VOCAB, rms_norm_eps=1e-5, norm_one_plus_w=True,
+                      block="pre", streams=streams, residual_mult=0.8, hidden_act="silu", embedding_scale=s["hidden"] ** 0.5,
+                      max_position_embeddings=1 << 16, layer_specs=specs)
+    cfg.set_hybrid_dims()
+    return cfg
+
+
+def lightning_config(s: dict) -> ModelConfig:
+    """Attention with capped and biased scores and lightning attention, with the heads of ``tomopel_config``'s layers."""
+    att = MixerSpec("attention", heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5, head_qk_norm=True,
+                    qkv_bias=False, o_bias=False, softcap=30.0, bias_max=256, sink=True)
+    lin = MixerSpec("lightning", heads=s["ssd"], dim=128, vdim=64,
+                    decay=tuple(1 - 2.0 ** -(1 + 8 * h / s["ssd"]) for h in range(s["ssd"])))
+    cfg = ModelConfig(arch="ritirax", hidden_size=s["hidden"], num_layers=2, vocab_size=VOCAB, rms_norm_eps=1e-5, norm_one_plus_w=True,
+                      block="parallel", hidden_act="silu", embedding_scale=1.0, max_position_embeddings=1 << 16,
+                      layer_specs=[LayerSpec(att, ff=s["dense"], act="relu2", gated=False), LayerSpec(lin, act="silu")])
+    cfg.set_hybrid_dims()
+    return cfg
+
+
+def rglru_config(s: dict) -> ModelConfig:
+    """RG-LRU layers as wide as ``tomopel_config``'s minGRU layers, and its dense feed-forward."""
+    lru = MixerSpec("rglru", width=s["gru"], blocks=16, taps=4)
+    cfg = ModelConfig(arch="zenevik", hidden_size=s["hidden"], num_layers=2, vocab_size=VOCAB, rms_norm_eps=1e-5, postln_alpha=2.0,
+                      hidden_act="silu", max_position_embeddings=1 << 16, layer_specs=[LayerSpec(lru, ff=s["dense"], act="silu"), LayerSpec(lru)])
     cfg.set_hybrid_dims()
     return cfg
 
@@ -174,14 +218,47 @@ def work(cfg: ModelConfig, T: int, decode: bool, rows: int) -> Dict[str, tuple]:
         else:
             add("attention", (T * (2 * heads + 2 * kv) * d * 2, 4 * T * n * heads * d))
 
-    def experts(E, top, ff):
+    def experts(E, top, ff, gated=True):
         used = E * (1 - (1 - top / E) ** T)
-        rows = T * top
+        rows, n = T * top, 2 if gated else 1
         add("moe_route", _gemm(T, E, H, 4))
         add("moe_permute", ((T + rows) * H * 2, 0))
-        add("moe_gate_up", (rows * (H + ff) * 2 + used * 2 * ff * H * 2, 4 * rows * ff * H))
+        add("moe_gate_up" if gated else "moe_up", (rows * (H + ff) * 2 + used * n * ff * H * 2, 2 * n * rows * ff * H))
         add("moe_down", (rows * (H + ff) * 2 + used * ff * H * 2, 2 * rows * ff * H))
-    if cfg.block == "parallel":
+    if cfg.block == "pre":
+        S = max(cfg.streams, 1)
+        norm = lambda extra: add("norm", (T * H * (8 * S + 2 + extra), 0))      # the streams read and written, the next operand
+        for l in cfg.layer_specs:
+            m, moe = l.mixer, l.moe
+            if m.kind == "mingru":
+                add("in_gemm", _gemm(T, 3 * m.width, H))
+                add("mingru", (T * m.width * (8 + (8 if decode else 0)), 0))
+                add("out_gemm", _gemm(T, H, m.width, 4))
+            else:
+                a, r = m.left, m.right
+                nq, nk, inner, ch = a.heads * a.dim, a.kv_heads * a.dim, r.heads * r.vdim, r.conv_channels
+                add("in_gemm", _gemm(T, nq + 2 * nk + a.heads + inner + ch + r.heads, H))
+                add("qk_prep", (T * (2 * nq + 4 * nk) * 2, 0))
+                attend(a.heads, a.kv_heads, a.dim)
+                add("head_gate", (T * nq * 4, 0))
+                add("ssd_conv", (T * ch * (4 + (4 * (r.taps + 1) if decode else 0)), 0))
+                if decode:
+                    add("ssd", (T * r.heads * r.dim * r.vdim * 8 + T * ch * 2 + T * inner * 4, 0))
+                else:      # as for linear attention below
+                    add("ssd", (T * ch * 2 + T * inner * 4, 2 * T * r.heads * (2 * r.dim * r.vdim + 32 * (r.dim + r.vdim))))
+                add("ssd_gate", (T * inner * 8, 0))
+                add("out_gemm", _gemm(T, H, nq + inner, 4))
+            norm(4)
+            if l.ff:
+                add("gate_up_gemm", (T * H * 2 + 2 * l.ff * H * 2 + T * l.ff * 2, 4 * T * l.ff * H))
+                add("down_gemm", _gemm(T, H, l.ff, 4))
+                norm(4)
+            elif moe:
+                experts(moe.experts, moe.top, moe.ff, moe.gated)
+                add("shared_up", _gemm(T, moe.shared_ff, H))
+                add("shared_down", _gemm(T, H, moe.shared_ff, 4))
+                norm(4 + 2 * moe.top)
+    elif cfg.block == "parallel":
         for l in cfg.layer_specs:
             m, moe = l.mixer, l.moe
             if m.kind == "attention":
@@ -214,12 +291,12 @@ def work(cfg: ModelConfig, T: int, decode: bool, rows: int) -> Dict[str, tuple]:
             if l.ff:
                 add("up_gemm", _gemm(T, l.ff, H))
                 add("down_gemm", _gemm(T, H, l.ff, 4))
-            else:
+            elif moe:
                 experts(moe.experts, moe.top, moe.ff)
                 add("shared_gate_up", (T * H * 2 + 2 * moe.shared_ff * H * 2 + T * moe.shared_ff * 2, 4 * T * moe.shared_ff * H))
                 add("shared_down", _gemm(T, H, moe.shared_ff, 4))
             # the stream read and written, the next operand written, the sublayers' outputs read
-            add("norm", (T * H * (4 + 4 + 2 + 4 + (4 if l.ff else 4 + 2 * moe.top)), 0))
+            add("norm", (T * H * (4 + 4 + 2 + 4 + (4 if l.ff else 4 + 2 * moe.top if moe else 0)), 0))
     elif cfg.block == "sandwich":
         stream = T * H * (4 + 4 + 2)          # the residual sum read and written, the next operand written
         for i, _ in cfg.layer_runs():
@@ -434,6 +511,20 @@ def main(sizes=("2048", "2048d64", "4096"), steps: int = 10, warmup: int = 3) ->
     for size in sizes:
         for name, cls, cfg in (("zenevik", HybridDecoder, hybrid_config(SIZES[size])),
                                ("dense", DecoderModel, dense_config(SIZES[size]))):
+            src = RandomWeights(cfg, "cuda", torch.bfloat16, seed=0)
+            model = cls(cfg, src, device="cuda", dtype=torch.bfloat16, max_positions=PROMPT)
+            out[f"{name}-{size}"] = bench_model(model, steps, warmup)
+            del model, src
+            torch.cuda.empty_cache()
+    return out
+
+
+def tomopel_main(sizes=tuple(TOMOPEL_SIZES), steps: int = 10, warmup: int = 3) -> dict:
+    out = {}
+    for size in sizes:
+        s = TOMOPEL_SIZES[size]
+        for name, cls, cfg in (("tomopel", HybridDecoder, tomopel_config(s)), ("moe", DecoderModel, moe_config(s, 6, 0)),
+                               ("lightning", HybridDecoder, lightning_config(s)), ("rglru", HybridDecoder, rglru_config(s))):
             src = RandomWeights(cfg, "cuda", torch.bfloat16, seed=0)
             model = cls(cfg, src, device="cuda", dtype=torch.bfloat16, max_positions=PROMPT)
             out[f"{name}-{size}"] = bench_model(model, steps, warmup)

@@ -222,3 +222,127 @@ def greedy(cfg, weights, prompt, n):
     for _ in range(n):
         toks.append(int(forward(cfg, weights, toks)[-1].argmax()))
     return toks[len(prompt):]
+
+
+# ------------------------------------------------------------------------------------------------
+# configurations and weights of the tests
+# ------------------------------------------------------------------------------------------------
+def dense_ff(ff=72):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(ff=24, experts=6, top=2, shared=40):
+    return {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": shared}, "router": {"experts": experts, "top": top}}
+
+
+def att(heads=4, kv_heads=2, dim=16, vdim=24, far=50, scale=None, coef=0.4, every=24):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or dim ** -0.5, "bias_max": far,
+            "q_temp": {"coef": coef, "every": every}}
+
+
+def state_space(heads=4, vdim=16, state=16, groups=2, conv=4, norm_groups=2):
+    return {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": norm_groups}
+
+
+def par(left=None, right=None, scales=(0.7, 1.3), mlp=None):
+    return {"type": "parallel", "mlp": mlp, "mixer": {"left": left or att(), "right": right or state_space(), "left_scale": scales[0],
+                                                      "right_scale": scales[1]}}
+
+
+def gru(width=72, mlp=None):
+    return {"type": "mingru", "mlp": mlp, "mixer": {"width": width}}
+
+
+def config(layers, width=64, vocab=96, eps=1e-6, embed=6.5, streams=3, mult=0.8):
+    return {"architecture": "Tomopel", "layers": layers, "width": width, "vocab": vocab, "norm": {"eps": eps},
+            "embedding": {"scale": embed}, "streams": streams, "residual_mult": mult}
+
+
+def weights(cfg, seed=0, sharp=2.0, rows=12):
+    """Random weights, rounded to bf16. ``sharp`` scales the queries (one key then stands out in a softmax), ``rows`` is the
+    length of the distance tables. With experts every token id has one of four kinds, a strong direction of its embedding, and the
+    router separates the experts of each kind: some are chosen by their score, some only through their correction, past one whose
+    score is higher; and rounding decides about none of them."""
+    gen = torch.Generator().manual_seed(seed)
+    rn = lambda *shape, s=1.0: torch.randn(shape, generator=gen) * s
+    lin = lambda o, i, s=1.0: rn(o, i, s=s / math.sqrt(i))
+    one = lambda n, s=1.0: s * (1 + 0.2 * rn(n))
+    zero = lambda n: 0.2 * rn(n)
+    Wd, V, scale, S = cfg["width"], cfg["vocab"], cfg["embedding"]["scale"], cfg["streams"]
+    w = {"embed": rn(V, Wd), "head": lin(V, Wd, 2.0), "final.norm": zero(Wd)}
+    kinds = torch.linalg.qr(rn(Wd, 4)).Q.T
+    if any(l["mlp"] and l["mlp"]["kind"] == "moe" for l in cfg["layers"]):
+        w["embed"] += 12 * math.sqrt(Wd) * kinds[torch.arange(V) % 4]
+    w["embed"] /= scale
+
+    def router(E, top):
+        helped = torch.randperm(E, generator=gen)[:E // 2].tolist()
+        na = min(len(helped), (top + 1) // 2)
+        nb = min(top - na, E - len(helped))
+        na = top - nb
+        z = torch.zeros(4, E)
+        for k in range(4):
+            order = torch.randperm(E, generator=gen).tolist()
+            inside, outside = [e for e in order if e in helped], [e for e in order if e not in helped]
+            u = torch.full((E,), 0.03)
+            u[inside[:na]], u[outside[:nb]], u[outside[nb:nb + 1]] = 0.7, 3.0, 1.1
+            z[k] = torch.log(u * (1 + 0.1 * torch.rand(E, generator=gen)))
+        correction = torch.zeros(E)
+        correction[helped] = 1.9 / float(u.sum())
+        return z.T @ kinds / math.sqrt(Wd) + lin(E, Wd, 0.01), correction
+    for n, layer in enumerate(cfg["layers"]):
+        m, p = layer["mixer"], f"l{n}.mix."
+        if layer["type"] == "mingru":
+            W = m["width"]
+            w.update({p + "z": lin(W, Wd, 0.7), p + "x": lin(W, Wd), p + "g": lin(W, Wd), p + "o": lin(Wd, W), p + "x.b": 0.5 * rn(W),
+                      p + "z.b": torch.tensor([-7.0, -3.0, 0.0, 1.5])[torch.arange(W) % 4] + 0.3 * rn(W)})
+        else:
+            a, r = m["left"], m["right"]
+            H, G, d, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            w.update({p + "left." + k: t for k, t in {
+                "q": lin(H * d, Wd), "k": lin(G * d, Wd), "v": lin(G * dv, Wd), "q.norm": one(d, sharp), "k.norm": one(d),
+                "rel": 1.5 * rn(rows, H), "g": lin(H, Wd, 2.0), "o": lin(Wd, H * dv)}.items()})
+            H, P, N, G = r["heads"], r["vdim"], r["state"], r["groups"]
+            ch = H * P + 2 * G * N
+            w.update({p + "right." + k: t for k, t in {
+                "in": lin(2 * H * P + 2 * G * N + H, Wd), "conv": 0.6 * rn(ch, r["conv"]), "conv.b": 0.3 * rn(ch), "dt_bias": rn(H) - 1.0,
+                "A_log": torch.tensor([-5.0, 0.0, 1.0, -2.0])[torch.arange(H) % 4] + 0.2 * rn(H), "D": one(H), "norm": one(H * P),
+                "o": lin(Wd, H * P)}.items()})
+        mlp, q = layer["mlp"], f"l{n}.mlp."
+        w[f"l{n}.norm1"] = zero(Wd)
+        for sub in (1, 2) if mlp else (1,):
+            h = f"l{n}.hc{sub}."
+            w.update({h + "in": 0.6 + 0.3 * rn(S), h + "out": 1 + 0.3 * rn(S), h + "mix": 0.6 * torch.eye(S) + 0.4 / S + 0.15 * rn(S, S)})
+        if mlp:
+            w[f"l{n}.norm2"] = zero(Wd) if mlp["kind"] == "dense" else 0.05 * rn(Wd)
+        if mlp and mlp["kind"] == "dense":
+            w.update({q + "gate": lin(mlp["ff"], Wd, 1.5), q + "up": lin(mlp["ff"], Wd, 1.5), q + "down": lin(Wd, mlp["ff"])})
+        elif mlp:
+            w[q + "router"], w[q + "correction"] = router(mlp["router"]["experts"], mlp["router"]["top"])
+            for e, f in [(f"e{e}", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])] + [("shared", mlp["shared"]["ff"])]:
+                w.update({f"{q}{e}.up": lin(f, Wd), f"{q}{e}.down": lin(Wd, f)})
+    return {k: v.to(torch.bfloat16) for k, v in w.items()}
+
+
+def tokens(cfg, n, seed=0):
+    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(1000 + seed)).tolist()
+
+
+def save(folder, cfg, w):
+    """config.json and model.safetensors (bf16)."""
+    (folder / "config.json").write_text(json.dumps(cfg))
+    head, data = {}, b""
+    for k, v in w.items():
+        raw = v.contiguous().view(torch.int16).numpy().tobytes()
+        head[k] = {"dtype": "BF16", "shape": list(v.shape), "data_offsets": [len(data), len(data) + len(raw)]}
+        data += raw
+    h = json.dumps(head).encode()
+    (folder / "model.safetensors").write_bytes(struct.pack("<Q", len(h)) + h + data)
+    return folder
+
+
+def error(got, want):
+    """Largest over the rows of rms(difference of centred logits) / rms(centred logits)."""
+    c = lambda t: t.to(D) - t.to(D).mean(-1, keepdim=True)
+    g, w = c(torch.as_tensor(got)), c(torch.as_tensor(want))
+    return float(((g - w).pow(2).mean(-1).sqrt() / w.pow(2).mean(-1).sqrt()).max())
