@@ -6,7 +6,8 @@
 //                          projected from the token; q and k (C and B there) are shared by a group of heads
 //
 //   lightning_chunk_kernel    bf16 prompts in chunks of 64 tokens on tensor cores; a CTA owns one (sequence, head, 64 value
-//                             columns) and keeps its slice of the state in fp32 registers from chunk to chunk
+//                             columns) and keeps its slice of the state in fp32 registers from chunk to chunk (state-space layers
+//                             of the usual sizes: ssd_chunk.cu)
 //   lightning_decode_kernel   one token per sequence; a CTA streams the fp32 state [dim][vdim] of one (sequence, head) once
 //   lightning_step_kernel     any sizes, bf16 or fp32, token by token
 //   row_norm_gate_kernel      RMS norm over a whole row times a weight times sigmoid(gate)
@@ -18,52 +19,15 @@
 // core as a (value, remainder) pair. The powers a^0 .. a^64 of every head come from a table, 1 - a as a number of its own: a
 // state remembers 1 / (1 - a) tokens, so the distance of a decay to 1 has to keep its relative accuracy. With decays per token
 // a^(i-j) becomes the exponential of a difference of running sums, and the values are scaled by d_j.
-#include "mma.cuh"
-#include "recurrent.cuh"
+#include "linear_attention.cuh"
 
 namespace gllm {
 
-using bf16_t = __nv_bfloat16;
-constexpr int kLiC = 64, kLiV = 64, kLiThreads = 256, kLiSlice = 128;
+constexpr int kLiV = 64, kLiThreads = 256, kLiSlice = 128;
 constexpr int kLiVP = kLiV + 8, kLiAP = kLiC + 8;          // bf16 per row of the value and score tiles
 
-struct LightningParams {
-  SeqView sv;
-  const void *q, *k, *v;
-  long long ld;
-  int heads, dim, vdim;
-  const float* forget;     // [heads] 1 - decay
-  const float* powers;     // [heads][kLiC + 1] decay^n
-  float* state;            // [slots][heads][dim][vdim]
-  float* out;              // [rows, heads * vdim]
-  // SSD: the steps [rows, heads] (type and rows of q, pitch ldt), [heads] each of the others, heads per q / k head
-  const void* dt;
-  long long ldt;
-  const float *dt_bias, *neg_a, *skip;
-  int group;
-};
-
-template <typename T> __device__ __forceinline__ float ssd_step(const LightningParams& p, long long row, int head) {
-  return softplus_f(to_f(static_cast<const T*>(p.dt)[row * p.ldt + head]) + p.dt_bias[head]);
-}
-__device__ __forceinline__ float li_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-constexpr float kLiLog2e = 1.4426950408889634f;
-
-__device__ __forceinline__ void li_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(x, y);
-  lo = pack_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xFFFF0000u));
-}
 // Element offset in a state tile [rows][64] bf16: 16-byte groups XOR-swizzled by the row.
 __device__ __forceinline__ int li_state_off(int row, int col) { return row * kLiV + ((((col >> 3) ^ row) & 7) << 3) + (col & 7); }
-// 16 bytes, or zeros when there is nothing to copy.
-__device__ __forceinline__ void li_cp16(void* dst, const void* src, bool there) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(there ? 16 : 0) : "memory");
-}
-
 // NSL: key dimensions in slices of 128 (1 or 2); ST: chunks in flight (the next one loads while one is computed)
 template <int NSL, int ST> struct LiShape {
   static constexpr int KP = NSL * kLiSlice + 8;
@@ -583,6 +547,7 @@ static int li_run(const LightningParams& p, int is_f32, int general, cudaStream_
     return li_done(is_f32 ? launch_kernel(lightning_decode_kernel<float, SSD>, grid, dim3(256), decode_smem, s, true, 0, p)
                           : launch_kernel(lightning_decode_kernel<bf16_t, SSD>, grid, dim3(256), decode_smem, s, true, 0, p), "decode");
   }
+  if (SSD && !general && p.sv.q_start && !is_f32 && ssd_chunks_ok(p)) return li_done(ssd_chunks(p, s), "ssd chunks");
   if (!general && p.sv.q_start && !is_f32 && dim % 16 == 0 && dim <= 2 * kLiSlice && vdim % 8 == 0 && p.ld % 8 == 0 && li_al16(p.q) &&
       li_al16(p.k) && li_al16(p.v))
     return dim <= kLiSlice ? li_chunks<1, 2, SSD>(p, s) : li_chunks<2, 1, SSD>(p, s);

@@ -29,7 +29,6 @@ struct MinGruParams {
   const float* seg_init;     // [seqs, n_seg, W] start states, or null (one segment: the slot's state)
 };
 
-__device__ __forceinline__ float mg_candidate(float u) { return u >= 0.f ? u + 0.5f : sigmoid_f(u); }
 // first (f, b), then (f2, b2)
 __device__ __forceinline__ void mg_then(float& f, float& b, float f2, float b2) {
   b = fmaf(-f2, b, b) + b2;
@@ -44,17 +43,12 @@ __device__ __forceinline__ void mg_segment(int len, int n_seg, int seg, int& t0,
 }
 
 template <bool SUMMARY>
-__global__ void __launch_bounds__(kMgThreads, 2) mingru_tile_kernel(const MinGruParams p) {
-  __shared__ float fs[8][kMgCh], bs[8][kMgCh], carry[2][2][kMgCh];      // per warp; state (summary: also F) by tile parity
+__global__ void __launch_bounds__(kMgThreads, 3) mingru_tile_kernel(const MinGruParams p) {
+  __shared__ __align__(16) float fs[8][kMgCh], bs[8][kMgCh], start[9][kMgCh];   // of each warp: (F, B); state in front of it ([8]: behind the tile)
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int cv = lane & 3, sub = lane >> 2;        // 8-channel group, place among the warp's 8 token pairs
   const int c0 = blockIdx.x * kMgCh + cv * 8;
   const bool live = c0 < p.W;
-  float bz[8] = {}, bx[8] = {};
-  if (live) {
-    load8(p.bz + c0, bz);
-    load8(p.bx + c0, bx);
-  }
   pdl_wait();
   pdl_launch_dependents();
   const int seq = blockIdx.y / p.n_seg, seg = blockIdx.y % p.n_seg;
@@ -63,6 +57,7 @@ __global__ void __launch_bounds__(kMgThreads, 2) mingru_tile_kernel(const MinGru
   int t0, t1;
   mg_segment(s.len, p.n_seg, seg, t0, t1);
   const long long seg_at = (static_cast<long long>(seq) * p.n_seg + seg) * p.W;
+  float total = 0.f;                               // summary: F of the segment so far (one thread per channel)
   if (tid < kMgCh) {
     const int c = blockIdx.x * kMgCh + tid;
     float S = 0.f;
@@ -70,19 +65,20 @@ __global__ void __launch_bounds__(kMgThreads, 2) mingru_tile_kernel(const MinGru
       if (p.seg_init) S = p.seg_init[seg_at + c];
       else if (s.start > 0) S = p.state[static_cast<long long>(s.slot) * p.W + c];
     }
-    carry[0][0][tid] = S;
-    carry[0][1][tid] = 0.f;
+    start[8][tid] = S;
   }
-  const bf16_t* zx = static_cast<const bf16_t*>(p.zx) + static_cast<long long>(s.row0) * p.ld + c0;
-  const bf16_t* cx = static_cast<const bf16_t*>(p.cx) + static_cast<long long>(s.row0) * p.ld + c0;
-  const bf16_t* gx = static_cast<const bf16_t*>(p.g) + static_cast<long long>(s.row0) * p.ld + c0;
   const int mine = (warp * 8 + sub) * 2;           // the thread's two tokens of a tile
+  const long long at0 = static_cast<long long>(s.row0 + mine) * p.ld + c0;
+  const bf16_t* zx = static_cast<const bf16_t*>(p.zx) + at0;
+  const bf16_t* cx = static_cast<const bf16_t*>(p.cx) + at0;
+  const bf16_t* gx = static_cast<const bf16_t*>(p.g) + at0;
+  bf16_t* out = static_cast<bf16_t*>(p.out) + static_cast<long long>(s.row0 + mine) * p.W + c0;
   uint4 zr[2], cr[2], gr[2];
   auto fetch = [&](int t) {
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const bool ok = live && t + mine + i < t1;
-      const long long at = static_cast<long long>(t + mine + i) * p.ld;
+      const long long at = static_cast<long long>(t + i) * p.ld;
       zr[i] = ok ? *reinterpret_cast<const uint4*>(zx + at) : make_uint4(0, 0, 0, 0);
       cr[i] = ok ? *reinterpret_cast<const uint4*>(cx + at) : make_uint4(0, 0, 0, 0);
       if (!SUMMARY) gr[i] = ok ? *reinterpret_cast<const uint4*>(gx + at) : make_uint4(0, 0, 0, 0);
@@ -97,29 +93,31 @@ __global__ void __launch_bounds__(kMgThreads, 2) mingru_tile_kernel(const MinGru
     }
   };
   fetch(t0);
-  int par = 0;
-  for (int t = t0; t < t1; t += kMgTok, par ^= 1) {
-    float F[2][8], B[2][8], gate[2][8];            // of each token
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const bool ok = t + mine + i < t1;
-      float a[8], u[8];
-      expand(zr[i], a);
-      expand(cr[i], u);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        F[i][e] = ok ? sigmoid_f(a[e] + bz[e]) : 0.f;
-        B[i][e] = F[i][e] * mg_candidate(u[e] + bx[e]);
+  for (int t = t0; t < t1; t += kMgTok) {
+    float F[2][8], B[2][8], f[8], b[8];            // of each token; of the pair
+    uint4 gate[2];
+    {
+      float bz[8] = {}, bx[8] = {};                // from L1: not worth the registers
+      if (live) {
+        load8(p.bz + c0, bz);
+        load8(p.bx + c0, bx);
       }
-      if (!SUMMARY) {
-        expand(gr[i], gate[i]);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) gate[i][e] = silu_exact(gate[i][e]);
+      for (int i = 0; i < 2; ++i) {
+        const bool ok = t + mine + i < t1;
+        float a[8], u[8];
+        expand(zr[i], a);
+        expand(cr[i], u);
+        gate[i] = gr[i];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          F[i][e] = ok ? sigmoid_t<bf16_t>(a[e] + bz[e]) : 0.f;
+          const float v = u[e] + bx[e];
+          B[i][e] = F[i][e] * (v >= 0.f ? v + 0.5f : sigmoid_t<bf16_t>(v));
+        }
       }
     }
     if (t + kMgTok < t1) fetch(t + kMgTok);
-    // inclusive over the warp's token pairs, then what is in front of this thread's pair
-    float f[8], b[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       f[e] = F[0][e];
@@ -127,7 +125,7 @@ __global__ void __launch_bounds__(kMgThreads, 2) mingru_tile_kernel(const MinGru
       mg_then(f[e], b[e], F[1][e], B[1][e]);
     }
 #pragma unroll
-    for (int o = 1; o < 8; o <<= 1)
+    for (int o = 1; o < 8; o <<= 1)                // inclusive over the warp's token pairs
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         float fu = __shfl_up_sync(0xffffffffu, f[e], o * 4), bu = __shfl_up_sync(0xffffffffu, b[e], o * 4);
@@ -138,30 +136,26 @@ __global__ void __launch_bounds__(kMgThreads, 2) mingru_tile_kernel(const MinGru
         }
       }
     if (sub == 7) {
-#pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        fs[warp][cv * 8 + e] = f[e];
-        bs[warp][cv * 8 + e] = b[e];
-      }
+      store8(&fs[warp][cv * 8], f);
+      store8(&bs[warp][cv * 8], b);
     }
     __syncthreads();
-    if (tid < kMgCh) {                             // the tile's carry for the next one
-      float S = carry[par][0][tid], G = carry[par][1][tid];
+    if (tid < kMgCh) {
+      float S = start[8][tid];
 #pragma unroll
       for (int w = 0; w < 8; ++w) {
-        if (SUMMARY) G = fmaf(-fs[w][tid], G, G) + fs[w][tid];
+        start[w][tid] = S;
+        if (SUMMARY) total = fmaf(-fs[w][tid], total, total) + fs[w][tid];
         S = fmaf(-fs[w][tid], S, S) + bs[w][tid];
       }
-      carry[par ^ 1][0][tid] = S;
-      carry[par ^ 1][1][tid] = G;
+      start[8][tid] = S;
     }
+    __syncthreads();
     if constexpr (!SUMMARY) {
-      float S[8];
-#pragma unroll
-      for (int e = 0; e < 8; ++e) S[e] = carry[par][0][cv * 8 + e];
-      for (int w = 0; w < warp; ++w)
-#pragma unroll
-        for (int e = 0; e < 8; ++e) S[e] = fmaf(-fs[w][cv * 8 + e], S[e], S[e]) + bs[w][cv * 8 + e];
+      float S[8], g[2][8];
+      load8(&start[warp][cv * 8], S);
+      expand(gate[0], g[0]);
+      expand(gate[1], g[1]);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {                // the pairs of the warp in front of this one
         const float fu = __shfl_up_sync(0xffffffffu, f[e], 4), bu = __shfl_up_sync(0xffffffffu, b[e], 4);
@@ -173,19 +167,17 @@ __global__ void __launch_bounds__(kMgThreads, 2) mingru_tile_kernel(const MinGru
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           S[e] = fmaf(-F[i][e], S[e], S[e]) + B[i][e];
-          o[e] = S[e] * gate[i][e];
+          o[e] = S[e] * silu_t<bf16_t>(g[i][e]);
         }
-        if (live && t + mine + i < t1) store8(static_cast<bf16_t*>(p.out) + static_cast<long long>(s.row0 + t + mine + i) * p.W + c0, o);
+        if (live && t + mine + i < t1) store8(out + static_cast<long long>(t + i) * p.W, o);
       }
     }
-    __syncthreads();                               // the next tile writes fs and bs again
   }
-  __syncthreads();
   if (tid < kMgCh) {
     const int c = blockIdx.x * kMgCh + tid;
     if (c < p.W) {
-      if (SUMMARY) p.seg_sum[seg_at + c] = make_float2(carry[par][1][tid], carry[par][0][tid]);
-      else if (t1 == s.len && (t0 < t1)) p.state[static_cast<long long>(s.slot) * p.W + c] = carry[par][0][tid];
+      if (SUMMARY) p.seg_sum[seg_at + c] = make_float2(total, start[8][tid]);
+      else if (t1 == s.len && t0 < t1) p.state[static_cast<long long>(s.slot) * p.W + c] = start[8][tid];
     }
   }
 }
@@ -220,10 +212,9 @@ __global__ void __launch_bounds__(128) mingru_step_kernel(const MinGruParams p) 
 #pragma unroll 4
   for (int i = 0; i < s.len; ++i) {
     const long long at = static_cast<long long>(s.row0 + i) * p.ld + c;
-    const float z = sigmoid_f(to_f(static_cast<const T*>(p.zx)[at]) + bz);
-    const float v = mg_candidate(to_f(static_cast<const T*>(p.cx)[at]) + bx);
-    S = fmaf(-z, S, S) + z * v;
-    static_cast<T*>(p.out)[static_cast<long long>(s.row0 + i) * p.W + c] = from_f<T>(S * silu_exact(to_f(static_cast<const T*>(p.g)[at])));
+    const float z = sigmoid_t<T>(to_f(static_cast<const T*>(p.zx)[at]) + bz), u = to_f(static_cast<const T*>(p.cx)[at]) + bx;
+    S = fmaf(-z, S, S) + z * (u >= 0.f ? u + 0.5f : sigmoid_t<T>(u));
+    static_cast<T*>(p.out)[static_cast<long long>(s.row0 + i) * p.W + c] = from_f<T>(S * silu_t<T>(to_f(static_cast<const T*>(p.g)[at])));
   }
   *st = S;
 }

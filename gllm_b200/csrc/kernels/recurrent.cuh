@@ -75,6 +75,18 @@ template <typename T> __device__ __forceinline__ void store8(T* p, const float (
 }
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+// Sigmoid and silu of tensors of type T: exact for fp32; for bf16 on the fast units (relative errors of a few 1e-7).
+template <typename T> __device__ __forceinline__ float sigmoid_t(float x) {
+  if constexpr (sizeof(T) == 4) {
+    return sigmoid_f(x);
+  } else {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * -1.4426950408889634f));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+    return r;
+  }
+}
+template <typename T> __device__ __forceinline__ float silu_t(float x) { return x * sigmoid_t<T>(x); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float log_sigmoid_f(float x) { return -softplus_f(-x); }
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.f + expf(-x)); }

@@ -81,7 +81,7 @@ __global__ void __launch_bounds__(kConvThreads) conv_act8_kernel(const ConvActPa
 #pragma unroll
       for (int k = TAPS - 2; k > 0; --k) hist[k][e] = hist[k - 1][e];
       if constexpr (TAPS > 1) hist[0][e] = v[e];
-      y[e] = silu_exact(a);
+      y[e] = silu_t<T>(a);
     }
     store8(static_cast<T*>(p.out) + m * p.channels + c, y);
   }
@@ -112,7 +112,7 @@ __global__ void __launch_bounds__(kConvThreads) conv_act_any_kernel(const ConvAc
                              : conv_history(p.ring, s.slot, p.taps, p.channels, s.start + k, c);
       a = fmaf(w[j], v, a);
     }
-    static_cast<T*>(p.out)[static_cast<long long>(s.row0 + i) * p.channels + c] = from_f<T>(silu_exact(a));
+    static_cast<T*>(p.out)[static_cast<long long>(s.row0 + i) * p.channels + c] = from_f<T>(silu_t<T>(a));
   }
   if (p.taps > 1 && t0 == 0 && n > 0) advance_conv_ring(s, x, p.ld, p.ring, p.channels, p.taps, c);
 }
@@ -139,13 +139,13 @@ __global__ void __launch_bounds__(THREADS) gate_norm_kernel(const float* y, cons
       const int c = (i * THREADS + tid) * 4;
       if (c < n) {
         const float4 a = load4(src + c), g = load4(zr + c);
-        x[i] = make_float4(a.x * silu_exact(g.x), a.y * silu_exact(g.y), a.z * silu_exact(g.z), a.w * silu_exact(g.w));
+        x[i] = make_float4(a.x * silu_t<T>(g.x), a.y * silu_t<T>(g.y), a.z * silu_t<T>(g.z), a.w * silu_t<T>(g.w));
         ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
       }
     }
   } else {
     for (int c = tid; c < n; c += THREADS) {
-      const float v = src[c] * silu_exact(to_f(zr[c]));
+      const float v = src[c] * silu_t<T>(to_f(zr[c]));
       ss = fmaf(v, v, ss);
     }
   }
@@ -165,7 +165,7 @@ __global__ void __launch_bounds__(THREADS) gate_norm_kernel(const float* y, cons
       store4(dst + c, make_float4(x[i].x * r * g.x, x[i].y * r * g.y, x[i].z * r * g.z, x[i].w * r * g.w));
     }
   } else {
-    for (int c = tid; c < n; c += THREADS) dst[c] = from_f<T>(src[c] * silu_exact(to_f(zr[c])) * r * w[c0 + c]);
+    for (int c = tid; c < n; c += THREADS) dst[c] = from_f<T>(src[c] * silu_t<T>(to_f(zr[c])) * r * w[c0 + c]);
   }
 }
 
@@ -182,7 +182,7 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const T* o, const T* g, 
   if (i >= rows * per) return;
   const long long m = i / per;
   const int c = static_cast<int>(i - m * per) * V;
-  const float f = g ? scale * sigmoid_f(to_f(g[m * ldg + c / vdim])) : scale;
+  const float f = g ? scale * sigmoid_t<T>(to_f(g[m * ldg + c / vdim])) : scale;
   if constexpr (V == 8) {
     float v[8];
     load8(o + m * width + c, v);
