@@ -229,8 +229,18 @@ __global__ void __launch_bounds__(THREADS) hyper_norm_kernel(const HyperNormPara
   auto fma4 = [](float w, float4 f, float4& o) {
     o.x = fmaf(w, f.x, o.x); o.y = fmaf(w, f.y, o.y); o.z = fmaf(w, f.z, o.z); o.w = fmaf(w, f.w, o.w);
   };
+  constexpr bool kAhead = N * MS <= 8;      // all streams of the row are in flight while the sublayer's output is summed
+  float4 xa[kAhead ? N : 1][MS];
+  auto load_streams = [&](int n, float4 (&v)[MS]) {
 #pragma unroll
-  for (int n = 0; n < N; ++n) h[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < MS; ++s) v[s] = load4(xr + static_cast<long long>(s) * H + idx(n));
+  };
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+    h[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if constexpr (kAhead)
+      if (idx(n) < H) load_streams(n, xa[n]);
+  }
   if (p.y) {
     const TY* y = static_cast<const TY*>(p.y);
     const int cnt = p.dest ? p.top : 1;
@@ -252,9 +262,9 @@ __global__ void __launch_bounds__(THREADS) hyper_norm_kernel(const HyperNormPara
 #pragma unroll
   for (int n = 0; n < N; ++n)
     if (idx(n) < H) {
-      float4 xs[MS], u = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-      for (int s = 0; s < MS; ++s) xs[s] = load4(xr + static_cast<long long>(s) * H + idx(n));
+      float4 here[MS], u = make_float4(0.f, 0.f, 0.f, 0.f);
+      if constexpr (!kAhead) load_streams(n, here);
+      const float4(&xs)[MS] = kAhead ? xa[kAhead ? n : 0] : here;
       if (p.y) {
 #pragma unroll
         for (int t = 0; t < MS; ++t) {
